@@ -516,6 +516,73 @@ RLT_API int rlt_sandwich_norm(const void* x, const void* weight, const void* res
                       const void* weight2, void* norm_out, int rows, int hidden, float eps, int dtype,
                       rlt_stream_t stream);
 
+/* ------------------------------------------------------------------------
+ * Parallel-block models with recurrent layers (no counterpart in the reference).
+ *
+ * Packed sequences: sequence s owns rows cu_seqlens[s] .. cu_seqlens[s + 1] - 1 of every row tensor, its
+ * portion starts at position starts[s] of the sequence, and what it carries from step to step lies in
+ * state slot slot_of[s] (a portion that starts at 0 ignores the slot's old content).  `max_tokens` is a
+ * host-side bound on the longest portion: it sizes the launches.
+ * ---------------------------------------------------------------------- */
+
+/* Paged attention with score terms.  Query row at position p (it sees keys 0 .. p), query head h of H:
+ *   score_j = (q . k_j) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
+ *             - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
+ * softmax over the visible keys, weighted sum of the values.  Keys and values may have different head
+ * sizes and cache strides; query and output rows may be column slices (strides in elements).
+ * context_lengths[s]: tokens of sequence s after this portion.  planned != 0: the workspace holds the
+ * plan of rlt_verify_attention_plan for the same tables, lengths and packing (max_new <= 16 only). */
+RLT_API size_t rlt_scored_attention_workspace_bytes(int rows, int sequences, int max_new, int q_heads, int kv_heads,
+                                            int key_dim, int value_dim, int block_size, int table_width, int dtype);
+RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, void* out, int64_t out_stride,
+                         const void* key_cache, int64_t k_block_stride, int64_t k_token_stride,
+                         const void* value_cache, int64_t v_block_stride, int64_t v_token_stride,
+                         int64_t num_blocks, int block_size, int q_heads, int kv_heads, int key_dim,
+                         int value_dim, int dtype, const int32_t* block_tables, int sequences, int table_width,
+                         const int32_t* context_lengths, const int32_t* cu_seqlens_q, int rows, int max_new,
+                         float scale, float temp_coef, int temp_every, int distance_bias, int planned,
+                         void* workspace, size_t workspace_bytes, rlt_stream_t stream);
+
+/* The fp32 residual stream and the norm that opens a layer:
+ *   r = tokens ? embed[tokens[i]] : residual[i];  r += delta[i];  residual[i] = r (store_residual != 0)
+ *   out[row] = r / sqrt(mean(r^2) + eps) * (weight_offset + weight)
+ * i = row_index ? row_index[row] : row.  delta, embed, out: `dtype`; residual, weight: fp32. */
+RLT_API int rlt_residual_norm(float* residual, const void* delta, const int64_t* tokens, const void* embed, int64_t vocab,
+                      const int64_t* row_index, int store_residual, const float* weight, float weight_offset,
+                      void* out, int rows, int width, float eps, int dtype, rlt_stream_t stream);
+
+/* Columns of a stacked projection to where they are needed: k_width columns from k_col and v_width from v_col into
+ * the pages of (row_seq[row], positions[row]) — row_seq -1: a padding row, nothing is written — and act_width
+ * columns from act_col through the activation (1: erf gelu, 2: tanh gelu) into out[row, out_col ..]. */
+RLT_API int rlt_block_epilogue(const void* proj, int64_t proj_stride, int k_col, int k_width, int v_col, int v_width,
+                       void* key_cache, int64_t k_block_stride, int64_t k_token_stride,
+                       void* value_cache, int64_t v_block_stride, int64_t v_token_stride,
+                       int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
+                       const int32_t* row_seq, const int32_t* positions, int act_col, int act_width, int act,
+                       void* out, int64_t out_stride, int out_col, int rows, int dtype, rlt_stream_t stream);
+
+/* Causal convolution per channel with bias and silu; state: [slots][taps - 1][channels] of `dtype` (the last
+ * inputs).  act_*: feed-forward columns of the same projection (stride in_stride) through an activation. */
+RLT_API int rlt_causal_conv(const void* in, int64_t in_stride, const float* weight, const float* bias, void* out,
+                    int64_t out_stride, void* state, int64_t slots, int channels, int taps,
+                    const int32_t* cu_seqlens, const int32_t* starts, const int32_t* slot_of, int sequences,
+                    int max_tokens, const void* act_in, void* act_out, int64_t act_out_stride, int act_width,
+                    int act, int dtype, rlt_stream_t stream);
+
+/* Mamba-2 recurrence, fp32 or bf16 inputs, fp32 state [slots][heads][state_size][head_dim]:
+ *   dt = softplus(dt_raw + dt_bias);  S = exp(-exp(a_log) dt) S + dt B x^T;  y = S^T C + d x */
+RLT_API size_t rlt_ssd_scan_workspace_bytes(int sequences, int max_tokens, int heads, int state, int head_dim, int dtype);
+RLT_API int rlt_ssd_scan(const void* x, const void* b, const void* c, int64_t xbc_stride, const void* dt, int64_t dt_stride,
+                 const float* dt_bias, const float* a_log, const float* d, void* y, int64_t y_stride,
+                 float* state, int64_t slots, const int32_t* cu_seqlens, const int32_t* starts,
+                 const int32_t* slot_of, int sequences, int max_tokens, int heads, int groups, int state_size,
+                 int head_dim, int dtype, void* workspace, size_t workspace_bytes, rlt_stream_t stream);
+
+/* out = rmsnorm_parts(y * silu(z)) * weight: the row is normed in `parts` equal parts, each by its own root mean square. */
+RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight,
+                   void* out, int64_t out_stride, int rows, int width, int parts, float eps, int dtype,
+                   rlt_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

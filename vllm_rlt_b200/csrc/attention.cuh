@@ -1,9 +1,25 @@
 // Argument block and row addressing shared by the attention kernels.
 #pragma once
 
+#include <math.h>
+
 #include "common.cuh"
 
 namespace rlt {
+
+// What happens to q . k before the softmax.  Query row at position p (its visible keys are 0 .. p, so p is
+// the row's length minus one), query head h of H, key at position j:
+//   score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
+//           - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
+// The default is the plain 1 / sqrt(head_dim) of the looped models.
+struct ScoreTerms {
+  float scale = 0.0f;        // 0: 1 / sqrt(head_dim)
+  float temp_coef = 0.0f;
+  int temp_every = 1;
+  int distance_bias = 0;
+
+  __host__ __device__ bool plain() const { return temp_coef == 0.0f && distance_bias == 0; }
+};
 
 struct AttentionArgs {
   const void* q;
@@ -24,7 +40,36 @@ struct AttentionArgs {
   const int32_t* context_lengths;
   const int32_t* cu_seqlens_q;  // nullptr: one table row per query row
   int rows;
+  int value_dim;                // elements of a value head (key heads have head_dim)
+  int64_t v_block_stride;       // the value cache's own strides
+  int64_t v_token_stride;
+  int64_t q_stride;             // elements between consecutive query rows / output rows
+  int64_t out_stride;
+  ScoreTerms terms;
 };
+
+// The layout every entry without extra terms has: one head size, one cache layout, contiguous query and output rows.
+inline void set_plain_layout(AttentionArgs& a) {
+  a.value_dim = a.head_dim;
+  a.v_block_stride = a.block_stride;
+  a.v_token_stride = a.token_stride;
+  a.q_stride = a.out_stride = static_cast<int64_t>(a.q_heads) * a.head_dim;
+}
+
+inline float score_scale(const AttentionArgs& a) {
+  return a.terms.scale != 0.0f ? a.terms.scale : static_cast<float>(1.0 / sqrt(static_cast<double>(a.head_dim)));
+}
+
+// The query temperature of a row that sees `len` keys (position len - 1).
+__device__ __forceinline__ float query_temperature(const ScoreTerms& t, int len) {
+  if (t.temp_coef == 0.0f) return 1.0f;
+  return fmaf(t.temp_coef, logf(static_cast<float>(len / t.temp_every + 1)), 1.0f);
+}
+
+// The distance slope of query head `head`, 0 without a distance bias.
+__device__ __forceinline__ float distance_slope(const ScoreTerms& t, int head, int q_heads) {
+  return t.distance_bias == 0 ? 0.0f : exp2f(-8.0f * static_cast<float>(head + 1) / static_cast<float>(q_heads));
+}
 
 // Table row and number of visible keys of query row `row`.
 // Unpacked: its own table row and context length.  Packed: the sequence s that contains

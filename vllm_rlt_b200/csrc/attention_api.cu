@@ -61,6 +61,7 @@ extern "C" RLT_API int rlt_verify_attention(const void* q, void* out, const void
   a.block_size = block_size; a.q_heads = q_heads; a.kv_heads = kv_heads; a.head_dim = head_dim;
   a.dtype = dtype; a.block_tables = block_tables; a.table_rows = table_rows; a.table_width = table_width;
   a.context_lengths = context_lengths; a.cu_seqlens_q = cu_seqlens_q; a.rows = rows;
+  set_plain_layout(a);
   int status = check_args(a);
   if (status != RLT_OK || rows == 0) return status;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -82,6 +83,7 @@ extern "C" RLT_API int rlt_windowed_attention(const void* q, void* out, const vo
   a.block_size = block_size; a.q_heads = q_heads; a.kv_heads = kv_heads; a.head_dim = head_dim;
   a.dtype = dtype; a.block_tables = block_tables; a.table_rows = rows; a.table_width = table_width;
   a.context_lengths = context_lengths; a.cu_seqlens_q = nullptr; a.rows = rows;
+  set_plain_layout(a);
   int status = check_args(a);
   if (status != RLT_OK || rows == 0) return status;
   return launch_attention_generic(a, static_cast<cudaStream_t>(stream), window);
@@ -96,6 +98,7 @@ extern "C" RLT_API int rlt_verify_attention_plan(const int32_t* block_tables, in
   AttentionArgs a = {};
   a.block_tables = block_tables; a.table_rows = table_rows; a.table_width = table_width;
   a.context_lengths = context_lengths; a.cu_seqlens_q = cu_seqlens_q; a.rows = rows;
+  set_plain_layout(a);
   a.q_heads = q_heads; a.kv_heads = kv_heads; a.head_dim = head_dim; a.block_size = block_size; a.dtype = dtype;
   int status = check_metadata(a);
   if (status != RLT_OK || rows == 0) return status;
@@ -120,6 +123,7 @@ extern "C" RLT_API int rlt_verify_attention_run(const void* q, void* out, const 
   a.block_size = block_size; a.q_heads = q_heads; a.kv_heads = kv_heads; a.head_dim = head_dim;
   a.dtype = dtype; a.block_tables = block_tables; a.table_rows = table_rows; a.table_width = table_width;
   a.context_lengths = context_lengths; a.cu_seqlens_q = cu_seqlens_q; a.rows = rows;
+  set_plain_layout(a);
   int status = check_args(a);
   if (status != RLT_OK || rows == 0) return status;
   if (!attention_sm100_supported(a)) {
@@ -149,6 +153,7 @@ extern "C" RLT_API int rlt_verify_attention_noalloc(const void* q, void* out, co
   a.block_size = block_size; a.q_heads = q_heads; a.kv_heads = kv_heads; a.head_dim = head_dim;
   a.dtype = dtype; a.block_tables = block_tables; a.table_rows = table_rows; a.table_width = table_width;
   a.context_lengths = context_lengths; a.cu_seqlens_q = cu_seqlens_q; a.rows = rows;
+  set_plain_layout(a);
   int status = check_args(a);
   if (status != RLT_OK) return status;
   // A call without rows is the warm-up: it loads the library's device image (and with it the
@@ -181,6 +186,7 @@ extern "C" RLT_API int rlt_prefill_attention(const void* q, void* out, const voi
   a.block_size = block_size; a.q_heads = q_heads; a.kv_heads = kv_heads; a.head_dim = head_dim;
   a.dtype = dtype; a.block_tables = block_tables; a.table_rows = sequences; a.table_width = table_width;
   a.context_lengths = context_lengths; a.cu_seqlens_q = cu_seqlens_q; a.rows = rows;
+  set_plain_layout(a);
   RLT_REQUIRE(cu_seqlens_q != nullptr || rows == 0, "prefill_attention: cu_seqlens_q is required");
   int status = check_args(a);
   if (status != RLT_OK || rows == 0) return status;
@@ -192,5 +198,55 @@ extern "C" RLT_API int rlt_prefill_attention(const void* q, void* out, const voi
   // shapes or cache placements outside the tiled prefill kernel: the grouped verify kernel (which reports
   // RLT_ERR_WORKSPACE when the scratch was sized for the prompt kernels only), or the generic one
   if (attention_sm100_supported(a)) return launch_attention_sm100(a, workspace, workspace_bytes, s);
+  return launch_attention_generic(a, s);
+}
+
+extern "C" RLT_API size_t rlt_scored_attention_workspace_bytes(int rows, int sequences, int max_new, int q_heads, int kv_heads,
+                                                               int key_dim, int value_dim, int block_size, int table_width,
+                                                               int dtype) {
+  if (rows <= 0 || sequences <= 0 || q_heads <= 0 || kv_heads <= 0 || table_width <= 0) return 256;
+  if (dtype == RLT_F32 || key_dim != 128 || value_dim != 128 || block_size != 16) return 256;
+  if (max_new > 16) return rlt::prefill_sm100_workspace_bytes(rows, sequences);
+  return rlt_verify_attention_workspace_bytes(rows, q_heads, kv_heads, key_dim, block_size, table_width);
+}
+
+extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, void* out, int64_t out_stride,
+                                            const void* key_cache, int64_t k_block_stride, int64_t k_token_stride,
+                                            const void* value_cache, int64_t v_block_stride, int64_t v_token_stride,
+                                            int64_t num_blocks, int block_size, int q_heads, int kv_heads, int key_dim,
+                                            int value_dim, int dtype, const int32_t* block_tables, int sequences,
+                                            int table_width, const int32_t* context_lengths, const int32_t* cu_seqlens_q,
+                                            int rows, int max_new, float scale, float temp_coef, int temp_every,
+                                            int distance_bias, int planned, void* workspace, size_t workspace_bytes,
+                                            rlt_stream_t stream) {
+  using namespace rlt;
+  AttentionArgs a;
+  a.q = q; a.out = out; a.key_cache = key_cache; a.value_cache = value_cache;
+  a.block_stride = k_block_stride; a.token_stride = k_token_stride; a.num_blocks = num_blocks;
+  a.block_size = block_size; a.q_heads = q_heads; a.kv_heads = kv_heads; a.head_dim = key_dim;
+  a.dtype = dtype; a.block_tables = block_tables; a.table_rows = sequences; a.table_width = table_width;
+  a.context_lengths = context_lengths; a.cu_seqlens_q = cu_seqlens_q; a.rows = rows;
+  a.value_dim = value_dim; a.v_block_stride = v_block_stride; a.v_token_stride = v_token_stride;
+  a.q_stride = q_stride; a.out_stride = out_stride;
+  a.terms.scale = scale; a.terms.temp_coef = temp_coef; a.terms.temp_every = temp_every; a.terms.distance_bias = distance_bias;
+  RLT_REQUIRE(value_dim > 0 && temp_every > 0, "scored_attention: value_dim and temp_every must be positive");
+  RLT_REQUIRE(cu_seqlens_q != nullptr || rows == 0, "scored_attention: cu_seqlens_q is required");
+  int status = check_args(a);
+  if (status != RLT_OK || rows == 0) return status;
+  RLT_REQUIRE(v_token_stride >= static_cast<int64_t>(kv_heads) * value_dim && v_block_stride >= v_token_stride * block_size,
+              "scored_attention: the [kv_heads, value_dim] tail of the value cache must be contiguous");
+  RLT_REQUIRE(q_stride >= static_cast<int64_t>(q_heads) * key_dim && out_stride >= static_cast<int64_t>(q_heads) * value_dim,
+              "scored_attention: row strides smaller than a row");
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (attention_sm100_supported(a)) {
+    if (max_new > 16) {
+      if (prefill_sm100_supported(a)) {
+        status = launch_prefill_sm100(a, workspace, workspace_bytes, s);
+        if (status != RLT_ERR_UNSUPPORTED) return status;
+      }
+    } else {
+      return planned ? run_attention_sm100(a, workspace, workspace_bytes, s) : launch_attention_sm100(a, workspace, workspace_bytes, s);
+    }
+  }
   return launch_attention_generic(a, s);
 }

@@ -1,5 +1,5 @@
-// Shape-generic paged attention: any head_dim <= 256, any block size, any GQA ratio,
-// fp32 / fp16 / bf16.  One CTA per (query row, query head); four warps stride over the
+// Shape-generic paged attention: any head_dim <= 256 (keys and values may differ), any block size,
+// any GQA ratio, fp32 / fp16 / bf16, with the score terms of attention.cuh.  One CTA per (query row, query head); four warps stride over the
 // row's tokens with an fp32 online softmax each and are merged in warp order, so a row's
 // result depends on nothing but its own query, length and K/V.  This is the path for
 // shapes the tiled sm_100a kernel (attention_sm100.cu) does not cover — the fp32 tiny
@@ -22,14 +22,14 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
   const int row = blockIdx.x / a.q_heads;
   const int head = blockIdx.x % a.q_heads;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int D = a.head_dim;
-  const T* q = static_cast<const T*>(a.q);
-  T* out = static_cast<T*>(a.out) + (static_cast<int64_t>(row) * a.q_heads + head) * D;
+  const int D = a.head_dim, DV = a.value_dim;
+  const T* q = static_cast<const T*>(a.q) + row * a.q_stride + static_cast<int64_t>(head) * D;
+  T* out = static_cast<T*>(a.out) + row * a.out_stride + static_cast<int64_t>(head) * DV;
 
   int table_row, len;
   resolve_row(a, row, &table_row, &len);
   if (len <= 0) {
-    for (int d = threadIdx.x; d < D; d += kThreads) out[d] = Elem<T>::from_float(0.0f);
+    for (int d = threadIdx.x; d < DV; d += kThreads) out[d] = Elem<T>::from_float(0.0f);
     return;
   }
   const int32_t* table = a.block_tables + static_cast<int64_t>(table_row) * a.table_width;
@@ -41,9 +41,10 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
 #pragma unroll
   for (int j = 0; j < kMaxPerLane; ++j) {
     int d = lane + 32 * j;
-    qr[j] = d < D ? Elem<T>::to_float(q[(static_cast<int64_t>(row) * a.q_heads + head) * D + d]) : 0.0f;
+    qr[j] = d < D ? Elem<T>::to_float(q[d]) : 0.0f;
     o[j] = 0.0f;
   }
+  const float row_scale = scale * query_temperature(a.terms, len), slope = distance_slope(a.terms, head, a.q_heads);
   float m = -INFINITY, l = 0.0f;
   const int first = window > 0 && len > window ? len - window : 0;
   for (int t = first + warp; t < len; t += kWarps) {
@@ -51,6 +52,8 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
     if (page < 0 || page >= a.num_blocks) continue;  // corrupt table entry: never dereferenced
     const int64_t base = page * a.block_stride + static_cast<int64_t>(t % a.block_size) * a.token_stride +
                          static_cast<int64_t>(kv_head) * D;
+    const int64_t v_base = page * a.v_block_stride + static_cast<int64_t>(t % a.block_size) * a.v_token_stride +
+                           static_cast<int64_t>(kv_head) * DV;
     float s = 0.0f;
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) {
@@ -59,7 +62,7 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
     }
 #pragma unroll
     for (int x = 16; x > 0; x >>= 1) s += __shfl_xor_sync(0xffffffffu, s, x);
-    s *= scale;
+    s = fmaf(s, row_scale, -slope * static_cast<float>(len - 1 - t));
     const float m_new = fmaxf(m, s);
     const float alpha = m == -INFINITY ? 0.0f : expf(m - m_new);
     const float p = expf(s - m_new);
@@ -67,7 +70,7 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) {
       int d = lane + 32 * j;
-      if (d < D) o[j] = fmaf(o[j], alpha, p * Elem<T>::to_float(vc[base + d]));
+      if (d < DV) o[j] = fmaf(o[j], alpha, p * Elem<T>::to_float(vc[v_base + d]));
     }
     m = m_new;
   }
@@ -81,7 +84,7 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
   float big = -INFINITY;
 #pragma unroll
   for (int w = 0; w < kWarps; ++w) big = fmaxf(big, sm_m[w]);
-  for (int d = threadIdx.x; d < D; d += kThreads) {
+  for (int d = threadIdx.x; d < DV; d += kThreads) {
     float total = 0.0f, acc = 0.0f;
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) {
@@ -97,7 +100,7 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
 }  // namespace
 
 int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream, int window) {
-  if (a.head_dim > 32 * kMaxPerLane) {
+  if (a.head_dim > 32 * kMaxPerLane || a.value_dim > 32 * kMaxPerLane) {
     set_last_error_text("verify_attention supports head_dim <= 256");
     return RLT_ERR_UNSUPPORTED;
   }
@@ -106,7 +109,7 @@ int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream, int wi
     set_last_error_text("verify_attention: rows * q_heads exceeds the grid limit");
     return RLT_ERR_INVALID;
   }
-  const float scale = static_cast<float>(1.0 / sqrt(static_cast<double>(a.head_dim)));
+  const float scale = score_scale(a);
   RLT_DISPATCH_DTYPE(a.dtype, T,
                      (attention_generic_kernel<T><<<static_cast<unsigned>(ctas), kThreads, 0, stream>>>(a, scale, window)));
   return launch_status("attention_generic_kernel");

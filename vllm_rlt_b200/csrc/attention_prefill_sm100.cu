@@ -767,7 +767,9 @@ __device__ __forceinline__ bool pair_issue(PairShared& sm, uint32_t tmem, int mi
   return false;
 }
 
-template <bool kBF16>
+// kTerms: query temperature and distance bias (see the verify kernel): the stage's scores are brought to their
+// final log2-domain values in pairs, with the bias of the stage's first key as an exact integer distance.
+template <bool kBF16, bool kTerms>
 __global__ void __launch_bounds__(kPairThreads, 1)
 prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                     AttentionArgs a, const PrefillHeader* header, const PrefillTile* tiles, unsigned* error,
@@ -874,11 +876,10 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     // together would keep the load / store unit busy for thousands of cycles); a thread's own row goes through the
     // warp's staging rows in shared memory, whose 16-byte pieces are swizzled by the row.
     const int warp_row = (warp & 3) * 32, warp_count = min(max(count - warp_row, 0), 32);
-    const int64_t row_stride = static_cast<int64_t>(a.q_heads) * kHeadDim;
-    const int64_t warp_offset = ((static_cast<int64_t>(seq_first) + tile.first + t * kUmmaRows + warp_row) * a.q_heads + q_head) * kHeadDim;
+    const int64_t warp_first = static_cast<int64_t>(seq_first) + tile.first + t * kUmmaRows + warp_row;
     unsigned char* staging = &sm.rows[warp][0];
     if (my_stages > 0) {   // Q: tile 0 into tensor memory (two 16-bit values per column, a thread stores its row), tile 1 into shared memory
-      const T* src = static_cast<const T*>(a.q) + warp_offset;
+      const T* src = static_cast<const T*>(a.q) + warp_first * a.q_stride + static_cast<int64_t>(q_head) * kHeadDim;
       const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
       if (t == 0) {
         uint4 piece[2][8];
@@ -887,7 +888,7 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const int r = 4 * i + (lane >> 3);
-            piece[h][i] = r < warp_count ? __ldg(reinterpret_cast<const uint4*>(src + r * row_stride + h * 64) + (lane & 7)) : zero;
+            piece[h][i] = r < warp_count ? __ldg(reinterpret_cast<const uint4*>(src + r * a.q_stride + h * 64) + (lane & 7)) : zero;
           }
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
@@ -911,7 +912,7 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           const int r = 2 * i + (lane >> 4), c = lane & 15;
-          const uint4 value = r < warp_count ? __ldg(reinterpret_cast<const uint4*>(src + r * row_stride) + c) : zero;
+          const uint4 value = r < warp_count ? __ldg(reinterpret_cast<const uint4*>(src + r * a.q_stride) + c) : zero;
           *reinterpret_cast<uint4*>(&sm.q[c >> 3][(warp_row + r) * 128 + (((c & 7) ^ (r & 7)) << 4)]) = value;
         }
         fence_async_proxy();
@@ -921,6 +922,12 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
       if (lane == 0) mbar_arrive(smem_u32(&sm.p_ready[t]));
     }
     constexpr float kRaise = 8.0f;
+    float row_scale = 0.f, slope = 0.f;
+    if constexpr (kTerms) {
+      row_scale = scale_log2 * query_temperature(a.terms, len);
+      slope = kLog2e * distance_slope(a.terms, q_head, a.q_heads);
+    }
+    const float step_scale = kTerms ? 1.0f : scale_log2;
     const bool alternate = take_turns != 0 && stages0 > 0 && stages1 > 0;
     float m = -INFINITY, l = 0.f;
     const uint32_t s_col = tmem_row + kColS + t * kTileCols, p_col = s_col + kColP, o_col = tmem_row + kColO + t * kHeadDim;
@@ -940,6 +947,18 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&sm.s_free[t]));   // the scores are in registers: the next stage's may be written
       const int first_key = j * kUmmaKeys;
+      if constexpr (kTerms) {
+        const float first_bias = slope * static_cast<float>(first_key - len + 1);
+        const float2 row_scale2 = make_float2(row_scale, row_scale), slope2 = make_float2(slope, slope);
+        const float2 first2 = make_float2(first_bias, first_bias);
+#pragma unroll
+        for (int e = 0; e < kUmmaKeys / 2; ++e) {
+          const float2 bias = fma_pair(slope2, make_float2(2.0f * e, 2.0f * e + 1.0f), first2);
+          const float2 v = fma_pair(make_float2(s[2 * e], s[2 * e + 1]), row_scale2, bias);
+          s[2 * e] = v.x;
+          s[2 * e + 1] = v.y;
+        }
+      }
       if (first_key + kUmmaKeys > len) {
 #pragma unroll
         for (int i = 0; i < kUmmaKeys; ++i)
@@ -951,14 +970,14 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
 #pragma unroll
         for (int c = 0; c < 4; ++c) mx4[c] = max3(mx4[c], s[i + 2 * c], s[i + 2 * c + 1]);
       }
-      const float candidate = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+      const float candidate = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * step_scale;
       const bool raise = candidate > m + kRaise || (m == -INFINITY && candidate > -INFINITY);
       const float alpha = (raise && m != -INFINITY) ? fast_exp2(m - candidate) : 1.0f;
       if (raise) m = candidate;
       const float mu = m == -INFINITY ? 0.f : m;
       float2 sum4[4] = {{0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}};
       uint32_t packed[32];
-      const float2 scale2 = make_float2(scale_log2, scale_log2), shift2 = make_float2(-mu, -mu);
+      const float2 scale2 = make_float2(step_scale, step_scale), shift2 = make_float2(-mu, -mu);
       // On long prompts the two tiles' warps of one scheduler take turns at its exponential unit (tile 0 first
       // in every stage): left alone they fall into step, and one warp's loads, maxima and stores then no
       // longer run under the other's exponentials.
@@ -1005,7 +1024,7 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     failed = __any_sync(0xffffffffu, failed);
     if (!failed && count > 0) {
       const float inv = l > 0.f ? 1.0f / l : 0.f;
-      T* dst = static_cast<T*>(a.out) + warp_offset;
+      T* dst = static_cast<T*>(a.out) + warp_first * a.out_stride + static_cast<int64_t>(q_head) * kHeadDim;
 #pragma unroll
       for (int h = 0; h < 2; ++h) {   // 64 output columns at a time
         uint32_t lo[32], hi[32];
@@ -1029,7 +1048,7 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
         for (int i = 0; i < 8; ++i) {
           const int r = 4 * i + (lane >> 3);
           if (r < warp_count)
-            reinterpret_cast<uint4*>(dst + r * row_stride + h * 64)[lane & 7] =
+            reinterpret_cast<uint4*>(dst + r * a.out_stride + h * 64)[lane & 7] =
                 *reinterpret_cast<const uint4*>(staging + r * 128 + (((lane & 7) ^ (r & 7)) << 4));
         }
         __syncwarp();
@@ -1047,7 +1066,7 @@ size_t tile_capacity(int rows, int seqs) { return static_cast<size_t>(rows) / kT
 }  // namespace
 
 bool prefill_sm100_supported(const AttentionArgs& a) {
-  return a.cu_seqlens_q != nullptr && attention_sm100_supported(a);
+  return a.cu_seqlens_q != nullptr && attention_sm100_supported(a) && a.q_stride % 8 == 0 && aligned16(a.q);
 }
 
 size_t prefill_sm100_workspace_bytes(int rows, int seqs) {
@@ -1067,11 +1086,13 @@ int launch_prefill_sm100(const AttentionArgs& a, void* workspace, size_t workspa
   // where its second tile stays empty (chunks of 128 new tokens per sequence: 48 against 66 and 80 us at 16 sequences
   // on 1024-token contexts, 70 against 138 and 147 us at 4 sequences on 4096-token ones).
   const char* forced = getenv("RLT_PREFILL_KERNEL");
-  const char kernel_choice = forced != nullptr && forced[0] != 0 ? forced[0] : 'p';
+  // Only the pair kernel has score terms and strided query / output rows.
+  const bool plain = a.terms.plain() && a.q_stride == static_cast<int64_t>(a.q_heads) * kHeadDim && a.out_stride == a.q_stride;
+  const char kernel_choice = plain && forced != nullptr && forced[0] != 0 ? forced[0] : 'p';
   const bool use_mma_sync = kernel_choice == 'm';
   PrefillHeader* header = static_cast<PrefillHeader*>(workspace);
   PrefillTile* tiles = reinterpret_cast<PrefillTile*>(static_cast<unsigned char*>(workspace) + 256);
-  const float scale_log2 = static_cast<float>(1.4426950408889634 / sqrt(static_cast<double>(kHeadDim)));
+  const float scale_log2 = log2_scale(a);
   CUtensorMap k_map, v_map;
   if (kernel_choice == 'p' && make_page_map(&k_map, a.key_cache, a) == RLT_OK && make_page_map(&v_map, a.value_cache, a) == RLT_OK) {
     prefill_plan_kernel<<<1, kPrefillPlanThreads, 0, stream>>>(a.cu_seqlens_q, a.context_lengths, a.table_width, a.table_rows, kPairRows, header, tiles);
@@ -1081,17 +1102,14 @@ int launch_prefill_sm100(const AttentionArgs& a, void* workspace, size_t workspa
     const int take_turns = static_cast<int64_t>(a.rows) >= 2048ll * a.table_rows ? 1 : 0;   // prompts of 2048 tokens and more on average
     const dim3 grid(static_cast<unsigned>(static_cast<size_t>(a.rows) / kPairRows + static_cast<size_t>(a.table_rows) + 1),
                     static_cast<unsigned>(a.q_heads));
-    if (a.dtype == RLT_BF16) {
-      auto kernel = prefill_pair_kernel<true>;
-      RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-      kernel<<<grid, kPairThreads, smem, stream>>>(k_map, v_map, a, header, tiles, &header->error, scale_log2, take_turns);
-    } else {
-      auto kernel = prefill_pair_kernel<false>;
-      RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-      kernel<<<grid, kPairThreads, smem, stream>>>(k_map, v_map, a, header, tiles, &header->error, scale_log2, take_turns);
-    }
+    const bool terms = !a.terms.plain();
+    auto kernel = a.dtype == RLT_BF16 ? (terms ? prefill_pair_kernel<true, true> : prefill_pair_kernel<true, false>)
+                                      : (terms ? prefill_pair_kernel<false, true> : prefill_pair_kernel<false, false>);
+    RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    kernel<<<grid, kPairThreads, smem, stream>>>(k_map, v_map, a, header, tiles, &header->error, scale_log2, take_turns);
     return launch_status("prefill_pair_kernel");
   }
+  if (!plain) return RLT_ERR_UNSUPPORTED;   // the caches' maps were refused: the grouped verify kernel scores these rows
   if (!use_mma_sync && make_page_map(&k_map, a.key_cache, a) == RLT_OK && make_page_map(&v_map, a.value_cache, a) == RLT_OK) {
     prefill_plan_kernel<<<1, kPrefillPlanThreads, 0, stream>>>(a.cu_seqlens_q, a.context_lengths, a.table_width, a.table_rows, kUmmaRows, header, tiles);
     int status = launch_status("prefill_plan_kernel");

@@ -478,14 +478,16 @@ merge_kernel(AttentionArgs a, Workspace ws) {
   uint2 packed;
   packed.x = pack2<kBF16>(acc.x * inv, acc.y * inv);
   packed.y = pack2<kBF16>(acc.z * inv, acc.w * inv);
-  reinterpret_cast<uint2*>(static_cast<T*>(a.out) + pair * kHeadDim)[lane] = packed;
+  reinterpret_cast<uint2*>(static_cast<T*>(a.out) + row * a.out_stride + (pair - row * a.q_heads) * kHeadDim)[lane] = packed;
 }
 
 // kCopies: TMA copies per page.  4: 3-D maps, one copy per 64-dim half of K and of V.  2: 4-D
 // maps, one copy per K or V head slice.  1: one 5-D map over both caches (k_map; v_map unused),
 // one copy per page; `k_first` tells which cache lies at the lower address and therefore lands
 // in the first half of a stage.
-template <bool kBF16, int kWarps, int kStages, int kCopies>
+// kTerms: the rows have score terms beyond a constant scale (query temperature, distance bias): a score is
+// brought to its final log2-domain value right after Q K^T, before the masks and the row maximum.
+template <bool kBF16, int kWarps, int kStages, int kCopies, bool kTerms>
 __global__ void __launch_bounds__(kWarps * 32, 1)
 verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                         AttentionArgs a, Workspace ws, float scale_log2, int k_first) {
@@ -507,7 +509,7 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     const unsigned zero_rows = ws.header->zero_rows;
     const int row_elems = a.q_heads * kHeadDim;  // multiple of 4 elements = 8 bytes
     for (unsigned z = blockIdx.x * kWarps + warp; z < zero_rows; z += gridDim.x * kWarps) {
-      uint2* dst = reinterpret_cast<uint2*>(static_cast<T*>(a.out) + static_cast<int64_t>(ws.zero_list[z]) * row_elems);
+      uint2* dst = reinterpret_cast<uint2*>(static_cast<T*>(a.out) + static_cast<int64_t>(ws.zero_list[z]) * a.out_stride);
       for (int i = lane; i < row_elems / 4; i += 32) dst[i] = make_uint2(0u, 0u);
     }
   }
@@ -553,7 +555,7 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     const bool live0 = it.valid && r0 < rows && l0 > 0, live1 = it.valid && r1 < rows && l1 > 0;
     const int64_t row0 = it.row_start + r0 / gqa, row1 = it.row_start + r1 / gqa;
     const int head0 = it.kv_head * gqa + r0 % gqa, head1 = it.kv_head * gqa + r1 % gqa;
-    const int64_t e0 = (row0 * a.q_heads + head0) * kHeadDim, e1 = (row1 * a.q_heads + head1) * kHeadDim;
+    const int64_t e0 = row0 * a.q_stride + head0 * kHeadDim, e1 = row1 * a.q_stride + head1 * kHeadDim;
     const uint32_t* qp = reinterpret_cast<const uint32_t*>(a.q);
 #pragma unroll
     for (int ks = 0; ks < 8; ++ks) {
@@ -629,9 +631,14 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     nxt_ready = false;  // `nxt` still names this item until the new claim below completes
     top_up();
 
-    const int64_t qrow0 = cur.row_start + r0 / gqa, qrow1 = cur.row_start + r1 / gqa;
-    const int qhead0 = cur.kv_head * gqa + r0 % gqa, qhead1 = cur.kv_head * gqa + r1 % gqa;
-    const int64_t q0 = (qrow0 * a.q_heads + qhead0) * kHeadDim, q1 = (qrow1 * a.q_heads + qhead1) * kHeadDim;
+    float rs0 = 0.f, rs1 = 0.f, slope0 = 0.f, slope1 = 0.f;   // log2-domain scale and distance slope of the two rows
+    if constexpr (kTerms) {
+      rs0 = scale_log2 * query_temperature(a.terms, len0);
+      rs1 = scale_log2 * query_temperature(a.terms, len1);
+      slope0 = kLog2e * distance_slope(a.terms, cur.kv_head * gqa + r0 % gqa, a.q_heads);
+      slope1 = kLog2e * distance_slope(a.terms, cur.kv_head * gqa + r1 % gqa, a.q_heads);
+    }
+    const float step_scale = kTerms ? 1.0f : scale_log2;
     // nxt: the atomic now, its record after cur's first page, its rows after the second, the warp
     // reductions and the Q fragments after the third (or at the end of a shorter item).
     uint32_t qb[8][4];
@@ -692,8 +699,19 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[nt][e] += s2[nt][e];
       }
-      // mask by each row's own length (only tiles that reach past the shortest member)
       const int tile_start = cur.chunk_start + j * kPage;
+      if constexpr (kTerms) {
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int pos = tile_start + 2 * t + nt * 8 + e;
+            s[nt][e] = fmaf(s[nt][e], rs0, slope0 * static_cast<float>(pos - len0 + 1));
+            s[nt][2 + e] = fmaf(s[nt][2 + e], rs1, slope1 * static_cast<float>(pos - len1 + 1));
+          }
+        }
+      }
+      // mask by each row's own length (only tiles that reach past the shortest member)
       if (padded_rows || tile_start + kPage > shortest) {
         const int tok = tile_start + 2 * t;
 #pragma unroll
@@ -712,17 +730,17 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-      const float mn0 = fmaxf(m0, mx0 * scale_log2), mn1 = fmaxf(m1, mx1 * scale_log2);
+      const float mn0 = fmaxf(m0, mx0 * step_scale), mn1 = fmaxf(m1, mx1 * step_scale);
       const float mu0 = mn0 == -INFINITY ? 0.f : mn0, mu1 = mn1 == -INFINITY ? 0.f : mn1;
       const bool moved = (mn0 != m0) || (mn1 != m1);
       const float al0 = fast_exp2(m0 - mu0), al1 = fast_exp2(m1 - mu1);
       m0 = mn0; m1 = mn1;
       uint32_t pa[4];
       {
-        const float p00 = fast_exp2(fmaf(s[0][0], scale_log2, -mu0)), p01 = fast_exp2(fmaf(s[0][1], scale_log2, -mu0));
-        const float p02 = fast_exp2(fmaf(s[0][2], scale_log2, -mu1)), p03 = fast_exp2(fmaf(s[0][3], scale_log2, -mu1));
-        const float p10 = fast_exp2(fmaf(s[1][0], scale_log2, -mu0)), p11 = fast_exp2(fmaf(s[1][1], scale_log2, -mu0));
-        const float p12 = fast_exp2(fmaf(s[1][2], scale_log2, -mu1)), p13 = fast_exp2(fmaf(s[1][3], scale_log2, -mu1));
+        const float p00 = fast_exp2(fmaf(s[0][0], step_scale, -mu0)), p01 = fast_exp2(fmaf(s[0][1], step_scale, -mu0));
+        const float p02 = fast_exp2(fmaf(s[0][2], step_scale, -mu1)), p03 = fast_exp2(fmaf(s[0][3], step_scale, -mu1));
+        const float p10 = fast_exp2(fmaf(s[1][0], step_scale, -mu0)), p11 = fast_exp2(fmaf(s[1][1], step_scale, -mu0));
+        const float p12 = fast_exp2(fmaf(s[1][2], step_scale, -mu1)), p13 = fast_exp2(fmaf(s[1][3], step_scale, -mu1));
         l0 = l0 * al0 + ((p00 + p01) + (p10 + p11));
         l1 = l1 * al1 + ((p02 + p03) + (p12 + p13));
         pa[0] = pack2<kBF16>(p00, p01);
@@ -761,11 +779,13 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     const int chunks0 = chunk_count(len0), chunks1 = chunk_count(len1);
+    const int64_t qrow0 = cur.row_start + r0 / gqa, qrow1 = cur.row_start + r1 / gqa;
+    const int qhead0 = cur.kv_head * gqa + r0 % gqa, qhead1 = cur.kv_head * gqa + r1 % gqa;
     T* out = static_cast<T*>(a.out);
     if (cur.chunk < chunks0) {
       if (chunks0 == 1) {
         const float inv = 1.0f / l0;
-        uint32_t* dst = reinterpret_cast<uint32_t*>(out + q0);
+        uint32_t* dst = reinterpret_cast<uint32_t*>(out + qrow0 * a.out_stride + qhead0 * kHeadDim);
 #pragma unroll
         for (int jn = 0; jn < 16; ++jn) dst[jn * 4 + t] = pack2<kBF16>(o[jn][0] * inv, o[jn][1] * inv);
       } else {
@@ -778,7 +798,7 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     if (cur.chunk < chunks1) {
       if (chunks1 == 1) {
         const float inv = 1.0f / l1;
-        uint32_t* dst = reinterpret_cast<uint32_t*>(out + q1);
+        uint32_t* dst = reinterpret_cast<uint32_t*>(out + qrow1 * a.out_stride + qhead1 * kHeadDim);
 #pragma unroll
         for (int jn = 0; jn < 16; ++jn) dst[jn * 4 + t] = pack2<kBF16>(o[jn][2] * inv, o[jn][3] * inv);
       } else {
@@ -820,12 +840,12 @@ verify_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
 // ---- host side ----------------------------------------------------------------------------
 int gqa_cap(const AttentionArgs& a) { return kMaxGroupRows / (a.q_heads / a.kv_heads); }
 
-template <bool kBF16, int kWarps, int kStages, int kCopies>
+template <bool kBF16, int kWarps, int kStages, int kCopies, bool kTerms>
 int launch_main(const CUtensorMap& k_map, const CUtensorMap& v_map, const AttentionArgs& a, const Workspace& ws,
                 int sm_count, cudaStream_t stream, bool k_first = true) {
   const size_t smem = sizeof(SharedStorage<kWarps, kStages>) + 1024;
-  const float scale_log2 = static_cast<float>(1.4426950408889634 / sqrt(static_cast<double>(kHeadDim)));
-  auto kernel = verify_attention_kernel<kBF16, kWarps, kStages, kCopies>;
+  const float scale_log2 = log2_scale(a);
+  auto kernel = verify_attention_kernel<kBF16, kWarps, kStages, kCopies, kTerms>;
   RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   kernel<<<sm_count, kWarps * 32, smem, stream>>>(k_map, v_map, a, ws, scale_log2, k_first ? 1 : 0);
   int status = launch_status("verify_attention_kernel");
@@ -854,6 +874,8 @@ bool attention_sm100_supported(const AttentionArgs& a) {
   if ((a.token_stride * 2) % 16 != 0 || (a.block_stride * 2) % 16 != 0) return false;
   if (a.block_stride < a.token_stride * kPage) return false;
   if (!aligned16(a.key_cache) || !aligned16(a.value_cache)) return false;
+  if (a.value_dim != kHeadDim || a.v_block_stride != a.block_stride || a.v_token_stride != a.token_stride) return false;
+  if (a.q_stride % 2 != 0 || a.out_stride % 8 != 0) return false;
   if ((reinterpret_cast<uintptr_t>(a.q) & 3u) != 0 || (reinterpret_cast<uintptr_t>(a.out) & 15u) != 0) return false;
   if (a.num_blocks > 0xffffffffll) return false;
   return true;
@@ -938,14 +960,28 @@ int run_attention_sm100(const AttentionArgs& a, void* workspace, size_t workspac
     status = make_page_map(&v_map, a.value_cache, a);
     if (status != RLT_OK) return status;
   }
-  if (a.dtype == RLT_BF16) {
-    if (copies == 1) return launch_main<true, 8, 3, 1>(k_map, v_map, a, ws, info.sm_count, stream, k_first);
-    if (copies == 2) return launch_main<true, 8, 3, 2>(k_map, v_map, a, ws, info.sm_count, stream);
-    return launch_main<true, 8, 3, 4>(k_map, v_map, a, ws, info.sm_count, stream);
+  if (!a.terms.plain()) {
+    // two variants are enough here: one copy per page, or four through the plain 3-D maps
+    if (copies == 2) {
+      status = make_page_map(&k_map, a.key_cache, a);
+      if (status == RLT_OK) status = make_page_map(&v_map, a.value_cache, a);
+      if (status != RLT_OK) return status;
+    }
+    if (a.dtype == RLT_BF16) {
+      if (copies == 1) return launch_main<true, 8, 3, 1, true>(k_map, v_map, a, ws, info.sm_count, stream, k_first);
+      return launch_main<true, 8, 3, 4, true>(k_map, v_map, a, ws, info.sm_count, stream);
+    }
+    if (copies == 1) return launch_main<false, 8, 3, 1, true>(k_map, v_map, a, ws, info.sm_count, stream, k_first);
+    return launch_main<false, 8, 3, 4, true>(k_map, v_map, a, ws, info.sm_count, stream);
   }
-  if (copies == 1) return launch_main<false, 8, 3, 1>(k_map, v_map, a, ws, info.sm_count, stream, k_first);
-  if (copies == 2) return launch_main<false, 8, 3, 2>(k_map, v_map, a, ws, info.sm_count, stream);
-  return launch_main<false, 8, 3, 4>(k_map, v_map, a, ws, info.sm_count, stream);
+  if (a.dtype == RLT_BF16) {
+    if (copies == 1) return launch_main<true, 8, 3, 1, false>(k_map, v_map, a, ws, info.sm_count, stream, k_first);
+    if (copies == 2) return launch_main<true, 8, 3, 2, false>(k_map, v_map, a, ws, info.sm_count, stream);
+    return launch_main<true, 8, 3, 4, false>(k_map, v_map, a, ws, info.sm_count, stream);
+  }
+  if (copies == 1) return launch_main<false, 8, 3, 1, false>(k_map, v_map, a, ws, info.sm_count, stream, k_first);
+  if (copies == 2) return launch_main<false, 8, 3, 2, false>(k_map, v_map, a, ws, info.sm_count, stream);
+  return launch_main<false, 8, 3, 4, false>(k_map, v_map, a, ws, info.sm_count, stream);
 }
 
 int launch_attention_sm100(const AttentionArgs& a, void* workspace, size_t workspace_bytes, cudaStream_t stream) {

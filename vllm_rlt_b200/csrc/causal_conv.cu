@@ -1,0 +1,137 @@
+// Short causal convolution per channel over packed sequences, with the last taps - 1 inputs of every sequence
+// kept in its state slot:
+//
+//   out[i, c] = silu(bias[c] + sum_j w[c, j] * in[i - taps + 1 + j, c])
+//
+// Inputs before a portion's first token come from the slot (zeros when the portion starts the sequence).  A
+// sequence's tokens are cut into tiles of `tile` >= taps - 1 tokens; only the first tile reads the slot, and
+// the same threads write the new one (the last taps - 1 of old inputs followed by the portion), each for its own
+// channel, after they have read it.  The feed-forward columns of the stacked projection ride along in the same
+// launch (extra column blocks: activation instead of convolution).
+#include <math.h>
+
+#include "layer_math.cuh"
+
+namespace rlt {
+namespace {
+
+constexpr int kThreads = 128;
+constexpr int kTile = 32;
+constexpr int kMaxTaps = kTile + 1;
+
+struct ConvArgs {
+  const void* in; int64_t in_stride;      // the convolved columns of the projection
+  const float* weight; const float* bias; // [channels, taps], [channels]
+  void* out; int64_t out_stride;
+  void* state;                            // [slots][taps - 1][channels]
+  int64_t slots;
+  int channels, taps;
+  const int32_t* cu; const int32_t* starts; const int32_t* slot_of;
+  const void* act_in; void* act_out; int64_t act_out_stride;   // activation columns (act_in shares in_stride)
+  int act_width, act, conv_blocks;
+};
+
+// kTaps 0: any number of taps, inputs re-read (from L1) for every output.
+template <typename T, int kTaps>
+__global__ void __launch_bounds__(kThreads)
+causal_conv_kernel(ConvArgs a) {
+  const int seq = blockIdx.z, first = blockIdx.y * kTile;
+  const int row0 = a.cu[seq], n = a.cu[seq + 1] - row0;
+  if (first >= n) return;
+  const int count = min(kTile, n - first);
+  if (static_cast<int>(blockIdx.x) >= a.conv_blocks) {
+    const int c = (blockIdx.x - a.conv_blocks) * kThreads + threadIdx.x;
+    if (c >= a.act_width) return;
+    const T* src = static_cast<const T*>(a.act_in) + (row0 + first) * a.in_stride + c;
+    T* dst = static_cast<T*>(a.act_out) + (row0 + first) * a.act_out_stride + c;
+#pragma unroll 4
+    for (int i = 0; i < count; ++i)
+      dst[i * a.act_out_stride] = Elem<T>::from_float(activate(Elem<T>::to_float(src[i * a.in_stride]), a.act));
+    return;
+  }
+  const int c = blockIdx.x * kThreads + threadIdx.x;
+  if (c >= a.channels) return;
+  const int taps = kTaps > 0 ? kTaps : a.taps;
+  const T* in = static_cast<const T*>(a.in) + static_cast<int64_t>(row0) * a.in_stride + c;   // in[i * stride]: token i of the portion
+  T* out = static_cast<T*>(a.out) + static_cast<int64_t>(row0) * a.out_stride + c;
+  const bool resumed = a.starts[seq] > 0;
+  const int64_t slot = a.slot_of[seq];
+  const bool slot_ok = slot >= 0 && slot < a.slots;
+  T* state = static_cast<T*>(a.state) + slot * (taps - 1) * static_cast<int64_t>(a.channels) + c;
+  auto old_input = [&](int k) {   // k-th of the taps - 1 inputs before the portion, oldest first
+    return resumed && slot_ok ? state[static_cast<int64_t>(k) * a.channels] : Elem<T>::from_float(0.0f);
+  };
+  auto input = [&](int i) { return i >= 0 ? in[i * a.in_stride] : old_input(i + taps - 1); };
+  const float bias = a.bias[c];
+  const float* w = a.weight + static_cast<int64_t>(c) * taps;
+  if constexpr (kTaps > 0) {
+    float wr[kTaps], window[kTaps];
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j) wr[j] = w[j];
+#pragma unroll
+    for (int j = 0; j + 1 < kTaps; ++j) window[j + 1] = Elem<T>::to_float(input(first - kTaps + 1 + j));
+    T next[8];
+    for (int base = 0; base < count; base += 8) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (base + i < count) next[i] = in[(first + base + i) * a.in_stride];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        if (base + i < count) {
+#pragma unroll
+          for (int j = 0; j + 1 < kTaps; ++j) window[j] = window[j + 1];
+          window[kTaps - 1] = Elem<T>::to_float(next[i]);
+          float sum = 0.0f;
+#pragma unroll
+          for (int j = 0; j < kTaps; ++j) sum = fmaf(wr[j], window[j], sum);
+          out[(first + base + i) * a.out_stride] = Elem<T>::from_float(silu(sum + bias));
+        }
+      }
+    }
+  } else {
+    for (int i = 0; i < count; ++i) {
+      float sum = 0.0f;
+      for (int j = 0; j < taps; ++j) sum = fmaf(w[j], Elem<T>::to_float(input(first + i - taps + 1 + j)), sum);
+      out[(first + i) * a.out_stride] = Elem<T>::from_float(silu(sum + bias));
+    }
+  }
+  if (first == 0 && slot_ok)   // ascending: entry k is written after every entry it is shifted from has been read
+    for (int k = 0; k + 1 < taps; ++k) state[static_cast<int64_t>(k) * a.channels] = input(n + k - taps + 1);
+}
+
+template <typename T>
+void launch(const ConvArgs& a, dim3 grid, cudaStream_t s) {
+  if (a.taps == 4) causal_conv_kernel<T, 4><<<grid, kThreads, 0, s>>>(a);
+  else causal_conv_kernel<T, 0><<<grid, kThreads, 0, s>>>(a);
+}
+
+}  // namespace
+}  // namespace rlt
+
+extern "C" RLT_API int rlt_causal_conv(const void* in, int64_t in_stride, const float* weight, const float* bias, void* out,
+                                       int64_t out_stride, void* state, int64_t slots, int channels, int taps,
+                                       const int32_t* cu_seqlens, const int32_t* starts, const int32_t* slot_of,
+                                       int sequences, int max_tokens, const void* act_in, void* act_out,
+                                       int64_t act_out_stride, int act_width, int act, int dtype, rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype_valid(dtype), "causal_conv: dtype must be float32, float16 or bfloat16");
+  RLT_REQUIRE(channels > 0 && taps > 0 && sequences >= 0 && max_tokens >= 0 && act_width >= 0 && slots > 0, "causal_conv: invalid shape");
+  if (taps > kMaxTaps) {
+    set_last_error_text("causal_conv: more than 33 taps are not supported");
+    return RLT_ERR_UNSUPPORTED;
+  }
+  if (sequences == 0 || max_tokens == 0) return RLT_OK;
+  RLT_REQUIRE(in && weight && bias && out && (state || taps == 1) && cu_seqlens && starts && slot_of, "causal_conv: null pointer");
+  RLT_REQUIRE(sequences <= 65535 && (max_tokens + kTile - 1) / kTile <= 65535, "causal_conv: batch exceeds the grid limits");
+  RLT_REQUIRE(act_width == 0 || (act_in && act_out && act_valid(act)), "causal_conv: activation columns need a kind and an output");
+  ConvArgs a;
+  a.in = in; a.in_stride = in_stride; a.weight = weight; a.bias = bias; a.out = out; a.out_stride = out_stride;
+  a.state = state; a.slots = slots; a.channels = channels; a.taps = taps;
+  a.cu = cu_seqlens; a.starts = starts; a.slot_of = slot_of;
+  a.act_in = act_in; a.act_out = act_out; a.act_out_stride = act_out_stride; a.act_width = act_width; a.act = act;
+  a.conv_blocks = (channels + kThreads - 1) / kThreads;
+  const dim3 grid(static_cast<unsigned>(a.conv_blocks + (act_width + kThreads - 1) / kThreads),
+                  static_cast<unsigned>((max_tokens + kTile - 1) / kTile), static_cast<unsigned>(sequences));
+  RLT_DISPATCH_DTYPE(dtype, T, launch<T>(a, grid, static_cast<cudaStream_t>(stream)));
+  return launch_status("causal_conv_kernel");
+}

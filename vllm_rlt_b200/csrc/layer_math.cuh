@@ -1,0 +1,37 @@
+// Scalar functions and vector loads shared by the layer kernels (fp32 arithmetic, storage type T).
+#pragma once
+
+#include <math.h>
+
+#include "common.cuh"
+
+namespace rlt {
+
+enum Activation { kActGeluErf = 1, kActGeluTanh = 2 };
+inline bool act_valid(int act) { return act == kActGeluErf || act == kActGeluTanh; }
+
+__device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float activate(float x, int act) {
+  if (act == kActGeluErf) return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
+  return 0.5f * x * (1.0f + tanhf(0.79788456080286536f * (x + 0.044715f * x * x * x)));
+}
+
+// kVec consecutive elements as fp32, in one access of kVec * sizeof(T) bytes (the caller guarantees the alignment).
+template <typename T, int kVec>
+__device__ __forceinline__ void load_floats(const T* p, float (&v)[kVec]) {
+  struct alignas(sizeof(T) * kVec) Vec { T e[kVec]; };
+  const Vec x = *reinterpret_cast<const Vec*>(p);
+#pragma unroll
+  for (int e = 0; e < kVec; ++e) v[e] = Elem<T>::to_float(x.e[e]);
+}
+template <typename T, int kVec>
+__device__ __forceinline__ void store_floats(T* p, const float (&v)[kVec]) {
+  struct alignas(sizeof(T) * kVec) Vec { T e[kVec]; };
+  Vec x;
+#pragma unroll
+  for (int e = 0; e < kVec; ++e) x.e[e] = Elem<T>::from_float(v[e]);
+  *reinterpret_cast<Vec*>(p) = x;
+}
+
+}  // namespace rlt

@@ -1,0 +1,240 @@
+// Elementwise work of a parallel decoder block, where mixer and feed-forward read one norm and add into one
+// 32-bit residual stream.  A layer is two GEMMs — one over the stacked input projections, one over the
+// stacked output projections — and between them
+//
+//   residual_norm_kernel   residual += delta (or residual = embed[token]), h = rmsnorm(residual) * (offset + w):
+//                          the tail of one layer and the head of the next in one pass over the row
+//   block_epilogue_kernel  columns of the stacked input projection: keys and values to their pages,
+//                          the feed-forward columns through their activation into the stacked output operand
+//   gated_norm_kernel      y * silu(z), RMS-normed in equal parts, into the stacked output operand
+//
+// All three are streaming kernels: every input is read once and every output written once.  Sums, norms
+// and activations are fp32; only the stored operand of the next GEMM is rounded to the model dtype.
+#include <math.h>
+
+#include "layer_math.cuh"
+
+namespace rlt {
+namespace {
+
+constexpr int kThreads = 256;
+
+__device__ __forceinline__ float block_sum(float v, float* scratch) {
+#pragma unroll
+  for (int x = 16; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  v = (threadIdx.x & 31) < kThreads / 32 ? scratch[threadIdx.x & 31] : 0.0f;
+#pragma unroll
+  for (int x = 4; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
+  return __shfl_sync(0xffffffffu, v, 0);
+}
+
+template <typename T, int kVec>
+__global__ void __launch_bounds__(kThreads)
+residual_norm_kernel(float* residual, const T* __restrict__ delta, const int64_t* __restrict__ tokens,
+                     const T* __restrict__ embed, int64_t vocab, const int64_t* __restrict__ row_index, int store_residual,
+                     const float* __restrict__ weight, float weight_offset, T* __restrict__ out, int width, float eps) {
+  extern __shared__ float row_values[];
+  __shared__ float scratch[kThreads / 32];
+  const int64_t source = row_index != nullptr ? row_index[blockIdx.x] : static_cast<int64_t>(blockIdx.x);
+  float* res = residual + source * width;
+  const T* del = delta == nullptr ? nullptr : delta + source * width;
+  const T* emb = nullptr;
+  if (tokens != nullptr) {
+    int64_t token = tokens[source];
+    token = token < 0 ? 0 : (token >= vocab ? vocab - 1 : token);   // the host refuses such tokens; a device id never leaves the table
+    emb = embed + token * width;
+  }
+  float ss = 0.0f;
+  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
+    float v[kVec];
+    if (emb != nullptr) load_floats<T, kVec>(emb + i, v);
+    else load_floats<float, kVec>(res + i, v);
+    if (del != nullptr) {
+      float d[kVec];
+      load_floats<T, kVec>(del + i, d);
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) v[e] += d[e];
+    }
+    if (store_residual) store_floats<float, kVec>(res + i, v);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) {
+      row_values[i + e] = v[e];
+      ss = fmaf(v[e], v[e], ss);
+    }
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + eps);
+  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
+    float v[kVec], w[kVec];
+    load_floats<float, kVec>(weight + i, w);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) v[e] = row_values[i + e] * r * (weight_offset + w[e]);
+    store_floats<T, kVec>(out + static_cast<int64_t>(blockIdx.x) * width + i, v);
+  }
+}
+
+struct EpilogueArgs {
+  const void* proj; int64_t proj_stride;
+  int k_col, k_width, v_col, v_width;       // key / value columns of the projection (width 0: none)
+  void* key_cache; int64_t k_block_stride, k_token_stride;
+  void* value_cache; int64_t v_block_stride, v_token_stride;
+  int64_t num_blocks; int block_size;
+  const int32_t* tables; int table_width;
+  const int32_t* row_seq; const int32_t* positions;
+  int act_col, act_width, act;              // feed-forward columns and their activation
+  void* out; int64_t out_stride; int out_col;
+};
+
+// Items of a row, kVec elements each: keys, values, activations.
+template <typename T, int kVec>
+__global__ void __launch_bounds__(kThreads)
+block_epilogue_kernel(EpilogueArgs a) {
+  struct alignas(sizeof(T) * kVec) Vec { T e[kVec]; };
+  const int row = blockIdx.x;
+  const T* proj = static_cast<const T*>(a.proj) + row * a.proj_stride;
+  const int k_items = a.k_width / kVec, v_items = a.v_width / kVec, act_items = a.act_width / kVec;
+  const int item = blockIdx.y * kThreads + threadIdx.x;
+  if (item < k_items + v_items) {
+    const int seq = a.row_seq[row];
+    if (seq < 0) return;                    // a padding row of a captured step
+    const int position = a.positions[row];
+    const int page_index = position / a.block_size;
+    if (position < 0 || page_index >= a.table_width) return;
+    const int64_t page = a.tables[static_cast<int64_t>(seq) * a.table_width + page_index];
+    if (page < 0 || page >= a.num_blocks) return;
+    const int offset = position % a.block_size;
+    const bool key = item < k_items;
+    const int c = (key ? item : item - k_items) * kVec;
+    T* dst = key ? static_cast<T*>(a.key_cache) + page * a.k_block_stride + offset * a.k_token_stride
+                 : static_cast<T*>(a.value_cache) + page * a.v_block_stride + offset * a.v_token_stride;
+    *reinterpret_cast<Vec*>(dst + c) = *reinterpret_cast<const Vec*>(proj + (key ? a.k_col : a.v_col) + c);
+  } else if (item < k_items + v_items + act_items) {
+    const int c = (item - k_items - v_items) * kVec;
+    float v[kVec];
+    load_floats<T, kVec>(proj + a.act_col + c, v);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) v[e] = activate(v[e], a.act);
+    store_floats<T, kVec>(static_cast<T*>(a.out) + row * a.out_stride + a.out_col + c, v);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z, int64_t z_stride,
+                  const float* __restrict__ weight, T* __restrict__ out, int64_t out_stride, int part, float eps) {
+  extern __shared__ float row_values[];
+  __shared__ float scratch[kThreads / 32];
+  const int64_t row = blockIdx.x;
+  const int first = blockIdx.y * part;
+  const T* yr = y + row * y_stride + first;
+  const T* zr = z + row * z_stride + first;
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < part; i += kThreads) {
+    const float v = Elem<T>::to_float(yr[i]) * silu(Elem<T>::to_float(zr[i]));
+    row_values[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(part) + eps);
+  T* dst = out + row * out_stride + first;
+  for (int i = threadIdx.x; i < part; i += kThreads)
+    dst[i] = Elem<T>::from_float(row_values[i] * r * weight[first + i]);
+}
+
+constexpr size_t kMaxRowBytes = 48u * 1024u;   // a staged row of fp32 values
+
+}  // namespace
+}  // namespace rlt
+
+extern "C" RLT_API int rlt_residual_norm(float* residual, const void* delta, const int64_t* tokens, const void* embed,
+                                         int64_t vocab, const int64_t* row_index, int store_residual, const float* weight,
+                                         float weight_offset, void* out, int rows, int width, float eps, int dtype,
+                                         rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype_valid(dtype), "residual_norm: dtype must be float32, float16 or bfloat16");
+  RLT_REQUIRE(rows >= 0 && width > 0 && eps >= 0.0f, "residual_norm: invalid shape or eps");
+  if (rows == 0) return RLT_OK;
+  RLT_REQUIRE(residual && weight && out, "residual_norm: null pointer");
+  RLT_REQUIRE((tokens == nullptr) == (embed == nullptr) && (tokens == nullptr || vocab > 0), "residual_norm: tokens and embed go together");
+  const size_t smem = static_cast<size_t>(width) * sizeof(float);
+  if (smem > kMaxRowBytes - 1024) {
+    set_last_error_text("residual_norm: widths above 12032 are not supported");
+    return RLT_ERR_UNSUPPORTED;
+  }
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool wide = width % 4 == 0 && aligned16(residual) && aligned16(weight) && aligned16(delta) && aligned16(embed) && aligned16(out);
+#define RLT_LAUNCH(T, V)                                                                                              \
+  residual_norm_kernel<T, V><<<rows, kThreads, smem, s>>>(residual, static_cast<const T*>(delta), tokens,             \
+      static_cast<const T*>(embed), vocab, row_index, store_residual, weight, weight_offset, static_cast<T*>(out), width, eps)
+  RLT_DISPATCH_DTYPE(dtype, T, { if (wide) RLT_LAUNCH(T, 4); else RLT_LAUNCH(T, 1); });
+#undef RLT_LAUNCH
+  return launch_status("residual_norm_kernel");
+}
+
+extern "C" RLT_API int rlt_block_epilogue(const void* proj, int64_t proj_stride, int k_col, int k_width, int v_col,
+                                          int v_width, void* key_cache, int64_t k_block_stride, int64_t k_token_stride,
+                                          void* value_cache, int64_t v_block_stride, int64_t v_token_stride,
+                                          int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
+                                          const int32_t* row_seq, const int32_t* positions, int act_col, int act_width,
+                                          int act, void* out, int64_t out_stride, int out_col, int rows, int dtype,
+                                          rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype_valid(dtype), "block_epilogue: dtype must be float32, float16 or bfloat16");
+  RLT_REQUIRE(rows >= 0 && k_width >= 0 && v_width >= 0 && act_width >= 0, "block_epilogue: invalid shape");
+  if (rows == 0 || k_width + v_width + act_width == 0) return RLT_OK;
+  RLT_REQUIRE(proj, "block_epilogue: null projection");
+  RLT_REQUIRE(k_width + v_width == 0 || (key_cache && value_cache && tables && row_seq && positions && block_size > 0 &&
+                                         table_width > 0 && num_blocks > 0),
+              "block_epilogue: keys and values need a cache");
+  RLT_REQUIRE(k_token_stride >= k_width && v_token_stride >= v_width, "block_epilogue: the [kv_heads, dim] tail of the cache must be contiguous");
+  RLT_REQUIRE(act_width == 0 || (out && act_valid(act)), "block_epilogue: activation output or kind missing");
+  EpilogueArgs a;
+  a.proj = proj; a.proj_stride = proj_stride;
+  a.k_col = k_col; a.k_width = k_width; a.v_col = v_col; a.v_width = v_width;
+  a.key_cache = key_cache; a.k_block_stride = k_block_stride; a.k_token_stride = k_token_stride;
+  a.value_cache = value_cache; a.v_block_stride = v_block_stride; a.v_token_stride = v_token_stride;
+  a.num_blocks = num_blocks; a.block_size = block_size; a.tables = tables; a.table_width = table_width;
+  a.row_seq = row_seq; a.positions = positions;
+  a.act_col = act_col; a.act_width = act_width; a.act = act;
+  a.out = out; a.out_stride = out_stride; a.out_col = out_col;
+  const int vec = static_cast<int>(16 / dtype_size(dtype));
+  auto whole = [&](int64_t n) { return n % vec == 0; };
+  bool wide = whole(proj_stride) && aligned16(proj);
+  if (k_width + v_width > 0)
+    wide = wide && whole(k_col) && whole(k_width) && whole(v_col) && whole(v_width) && whole(k_block_stride) && whole(k_token_stride) &&
+           whole(v_block_stride) && whole(v_token_stride) && aligned16(key_cache) && aligned16(value_cache);
+  if (act_width > 0) wide = wide && whole(act_col) && whole(act_width) && whole(out_stride) && whole(out_col) && aligned16(out);
+  const int items = (k_width + v_width + act_width) / (wide ? vec : 1);
+  const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>((items + kThreads - 1) / kThreads));
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == RLT_F32) {
+    if (wide) block_epilogue_kernel<float, 4><<<grid, kThreads, 0, s>>>(a); else block_epilogue_kernel<float, 1><<<grid, kThreads, 0, s>>>(a);
+  } else if (dtype == RLT_F16) {
+    if (wide) block_epilogue_kernel<__half, 8><<<grid, kThreads, 0, s>>>(a); else block_epilogue_kernel<__half, 1><<<grid, kThreads, 0, s>>>(a);
+  } else {
+    if (wide) block_epilogue_kernel<__nv_bfloat16, 8><<<grid, kThreads, 0, s>>>(a);
+    else block_epilogue_kernel<__nv_bfloat16, 1><<<grid, kThreads, 0, s>>>(a);
+  }
+  return launch_status("block_epilogue_kernel");
+}
+
+extern "C" RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight,
+                                      void* out, int64_t out_stride, int rows, int width, int parts, float eps, int dtype,
+                                      rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype_valid(dtype), "gated_norm: dtype must be float32, float16 or bfloat16");
+  RLT_REQUIRE(rows >= 0 && width > 0 && parts > 0 && width % parts == 0 && eps >= 0.0f, "gated_norm: the width must be a whole number of parts");
+  if (rows == 0) return RLT_OK;
+  RLT_REQUIRE(y && z && weight && out, "gated_norm: null pointer");
+  const int part = width / parts;
+  const size_t smem = static_cast<size_t>(part) * sizeof(float);
+  if (smem > kMaxRowBytes - 1024) {
+    set_last_error_text("gated_norm: parts above 12032 elements are not supported");
+    return RLT_ERR_UNSUPPORTED;
+  }
+  const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>(parts));
+  RLT_DISPATCH_DTYPE(dtype, T, (gated_norm_kernel<T><<<grid, kThreads, smem, static_cast<cudaStream_t>(stream)>>>(
+                                   static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride, weight,
+                                   static_cast<T*>(out), out_stride, part, eps)));
+  return launch_status("gated_norm_kernel");
+}

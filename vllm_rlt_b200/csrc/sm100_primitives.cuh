@@ -16,7 +16,14 @@ constexpr int kHeadDim = 128;
 constexpr int kPage = 16;
 constexpr int kTileBytes = kPage * kHeadDim * 2;  // one page of one head: 4 KiB
 constexpr int kStageBytes = 2 * kTileBytes;       // K page + V page
+constexpr float kLog2e = 1.4426950408889634f;
 constexpr long long kWaitCycles = 4000000000ll;   // bounded waits (about 2 s): give up instead of hanging
+
+// The scale of the plain 1 / sqrt(128) in the log2 domain, or the call's own.
+inline float log2_scale(const AttentionArgs& a) {
+  const double scale = a.terms.scale != 0.0f ? static_cast<double>(a.terms.scale) : 1.0 / sqrt(static_cast<double>(kHeadDim));
+  return static_cast<float>(1.4426950408889634 * scale);
+}
 
 // ---- PTX wrappers -----------------------------------------------------------------------
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {
