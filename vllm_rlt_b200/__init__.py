@@ -10,14 +10,20 @@ raises if the CUDA library has not been built.
 from ._capi import NativeLibraryMissing, load as load_library
 from .activation import register_torch_op, silu_and_mul, silu_and_mul_packed
 from .attention import (B200_CAPABILITIES, AttentionBackend, B200PagedAttention, BackendCapabilities,
-                        create_backend)
+                        ScoreTerms, create_backend)
+from .checkpoint import read_safetensors, read_weights
 from .decoder import DecodeStats, GraphedLoops, PagedKV, SelfSpeculativeDecoder
 from .prefix_cache import PrefixIndex
+from .engine import Engine, StepEntry
+from .hybrid_lm import HybridLM, HybridLMConfig
 from .kv_cache import RollbackResult, finalize_tokens, kv_write, rollback
-from .layers import rope_kv_write, sandwich_norm
+from .layers import block_epilogue, residual_norm, rope_kv_write, sandwich_norm
 from .looped_lm import LoopedLM, LoopedLMConfig, seeded_state_dict
+from .recurrent import causal_conv, gated_norm, ssd_scan
+from .registry import load_model, register_model, registered_architectures
 from .runner import (B200SpeculativeRunner, KVCacheManagerView, ModelRunnerOutput, Request, SamplingParams, ScheduledRequest,
                      SchedulerOutput, SpeculativeConfig, SpeculativeRoundTicket, SpeculativeStats)
+from .sequence_cache import CacheFull, CacheSpec, KVSpec, SequenceCache, StateSpec
 from .speculative import (PipelineState, SpeculativeResult, accept_greedy, accept_rejection, argmax_rows,
                           decode_result, pipeline_shift, probabilities, raise_for_status, round_uniforms,
                           sample_rows)
@@ -30,5 +36,7 @@ __all__ = [
     "register_torch_op", "rollback", "rope_kv_write", "sample_rows", "sandwich_norm", "silu_and_mul",
     "B200SpeculativeRunner", "ModelRunnerOutput", "Request", "SamplingParams", "ScheduledRequest", "SchedulerOutput",
     "SpeculativeConfig", "SpeculativeRoundTicket", "SpeculativeStats", "round_uniforms", "silu_and_mul_packed",
-    "KVCacheManagerView",
+    "KVCacheManagerView", "CacheFull", "CacheSpec", "Engine", "HybridLM", "HybridLMConfig", "KVSpec", "ScoreTerms",
+    "SequenceCache", "StateSpec", "StepEntry", "block_epilogue", "causal_conv", "gated_norm", "load_model", "read_safetensors",
+    "read_weights", "register_model", "registered_architectures", "residual_norm", "ssd_scan",
 ]

@@ -41,6 +41,20 @@ class BackendCapabilities:
     sliding_window: bool = False
 
 
+@dataclass(frozen=True)
+class ScoreTerms:
+    """What becomes of `q . k` before the softmax: at query position p, key position j, query head h of H,
+
+        score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
+                - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
+    """
+
+    scale: float
+    temp_coef: float = 0.0
+    temp_every: int = 1
+    distance_bias: bool = False
+
+
 @dataclass
 class AttentionBackend:
     """Same shape as the reference's ``AttentionBackend`` adapter (attention/backend.py:30-55)."""
@@ -109,7 +123,7 @@ class B200PagedAttention:
             if self._sharing == 0:
                 self._planned.clear()
 
-    def _workspace(self, device: torch.device, stream: int, nbytes: int) -> torch.Tensor:
+    def _workspace(self, device: torch.device, stream, nbytes: int) -> torch.Tensor:
         # One scratch buffer per (device, stream): calls on one stream are ordered, calls on
         # different streams never share scratch.  Grown (doubling, by at most 256 MiB beyond the need),
         # never shrunk — and an outgrown buffer is kept, not freed: a caller's captured CUDA graph may have
@@ -301,6 +315,71 @@ class B200PagedAttention:
                 # the rows fall back to the grouped kernel (32-bit dtype, or caches the tensor map cannot express)
                 nbytes = lib.rlt_verify_attention_workspace_bytes(rows, q.shape[1], kv_heads, head_dim, block_size, max(width, 1))
         _capi.check(status, "prefill_attention")
+        return out
+
+    def scored(self, q, out, key_cache, value_cache, block_tables, context_lengths, cu_seqlens_q, max_new: int,
+               terms: ScoreTerms):
+        """Packed causal attention with score terms, into `out` (`rlt_scored_attention`).
+
+        q `[rows, heads, key_dim]` and out `[rows, heads, value_dim]` may be column slices of wider rows; the
+        caches are `[pages, block, kv_heads, dim]` views with sizes and strides of their own.  One table row and
+        one context length per sequence, rows of a sequence consecutive, `max_new` the longest portion.  128-wide
+        heads over 16-token pages in 16 bits run on the tiled kernels (portions of at most 16 tokens on the verify
+        kernel, whose plan a `shared_plan` block reuses; longer ones on the prompt kernel), everything else on
+        the shape-generic ones."""
+        device = _capi.require_cuda(q, out, key_cache, value_cache, block_tables, context_lengths, cu_seqlens_q)
+        rows, heads, key_dim = q.shape
+        if q.dtype not in _capi.DTYPE_CODES or any(t.dtype != q.dtype for t in (out, key_cache, value_cache)):
+            raise ValueError("q, out and the caches must share a float32/float16/bfloat16 dtype")
+        if key_cache.dim() != 4 or value_cache.dim() != 4 or key_cache.shape[:3] != value_cache.shape[:3] \
+                or key_cache.shape[3] != key_dim or out.shape != (rows, heads, value_cache.shape[3]):
+            raise ValueError("caches must be [pages, block, kv_heads, dim]; q and out [rows, heads, key_dim / value_dim]")
+        for name, t in (("q", q), ("out", out)):
+            if t.stride(2) != 1 or t.stride(1) != t.shape[2]:
+                raise ValueError(f"the [heads, dim] tail of {name} must be contiguous")
+        for cache in (key_cache, value_cache):
+            if cache.stride(3) != 1 or cache.stride(2) != cache.shape[3]:
+                raise ValueError("the [kv_heads, dim] tail of the caches must be contiguous")
+        sequences, width = block_tables.shape
+        if block_tables.dtype != torch.int32 or not block_tables.is_contiguous() or context_lengths.dtype != torch.int32 \
+                or context_lengths.shape != (sequences,) or cu_seqlens_q.dtype != torch.int32 or cu_seqlens_q.shape != (sequences + 1,):
+            raise ValueError("tables int32 [sequences, pages], context_lengths int32 [sequences], cu_seqlens_q int32 [sequences + 1]")
+        if heads % key_cache.shape[2]:
+            raise ValueError("query heads must be a positive multiple of KV heads")
+        if rows == 0:
+            return out
+        blocks, block, kv_heads, value_dim = value_cache.shape
+        lib, dtype = _capi.load(), _capi.DTYPE_CODES[q.dtype]
+        with torch.cuda.device(device):
+            stream = _capi.stream_of(q)
+            nbytes = lib.rlt_scored_attention_workspace_bytes(rows, sequences, max_new, heads, kv_heads, key_dim, value_dim, block,
+                                                              width, dtype)
+            ws_key = (device.index if device.index is not None else torch.cuda.current_device(), stream.value or 0)
+            # prompt calls have scratch of their own: a mixed step's plan for its short portions survives them
+            workspace = self._workspace(device, stream.value or 0 if max_new <= 16 else ("prompt", stream.value or 0), nbytes)
+            planned = False
+            tiled = max_new <= 16 and q.dtype != torch.float32 and key_dim == value_dim == 128 and block == 16
+            versions = self._versions(block_tables, context_lengths, cu_seqlens_q) if self._sharing and tiled else None
+            if versions is not None:
+                plan_key = (block_tables.data_ptr(), sequences, width, context_lengths.data_ptr(), cu_seqlens_q.data_ptr(), rows,
+                            heads, kv_heads, key_dim, block, dtype, versions)
+                if self._planned.get(ws_key) != plan_key:
+                    self._planned.pop(ws_key, None)
+                    status = lib.rlt_verify_attention_plan(
+                        _capi.ptr(block_tables), sequences, width, _capi.ptr(context_lengths), _capi.ptr(cu_seqlens_q), rows, heads,
+                        kv_heads, key_dim, block, dtype, _capi.ptr(workspace), workspace.numel(), stream)
+                    if status == _capi.OK:
+                        self._planned[ws_key] = plan_key
+                planned = self._planned.get(ws_key) == plan_key
+            elif max_new <= 16:
+                self._planned.pop(ws_key, None)       # the call overwrites the scratch a plan may lie in
+            status = lib.rlt_scored_attention(
+                _capi.ptr(q), q.stride(0), _capi.ptr(out), out.stride(0), _capi.ptr(key_cache), key_cache.stride(0),
+                key_cache.stride(1), _capi.ptr(value_cache), value_cache.stride(0), value_cache.stride(1), blocks, block, heads,
+                kv_heads, key_dim, value_dim, dtype, _capi.ptr(block_tables), sequences, width, _capi.ptr(context_lengths),
+                _capi.ptr(cu_seqlens_q), rows, int(max_new), float(terms.scale), float(terms.temp_coef), int(terms.temp_every),
+                int(terms.distance_bias), int(planned), _capi.ptr(workspace), workspace.numel(), stream)
+        _capi.check(status, "scored_attention")
         return out
 
 

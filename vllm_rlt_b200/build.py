@@ -9,6 +9,7 @@ dependency on PyTorch and can be bound from any host language through `include/r
 
 from __future__ import annotations
 
+import fcntl
 import os
 import shutil
 import subprocess
@@ -51,9 +52,17 @@ def stale() -> bool:
 def build(force: bool = False, verbose: bool = False) -> Path:
     if not force and not stale():
         return LIBRARY
-    objects = []
     build_dir = PACKAGE / "build"
     build_dir.mkdir(exist_ok=True)
+    with open(build_dir / ".lock", "w") as lock:       # processes that find no library at the same time: one builds
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if force or stale():
+            _compile(build_dir, verbose)
+    return LIBRARY
+
+
+def _compile(build_dir: Path, verbose: bool) -> None:
+    objects = []
     compile_flags = [f for f in NVCC_FLAGS if f not in ("--shared",)]
     procs = []
     for src in sources():
@@ -72,9 +81,9 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         print("\n".join(log))
     if failed:
         raise RuntimeError("nvcc failed; see output above")
-    link = [nvcc(), *NVCC_FLAGS, *map(str, objects), "-o", str(LIBRARY)]
-    subprocess.run(link, check=True)
-    return LIBRARY
+    linked = build_dir / LIBRARY.name
+    subprocess.run([nvcc(), *NVCC_FLAGS, *map(str, objects), "-o", str(linked)], check=True)
+    os.replace(linked, LIBRARY)
 
 
 if __name__ == "__main__":

@@ -99,3 +99,97 @@ def sandwich_norm(x, weight, eps: float, residual=None, weight2=None, *, in_plac
                                               _capi.DTYPE_CODES[x.dtype], _capi.stream_of(x))
     _capi.check(code, "sandwich_norm")
     return total, norm
+
+
+ACTIVATIONS = {"gelu": 1, "gelu_tanh": 2}      # the erf form and the tanh form
+
+
+def residual_norm(residual, weight, eps: float, dtype, *, delta=None, tokens=None, embed=None, row_index=None,
+                  weight_offset: float = 0.0, store: bool = True):
+    """The 32-bit residual stream of a parallel-block model and the norm that opens a layer, in one pass:
+
+        r = embed[tokens] or residual;  r += delta;  residual <- r (with `store`)
+        returns r / sqrt(mean(r^2) + eps) * (weight_offset + weight), in `dtype`
+
+    residual: float32 [rows, width], updated in place.  `row_index` (int64) selects rows: the result has one
+    row per entry, and the residual is not stored.  `weight`: float32 [width] (`weight_offset` 1 for weights
+    stored around zero)."""
+    _capi.require_cuda(residual, weight, delta, tokens, embed, row_index)
+    if residual.dim() != 2 or residual.dtype != torch.float32 or not residual.is_contiguous():
+        raise ValueError("residual must be contiguous float32 [rows, width]")
+    rows, width = residual.shape
+    if weight.dtype != torch.float32 or weight.shape != (width,) or not weight.is_contiguous():
+        raise ValueError("weight must be contiguous float32 [width]")
+    if dtype not in _capi.DTYPE_CODES:
+        raise ValueError("dtype must be float32 / float16 / bfloat16")
+    if delta is not None and (delta.shape != residual.shape or delta.dtype != dtype or not delta.is_contiguous()):
+        raise ValueError("delta must be a contiguous tensor of the model dtype, shaped like the residual")
+    if (tokens is None) != (embed is None):
+        raise ValueError("tokens and embed go together")
+    if tokens is not None and (tokens.dtype != torch.int64 or tokens.shape != (rows,) or embed.dtype != dtype
+                               or embed.dim() != 2 or embed.shape[1] != width or not embed.is_contiguous()):
+        raise ValueError("tokens must be int64 [rows] and embed contiguous [vocab, width] of the model dtype")
+    if row_index is not None:
+        if row_index.dtype != torch.int64 or row_index.dim() != 1:
+            raise ValueError("row_index must be int64")
+        if store:
+            raise ValueError("selected rows are not stored: pass store=False")
+        row_index = row_index.contiguous()
+    count = rows if row_index is None else row_index.numel()
+    out = torch.empty(count, width, dtype=dtype, device=residual.device)
+    if count == 0:
+        return out
+    tokens = None if tokens is None else tokens.contiguous()
+    with torch.cuda.device(residual.device):
+        code = _capi.load().rlt_residual_norm(
+            _capi.ptr(residual), _capi.ptr(delta), _capi.ptr(tokens), _capi.ptr(embed), 0 if embed is None else embed.shape[0],
+            _capi.ptr(row_index), int(store), _capi.ptr(weight), float(weight_offset), _capi.ptr(out), count, width, float(eps),
+            _capi.DTYPE_CODES[dtype], _capi.stream_of(residual))
+    _capi.check(code, "residual_norm")
+    return out
+
+
+def block_epilogue(proj, batch, *, kv=None, act=None):
+    """Columns of a stacked projection to where they are needed, in one launch.
+
+    kv = (key column, value column, key cache, value cache): the rows' keys and values into the pages of
+    (batch.row_seq, batch.positions); the caches are `[pages, block, kv_heads, dim]` views.
+    act = (first column, width, kind, out, out column): `out[:, out column + c] = kind(proj[:, first column + c])`."""
+    rows = proj.shape[0]
+    if proj.dim() != 2 or proj.stride(1) != 1 or proj.dtype not in _capi.DTYPE_CODES:
+        raise ValueError("proj must be [rows, columns] with unit inner stride")
+    if rows == 0 or (kv is None and act is None):
+        return
+    k_col = k_width = v_col = v_width = 0
+    key = value = tables = None
+    k_strides = v_strides = (0, 0)
+    pages = block = width = 0
+    if kv is not None:
+        k_col, v_col, key, value = kv
+        _capi.require_cuda(proj, key, value, batch.row_seq, batch.positions)
+        for name, cache in (("key", key), ("value", value)):
+            if cache.dim() != 4 or cache.dtype != proj.dtype or cache.stride(3) != 1 or cache.stride(2) != cache.shape[3]:
+                raise ValueError(f"the {name} cache must be [pages, block, kv_heads, dim] of the model dtype with a contiguous tail")
+        k_width, v_width = key.shape[2] * key.shape[3], value.shape[2] * value.shape[3]
+        if k_col + k_width > proj.shape[1] or v_col + v_width > proj.shape[1] or value.shape[:3] != key.shape[:3]:
+            raise ValueError("key or value columns lie outside the projection, or the caches do not match")
+        k_strides, v_strides = (key.stride(0), key.stride(1)), (value.stride(0), value.stride(1))
+        tables = batch.tables[0]
+        pages, block, width = key.shape[0], key.shape[1], tables.shape[1]
+    act_col = act_width = kind = out_col = out_stride = 0
+    out = None
+    if act is not None:
+        act_col, act_width, name, out, out_col = act
+        _capi.require_cuda(proj, out)
+        kind = ACTIVATIONS[name]
+        if out.dtype != proj.dtype or out.shape[0] != rows or out.stride(1) != 1 or out_col + act_width > out.shape[1] \
+                or act_col + act_width > proj.shape[1]:
+            raise ValueError("activation columns lie outside the projection or the output")
+        out_stride = out.stride(0)
+    with torch.cuda.device(proj.device):
+        code = _capi.load().rlt_block_epilogue(
+            _capi.ptr(proj), proj.stride(0), k_col, k_width, v_col, v_width, _capi.ptr(key), *k_strides, _capi.ptr(value),
+            *v_strides, pages, block, _capi.ptr(tables), width, _capi.ptr(None if kv is None else batch.row_seq),
+            _capi.ptr(None if kv is None else batch.positions), act_col, act_width, kind, _capi.ptr(out), out_stride, out_col,
+            rows, _capi.DTYPE_CODES[proj.dtype], _capi.stream_of(proj))
+    _capi.check(code, "block_epilogue")

@@ -12,7 +12,7 @@ the reference's (checkpoint-compatible), so a reference `state_dict()` loads unc
 from __future__ import annotations
 
 import hashlib
-from dataclasses import dataclass
+from dataclasses import dataclass, fields
 
 import torch
 import torch.nn.functional as F
@@ -21,6 +21,7 @@ from .activation import silu_and_mul, silu_and_mul_packed
 from .attention import B200PagedAttention
 from .kv_cache import kv_write
 from .layers import rope_kv_write, sandwich_norm
+from .sequence_cache import CacheSpec, KVSpec
 
 
 @dataclass(frozen=True)
@@ -38,6 +39,15 @@ class LoopedLMConfig:
     rope_theta: float = 1_000_000.0
     total_ut_steps: int = 4
     initializer_range: float = 0.02
+
+    @classmethod
+    def from_json(cls, config: dict) -> "LoopedLMConfig":
+        """The fields of a config.json (OuroConfig's names); what it leaves out keeps its default."""
+        known = {f.name for f in fields(cls)}
+        values = {k: v for k, v in config.items() if k in known and v is not None}
+        if "head_dim" not in values and {"hidden_size", "num_attention_heads"} <= values.keys():
+            values["head_dim"] = values["hidden_size"] // values["num_attention_heads"]
+        return cls(**values)
 
 
 def parameter_shapes(config: LoopedLMConfig) -> dict[str, tuple]:
@@ -200,6 +210,33 @@ class LoopedLM:
                 stream, x = sandwich_norm(mlp, w[p + "post_attention_layernorm_2.weight"], c.rms_norm_eps, stream,
                                           following, in_place=True)
         return x
+
+    # ---- serving through the engine (registry.py) ----------------------------------------------
+    @property
+    def vocab_size(self) -> int:
+        return self.config.vocab_size
+
+    def cache_spec(self) -> CacheSpec:
+        c = self.config
+        kind = KVSpec(c.num_key_value_heads, c.head_dim, c.head_dim)
+        return CacheSpec(planes=c.total_ut_steps, layers={i: kind for i in range(c.num_hidden_layers)}, pooled=True)
+
+    def forward_step(self, batch, cache):
+        """All rows of an engine step through every loop at full depth, each sequence's portion packed."""
+        active = batch.row_seq >= 0
+        owner = batch.row_seq.clamp_min(0).long()
+        positions = batch.positions.long()
+        offsets = positions % cache.block
+        hidden = self.prelude(batch.tokens)
+        for depth in range(self.config.total_ut_steps):
+            tables = batch.tables[depth]
+            blocks = tables[owner].gather(1, (positions // cache.block)[:, None]).squeeze(1).long()
+            hidden = self.recurrent(hidden, positions, cache.key_pool, cache.value_pool, blocks, offsets, tables,
+                                    batch.lengths, packed=(batch.cu, batch.max_new), write_mask=active)
+        return hidden
+
+    def step_logits(self, hidden, rows=None):
+        return self.coda(hidden if rows is None else hidden[rows]).float()
 
     def coda(self, hidden: torch.Tensor) -> torch.Tensor:
         return F.linear(hidden, self.w["lm_head.weight"])

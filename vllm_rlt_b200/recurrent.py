@@ -1,0 +1,98 @@
+"""Recurrent layers over packed sequences with per-sequence state slots: short causal convolution, the Mamba-2
+state-space recurrence, and the gated norm behind it.
+
+`group` arguments are a step's sequence group (`StepGroup`): `cu` (int32 [n + 1], row offsets into the step's
+rows), `starts` (position of each portion's first token), `slots`, and the host-side bound `max_new`.
+"""
+
+from __future__ import annotations
+
+import torch
+
+from . import _capi
+from .layers import ACTIVATIONS
+
+
+def causal_conv(x, weight, bias, state, out, group, act=None):
+    """`out[i, c] = silu(bias[c] + sum_j weight[c, j] * x[i - taps + 1 + j, c])`, inputs before a portion from `state`.
+
+    x `[rows, channels]` (any row stride), weight float32 `[channels, taps]`, bias float32 `[channels]`, state
+    `[slots, taps - 1, channels]` of x's dtype, updated in place.  act = (columns, kind, destination): feed-forward
+    columns of the same rows through an activation in the same launch."""
+    device = _capi.require_cuda(x, weight, bias, state, out, group.cu, group.starts, group.slots)
+    channels, taps = weight.shape
+    if weight.dtype != torch.float32 or bias.dtype != torch.float32 or bias.shape != (channels,) or not weight.is_contiguous():
+        raise ValueError("weight must be contiguous float32 [channels, taps] and bias float32 [channels]")
+    if x.dim() != 2 or x.shape[1] != channels or out.shape != x.shape or x.stride(1) != 1 or out.stride(1) != 1 \
+            or x.dtype not in _capi.DTYPE_CODES or out.dtype != x.dtype:
+        raise ValueError("x and out must be [rows, channels] of one dtype with unit inner stride")
+    if state.shape[1:] != (taps - 1, channels) or state.dtype != x.dtype or not state.is_contiguous():
+        raise ValueError("state must be contiguous [slots, taps - 1, channels] of the model dtype")
+    act_in, act_out, act_width, kind = None, None, 0, 0
+    if act is not None:
+        act_in, name, act_out = act
+        kind, act_width = ACTIVATIONS[name], act_in.shape[1]
+        if act_in.stride(0) != x.stride(0) or act_in.stride(1) != 1 or act_out.shape != act_in.shape or act_out.stride(1) != 1 \
+                or act_in.dtype != x.dtype or act_out.dtype != x.dtype:
+            raise ValueError("activation columns must come from the projection that holds x")
+    if group.sequences == 0:
+        return out
+    with torch.cuda.device(device):
+        code = _capi.load().rlt_causal_conv(
+            _capi.ptr(x), x.stride(0), _capi.ptr(weight), _capi.ptr(bias), _capi.ptr(out), out.stride(0), _capi.ptr(state),
+            state.shape[0], channels, taps, _capi.ptr(group.cu), _capi.ptr(group.starts), _capi.ptr(group.slots), group.sequences,
+            group.max_new, _capi.ptr(act_in), _capi.ptr(act_out), 0 if act_out is None else act_out.stride(0), act_width, kind,
+            _capi.DTYPE_CODES[x.dtype], _capi.stream_of(x))
+    _capi.check(code, "causal_conv")
+    return out
+
+
+def ssd_scan(x, b, c, dt, dt_bias, a_log, d, state, out, group):
+    """The Mamba-2 recurrence (`rlt_ssd_scan`): x, out `[rows, heads * head_dim]`, b, c `[rows, groups * state_size]`
+    (slices of rows of one stride), dt `[rows, heads]` raw, parameters float32 `[heads]`, state float32
+    `[slots, heads, state_size, head_dim]`, updated in place."""
+    device = _capi.require_cuda(x, b, c, dt, dt_bias, a_log, d, state, out, group.cu, group.starts, group.slots)
+    if state.dim() != 4 or state.dtype != torch.float32 or not state.is_contiguous():
+        raise ValueError("state must be contiguous float32 [slots, heads, state_size, head_dim]")
+    slots, heads, size, head_dim = state.shape
+    rows = x.shape[0]
+    if x.shape != (rows, heads * head_dim) or out.shape != x.shape or b.shape != c.shape or b.shape[1] % size or dt.shape != (rows, heads):
+        raise ValueError("x / out [rows, heads * head_dim], b / c [rows, groups * state_size], dt [rows, heads]")
+    groups = b.shape[1] // size
+    if x.stride(0) != b.stride(0) or b.stride(0) != c.stride(0) or any(t.stride(1) != 1 for t in (x, b, c, dt, out)):
+        raise ValueError("x, b and c must be column slices of the same rows")
+    if x.dtype not in (torch.float32, torch.bfloat16) or any(t.dtype != x.dtype for t in (b, c, dt, out)):
+        raise ValueError("x, b, c, dt and out must share float32 or bfloat16")
+    for name, t in (("dt_bias", dt_bias), ("a_log", a_log), ("d", d)):
+        if t.dtype != torch.float32 or t.shape != (heads,):
+            raise ValueError(f"{name} must be float32 [heads]")
+    if group.sequences == 0:
+        return out
+    lib, dtype = _capi.load(), _capi.DTYPE_CODES[x.dtype]
+    with torch.cuda.device(device):
+        nbytes = lib.rlt_ssd_scan_workspace_bytes(group.sequences, group.max_new, heads, size, head_dim, dtype)
+        workspace = torch.empty(nbytes, dtype=torch.uint8, device=device)
+        code = lib.rlt_ssd_scan(
+            _capi.ptr(x), _capi.ptr(b), _capi.ptr(c), x.stride(0), _capi.ptr(dt), dt.stride(0), _capi.ptr(dt_bias),
+            _capi.ptr(a_log), _capi.ptr(d), _capi.ptr(out), out.stride(0), _capi.ptr(state), slots, _capi.ptr(group.cu),
+            _capi.ptr(group.starts), _capi.ptr(group.slots), group.sequences, group.max_new, heads, groups, size, head_dim, dtype,
+            _capi.ptr(workspace), nbytes, _capi.stream_of(x))
+    _capi.check(code, "ssd_scan")
+    return out
+
+
+def gated_norm(y, z, weight, out, parts: int, eps: float):
+    """`out = rmsnorm(y * silu(z)) * weight`, the row normed in `parts` equal parts; all `[rows, width]`, any row stride."""
+    device = _capi.require_cuda(y, z, weight, out)
+    rows, width = y.shape
+    if z.shape != y.shape or out.shape != y.shape or weight.shape != (width,) or weight.dtype != torch.float32 \
+            or any(t.stride(1) != 1 for t in (y, z, out)) or y.dtype not in _capi.DTYPE_CODES or z.dtype != y.dtype or out.dtype != y.dtype:
+        raise ValueError("y, z and out must be [rows, width] of one dtype with unit inner stride, weight float32 [width]")
+    if rows == 0:
+        return out
+    with torch.cuda.device(device):
+        code = _capi.load().rlt_gated_norm(_capi.ptr(y), y.stride(0), _capi.ptr(z), z.stride(0), _capi.ptr(weight), _capi.ptr(out),
+                                           out.stride(0), rows, width, parts, float(eps), _capi.DTYPE_CODES[y.dtype],
+                                           _capi.stream_of(y))
+    _capi.check(code, "gated_norm")
+    return out
