@@ -106,6 +106,11 @@ __device__ __forceinline__ void resolve_row(const AttentionArgs& a, int row, int
 // attention_generic.cu: any shape, one CTA per (row, head).
 int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream, int window = 0);   // window > 0: the row's last `window` keys only
 
+// attention_tiles.cu: tensor cores for other head sizes (bf16, multiples of 8 up to 256), packed rows only.
+bool attention_tiles_supported(const AttentionArgs& a);
+size_t attention_tiles_workspace_bytes(int rows, int sequences, int max_new, int q_heads, int kv_heads, int value_dim, int64_t capacity);
+int launch_attention_tiles(const AttentionArgs& a, int max_new, void* workspace, size_t workspace_bytes, cudaStream_t stream);
+
 // attention_sm100.cu: head_dim 128, 16-token pages, fp16/bf16 — TMA page streaming,
 // request-grouped rows on tensor cores, split-KV with a deterministic merge.
 bool attention_sm100_supported(const AttentionArgs& a);        // shape and cache view

@@ -205,9 +205,14 @@ extern "C" RLT_API size_t rlt_scored_attention_workspace_bytes(int rows, int seq
                                                                int key_dim, int value_dim, int block_size, int table_width,
                                                                int dtype) {
   if (rows <= 0 || sequences <= 0 || q_heads <= 0 || kv_heads <= 0 || table_width <= 0) return 256;
-  if (dtype == RLT_F32 || key_dim != 128 || value_dim != 128 || block_size != 16) return 256;
-  if (max_new > 16) return rlt::prefill_sm100_workspace_bytes(rows, sequences);
-  return rlt_verify_attention_workspace_bytes(rows, q_heads, kv_heads, key_dim, block_size, table_width);
+  if (dtype == RLT_F32) return 256;
+  // the tile kernel's own scratch also where the page kernels are expected: they may refuse a cache's placement
+  const size_t tiles = rlt::attention_tiles_workspace_bytes(rows, sequences, max_new, q_heads, kv_heads, value_dim,
+                                                            static_cast<int64_t>(table_width) * block_size);
+  if (key_dim != 128 || value_dim != 128 || block_size != 16) return tiles;
+  const size_t pages = max_new > 16 ? rlt::prefill_sm100_workspace_bytes(rows, sequences)
+                                    : rlt_verify_attention_workspace_bytes(rows, q_heads, kv_heads, key_dim, block_size, table_width);
+  return tiles > pages ? tiles : pages;
 }
 
 extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, void* out, int64_t out_stride,
@@ -248,5 +253,6 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
       return planned ? run_attention_sm100(a, workspace, workspace_bytes, s) : launch_attention_sm100(a, workspace, workspace_bytes, s);
     }
   }
+  if (attention_tiles_supported(a)) return launch_attention_tiles(a, max_new, workspace, workspace_bytes, s);
   return launch_attention_generic(a, s);
 }
