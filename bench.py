@@ -39,6 +39,10 @@ Other entry points (each prints its own JSON line; none is the contract line abo
                       R requests in total (default 1024, prompts U[256, 2048], 512 output tokens, k = 6, T = 0.8),
                       length-balanced over the ranks and decoded to completion in waves that fit the KV
                       pool: whole-job strong scaling
+    --workload hybrid [--steps K --warmup W]
+                      prefill and decode of Sobipel-shaped models (parallel attention / Mamba-2 blocks, random weights)
+                      beside the looped model at equal size with one loop, through the same engine, and every kernel
+                      of a layer against its roofline beside the like kernel of the looped model
     --only attention  [--requests --layers --tokens --depths --kv-heads --context-min --context-max --shared-plan]
     --only prefill    [--requests --tokens --kv-heads --eager]   packed causal prefill, TFLOP/s
     --only accept | --only silu                                  the small kernels at the step's shapes
@@ -898,6 +902,247 @@ def run_reference_engine_workload(args):
         "finished_requests": finished}))
 
 
+# Layer shapes of the hybrid workload: width, attention (heads, kv heads), feed-forward width of the two-matrix MLP (and of
+# the looped model's three-matrix one: the same parameters), Mamba-2 (heads, head size, state, groups), layers, vocabulary.
+HYBRID_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=16, ff=8448, looped_ff=5632, mamba=(64, 64, 128, 1), layers=12, vocab=49152),
+    "4096": dict(width=4096, heads=32, kv_heads=8, ff=14336, looped_ff=9600, mamba=(128, 64, 128, 8), layers=8, vocab=49152),
+}
+
+
+def hybrid_config(size, pattern: str):
+    """config.json of a Sobipel model whose layers repeat `pattern` ('a' attention, 'm' Mamba-2)."""
+    heads, vdim, state, groups = size["mamba"]
+    kinds = {"a": {"type": "attention", "mixer": {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": HEAD_DIM, "vdim": HEAD_DIM,
+                                                  "scale": HEAD_DIM ** -0.5, "q_temp": {"coef": 0.1, "every": 2048}}},
+             "m": {"type": "mamba2", "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": 4,
+                                               "norm_groups": groups}}}
+    layers = [dict(kinds[pattern[i % len(pattern)]], mlp={"kind": "dense", "ff": size["ff"]}) for i in range(size["layers"])]
+    return {"architecture": "Sobipel", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6}, "layers": layers}
+
+
+def device_weights(shapes, device, seed=0):
+    g = torch.Generator(device=device).manual_seed(seed)
+    out = {}
+    for name, shape in shapes.items():
+        w = torch.randn(shape, device=device, generator=g) * (0.02 if len(shape) == 2 else 0.1)
+        if "layernorm" in name or name in ("model.norm.weight",) or name.endswith("mix.norm"):
+            w = w + 1
+        out[name] = w.to(torch.bfloat16)
+    return out
+
+
+def timed_ms(run, steps: int, warmup: int) -> float:
+    for _ in range(warmup):
+        run()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    a.record()
+    for _ in range(steps):
+        run()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / steps
+
+
+@torch.no_grad()
+def hybrid_model_rows(name, model, steps, warmup):
+    """Prefill and decode of one model through the engine: device time of a step, weights and caches larger than L2."""
+    import vllm_rlt_b200 as rlt
+
+    rows = []
+    for requests, tokens in ((8, 2048), (1, 16384)):
+        engine = rlt.Engine(model, max_tokens=requests * (tokens + BLOCK), max_sequences=requests, cuda_graphs=False)
+        entries = [rlt.StepEntry(i, torch.randint(0, model.vocab_size, (tokens,)).tolist(), [tokens - 1]) for i in range(requests)]
+        engine._claim(entries)
+        batch = engine._batch(entries)
+        last = batch.cu[1:].long() - 1
+        ms = timed_ms(lambda: model.step_logits(model.forward_step(batch, engine.cache), last), steps, warmup)
+        rows.append({"model": name, "phase": "prefill", "requests": requests, "tokens": tokens, "ms": ms, "tokens_per_s": requests * tokens / ms * 1e3})
+        del engine, batch
+    for requests, context in ((1, 4096), (16, 4096), (64, 2048)):
+        engine = rlt.Engine(model, max_tokens=requests * (context + BLOCK), max_sequences=requests, max_sequence_tokens=context + BLOCK,
+                            capture_sizes=[requests])
+        for i in range(requests):
+            engine.step([rlt.StepEntry(i, torch.randint(0, model.vocab_size, (context,)).tolist())])
+        engine.step([rlt.StepEntry(i, [1], [0]) for i in range(requests)])
+        (graph, *_), = engine._graphs.values()
+        ms = timed_ms(graph.replay, steps * 4, warmup)
+        rows.append({"model": name, "phase": "decode", "requests": requests, "tokens": context, "ms": ms, "tokens_per_s": requests / ms * 1e3})
+        del engine, graph
+    torch.cuda.empty_cache()
+    return rows
+
+
+def ring_us(calls, replays: int) -> float:
+    """Microseconds per call of a ring of calls whose tensors together exceed L2, replayed from a CUDA graph."""
+    for call in calls:
+        call()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        kept = [call() for call in calls]
+    ms = timed_ms(graph.replay, replays, 2)
+    del kept
+    return ms / len(calls) * 1e3
+
+
+@torch.no_grad()
+def hybrid_kernel_rows(size, steps):
+    """Every kernel of a hybrid layer at prefill (16384 rows: 8 x 2048) and decode (64 rows, context 2048), with its
+    algorithmic bytes or flops against the measured peak, beside the like kernel of the looped model."""
+    from types import SimpleNamespace
+
+    import vllm_rlt_b200 as rlt
+
+    device = torch.device("cuda", 0)
+    peak_gbs, _ = measured_peaks()
+    peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+    peak_tflops = float(peaks.get("bf16_tflops", 1590.0))
+    width, heads, kv_heads, ff = size["width"], size["heads"], size["kv_heads"], size["ff"]
+    m_heads, vdim, state, groups = size["mamba"]
+    inner, gn = m_heads * vdim, groups * state
+    channels = inner + 2 * gn
+    bf16 = lambda *shape: torch.randn(*shape, device=device).to(torch.bfloat16)
+    f32 = lambda *shape: torch.randn(*shape, device=device)
+    rows_out = []
+
+    def add(kernel, phase, like, make, nbytes=0.0, flops=0.0, copies=None):
+        """make(i) -> a call on the i-th set of tensors."""
+        copies = copies or max(2, min(48, int(400e6 // max(nbytes, 1)) + 1))
+        us = ring_us([make(i) for i in range(copies)], steps)
+        frac = flops / us / 1e6 / peak_tflops if flops else nbytes / us / 1e3 / peak_gbs
+        rows_out.append({"kernel": kernel, "phase": phase, "like": like, "us": us, "bound": "tensor" if flops else "hbm",
+                         "roofline_frac": frac})
+        torch.cuda.empty_cache()
+
+    for phase, seqs, new, context in (("prefill", 8, 2048, 2048), ("decode", 64, 1, 2048)):
+        rows = seqs * new
+        pages = context // BLOCK
+        tables = torch.randperm(seqs * pages, device=device).int().view(seqs, pages)
+        lengths = torch.full((seqs,), context, dtype=torch.int32, device=device)
+        cu = (torch.arange(seqs + 1, device=device) * new).int()
+        starts = lengths - new
+        slots = torch.arange(seqs, device=device, dtype=torch.int32)
+        row_seq = torch.arange(seqs, device=device, dtype=torch.int32).repeat_interleave(new)
+        positions = (torch.arange(rows, device=device) % new).int() + (context - new)
+        batch = SimpleNamespace(tables=tables[None], row_seq=row_seq, positions=positions)
+        group = SimpleNamespace(sequences=seqs, max_new=new, cu=cu, starts=starts, slots=slots)
+        terms = rlt.ScoreTerms(HEAD_DIM ** -0.5, 0.1, 2048, True)
+
+        # attention: score terms against none, on the same cache
+        kv_bytes = 2 * seqs * context * kv_heads * HEAD_DIM * 2
+        qo_bytes = 2 * rows * heads * HEAD_DIM * 2
+        visible = seqs * sum(range(context - new + 1, context + 1))
+        flops = 4.0 * HEAD_DIM * heads * visible if new > 16 else 0.0
+        sets = 2
+        pools = [bf16(2, seqs * pages, BLOCK, kv_heads, HEAD_DIM) for _ in range(sets)]
+        proj_width = (heads + 2 * kv_heads) * HEAD_DIM + ff
+        q_wide = [bf16(rows, proj_width) for _ in range(sets)]
+        out_wide = bf16(rows, heads * HEAD_DIM + ff)
+        kernels = rlt.B200PagedAttention()
+
+        def scored(i):
+            q = q_wide[i % sets][:, :heads * HEAD_DIM].view(rows, heads, HEAD_DIM)
+            out = out_wide[:, :heads * HEAD_DIM].view(rows, heads, HEAD_DIM)
+            return lambda: kernels.scored(q, out, pools[i % sets][0], pools[i % sets][1], tables, lengths, cu, new, terms)
+
+        q_plain = [bf16(rows, heads, HEAD_DIM) for _ in range(sets)]
+        plain = lambda i: (lambda: kernels.prefill(q_plain[i % sets], pools[i % sets][0], pools[i % sets][1], tables, lengths, cu, new))
+        add("scored attention", phase, None, scored, kv_bytes + qo_bytes, flops, copies=4)
+        add("attention of the looped model", phase, "scored attention", plain, kv_bytes + qo_bytes, flops, copies=4)
+        del pools, q_plain
+
+        # the norm that opens a layer: 32-bit residual read and written, 16-bit contribution read, 16-bit row written
+        copies = max(2, min(48, int(400e6 // (rows * width * 12)) + 1))
+        res, delta, weight = [f32(rows, width) for _ in range(copies)], [bf16(rows, width) for _ in range(copies)], f32(width)
+        add("residual_norm", phase, None, lambda i: (lambda: rlt.residual_norm(res[i], weight, 1e-6, torch.bfloat16, delta=delta[i], weight_offset=1.0)),
+            rows * width * 12.0, copies=copies)
+        res16, w16 = [bf16(rows, width) for _ in range(copies)], bf16(width)
+        add("sandwich_norm", phase, "residual_norm",
+            lambda i: (lambda: rlt.sandwich_norm(delta[i], w16, 1e-6, res16[i], w16, in_place=True)), rows * width * 8.0, copies=copies)
+        del res, res16, delta
+
+        # keys and values to their pages and gelu, against rope + KV write and silu-and-mul
+        cache = bf16(2, seqs * pages, BLOCK, kv_heads, HEAD_DIM)
+        kv_width = kv_heads * HEAD_DIM
+        copies = max(2, min(48, int(400e6 // (rows * (2 * kv_width + ff) * 4)) + 1))
+        projs = [bf16(rows, proj_width) for _ in range(copies)]
+        add("block_epilogue", phase, None, lambda i: (lambda: rlt.block_epilogue(
+            projs[i], batch, kv=(heads * HEAD_DIM, heads * HEAD_DIM + kv_width, cache[0], cache[1]),
+            act=(heads * HEAD_DIM + 2 * kv_width, ff, "gelu", out_wide, heads * HEAD_DIM))), rows * (2 * kv_width + ff) * 4.0, copies=copies)
+        cos = bf16(rows, HEAD_DIM)
+        blocks = tables[row_seq.long(), (positions // BLOCK).long()].long()
+        offsets = (positions % BLOCK).long()
+        cut = lambda p, a, n: p[:, a * HEAD_DIM:(a + n) * HEAD_DIM].view(rows, n, HEAD_DIM)
+        add("rope_kv_write", phase, "block_epilogue", lambda i: (lambda: rlt.rope_kv_write(
+            cut(projs[i], 0, heads), cut(projs[i], heads, kv_heads), cut(projs[i], heads + kv_heads, kv_heads), cos, cos, cache[0], cache[1],
+            blocks, offsets)), rows * ((heads + 2 * kv_heads) * HEAD_DIM * 4.0 + HEAD_DIM * 4), copies=copies)
+        gate_up = [bf16(rows, 2 * size["looped_ff"]) for _ in range(copies)]
+        add("silu_and_mul", phase, "block_epilogue", lambda i: (lambda: rlt.silu_and_mul_packed(gate_up[i])), rows * size["looped_ff"] * 6.0, copies=copies)
+        del projs, gate_up, cache, q_wide, out_wide
+
+        # the recurrent layer
+        in_width = inner + channels + m_heads + ff
+        conv_bytes = rows * (channels + ff) * 4.0
+        copies = max(2, min(24, int(400e6 // conv_bytes) + 1))
+        projs = [bf16(rows, in_width) for _ in range(copies)]
+        mixed = [bf16(rows, channels) for _ in range(copies)]
+        acted, y = bf16(rows, ff), bf16(rows, inner)
+        conv_state = torch.zeros(seqs, 3, channels, device=device, dtype=torch.bfloat16)
+        conv_w, conv_b = f32(channels, 4), f32(channels)
+        add("causal_conv + gelu", phase, None, lambda i: (lambda: rlt.causal_conv(
+            projs[i][:, inner:inner + channels], conv_w, conv_b, conv_state, mixed[i], group,
+            act=(projs[i][:, inner + channels + m_heads:], "gelu", acted))), conv_bytes, copies=copies)
+        dt_bias, a_log, d = f32(m_heads) - 3, f32(m_heads), f32(m_heads)
+        ssm_sets = 2 if new > 1 else 4
+        ssm = [torch.zeros(seqs, m_heads, state, vdim, device=device) for _ in range(ssm_sets)]
+
+        def scan(i):
+            x, b, c = mixed[i % copies].split((inner, gn, gn), 1)
+            dt = projs[i % copies][:, inner + channels:inner + channels + m_heads]
+            return lambda: rlt.ssd_scan(x, b, c, dt, dt_bias, a_log, d, ssm[i % ssm_sets], y, group)
+
+        scan_bytes = rows * (channels + inner + m_heads) * 2.0 + 2 * ssm[0].numel() * 4.0
+        add("ssd_scan", phase, None, scan, scan_bytes, copies=4)
+        norm_w = f32(inner)
+        outs = bf16(rows, inner + ff)
+        add("gated_norm", phase, "sandwich_norm", lambda i: (lambda: rlt.gated_norm(
+            y, projs[i][:, :inner], norm_w, outs[:, :inner], groups, 1e-6)), rows * inner * 6.0, copies=copies)
+        del projs, mixed, acted, y, ssm, outs
+    return rows_out
+
+
+def run_hybrid_workload(args):
+    """`--workload hybrid`: one JSON line with throughput rows, kernel rows and the clocks under them."""
+    import vllm_rlt_b200 as rlt
+    from vllm_rlt_b200.hybrid_lm import parameter_shapes as hybrid_shapes
+    from vllm_rlt_b200.looped_lm import parameter_shapes as looped_shapes
+
+    torch.cuda.set_device(0)
+    device = torch.device("cuda", 0)
+    report = {"workload": "hybrid", "data": "synthetic, random weights", "dtype": "bf16", "steps": args.steps, "sizes": {}}
+    with ClockSampler(0) as clocks:
+        for name, size in HYBRID_SIZES.items():
+            rows = []
+            for label, pattern in (("Sobipel, attention layers", "a"), ("Sobipel, Mamba-2 layers", "m"), ("Sobipel, 1 attention : 3 Mamba-2", "ammm")):
+                config = rlt.HybridLMConfig.from_json(hybrid_config(size, pattern))
+                model = rlt.HybridLM(config, device_weights(hybrid_shapes(config), device), device)
+                rows += hybrid_model_rows(label, model, args.steps, args.warmup)
+                del model
+            looped = rlt.LoopedLMConfig(vocab_size=size["vocab"], hidden_size=size["width"], intermediate_size=size["looped_ff"],
+                                        num_hidden_layers=size["layers"], num_attention_heads=size["heads"],
+                                        num_key_value_heads=size["kv_heads"], head_dim=HEAD_DIM, total_ut_steps=1)
+            model = rlt.LoopedLM(looped, device_weights(looped_shapes(looped), device), device, torch.bfloat16)
+            rows += hybrid_model_rows("looped model, one loop", model, args.steps, args.warmup)
+            del model
+            torch.cuda.empty_cache()
+            report["sizes"][name] = {"shape": {k: v for k, v in size.items()}, "throughput": rows, "kernels": hybrid_kernel_rows(size, args.steps)}
+            torch.cuda.empty_cache()
+    report["clocks"] = clocks.summary()
+    print(json.dumps(report))
+
+
 def balanced_shards(lengths, world: int):
     """Longest-first greedy assignment of requests to ranks by prompt length: returns one list of request
     indices per rank whose total lengths differ by at most one request's length."""
@@ -1190,7 +1435,7 @@ def main():
     parser.add_argument("--no-cpu-baseline", action="store_true")
     parser.add_argument("--only", default=None, choices=["attention", "accept", "silu", "prefill"],
                         help="profiling aid: run only this kernel family (not a bench line)")
-    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded"],
+    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded", "hybrid"],
                         help="rounds: timed speculative rounds (the bench line); decode: one complete generation; "
                              "sharded: a fixed request set shared out over the ranks, decoded to completion")
     parser.add_argument("--engine", default="b200", choices=["b200", "reference"],
@@ -1238,6 +1483,9 @@ def main():
             setattr(args, name, sharded_default if sharded else decode_default)
     if sharded:
         run_sharded_workload(args)
+        return
+    if args.workload == "hybrid":
+        run_hybrid_workload(args)
         return
     if args.workload == "decode":
         if args.engine == "reference":

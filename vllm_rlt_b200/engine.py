@@ -204,18 +204,20 @@ class Engine:
         # from the caching host allocator: reused only after the copy that reads it has run
         return torch.zeros(size, dtype=torch.int32, pin_memory=self.device.type == "cuda")
 
-    def _eager_step(self, ordered, entries):
+    def _batch(self, ordered) -> StepBatch:
+        """The uploaded metadata of entries whose pages are reserved; short portions come first."""
         cache = self.cache
-        short = sum(len(e.tokens) <= SHORT_PORTION for e in ordered)
-        rows = sum(len(e.tokens) for e in ordered)
-        width = max(-(-(cache.length(e.name) + len(e.tokens)) // cache.block) for e in ordered)
-        layout = _Layout(rows, len(ordered), cache.spec.planes, width, short)
+        counts = [len(e.tokens) for e in ordered]
+        short = sum(n <= SHORT_PORTION for n in counts)
+        width = max(-(-(cache.length(e.name) + n) // cache.block) for e, n in zip(ordered, counts))
+        layout = _Layout(sum(counts), len(ordered), cache.spec.planes, width, short)
         host = self._host_buffer(layout.size)
         self._fill(layout, host, ordered)
-        short_rows = sum(len(e.tokens) for e in ordered[:short])
-        batch = layout.batch(host.to(self.device, non_blocking=True), short_rows, max((len(e.tokens) for e in ordered[:short]), default=0),
-                             max((len(e.tokens) for e in ordered[short:]), default=0))
-        hidden = self.model.forward_step(batch, cache)
+        return layout.batch(host.to(self.device, non_blocking=True), sum(counts[:short]), max(counts[:short], default=0),
+                            max(counts[short:], default=0))
+
+    def _eager_step(self, ordered, entries):
+        hidden = self.model.forward_step(self._batch(ordered), self.cache)
         first, at = {}, 0
         for e in ordered:
             first[e.name] = at
