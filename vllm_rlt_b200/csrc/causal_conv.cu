@@ -31,8 +31,9 @@ struct ConvArgs {
   int act_width, act, conv_blocks;
 };
 
-// kTaps 0: any number of taps, inputs re-read (from L1) for every output.
-template <typename T, int kTaps>
+// A thread owns kVec neighbouring channels (or kActVec activation columns) for a tile of tokens.
+// kTaps 0: any number of taps, inputs re-read (from L1) for every output, one channel per thread.
+template <typename T, int kTaps, int kVec, int kActVec>
 __global__ void __launch_bounds__(kThreads)
 causal_conv_kernel(ConvArgs a) {
   const int seq = blockIdx.z, first = blockIdx.y * kTile;
@@ -40,17 +41,23 @@ causal_conv_kernel(ConvArgs a) {
   if (first >= n) return;
   const int count = min(kTile, n - first);
   if (static_cast<int>(blockIdx.x) >= a.conv_blocks) {
-    const int c = (blockIdx.x - a.conv_blocks) * kThreads + threadIdx.x;
+    const int c = ((blockIdx.x - a.conv_blocks) * kThreads + threadIdx.x) * kActVec;
     if (c >= a.act_width) return;
     const T* src = static_cast<const T*>(a.act_in) + (row0 + first) * a.in_stride + c;
     T* dst = static_cast<T*>(a.act_out) + (row0 + first) * a.act_out_stride + c;
-#pragma unroll 4
-    for (int i = 0; i < count; ++i)
-      dst[i * a.act_out_stride] = Elem<T>::from_float(activate(Elem<T>::to_float(src[i * a.in_stride]), a.act));
+#pragma unroll 2
+    for (int i = 0; i < count; ++i) {
+      float v[kActVec];
+      load_floats<T, kActVec>(src + i * a.in_stride, v);
+#pragma unroll
+      for (int e = 0; e < kActVec; ++e) v[e] = activate(v[e], a.act);
+      store_floats<T, kActVec>(dst + i * a.act_out_stride, v);
+    }
     return;
   }
-  const int c = blockIdx.x * kThreads + threadIdx.x;
+  const int c = (blockIdx.x * kThreads + threadIdx.x) * kVec;
   if (c >= a.channels) return;
+  struct alignas(sizeof(T) * kVec) Vec { T e[kVec]; };
   const int taps = kTaps > 0 ? kTaps : a.taps;
   const T* in = static_cast<const T*>(a.in) + static_cast<int64_t>(row0) * a.in_stride + c;   // in[i * stride]: token i of the portion
   T* out = static_cast<T*>(a.out) + static_cast<int64_t>(row0) * a.out_stride + c;
@@ -58,51 +65,83 @@ causal_conv_kernel(ConvArgs a) {
   const int64_t slot = a.slot_of[seq];
   const bool slot_ok = slot >= 0 && slot < a.slots;
   T* state = static_cast<T*>(a.state) + slot * (taps - 1) * static_cast<int64_t>(a.channels) + c;
-  auto old_input = [&](int k) {   // k-th of the taps - 1 inputs before the portion, oldest first
-    return resumed && slot_ok ? state[static_cast<int64_t>(k) * a.channels] : Elem<T>::from_float(0.0f);
+  auto input = [&](int i) {   // token i of the portion; negative: one of the taps - 1 inputs before it
+    if (i >= 0) return *reinterpret_cast<const Vec*>(in + i * a.in_stride);
+    if (resumed && slot_ok) return *reinterpret_cast<const Vec*>(state + static_cast<int64_t>(i + taps - 1) * a.channels);
+    Vec zero;
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) zero.e[e] = Elem<T>::from_float(0.0f);
+    return zero;
   };
-  auto input = [&](int i) { return i >= 0 ? in[i * a.in_stride] : old_input(i + taps - 1); };
-  const float bias = a.bias[c];
   const float* w = a.weight + static_cast<int64_t>(c) * taps;
   if constexpr (kTaps > 0) {
-    float wr[kTaps], window[kTaps];
+    float wr[kVec][kTaps], bias[kVec], window[kTaps][kVec];
+    load_floats<float, kVec>(a.bias + c, bias);
 #pragma unroll
-    for (int j = 0; j < kTaps; ++j) wr[j] = w[j];
+    for (int e = 0; e < kVec; ++e)
 #pragma unroll
-    for (int j = 0; j + 1 < kTaps; ++j) window[j + 1] = Elem<T>::to_float(input(first - kTaps + 1 + j));
-    T next[8];
-    for (int base = 0; base < count; base += 8) {
+      for (int j = 0; j < kTaps; ++j) wr[e][j] = w[e * kTaps + j];
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
-        if (base + i < count) next[i] = in[(first + base + i) * a.in_stride];
+    for (int j = 0; j + 1 < kTaps; ++j) {
+      const Vec x = input(first - kTaps + 1 + j);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int e = 0; e < kVec; ++e) window[j + 1][e] = Elem<T>::to_float(x.e[e]);
+    }
+    constexpr int kAhead = 8;
+    Vec next[kAhead];
+    for (int base = 0; base < count; base += kAhead) {
+#pragma unroll
+      for (int i = 0; i < kAhead; ++i)
+        if (base + i < count) next[i] = *reinterpret_cast<const Vec*>(in + (first + base + i) * a.in_stride);
+#pragma unroll
+      for (int i = 0; i < kAhead; ++i) {
         if (base + i < count) {
+          float sum[kVec];
 #pragma unroll
-          for (int j = 0; j + 1 < kTaps; ++j) window[j] = window[j + 1];
-          window[kTaps - 1] = Elem<T>::to_float(next[i]);
-          float sum = 0.0f;
+          for (int e = 0; e < kVec; ++e) {
 #pragma unroll
-          for (int j = 0; j < kTaps; ++j) sum = fmaf(wr[j], window[j], sum);
-          out[(first + base + i) * a.out_stride] = Elem<T>::from_float(silu(sum + bias));
+            for (int j = 0; j + 1 < kTaps; ++j) window[j][e] = window[j + 1][e];
+            window[kTaps - 1][e] = Elem<T>::to_float(next[i].e[e]);
+            sum[e] = 0.0f;
+#pragma unroll
+            for (int j = 0; j < kTaps; ++j) sum[e] = fmaf(wr[e][j], window[j][e], sum[e]);
+            sum[e] = silu(sum[e] + bias[e]);
+          }
+          store_floats<T, kVec>(out + (first + base + i) * a.out_stride, sum);
         }
       }
     }
   } else {
+    static_assert(kTaps > 0 || kVec == 1, "the re-reading form handles one channel per thread");
     for (int i = 0; i < count; ++i) {
       float sum = 0.0f;
-      for (int j = 0; j < taps; ++j) sum = fmaf(w[j], Elem<T>::to_float(input(first + i - taps + 1 + j)), sum);
-      out[(first + i) * a.out_stride] = Elem<T>::from_float(silu(sum + bias));
+      for (int j = 0; j < taps; ++j) sum = fmaf(w[j], Elem<T>::to_float(input(first + i - taps + 1 + j).e[0]), sum);
+      out[(first + i) * a.out_stride] = Elem<T>::from_float(silu(sum + a.bias[c]));
     }
   }
   if (first == 0 && slot_ok)   // ascending: entry k is written after every entry it is shifted from has been read
-    for (int k = 0; k + 1 < taps; ++k) state[static_cast<int64_t>(k) * a.channels] = input(n + k - taps + 1);
+    for (int k = 0; k + 1 < taps; ++k)
+      *reinterpret_cast<Vec*>(state + static_cast<int64_t>(k) * a.channels) = input(n + k - taps + 1);
 }
 
 template <typename T>
-void launch(const ConvArgs& a, dim3 grid, cudaStream_t s) {
-  if (a.taps == 4) causal_conv_kernel<T, 4><<<grid, kThreads, 0, s>>>(a);
-  else causal_conv_kernel<T, 0><<<grid, kThreads, 0, s>>>(a);
+int launch(ConvArgs a, int sequences, int max_tokens, cudaStream_t s) {
+  constexpr int kVec = 4, kWide = static_cast<int>(16 / sizeof(T));
+  auto whole = [](int64_t n, int v) { return n % v == 0; };
+  auto aligned = [](const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
+  const bool vectors = a.taps == 4 && whole(a.channels, kVec) && whole(a.in_stride, kVec) && whole(a.out_stride, kVec) &&
+                       aligned(a.in, kVec * sizeof(T)) && aligned(a.out, kVec * sizeof(T)) && aligned(a.state, kVec * sizeof(T)) && aligned16(a.bias);
+  const bool wide = a.act_width > 0 && whole(a.act_width, kWide) && whole(a.in_stride, kWide) && whole(a.act_out_stride, kWide) &&
+                    aligned16(a.act_in) && aligned16(a.act_out);
+  const int vec = vectors ? kVec : 1, act_vec = wide ? kWide : 1;
+  a.conv_blocks = (a.channels + kThreads * vec - 1) / (kThreads * vec);
+  const dim3 grid(static_cast<unsigned>(a.conv_blocks + (a.act_width + kThreads * act_vec - 1) / (kThreads * act_vec)),
+                  static_cast<unsigned>((max_tokens + kTile - 1) / kTile), static_cast<unsigned>(sequences));
+  if (vectors && wide) causal_conv_kernel<T, 4, kVec, kWide><<<grid, kThreads, 0, s>>>(a);
+  else if (vectors) causal_conv_kernel<T, 4, kVec, 1><<<grid, kThreads, 0, s>>>(a);
+  else if (a.taps == 4) wide ? causal_conv_kernel<T, 4, 1, kWide><<<grid, kThreads, 0, s>>>(a) : causal_conv_kernel<T, 4, 1, 1><<<grid, kThreads, 0, s>>>(a);
+  else wide ? causal_conv_kernel<T, 0, 1, kWide><<<grid, kThreads, 0, s>>>(a) : causal_conv_kernel<T, 0, 1, 1><<<grid, kThreads, 0, s>>>(a);
+  return launch_status("causal_conv_kernel");
 }
 
 }  // namespace
@@ -129,9 +168,5 @@ extern "C" RLT_API int rlt_causal_conv(const void* in, int64_t in_stride, const 
   a.state = state; a.slots = slots; a.channels = channels; a.taps = taps;
   a.cu = cu_seqlens; a.starts = starts; a.slot_of = slot_of;
   a.act_in = act_in; a.act_out = act_out; a.act_out_stride = act_out_stride; a.act_width = act_width; a.act = act;
-  a.conv_blocks = (channels + kThreads - 1) / kThreads;
-  const dim3 grid(static_cast<unsigned>(a.conv_blocks + (act_width + kThreads - 1) / kThreads),
-                  static_cast<unsigned>((max_tokens + kTile - 1) / kTile), static_cast<unsigned>(sequences));
-  RLT_DISPATCH_DTYPE(dtype, T, launch<T>(a, grid, static_cast<cudaStream_t>(stream)));
-  return launch_status("causal_conv_kernel");
+  RLT_DISPATCH_DTYPE(dtype, T, return launch<T>(a, sequences, max_tokens, static_cast<cudaStream_t>(stream)));
 }

@@ -35,7 +35,7 @@ __global__ void __launch_bounds__(kThreads)
 residual_norm_kernel(float* residual, const T* __restrict__ delta, const int64_t* __restrict__ tokens,
                      const T* __restrict__ embed, int64_t vocab, const int64_t* __restrict__ row_index, int store_residual,
                      const float* __restrict__ weight, float weight_offset, T* __restrict__ out, int width, float eps) {
-  extern __shared__ float row_values[];
+  extern __shared__ __align__(16) float row_values[];
   __shared__ float scratch[kThreads / 32];
   const int64_t source = row_index != nullptr ? row_index[blockIdx.x] : static_cast<int64_t>(blockIdx.x);
   float* res = residual + source * width;
@@ -119,26 +119,38 @@ block_epilogue_kernel(EpilogueArgs a) {
   }
 }
 
-template <typename T>
+template <typename T, int kVec>
 __global__ void __launch_bounds__(kThreads)
 gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z, int64_t z_stride,
                   const float* __restrict__ weight, T* __restrict__ out, int64_t out_stride, int part, float eps) {
-  extern __shared__ float row_values[];
+  extern __shared__ __align__(16) float row_values[];
   __shared__ float scratch[kThreads / 32];
   const int64_t row = blockIdx.x;
   const int first = blockIdx.y * part;
   const T* yr = y + row * y_stride + first;
   const T* zr = z + row * z_stride + first;
   float ss = 0.0f;
-  for (int i = threadIdx.x; i < part; i += kThreads) {
-    const float v = Elem<T>::to_float(yr[i]) * silu(Elem<T>::to_float(zr[i]));
-    row_values[i] = v;
-    ss = fmaf(v, v, ss);
+  for (int i = threadIdx.x * kVec; i < part; i += kThreads * kVec) {
+    float v[kVec], g[kVec];
+    load_floats<T, kVec>(yr + i, v);
+    load_floats<T, kVec>(zr + i, g);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) {
+      v[e] *= silu(g[e]);
+      ss = fmaf(v[e], v[e], ss);
+    }
+    store_floats<float, kVec>(row_values + i, v);
   }
   const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(part) + eps);
   T* dst = out + row * out_stride + first;
-  for (int i = threadIdx.x; i < part; i += kThreads)
-    dst[i] = Elem<T>::from_float(row_values[i] * r * weight[first + i]);
+  for (int i = threadIdx.x * kVec; i < part; i += kThreads * kVec) {   // each thread reads back what it staged itself
+    float v[kVec], w[kVec];
+    load_floats<float, kVec>(row_values + i, v);
+    load_floats<float, kVec>(weight + first + i, w);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) v[e] *= r * w[e];
+    store_floats<T, kVec>(dst + i, v);
+  }
 }
 
 constexpr size_t kMaxRowBytes = 48u * 1024u;   // a staged row of fp32 values
@@ -233,8 +245,14 @@ extern "C" RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const voi
     return RLT_ERR_UNSUPPORTED;
   }
   const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>(parts));
-  RLT_DISPATCH_DTYPE(dtype, T, (gated_norm_kernel<T><<<grid, kThreads, smem, static_cast<cudaStream_t>(stream)>>>(
-                                   static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride, weight,
-                                   static_cast<T*>(out), out_stride, part, eps)));
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const size_t bytes = 4 * dtype_size(dtype);
+  auto aligned = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
+  const bool wide = part % 4 == 0 && y_stride % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 && aligned(y) && aligned(z) && aligned(out) && aligned16(weight);
+#define RLT_LAUNCH(T, V)                                                                                                  \
+  gated_norm_kernel<T, V><<<grid, kThreads, smem, s>>>(static_cast<const T*>(y), y_stride, static_cast<const T*>(z),       \
+      z_stride, weight, static_cast<T*>(out), out_stride, part, eps)
+  RLT_DISPATCH_DTYPE(dtype, T, { if (wide) RLT_LAUNCH(T, 4); else RLT_LAUNCH(T, 1); });
+#undef RLT_LAUNCH
   return launch_status("gated_norm_kernel");
 }

@@ -25,11 +25,12 @@ constexpr int kStepThreads = 256;
 
 // ---- one token after the other ---------------------------------------------------------------
 // Threads: lanes over the head's P columns (kVec each), slices over the N rows; row r of a thread is
-// slice + r * slices.
+// slice + r * slices.  Decoding is bound by the state's bytes: its loads are the first thing issued, and registers are
+// held to four CTAs per SM so that enough of them are in flight.
 template <typename T, int kVec, int kRows>
-__global__ void __launch_bounds__(kStepThreads)
+__global__ void __launch_bounds__(kStepThreads, kRows * kVec <= 32 ? 4 : (kRows * kVec <= 64 ? 2 : 1))
 scan_step_kernel(ScanArgs a, int tile_p, int lanes) {
-  extern __shared__ float partial[];             // [2][slices][tile_p]
+  extern __shared__ float partial[];             // [2][slices][tile_p], then [2][B | C][n]
   const int head = blockIdx.x, seq = blockIdx.y, p0 = blockIdx.z * tile_p;
   const int row0 = a.cu[seq], count = a.cu[seq + 1] - row0;
   if (count <= 0) return;
@@ -53,28 +54,37 @@ scan_step_kernel(ScanArgs a, int tile_p, int lanes) {
       for (int e = 0; e < kVec; ++e) s[r][e] = 0.0f;
     }
   }
-  const float rate = -expf(a.a_log[head]), dt_bias = a.dt_bias[head], skip = a.d[head];
   const T* xp = static_cast<const T*>(a.x) + static_cast<int64_t>(head) * a.p + p;
   const T* bp = static_cast<const T*>(a.b) + static_cast<int64_t>(group) * a.n;
   const T* cp = static_cast<const T*>(a.c) + static_cast<int64_t>(group) * a.n;
   const T* dtp = static_cast<const T*>(a.dt) + head;
   T* yp = static_cast<T*>(a.y) + static_cast<int64_t>(head) * a.p + p0;
+  float* staged = partial + 2 * slices * tile_p;
+  auto stage = [&](int t) {                       // B and C of a token as fp32
+    float* dst = staged + (t & 1) * 2 * a.n;
+    for (int i = threadIdx.x; i < 2 * a.n; i += kStepThreads)
+      dst[i] = Elem<T>::to_float(i < a.n ? bp[(row0 + t) * a.xbc_stride + i] : cp[(row0 + t) * a.xbc_stride + i - a.n]);
+  };
+  stage(0);
+  const float rate = -expf(a.a_log[head]), dt_bias = a.dt_bias[head], skip = a.d[head];
+  __syncthreads();
   for (int t = 0; t < count; ++t) {
     const int64_t row = row0 + t;
     const float dt = softplus(Elem<T>::to_float(dtp[row * a.dt_stride]) + dt_bias);
     const float decay = expf(rate * dt);
-    float x[kVec], y[kVec];
-#pragma unroll
-    for (int e = 0; e < kVec; ++e) { x[e] = 0.0f; y[e] = 0.0f; }
+    const float* bt = staged + (t & 1) * 2 * a.n;
+    const float* ct = bt + a.n;
+    float* buffer = partial + (t & 1) * slices * tile_p;   // two buffers each: one barrier per token
     if (active) {
+      float x[kVec], y[kVec];
       load_floats<T, kVec>(xp + row * a.xbc_stride, x);
 #pragma unroll
-      for (int e = 0; e < kVec; ++e) x[e] *= dt;
+      for (int e = 0; e < kVec; ++e) { x[e] *= dt; y[e] = 0.0f; }
 #pragma unroll
       for (int r = 0; r < kRows; ++r) {
         const int n = slice + r * slices;
         if (n < a.n) {
-          const float bn = Elem<T>::to_float(bp[row * a.xbc_stride + n]), cn = Elem<T>::to_float(cp[row * a.xbc_stride + n]);
+          const float bn = bt[n], cn = ct[n];
 #pragma unroll
           for (int e = 0; e < kVec; ++e) {
             s[r][e] = fmaf(decay, s[r][e], bn * x[e]);
@@ -82,12 +92,10 @@ scan_step_kernel(ScanArgs a, int tile_p, int lanes) {
           }
         }
       }
-    }
-    float* buffer = partial + (t & 1) * slices * tile_p;   // two buffers: one barrier per token
-    if (active) {
 #pragma unroll
       for (int e = 0; e < kVec; ++e) buffer[slice * tile_p + lane * kVec + e] = y[e];
     }
+    if (t + 1 < count) stage(t + 1);
     __syncthreads();
     for (int i = threadIdx.x; i < width; i += kStepThreads) {
       float sum = 0.0f;
@@ -108,7 +116,7 @@ template <typename T, int kVec>
 int launch_step_rows(const ScanArgs& a, int sequences, int tile_p, int lanes, cudaStream_t stream) {
   const int slices = kStepThreads / lanes, rows = (a.n + slices - 1) / slices;
   const dim3 grid(static_cast<unsigned>(a.heads), static_cast<unsigned>(sequences), static_cast<unsigned>((a.p + tile_p - 1) / tile_p));
-  const size_t smem = 2 * sizeof(float) * slices * tile_p;
+  const size_t smem = 2 * sizeof(float) * (static_cast<size_t>(slices) * tile_p + 2 * a.n);
 #define RLT_STEP(R) scan_step_kernel<T, kVec, R><<<grid, kStepThreads, smem, stream>>>(a, tile_p, lanes)
   if (rows <= 2) RLT_STEP(2);
   else if (rows <= 4) RLT_STEP(4);
