@@ -178,6 +178,18 @@ def test_block_epilogue(dtype, kv_heads, dim, vdim, ff, kind):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("kind", ["gelu", "gelu_tanh"])
+def test_activations_over_their_whole_range(dtype, kind):
+    x = torch.cat([torch.linspace(-40, 40, 4001), torch.linspace(-1e-3, 1e-3, 95)]).to(dtype).view(8, 512)
+    out = torch.empty(8, 512, dtype=dtype, device="cuda")
+    rlt.block_epilogue(x.cuda(), None, act=(0, 512, kind, out, 0))
+    want = (plain.gelu if kind == "gelu" else plain.gelu_tanh)(x.double())
+    error = (out.double().cpu() - want).abs()
+    relative = 2.0 ** -8 if dtype == torch.bfloat16 else 4e-6
+    assert bool((error <= relative * want.abs() + 2e-6).all())
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("width,parts", [(64, 1), (96, 4), (30, 3), (512, 8)])
 def test_gated_norm(dtype, width, parts):
     g = torch.Generator().manual_seed(7)

@@ -34,7 +34,7 @@ struct ConvArgs {
 // A thread owns kVec neighbouring channels (or kActVec activation columns) for a tile of tokens.
 // kTaps 0: any number of taps, inputs re-read (from L1) for every output, one channel per thread.
 template <typename T, int kTaps, int kVec, int kActVec>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, 8)
 causal_conv_kernel(ConvArgs a) {
   const int seq = blockIdx.z, first = blockIdx.y * kTile;
   const int row0 = a.cu[seq], n = a.cu[seq + 1] - row0;
@@ -50,7 +50,7 @@ causal_conv_kernel(ConvArgs a) {
       float v[kActVec];
       load_floats<T, kActVec>(src + i * a.in_stride, v);
 #pragma unroll
-      for (int e = 0; e < kActVec; ++e) v[e] = activate(v[e], a.act);
+      for (int e = 0; e < kActVec; ++e) v[e] = activate<T>(v[e], a.act);
       store_floats<T, kActVec>(dst + i * a.act_out_stride, v);
     }
     return;
@@ -87,7 +87,7 @@ causal_conv_kernel(ConvArgs a) {
 #pragma unroll
       for (int e = 0; e < kVec; ++e) window[j + 1][e] = Elem<T>::to_float(x.e[e]);
     }
-    constexpr int kAhead = 8;
+    constexpr int kAhead = 4;
     Vec next[kAhead];
     for (int base = 0; base < count; base += kAhead) {
 #pragma unroll

@@ -10,10 +10,22 @@ namespace rlt {
 enum Activation { kActGeluErf = 1, kActGeluTanh = 2 };
 inline bool act_valid(int act) { return act == kActGeluErf || act == kActGeluTanh; }
 
-__device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }   // a few ulp; 0 far on the left
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
+// erf to 1.5e-7: the rational approximation 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions.
+__device__ __forceinline__ float erf_approx(float x) {
+  const float z = fabsf(x), t = __fdividef(1.0f, fmaf(0.3275911f, z, 1.0f));
+  const float p = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+  return copysignf(fmaf(-p, __expf(-z * z), 1.0f), x);
+}
+
+// The activation of a value stored as T: 16-bit results do not show erf's last digits, 32-bit ones take erff.
+template <typename T>
 __device__ __forceinline__ float activate(float x, int act) {
-  if (act == kActGeluErf) return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
+  if (act == kActGeluErf) {
+    const float u = x * 0.70710678118654752f;
+    return 0.5f * x * (1.0f + (sizeof(T) == 4 ? erff(u) : erf_approx(u)));
+  }
   return 0.5f * x * (1.0f + tanhf(0.79788456080286536f * (x + 0.044715f * x * x * x)));
 }
 

@@ -114,7 +114,7 @@ block_epilogue_kernel(EpilogueArgs a) {
     float v[kVec];
     load_floats<T, kVec>(proj + a.act_col + c, v);
 #pragma unroll
-    for (int e = 0; e < kVec; ++e) v[e] = activate(v[e], a.act);
+    for (int e = 0; e < kVec; ++e) v[e] = activate<T>(v[e], a.act);
     store_floats<T, kVec>(static_cast<T*>(a.out) + row * a.out_stride + a.out_col + c, v);
   }
 }

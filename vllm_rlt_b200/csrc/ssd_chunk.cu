@@ -13,9 +13,9 @@ using T = __nv_bfloat16;
 
 // hi + lo of two fp32 values as packed 16-bit pairs: lo holds what rounding to hi left over.
 __device__ __forceinline__ void split2(float a, float b, uint32_t* hi, uint32_t* lo) {
-  const T ha = Elem<T>::from_float(a), hb = Elem<T>::from_float(b);
-  *hi = pack2<true>(a, b);
-  *lo = pack2<true>(a - Elem<T>::to_float(ha), b - Elem<T>::to_float(hb));
+  const uint32_t h = pack2<true>(a, b);
+  *hi = h;
+  *lo = pack2<true>(a - __uint_as_float(h << 16), b - __uint_as_float(h & 0xffff0000u));
 }
 
 // Shared memory of one CTA.  Rows are padded by 8 elements: eight consecutive rows then start in eight
