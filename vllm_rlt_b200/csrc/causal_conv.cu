@@ -124,6 +124,57 @@ causal_conv_kernel(ConvArgs a) {
       *reinterpret_cast<Vec*>(state + static_cast<int64_t>(k) * a.channels) = input(n + k - taps + 1);
 }
 
+// Decoding: one token per sequence, four taps, kVec channels per thread.  Nothing to tile or to keep in a window: all loads
+// of a thread are issued together, and few registers leave room for every CTA of a batch at once.
+template <typename T, int kVec>
+__global__ void __launch_bounds__(kThreads, 12)
+conv_step_kernel(ConvArgs a) {
+  struct alignas(sizeof(T) * kVec) Vec { T e[kVec]; };
+  const int seq = blockIdx.z;
+  const int row = a.cu[seq], next = a.cu[seq + 1], start = a.starts[seq];
+  const int64_t slot = a.slot_of[seq];
+  if (row >= next) return;
+  if (static_cast<int>(blockIdx.x) >= a.conv_blocks) {
+    const int c = ((blockIdx.x - a.conv_blocks) * kThreads + threadIdx.x) * kVec;
+    if (c >= a.act_width) return;
+    float v[kVec];
+    load_floats<T, kVec>(static_cast<const T*>(a.act_in) + row * a.in_stride + c, v);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) v[e] = activate<T>(v[e], a.act);
+    store_floats<T, kVec>(static_cast<T*>(a.act_out) + row * a.act_out_stride + c, v);
+    return;
+  }
+  const int c = (blockIdx.x * kThreads + threadIdx.x) * kVec;
+  if (c >= a.channels) return;
+  const bool slot_ok = slot >= 0 && slot < a.slots;
+  T* state = static_cast<T*>(a.state) + slot * 3 * a.channels + c;
+  Vec x[4];
+  x[3] = *reinterpret_cast<const Vec*>(static_cast<const T*>(a.in) + row * a.in_stride + c);
+#pragma unroll
+  for (int j = 0; j < 3; ++j) {
+    if (start > 0 && slot_ok) {
+      x[j] = *reinterpret_cast<const Vec*>(state + j * a.channels);
+    } else {
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) x[j].e[e] = Elem<T>::from_float(0.0f);
+    }
+  }
+  float y[kVec], bias[kVec];
+  load_floats<float, kVec>(a.bias + c, bias);
+#pragma unroll
+  for (int e = 0; e < kVec; ++e) {
+    float w[4], sum = 0.0f;
+    load_floats<float, 4>(a.weight + static_cast<int64_t>(c + e) * 4, w);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) sum = fmaf(w[j], Elem<T>::to_float(x[j].e[e]), sum);
+    y[e] = silu(sum + bias[e]);
+  }
+  store_floats<T, kVec>(static_cast<T*>(a.out) + row * a.out_stride + c, y);
+  if (!slot_ok) return;
+#pragma unroll
+  for (int j = 0; j < 3; ++j) *reinterpret_cast<Vec*>(state + j * a.channels) = x[j + 1];
+}
+
 template <typename T>
 int launch(ConvArgs a, int sequences, int max_tokens, cudaStream_t s) {
   constexpr int kVec = 4, kWide = static_cast<int>(16 / sizeof(T));
@@ -133,6 +184,12 @@ int launch(ConvArgs a, int sequences, int max_tokens, cudaStream_t s) {
                        aligned(a.in, kVec * sizeof(T)) && aligned(a.out, kVec * sizeof(T)) && aligned(a.state, kVec * sizeof(T)) && aligned16(a.bias);
   const bool wide = a.act_width > 0 && whole(a.act_width, kWide) && whole(a.in_stride, kWide) && whole(a.act_out_stride, kWide) &&
                     aligned16(a.act_in) && aligned16(a.act_out);
+  if (max_tokens == 1 && vectors && (a.act_width == 0 || wide) && aligned16(a.weight)) {
+    a.conv_blocks = (a.channels + kThreads * kVec - 1) / (kThreads * kVec);
+    const dim3 grid(static_cast<unsigned>(a.conv_blocks + (a.act_width + kThreads * kVec - 1) / (kThreads * kVec)), 1, static_cast<unsigned>(sequences));
+    conv_step_kernel<T, kVec><<<grid, kThreads, 0, s>>>(a);
+    return launch_status("conv_step_kernel");
+  }
   const int vec = vectors ? kVec : 1, act_vec = wide ? kWide : 1;
   a.conv_blocks = (a.channels + kThreads * vec - 1) / (kThreads * vec);
   const dim3 grid(static_cast<unsigned>(a.conv_blocks + (a.act_width + kThreads * act_vec - 1) / (kThreads * act_vec)),
