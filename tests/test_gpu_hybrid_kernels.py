@@ -233,7 +233,8 @@ def test_convolution_in_portions(dtype, channels, taps, cuts):
     assert bool((state[1] == 1e4).all())
 
 
-SCANS = [(4, 16, 20, 2), (3, 10, 12, 3), (2, 64, 128, 1), (2, 32, 48, 2), (2, 80, 144, 1), (1, 7, 9, 1), (2, 64, 256, 2), (4, 24, 64, 4)]
+SCANS = [(4, 16, 20, 2), (3, 10, 12, 3), (2, 64, 128, 1), (2, 32, 48, 2), (2, 80, 144, 1), (1, 7, 9, 1), (2, 64, 256, 2), (4, 24, 64, 4),
+         (4, 64, 96, 2), (2, 48, 72, 1), (3, 128, 128, 3)]
 
 
 def scan_inputs(total, heads, p, size, groups, dtype, seed):
@@ -262,7 +263,7 @@ def run_scan(inputs, cuts, heads, p, size, groups, dtype, state, slots, portions
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,p,size,groups", SCANS)
-@pytest.mark.parametrize("cuts", [[1] * 6, [2, 16, 17, 64, 3, 65], [167]])
+@pytest.mark.parametrize("cuts", [[1] * 6, [2, 16, 17, 64, 3, 65], [167], [129, 127, 20]])
 def test_scan_in_portions(dtype, heads, p, size, groups, cuts):
     total = sum(cuts)
     inputs = scan_inputs(2 * total, heads, p, size, groups, dtype, heads * p + size)
@@ -280,9 +281,10 @@ def test_scan_in_portions(dtype, heads, p, size, groups, cuts):
     assert bool((state[0] == 1e3).all()) and bool((state[2] == 1e3).all())
 
 
-def test_long_prompts_run_in_segments():
+@pytest.mark.parametrize("p,size", [(32, 64), (64, 128), (72, 104)])
+def test_long_prompts_run_in_segments(p, size):
     """One long sequence beside a short one: the long one is cut into segments that start from folded states."""
-    heads, p, size, groups, lengths = 2, 32, 64, 1, [1500, 300]
+    heads, groups, lengths = 2, 1, [1500, 300]
     inputs = scan_inputs(sum(lengths), heads, p, size, groups, torch.bfloat16, 5)
     x, b, c, dt, dt_bias, a_log, d = inputs
     state = torch.randn(3, heads, size, p, device="cuda")

@@ -6,7 +6,8 @@
 //
 // step kernel     one CTA per (sequence, head): the state in registers, one token after the other.  Decoding
 //                 (bytes: the state, read and written once), portions of a few tokens, and 32-bit models.
-// chunk kernels   portions of many tokens in bf16 models (ssd_chunk.cu): 64 tokens at a time on tensor cores.  With
+// chunk kernels   portions of many tokens in bf16 models: 128 tokens at a time with tcgen05 (ssd_chunk_sm100.cu: states of
+//                 65 .. 128 rows) or 64 with mma.sync (ssd_chunk.cu: every other shape).  With
 //                 L_i = sum of log-decays up to token i of the chunk, S the state before it,
 //                   Y = exp(L) o (C S) + M X,      M_ij = (C_i . B_j) exp(L_i - L_j) dt_j  (j <= i)
 //                   S' = exp(L_end) S + B^T W,     W_j = exp(L_end - L_j) dt_j X_j
@@ -183,6 +184,8 @@ extern "C" RLT_API int rlt_ssd_scan(const void* x, const void* b, const void* c,
   a.dt_bias = dt_bias; a.a_log = a_log; a.d = d; a.y = y; a.y_stride = y_stride; a.state = state; a.slots = slots;
   a.cu = cu_seqlens; a.starts = starts; a.slot_of = slot_of;
   a.heads = heads; a.groups = groups; a.n = state_size; a.p = head_dim;
+  // workspace: an error word (256 bytes), then the segments'
+  a.error = (reinterpret_cast<uintptr_t>(workspace) & 15u) == 0 && workspace_bytes >= 256 ? static_cast<unsigned*>(workspace) : nullptr;
   a.segments = nullptr; a.segment_decay = nullptr; a.segment_tokens = 1 << 30; a.segment_count = 1;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (!chunked(max_tokens, state_size, dtype)) {
@@ -201,9 +204,10 @@ extern "C" RLT_API int rlt_ssd_scan(const void* x, const void* b, const void* c,
       return RLT_ERR_WORKSPACE;
     }
     a.segment_count = count;
-    a.segment_tokens = ((max_tokens + count - 1) / count + 63) / 64 * 64;
-    a.segments = static_cast<float*>(workspace);
+    a.segment_tokens = ((max_tokens + count - 1) / count + 127) / 128 * 128;
+    a.segments = reinterpret_cast<float*>(static_cast<unsigned char*>(workspace) + 256);
     a.segment_decay = a.segments + static_cast<size_t>(sequences) * (kMaxSegments + 1) * heads * state_size * head_dim;
   }
+  if (scan_umma_supported(a)) return launch_scan_umma(a, sequences, s);
   return launch_scan_chunks(a, sequences, s);
 }

@@ -18,9 +18,14 @@ struct ScanArgs {
   int heads, groups, n, p;
   float* segments; float* segment_decay;         // [sequences][kMaxSegments + 1][heads][N][P], [sequences][kMaxSegments][heads]
   int segment_tokens, segment_count;
+  unsigned* error;                               // set when a bounded wait of the tcgen05 kernel gave up (workspace)
 };
 
 // ssd_chunk.cu: 64 tokens at a time on tensor cores, bf16, state sizes up to 256.
 int launch_scan_chunks(const ScanArgs& a, int sequences, cudaStream_t stream);
+
+// ssd_chunk_sm100.cu: 128 tokens at a time with tcgen05, for states of 65 .. 128 rows and aligned operands.
+bool scan_umma_supported(const ScanArgs& a);
+int launch_scan_umma(const ScanArgs& a, int sequences, cudaStream_t stream);
 
 }  // namespace rlt
