@@ -1051,7 +1051,18 @@ def hybrid_kernel_rows(size, steps):
         plain = lambda i: (lambda: kernels.prefill(q_plain[i % sets], pools[i % sets][0], pools[i % sets][1], tables, lengths, cu, new))
         add("scored attention", phase, None, scored, kv_bytes + qo_bytes, flops, copies=4)
         add("attention of the looped model", phase, "scored attention", plain, kv_bytes + qo_bytes, flops, copies=4)
-        del pools, q_plain
+        del q_plain
+
+        # the same bytes and flops in 64-wide heads: the shape-general tensor-core kernels
+        narrow = [pool.view(2, seqs * pages, BLOCK, 2 * kv_heads, HEAD_DIM // 2) for pool in pools]
+
+        def scored_narrow(i):
+            q = q_wide[i % sets][:, :heads * HEAD_DIM].view(rows, 2 * heads, HEAD_DIM // 2)
+            out = out_wide[:, :heads * HEAD_DIM].view(rows, 2 * heads, HEAD_DIM // 2)
+            return lambda: kernels.scored(q, out, narrow[i % sets][0], narrow[i % sets][1], tables, lengths, cu, new, terms)
+
+        add("scored attention, 64-wide heads", phase, None, scored_narrow, kv_bytes + qo_bytes, flops, copies=4)
+        del pools, narrow
 
         # the norm that opens a layer: 32-bit residual read and written, 16-bit contribution read, 16-bit row written
         copies = max(2, min(48, int(400e6 // (rows * width * 12)) + 1))
