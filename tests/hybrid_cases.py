@@ -42,6 +42,7 @@ CONFIGS = {
                         attention_layer(5, 5, 20, 12, kv_from=1)], vocab=83, width=52),
     "wide": make_config([attention_layer(4, 2, 128, 128, temp=(0.3, 64)),
                          mamba_layer(4, 64, 128, 2, norm_groups=2),
+                         attention_layer(6, 3, 64, 64, temp=(0.2, 40), ff=None),
                          attention_layer(4, 2, 128, 128, kv_from=0, temp=(0.2, 33)),
                          mamba_layer(2, 80, 144, 1, conv=5)], vocab=211, width=128),
 }

@@ -73,12 +73,12 @@ def run_scored(q, key, value, tables, contexts, portions, terms, heads, dim, vdi
     return wide_out[:, :heads * vdim].reshape(rows, heads, vdim)
 
 
-SHAPES = [(6, 2, 24, 40), (4, 4, 64, 64), (8, 2, 128, 128), (3, 1, 128, 128), (4, 1, 96, 160), (5, 5, 20, 12), (2, 2, 256, 64), (16, 1, 16, 8)]
+SHAPES = [(6, 2, 24, 40), (4, 4, 64, 64), (6, 2, 64, 64), (8, 2, 128, 128), (3, 1, 128, 128), (4, 1, 96, 160), (5, 5, 20, 12), (2, 2, 256, 64), (16, 1, 16, 8)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim", SHAPES)
-@pytest.mark.parametrize("portions,contexts", [([1, 1, 1], [1, 17, 530]), ([2, 16, 5], [2, 33, 300]), ([40, 70, 1], [40, 201, 64]), ([150], [150])])
+@pytest.mark.parametrize("portions,contexts", [([1, 1, 1], [1, 17, 530]), ([2, 16, 5], [2, 33, 300]), ([40, 70, 1], [40, 201, 64]), ([150], [150]), ([300, 17], [500, 17])])
 def test_scored_attention(dtype, heads, kv_heads, dim, vdim, portions, contexts):
     terms = rlt.ScoreTerms(0.8 * dim ** -0.5, 0.5, 37, True)
     q, k, v, key, value, tables = paged_case(portions, contexts, heads, kv_heads, dim, vdim, dtype, 3)
@@ -90,7 +90,7 @@ def test_scored_attention(dtype, heads, kv_heads, dim, vdim, portions, contexts)
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("coef,every,bias", [(0.0, 1, False), (0.0, 1, True), (0.9, 1, False), (0.25, 64, True)])
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 128, 128), (4, 2, 32, 48)])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 128, 128), (4, 2, 64, 64), (4, 2, 32, 48)])
 def test_every_score_term_alone(dtype, coef, every, bias, heads, kv_heads, dim, vdim):
     portions, contexts = [1, 90], [200, 130]
     terms = rlt.ScoreTerms(dim ** -0.5, coef, every, bias)
@@ -102,7 +102,7 @@ def test_every_score_term_alone(dtype, coef, every, bias, heads, kv_heads, dim, 
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 128, 128), (4, 2, 48, 64)])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 128, 128), (4, 2, 64, 64), (4, 2, 48, 64)])
 @pytest.mark.parametrize("position", [0, 1, 15, 16, 255, 256, 511, 512, 639])
 def test_one_key_that_stands_out_is_found_wherever_it_lies(dtype, heads, kv_heads, dim, vdim, position):
     """The query's match dominates its softmax at any distance and across page, stage and chunk borders: a row that

@@ -209,7 +209,8 @@ extern "C" RLT_API size_t rlt_scored_attention_workspace_bytes(int rows, int seq
   // the tile kernel's own scratch also where the page kernels are expected: they may refuse a cache's placement
   const size_t tiles = rlt::attention_tiles_workspace_bytes(rows, sequences, max_new, q_heads, kv_heads, value_dim,
                                                             static_cast<int64_t>(table_width) * block_size);
-  if (key_dim != 128 || value_dim != 128 || block_size != 16) return tiles;
+  const bool pages_kernel = key_dim == value_dim && block_size == 16 && (key_dim == 128 || (key_dim == 64 && max_new > 16));
+  if (!pages_kernel) return tiles;
   const size_t pages = max_new > 16 ? rlt::prefill_sm100_workspace_bytes(rows, sequences)
                                     : rlt_verify_attention_workspace_bytes(rows, q_heads, kv_heads, key_dim, block_size, table_width);
   return tiles > pages ? tiles : pages;
@@ -243,15 +244,13 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
   RLT_REQUIRE(q_stride >= static_cast<int64_t>(q_heads) * key_dim && out_stride >= static_cast<int64_t>(q_heads) * value_dim,
               "scored_attention: row strides smaller than a row");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (attention_sm100_supported(a)) {
-    if (max_new > 16) {
-      if (prefill_sm100_supported(a)) {
-        status = launch_prefill_sm100(a, workspace, workspace_bytes, s);
-        if (status != RLT_ERR_UNSUPPORTED) return status;
-      }
-    } else {
-      return planned ? run_attention_sm100(a, workspace, workspace_bytes, s) : launch_attention_sm100(a, workspace, workspace_bytes, s);
+  if (max_new > 16) {
+    if (prefill_sm100_supported(a)) {
+      status = launch_prefill_sm100(a, workspace, workspace_bytes, s);
+      if (status != RLT_ERR_UNSUPPORTED) return status;
     }
+  } else if (attention_sm100_supported(a)) {
+    return planned ? run_attention_sm100(a, workspace, workspace_bytes, s) : launch_attention_sm100(a, workspace, workspace_bytes, s);
   }
   if (attention_tiles_supported(a)) return launch_attention_tiles(a, max_new, workspace, workspace_bytes, s);
   return launch_attention_generic(a, s);

@@ -617,7 +617,7 @@ __device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {
 }
 
 // ---- two query tiles per CTA: K / V stages shared, A operands in tensor memory -----------------
-// 256 query tokens of one query head per CTA (one CTA per SM, all 512 TMEM columns), ten warps:
+// (128- or 64-wide heads.)  256 query tokens of one query head per CTA (one CTA per SM, all 512 TMEM columns), ten warps:
 //   warps 0..3 / 4..7  the softmax rows of query tile 0 / 1 (row = TMEM lane),
 //   warps 8, 9         issue the Q K^T MMAs of tile 0 / 1 (the warp runs the loop, an elected lane issues),
 //   warps 10, 11       issue the P V MMAs of tile 0 / 1,
@@ -634,10 +634,12 @@ constexpr int kPairThreads = 416;
 constexpr int kPairStages = 5;
 constexpr uint32_t kPairTmemColumns = 512;
 
+// kHalves: 64-wide column halves of a head (2: the 128-wide heads of the looped models, 1: 64-wide heads).
+template <int kHalves>
 struct __align__(1024) PairShared {
-  unsigned char q[2][kUmmaRows * 128];                   // tile 1: [half][row][64 dims], 128-byte swizzle
-  unsigned char k[kPairStages][2][kUmmaKeys * 128];      // [half][key][64 dims]
-  unsigned char v[kPairStages][2][kUmmaKeys * 128];
+  unsigned char q[kHalves][kUmmaRows * 128];                   // tile 1: [half][row][64 dims], 128-byte swizzle
+  unsigned char k[kPairStages][kHalves][kUmmaKeys * 128];      // [half][key][64 dims]
+  unsigned char v[kPairStages][kHalves][kUmmaKeys * 128];
   unsigned char rows[2 * kUmmaRows / 32][32 * 128];      // per softmax warp: its 32 rows, 64 columns of 16 bits, 16-byte pieces swizzled
   unsigned long long full_k[kPairStages], full_v[kPairStages], free_k[kPairStages], free_v[kPairStages];
   unsigned long long s_ready[2], s_free[2], p_ready[2], pv_done[2];
@@ -656,8 +658,8 @@ constexpr uint32_t kColQ = 0, kColS = 64, kTileCols = 96, kColP = 64, kColO = 25
 // The two products of a tile touch different TMEM columns, so their warps need no order between
 // them.  A stage is released to the copy warp by the commits of both tiles' warps; for a tile that
 // does not read the stage the other tile's warp arrives by hand.  Returns true when a wait gave up.
-template <bool kScores, int kTile>
-__device__ __forceinline__ bool pair_issue(PairShared& sm, uint32_t tmem, int mine, int other, uint32_t idesc,
+template <bool kScores, int kTile, int kHalves>
+__device__ __forceinline__ bool pair_issue(PairShared<kHalves>& sm, uint32_t tmem, int mine, int other, uint32_t idesc,
                                            int kv_end, int total_pages, int lane) {
   const uint32_t s_col = tmem + kColS + kTile * kTileCols, o_col = tmem + kColO + kTile * kHeadDim;
   // Q announced: from here on p_ready has completed its first phase, so a parity probe of it is unambiguous
@@ -680,7 +682,7 @@ __device__ __forceinline__ bool pair_issue(PairShared& sm, uint32_t tmem, int mi
       const uint64_t k_desc = umma_desc(smem_u32(&sm.k[stage][0][0]), 16, 1024);
       if (elect_one()) {
 #pragma unroll
-        for (int ks = 0; ks < 8; ++ks) {
+        for (int ks = 0; ks < 4 * kHalves; ++ks) {
           const uint64_t step = static_cast<uint64_t>(((ks >> 2) * (kUmmaKeys * 128) + (ks & 3) * 32) >> 4);   // address field, 16-byte units
           if (kTile == 0) umma_issue_ts(s_col, tmem + kColQ + ks * 8, k_desc + step, idesc, ks > 0);
           else umma_issue(s_col, q_desc + static_cast<uint64_t>(((ks >> 2) * (kUmmaRows * 128) + (ks & 3) * 32) >> 4), k_desc + step, idesc, ks > 0);
@@ -692,7 +694,7 @@ __device__ __forceinline__ bool pair_issue(PairShared& sm, uint32_t tmem, int mi
     } else {         // O += P(j) V(j) over the 64 keys
       const int rows = min(4, total_pages - j * 4) * kPage;
       if (kv_end - j * kUmmaKeys < rows)   // the last stage: slots behind the last key any row sees (both tiles' warps may clear them)
-        zero_rows_warp(&sm.v[stage][0][0], &sm.v[stage][1][0], kv_end - j * kUmmaKeys, rows, lane);
+        zero_rows_warp(&sm.v[stage][0][0], &sm.v[stage][kHalves - 1][0], kv_end - j * kUmmaKeys, rows, lane);
       const uint64_t v_desc = umma_desc(smem_u32(&sm.v[stage][0][0]), 8192, 1024);
       if (elect_one()) {
 #pragma unroll
@@ -714,7 +716,7 @@ __device__ __forceinline__ bool pair_issue(PairShared& sm, uint32_t tmem, int mi
 
 // kTerms: query temperature and distance bias (see the verify kernel): the stage's scores are brought to their
 // final log2-domain values in pairs, with the bias of the stage's first key as an exact integer distance.
-template <bool kBF16, bool kTerms>
+template <bool kBF16, bool kTerms, int kHalves>
 __global__ void __launch_bounds__(kPairThreads, 1)
 prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                     AttentionArgs a, const PrefillHeader* header, const PrefillTile* tiles, unsigned* error,
@@ -722,7 +724,9 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
   using T = typename std::conditional<kBF16, __nv_bfloat16, __half>::type;
   if (blockIdx.x >= header->tiles) return;
   extern __shared__ unsigned char smem_raw[];
-  PairShared& sm = *reinterpret_cast<PairShared*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  using Shared = PairShared<kHalves>;
+  constexpr int kDim = 64 * kHalves;
+  Shared& sm = *reinterpret_cast<Shared*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const int lane = threadIdx.x & 31, warp = __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0);   // warp-uniform for the compiler too
   const PrefillTile tile = tiles[blockIdx.x];   // everything the CTA needs to know about its rows: one load
   const int q_head = blockIdx.y, kv_head = q_head / (a.q_heads / a.kv_heads);
@@ -762,7 +766,7 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     const int pages_last = total_pages - (all_stages - 1) * 4;   // 1 .. 4
     const int tail = (4 - pages_last) * 2048 / 16;               // 16-byte words per half
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-    for (int i = threadIdx.x; i < 2 * tail; i += kPairThreads) {
+    for (int i = threadIdx.x; i < kHalves * tail; i += kPairThreads) {
       const int half = i / tail, word = i - half * tail;
       reinterpret_cast<uint4*>(&sm.v[all_stages - 1][half][pages_last * 2048])[word] = zero;
     }
@@ -775,7 +779,7 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
   constexpr uint32_t kFormat = kBF16 ? 1u : 0u;
   constexpr uint32_t kIdesc = (1u << 4) | (kFormat << 7) | (kFormat << 10) | (static_cast<uint32_t>(kUmmaRows >> 4) << 24);
   constexpr uint32_t kIdescQK = kIdesc | (static_cast<uint32_t>(kUmmaKeys >> 3) << 17);            // N = 64 keys
-  constexpr uint32_t kIdescPV = kIdesc | (static_cast<uint32_t>(kHeadDim >> 3) << 17) | (1u << 16);  // N = 128 dims, B MN-major
+  constexpr uint32_t kIdescPV = kIdesc | (static_cast<uint32_t>(kDim >> 3) << 17) | (1u << 16);      // N = the head's dims, B MN-major
   bool failed = false;
 
   if (warp == 12) {
@@ -785,8 +789,8 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     for (int j = 0; j < all_stages && !failed; ++j) {
       const int stage = j % kPairStages, use = j / kPairStages;
       const int pages = min(4, total_pages - j * 4);
-      const int page = (lane & 7) >> 1, half = lane & 1;
-      const int block = (lane < 8 && page < pages) ? table[j * 4 + page] : 0;
+      const int page = (lane / kHalves) & 3, half = lane % kHalves;
+      const int block = (lane < 4 * kHalves && page < pages) ? table[j * 4 + page] : 0;
 #pragma unroll
       for (int operand = 0; operand < 2; ++operand) {
         bool ok = true;
@@ -794,21 +798,21 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
         ok = __shfl_sync(0xffffffffu, ok, 0);
         if (!ok) { failed = true; break; }
         const uint32_t bar = smem_u32(operand == 0 ? &sm.full_k[stage] : &sm.full_v[stage]);
-        if (lane == 0) mbar_expect_tx(bar, pages * kTileBytes);
+        if (lane == 0) mbar_expect_tx(bar, pages * kHalves * 2048);
         __syncwarp();
-        if (lane < 8 && page < pages) {
+        if (lane < 4 * kHalves && page < pages) {
           unsigned char* dst = (operand == 0 ? &sm.k[stage][half][0] : &sm.v[stage][half][0]) + page * 2048;
-          tma_load_page_half(smem_u32(dst), operand == 0 ? &k_map : &v_map, kv_head * kHeadDim + half * 64, block, bar, policy);
+          tma_load_page_half(smem_u32(dst), operand == 0 ? &k_map : &v_map, kv_head * kDim + half * 64, block, bar, policy);
         }
       }
     }
   } else if (warp >= 8) {
     // ---- MMA issue: one warp per query tile and product ----
     const int kv_end = max(base_len + tile.first + tile.count - 1, 0);   // keys the pair's last row sees
-    if (warp == 8) failed = pair_issue<true, 0>(sm, tmem, stages0, stages1, kIdescQK, kv_end, total_pages, lane);
-    else if (warp == 9) failed = pair_issue<true, 1>(sm, tmem, stages1, stages0, kIdescQK, kv_end, total_pages, lane);
-    else if (warp == 10) failed = pair_issue<false, 0>(sm, tmem, stages0, stages1, kIdescPV, kv_end, total_pages, lane);
-    else failed = pair_issue<false, 1>(sm, tmem, stages1, stages0, kIdescPV, kv_end, total_pages, lane);
+    if (warp == 8) failed = pair_issue<true, 0, kHalves>(sm, tmem, stages0, stages1, kIdescQK, kv_end, total_pages, lane);
+    else if (warp == 9) failed = pair_issue<true, 1, kHalves>(sm, tmem, stages1, stages0, kIdescQK, kv_end, total_pages, lane);
+    else if (warp == 10) failed = pair_issue<false, 0, kHalves>(sm, tmem, stages0, stages1, kIdescPV, kv_end, total_pages, lane);
+    else failed = pair_issue<false, 1, kHalves>(sm, tmem, stages1, stages0, kIdescPV, kv_end, total_pages, lane);
   } else {
     // ---- softmax rows ----
     const int t = warp >> 2, row = threadIdx.x & (kUmmaRows - 1);
@@ -824,19 +828,19 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     const int64_t warp_first = static_cast<int64_t>(seq_first) + tile.first + t * kUmmaRows + warp_row;
     unsigned char* staging = &sm.rows[warp][0];
     if (my_stages > 0) {   // Q: tile 0 into tensor memory (two 16-bit values per column, a thread stores its row), tile 1 into shared memory
-      const T* src = static_cast<const T*>(a.q) + warp_first * a.q_stride + static_cast<int64_t>(q_head) * kHeadDim;
+      const T* src = static_cast<const T*>(a.q) + warp_first * a.q_stride + static_cast<int64_t>(q_head) * kDim;
       const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
       if (t == 0) {
-        uint4 piece[2][8];
+        uint4 piece[kHalves][8];
 #pragma unroll
-        for (int h = 0; h < 2; ++h)
+        for (int h = 0; h < kHalves; ++h)
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const int r = 4 * i + (lane >> 3);
             piece[h][i] = r < warp_count ? __ldg(reinterpret_cast<const uint4*>(src + r * a.q_stride + h * 64) + (lane & 7)) : zero;
           }
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
+        for (int h = 0; h < kHalves; ++h) {
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const int r = 4 * i + (lane >> 3);
@@ -855,8 +859,9 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
         tmem_store_wait();
       } else {
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const int r = 2 * i + (lane >> 4), c = lane & 15;
+        for (int i = 0; i < 8 * kHalves; ++i) {
+          constexpr int kPieces = 8 * kHalves;      // 16-byte pieces of a row
+          const int r = i * (32 / kPieces) + lane / kPieces, c = lane % kPieces;
           const uint4 value = r < warp_count ? __ldg(reinterpret_cast<const uint4*>(src + r * a.q_stride) + c) : zero;
           *reinterpret_cast<uint4*>(&sm.q[c >> 3][(warp_row + r) * 128 + (((c & 7) ^ (r & 7)) << 4)]) = value;
         }
@@ -948,7 +953,7 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
         tcgen05_after_sync();
         if (__any_sync(0xffffffffu, alpha != 1.0f)) {   // rescale this warp's 32 output rows in place
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < 2 * kHalves; ++c) {
             uint32_t r[32];
             tmem_load32(o_col + c * 32, r);
             tmem_load_wait();
@@ -969,9 +974,9 @@ prefill_pair_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     failed = __any_sync(0xffffffffu, failed);
     if (!failed && count > 0) {
       const float inv = l > 0.f ? 1.0f / l : 0.f;
-      T* dst = static_cast<T*>(a.out) + warp_first * a.out_stride + static_cast<int64_t>(q_head) * kHeadDim;
+      T* dst = static_cast<T*>(a.out) + warp_first * a.out_stride + static_cast<int64_t>(q_head) * kDim;
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {   // 64 output columns at a time
+      for (int h = 0; h < kHalves; ++h) {   // 64 output columns at a time
         uint32_t lo[32], hi[32];
         if (my_stages > 0) {
           tmem_load32(o_col + h * 64, lo);
@@ -1010,7 +1015,17 @@ size_t tile_capacity(int rows, int seqs) { return static_cast<size_t>(rows) / kT
 
 }  // namespace
 
+// 64-wide heads: the pair kernel only, bf16.
+bool prefill_narrow_supported(const AttentionArgs& a) {
+  if (a.dtype != RLT_BF16 || a.head_dim != 64 || a.value_dim != 64 || a.block_size != kPage || a.cu_seqlens_q == nullptr) return false;
+  if (a.v_block_stride != a.block_stride || a.v_token_stride != a.token_stride) return false;
+  if (a.token_stride % 8 != 0 || a.block_stride % 8 != 0 || a.block_stride < a.token_stride * kPage || a.num_blocks > 0xffffffffll) return false;
+  if (static_cast<long long>(a.table_width) * a.block_size > (1 << 26)) return false;
+  return a.q_stride % 8 == 0 && a.out_stride % 8 == 0 && aligned16(a.q) && aligned16(a.out) && aligned16(a.key_cache) && aligned16(a.value_cache);
+}
+
 bool prefill_sm100_supported(const AttentionArgs& a) {
+  if (prefill_narrow_supported(a)) return true;
   return a.cu_seqlens_q != nullptr && attention_sm100_supported(a) && a.q_stride % 8 == 0 && aligned16(a.q);
 }
 
@@ -1032,7 +1047,7 @@ int launch_prefill_sm100(const AttentionArgs& a, void* workspace, size_t workspa
   // on 1024-token contexts, 70 against 138 and 147 us at 4 sequences on 4096-token ones).
   const char* forced = getenv("RLT_PREFILL_KERNEL");
   // Only the pair kernel has score terms and strided query / output rows.
-  const bool plain = a.terms.plain() && a.q_stride == static_cast<int64_t>(a.q_heads) * kHeadDim && a.out_stride == a.q_stride;
+  const bool plain = a.head_dim == kHeadDim && a.terms.plain() && a.q_stride == static_cast<int64_t>(a.q_heads) * kHeadDim && a.out_stride == a.q_stride;
   const char kernel_choice = plain && forced != nullptr && forced[0] != 0 ? forced[0] : 'p';
   const bool use_mma_sync = kernel_choice == 'm';
   PrefillHeader* header = static_cast<PrefillHeader*>(workspace);
@@ -1043,13 +1058,15 @@ int launch_prefill_sm100(const AttentionArgs& a, void* workspace, size_t workspa
     prefill_plan_kernel<<<1, kPrefillPlanThreads, 0, stream>>>(a.cu_seqlens_q, a.context_lengths, a.table_width, a.table_rows, kPairRows, header, tiles);
     int status = launch_status("prefill_plan_kernel");
     if (status != RLT_OK) return status;
-    const size_t smem = sizeof(PairShared) + 1024;
+    const bool narrow = a.head_dim == 64;
+    const size_t smem = (narrow ? sizeof(PairShared<1>) : sizeof(PairShared<2>)) + 1024;
     const int take_turns = static_cast<int64_t>(a.rows) >= 2048ll * a.table_rows ? 1 : 0;   // prompts of 2048 tokens and more on average
     const dim3 grid(static_cast<unsigned>(static_cast<size_t>(a.rows) / kPairRows + static_cast<size_t>(a.table_rows) + 1),
                     static_cast<unsigned>(a.q_heads));
     const bool terms = !a.terms.plain();
-    auto kernel = a.dtype == RLT_BF16 ? (terms ? prefill_pair_kernel<true, true> : prefill_pair_kernel<true, false>)
-                                      : (terms ? prefill_pair_kernel<false, true> : prefill_pair_kernel<false, false>);
+    auto kernel = narrow ? prefill_pair_kernel<true, true, 1>
+                  : a.dtype == RLT_BF16 ? (terms ? prefill_pair_kernel<true, true, 2> : prefill_pair_kernel<true, false, 2>)
+                                        : (terms ? prefill_pair_kernel<false, true, 2> : prefill_pair_kernel<false, false, 2>);
     RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     kernel<<<grid, kPairThreads, smem, stream>>>(k_map, v_map, a, header, tiles, &header->error, scale_log2, take_turns);
     return launch_status("prefill_pair_kernel");

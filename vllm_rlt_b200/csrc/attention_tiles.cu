@@ -101,6 +101,7 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
   const float rs0 = scale_log2 * query_temperature(a.terms, len0), rs1 = scale_log2 * query_temperature(a.terms, len1);
   const float slope0 = kLog2e * distance_slope(a.terms, head0, a.q_heads), slope1 = kLog2e * distance_slope(a.terms, head1, a.q_heads);
   const int warp_end = kSplit ? key_end : row_len(min(all_rows - 1, r_base + warp * 16 + 15));   // keys any row of the warp sees
+  const int unmasked_end = min(row_len(r_base + (kSplit ? 0 : warp * 16)), key_end);   // keys every row of the warp sees
   float o[kD / 8][4];
 #pragma unroll
   for (int j = 0; j < kD / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
@@ -128,19 +129,32 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
           mma_16816<true>(s[2 * n + 1], q, f[2], f[3]);
         }
       }
-      float mx0 = -INFINITY, mx1 = -INFINITY;
+      const float first0 = slope0 * static_cast<float>(first_key + 2 * t - len0 + 1), first1 = slope1 * static_cast<float>(first_key + 2 * t - len1 + 1);
 #pragma unroll
       for (int n = 0; n < kMine / 8; ++n) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int pos = first_key + n * 8 + 2 * t + e;
-          const float v0 = fmaf(s[n][e], rs0, slope0 * static_cast<float>(pos - len0 + 1));
-          const float v1 = fmaf(s[n][2 + e], rs1, slope1 * static_cast<float>(pos - len1 + 1));
-          s[n][e] = pos < len0 && pos < key_end ? v0 : -INFINITY;
-          s[n][2 + e] = pos < len1 && pos < key_end ? v1 : -INFINITY;
-          mx0 = fmaxf(mx0, s[n][e]);
-          mx1 = fmaxf(mx1, s[n][2 + e]);
+          const float at = static_cast<float>(n * 8 + e);
+          s[n][e] = fmaf(s[n][e], rs0, fmaf(slope0, at, first0));
+          s[n][2 + e] = fmaf(s[n][2 + e], rs1, fmaf(slope1, at, first1));
         }
+      }
+      if (first_key + kMine > unmasked_end) {
+        const int left0 = min(len0, key_end) - first_key - 2 * t, left1 = min(len1, key_end) - first_key - 2 * t;
+#pragma unroll
+        for (int n = 0; n < kMine / 8; ++n) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            if (n * 8 + e >= left0) s[n][e] = -INFINITY;
+            if (n * 8 + e >= left1) s[n][2 + e] = -INFINITY;
+          }
+        }
+      }
+      float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+      for (int n = 0; n < kMine / 8; ++n) {
+        mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
+        mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
       }
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));

@@ -19,9 +19,9 @@ constexpr int kStageBytes = 2 * kTileBytes;       // K page + V page
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr long long kWaitCycles = 4000000000ll;   // bounded waits (about 2 s): give up instead of hanging
 
-// The scale of the plain 1 / sqrt(128) in the log2 domain, or the call's own.
+// The scale of the plain 1 / sqrt(head_dim) in the log2 domain, or the call's own.
 inline float log2_scale(const AttentionArgs& a) {
-  const double scale = a.terms.scale != 0.0f ? static_cast<double>(a.terms.scale) : 1.0 / sqrt(static_cast<double>(kHeadDim));
+  const double scale = a.terms.scale != 0.0f ? static_cast<double>(a.terms.scale) : 1.0 / sqrt(static_cast<double>(a.head_dim));
   return static_cast<float>(1.4426950408889634 * scale);
 }
 
@@ -223,7 +223,7 @@ inline EncodeTiledFn encode_tiled_fn() {
   return fn;
 }
 
-// Tensor map over one layer's cache view as [num_blocks][16 tokens][kv_heads * 128] elements,
+// Tensor map over one layer's cache view as [num_blocks][16 tokens][kv_heads * head_dim] elements,
 // box = 64 elements x 16 tokens x 1 block, 128-byte swizzle.
 inline int make_page_map(CUtensorMap* map, const void* base, const AttentionArgs& a) {
   EncodeTiledFn fn = encode_tiled_fn();
@@ -231,7 +231,7 @@ inline int make_page_map(CUtensorMap* map, const void* base, const AttentionArgs
     set_last_error_text("cuTensorMapEncodeTiled is not available from this driver");
     return RLT_ERR_CUDA;
   }
-  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(a.kv_heads) * kHeadDim, kPage,
+  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(a.kv_heads) * a.head_dim, kPage,
                               static_cast<cuuint64_t>(a.num_blocks)};
   const cuuint64_t strides[2] = {static_cast<cuuint64_t>(a.token_stride) * 2,
                                  static_cast<cuuint64_t>(a.block_stride) * 2};
