@@ -540,7 +540,7 @@ RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, void* out, int
                          int64_t num_blocks, int block_size, int q_heads, int kv_heads, int key_dim,
                          int value_dim, int dtype, const int32_t* block_tables, int sequences, int table_width,
                          const int32_t* context_lengths, const int32_t* cu_seqlens_q, int rows, int max_new,
-                         float scale, float temp_coef, int temp_every, int distance_bias, int planned,
+                         float scale, float temp_coef, int temp_every, int distance_bias, int window, int planned,
                          void* workspace, size_t workspace_bytes, rlt_stream_t stream);
 
 /* The fp32 residual stream and the norm that opens a layer:
@@ -578,10 +578,70 @@ RLT_API int rlt_ssd_scan(const void* x, const void* b, const void* c, int64_t xb
                  const int32_t* slot_of, int sequences, int max_tokens, int heads, int groups, int state_size,
                  int head_dim, int dtype, void* workspace, size_t workspace_bytes, rlt_stream_t stream);
 
-/* out = rmsnorm_parts(y * silu(z)) * weight: the row is normed in `parts` equal parts, each by its own root mean square. */
+/* out = rmsnorm_parts(y * silu(z)) * weight: the row is normed in `parts` equal parts, each by its own root mean square.
+ * gate_behind != 0: out = rmsnorm_parts(y) * weight * sigmoid(z). */
 RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight,
-                   void* out, int64_t out_stride, int rows, int width, int parts, float eps, int dtype,
-                   rlt_stream_t stream);
+                   void* out, int64_t out_stride, int rows, int width, int parts, float eps, int gate_behind,
+                   int dtype, rlt_stream_t stream);
+
+/* Linear attention with a constant decay per head: S_t = decay_h S_(t-1) + k_t v_t^T, out_t = S_t^T q_t.  q, k
+ * [rows, heads * key_dim] and v [rows, heads * value_dim] are column slices of rows of one stride; decay: fp32
+ * [2][heads], the decays and their base-2 logarithms; state: fp32 [slots][heads][key_dim][value_dim], updated in
+ * place.  Sequences, slots and workspace (rlt_ssd_scan_workspace_bytes with state = key_dim, head_dim = value_dim)
+ * as in rlt_ssd_scan. */
+RLT_API int rlt_decay_scan(const void* q, const void* k, const void* v, int64_t qkv_stride, const float* decay, void* out,
+                   int64_t out_stride, float* state, int64_t slots, const int32_t* cu_seqlens, const int32_t* starts,
+                   const int32_t* slot_of, int sequences, int max_tokens, int heads, int key_dim, int value_dim, int dtype,
+                   void* workspace, size_t workspace_bytes, rlt_stream_t stream);
+
+/* Hyper-connected residual streams, fp32 [rows][stream_count][width], between two sublayers:
+ *   x_t <- sum_s mix[s][t] x_s + out_coef[t] y   (with mix; stored when `store`)
+ *   u = sum_t in_coef[t] x_t  (null: plain sum),  out[row] = rmsnorm(u) * (weight_offset + weight)
+ * y: delta[i], or with parts > 0 the sum over p of part_weights[i][p] * delta[part_rows[i][p]].
+ * tokens != null starts a model instead: every stream becomes rmsnorm(embed[token] + bigram[bucket]) * embed_weight with
+ * bucket = (previous * mul_prev + token * mul_cur) mod buckets, row `buckets` where previous is negative (bigram null:
+ * no table).  i = row_index ? row_index[row] : row.  At most 8 streams. */
+RLT_API int rlt_stream_mix(float* streams, int stream_count, const void* delta, int parts, const int32_t* part_rows,
+                   const float* part_weights, const float* out_coef, const float* mix, const int64_t* tokens,
+                   const int32_t* previous, const void* embed, int64_t vocab, const void* bigram, int64_t buckets,
+                   int64_t mul_prev, int64_t mul_cur, const float* embed_weight, const float* in_coef,
+                   const int64_t* row_index, int store, const float* weight, float weight_offset, void* out, int rows,
+                   int width, float eps, int dtype, rlt_stream_t stream);
+
+/* The stacked down projections of latent attention: rmsnorm(proj[q_col ..]) * q_weight into q_out, and the cache row
+ * [rmsnorm(proj[kv_col .. + kv_rank]) * kv_weight | rotated proj[kv_col + kv_rank .. + rot_dim]] into the row's page.
+ * Pairs (2i, 2i + 1) of the first rot_dims dimensions are turned by position * frequencies[i]. */
+RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, int q_col, int q_rank, int kv_col, int kv_rank,
+                     int rot_dim, int rot_dims, const float* q_weight, const float* kv_weight, float eps,
+                     const double* frequencies, void* q_out, int64_t q_out_stride, void* cache, int64_t block_stride,
+                     int64_t token_stride, int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
+                     const int32_t* row_seq, const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
+
+/* The same rotation of `dim` elements of every head, from src to dst (which may be one); strides in elements. */
+RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head, void* dst, int64_t dst_row,
+                     int64_t dst_head, int heads, int dim, int rot_dims, const double* frequencies,
+                     const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
+
+/* Cache rows of positions first[s] .. of every sequence s, packed: row cu[s] + i holds position first[s] + i. */
+RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks,
+                      int block_size, int row_width, const int32_t* tables, int table_width, const int32_t* first,
+                      const int32_t* cu, int sequences, int rows, void* out, int dtype, rlt_stream_t stream);
+
+/* Mixture of experts.  route: s = softmax(logits) in fp32, the `top` largest of s + correction (null: none), weights =
+ * chosen s / (their sum + floor_sum); counts [experts] must be zero before.  gather: rows sorted by expert, and every
+ * choice's place among them.  gemm: y = act(x W_e^T) over sorted rows (act 0: none); workspace: 256 bytes for an error word. */
+RLT_API int rlt_expert_route(const float* logits, int64_t logit_stride, const float* correction, int rows, int experts,
+                     int top, float floor_sum, int32_t* counts, int32_t* chosen, int32_t* rank, float* weights,
+                     rlt_stream_t stream);
+RLT_API int rlt_expert_gather(const void* x, int64_t x_stride, const int32_t* counts, const int32_t* chosen,
+                      const int32_t* rank, int rows, int top, int width, void* sorted, int32_t* places, int dtype,
+                      rlt_stream_t stream);
+RLT_API int rlt_expert_gemm(const void* x, int64_t x_stride, const void* w, void* y, int64_t y_stride, const int32_t* counts,
+                    int rows, int experts, int in, int out, int act, int dtype, void* workspace, rlt_stream_t stream);
+
+/* g = min(gate, limit), u = clamp(up, -limit, limit): out = g * sigmoid(slope * g) * (u + 1); gate at column 0, up at up_col. */
+RLT_API int rlt_clamped_glu(const void* gate_up, int64_t row_stride, int up_col, void* out, int64_t out_stride, int64_t rows,
+                    int cols, float limit, float slope, int dtype, rlt_stream_t stream);
 
 #ifdef __cplusplus
 }

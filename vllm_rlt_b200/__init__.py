@@ -17,12 +17,15 @@ from .prefix_cache import PrefixIndex
 from .engine import Engine, StepEntry
 from .hybrid_lm import HybridLM, HybridLMConfig
 from .kv_cache import RollbackResult, finalize_tokens, kv_write, rollback
-from .layers import block_epilogue, residual_norm, rope_kv_write, sandwich_norm
+from .experts import expert_gather, expert_gemm, expert_route
+from .latent import latent_gather, latent_write, rotate_heads, rotation_frequencies
+from .layers import block_epilogue, clamped_glu, residual_norm, rope_kv_write, sandwich_norm, stream_mix
 from .looped_lm import LoopedLM, LoopedLMConfig, seeded_state_dict
-from .recurrent import causal_conv, gated_norm, ssd_scan
+from .recurrent import causal_conv, decay_scan, decay_table, gated_norm, ssd_scan
 from .registry import load_model, register_model, registered_architectures
 from .runner import (B200SpeculativeRunner, KVCacheManagerView, ModelRunnerOutput, Request, SamplingParams, ScheduledRequest,
                      SchedulerOutput, SpeculativeConfig, SpeculativeRoundTicket, SpeculativeStats)
+from .stream_lm import StreamLM, StreamLMConfig
 from .sequence_cache import CacheFull, CacheSpec, KVSpec, SequenceCache, StateSpec
 from .speculative import (PipelineState, SpeculativeResult, accept_greedy, accept_rejection, argmax_rows,
                           decode_result, pipeline_shift, probabilities, raise_for_status, round_uniforms,
@@ -39,4 +42,6 @@ __all__ = [
     "KVCacheManagerView", "CacheFull", "CacheSpec", "Engine", "HybridLM", "HybridLMConfig", "KVSpec", "ScoreTerms",
     "SequenceCache", "StateSpec", "StepEntry", "block_epilogue", "causal_conv", "gated_norm", "load_model", "read_safetensors",
     "read_weights", "register_model", "registered_architectures", "residual_norm", "ssd_scan",
+    "StreamLM", "StreamLMConfig", "clamped_glu", "decay_scan", "decay_table", "expert_gather", "expert_gemm", "expert_route",
+    "latent_gather", "latent_write", "rotate_heads", "rotation_frequencies", "stream_mix",
 ]

@@ -47,12 +47,15 @@ class ScoreTerms:
 
         score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
                 - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
+
+    over the keys j <= p, with `window` > 0 only those with p - j < window.
     """
 
     scale: float
     temp_coef: float = 0.0
     temp_every: int = 1
     distance_bias: bool = False
+    window: int = 0
 
 
 @dataclass
@@ -338,7 +341,7 @@ class B200PagedAttention:
             if t.stride(2) != 1 or t.stride(1) != t.shape[2]:
                 raise ValueError(f"the [heads, dim] tail of {name} must be contiguous")
         for cache in (key_cache, value_cache):
-            if cache.stride(3) != 1 or cache.stride(2) != cache.shape[3]:
+            if cache.stride(3) != 1 or (cache.shape[2] > 1 and cache.stride(2) != cache.shape[3]):
                 raise ValueError("the [kv_heads, dim] tail of the caches must be contiguous")
         sequences, width = block_tables.shape
         if block_tables.dtype != torch.int32 or not block_tables.is_contiguous() or context_lengths.dtype != torch.int32 \
@@ -358,7 +361,7 @@ class B200PagedAttention:
             # prompt calls have scratch of their own: a mixed step's plan for its short portions survives them
             workspace = self._workspace(device, stream.value or 0 if max_new <= 16 else ("prompt", stream.value or 0), nbytes)
             planned = False
-            tiled = max_new <= 16 and q.dtype != torch.float32 and key_dim == value_dim == 128 and block == 16
+            tiled = max_new <= 16 and not terms.window and q.dtype != torch.float32 and key_dim == value_dim == 128 and block == 16
             versions = self._versions(block_tables, context_lengths, cu_seqlens_q) if self._sharing and tiled else None
             if versions is not None:
                 plan_key = (block_tables.data_ptr(), sequences, width, context_lengths.data_ptr(), cu_seqlens_q.data_ptr(), rows,
@@ -378,7 +381,7 @@ class B200PagedAttention:
                 key_cache.stride(1), _capi.ptr(value_cache), value_cache.stride(0), value_cache.stride(1), blocks, block, heads,
                 kv_heads, key_dim, value_dim, dtype, _capi.ptr(block_tables), sequences, width, _capi.ptr(context_lengths),
                 _capi.ptr(cu_seqlens_q), rows, int(max_new), float(terms.scale), float(terms.temp_coef), int(terms.temp_every),
-                int(terms.distance_bias), int(planned), _capi.ptr(workspace), workspace.numel(), stream)
+                int(terms.distance_bias), int(terms.window), int(planned), _capi.ptr(workspace), workspace.numel(), stream)
         _capi.check(status, "scored_attention")
         return out
 

@@ -17,8 +17,9 @@ struct ScoreTerms {
   float temp_coef = 0.0f;
   int temp_every = 1;
   int distance_bias = 0;
+  int window = 0;            // 0: all keys before the row, else the last `window` of them (the row's own included)
 
-  __host__ __device__ bool plain() const { return temp_coef == 0.0f && distance_bias == 0; }
+  __host__ __device__ bool plain() const { return temp_coef == 0.0f && distance_bias == 0 && window == 0; }
 };
 
 struct AttentionArgs {
@@ -104,7 +105,7 @@ __device__ __forceinline__ void resolve_row(const AttentionArgs& a, int row, int
 }
 
 // attention_generic.cu: any shape, one CTA per (row, head).
-int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream, int window = 0);   // window > 0: the row's last `window` keys only
+int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream);
 
 // attention_tiles.cu: tensor cores for other head sizes (bf16, multiples of 8 up to 256), packed rows only.
 bool attention_tiles_supported(const AttentionArgs& a);

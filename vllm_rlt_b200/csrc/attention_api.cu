@@ -86,7 +86,8 @@ extern "C" RLT_API int rlt_windowed_attention(const void* q, void* out, const vo
   set_plain_layout(a);
   int status = check_args(a);
   if (status != RLT_OK || rows == 0) return status;
-  return launch_attention_generic(a, static_cast<cudaStream_t>(stream), window);
+  a.terms.window = window;
+  return launch_attention_generic(a, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" RLT_API int rlt_verify_attention_plan(const int32_t* block_tables, int table_rows, int table_width,
@@ -223,7 +224,7 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
                                             int value_dim, int dtype, const int32_t* block_tables, int sequences,
                                             int table_width, const int32_t* context_lengths, const int32_t* cu_seqlens_q,
                                             int rows, int max_new, float scale, float temp_coef, int temp_every,
-                                            int distance_bias, int planned, void* workspace, size_t workspace_bytes,
+                                            int distance_bias, int window, int planned, void* workspace, size_t workspace_bytes,
                                             rlt_stream_t stream) {
   using namespace rlt;
   AttentionArgs a;
@@ -235,7 +236,8 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
   a.value_dim = value_dim; a.v_block_stride = v_block_stride; a.v_token_stride = v_token_stride;
   a.q_stride = q_stride; a.out_stride = out_stride;
   a.terms.scale = scale; a.terms.temp_coef = temp_coef; a.terms.temp_every = temp_every; a.terms.distance_bias = distance_bias;
-  RLT_REQUIRE(value_dim > 0 && temp_every > 0, "scored_attention: value_dim and temp_every must be positive");
+  a.terms.window = window;
+  RLT_REQUIRE(value_dim > 0 && temp_every > 0 && window >= 0, "scored_attention: value_dim and temp_every must be positive, window not negative");
   RLT_REQUIRE(cu_seqlens_q != nullptr || rows == 0, "scored_attention: cu_seqlens_q is required");
   int status = check_args(a);
   if (status != RLT_OK || rows == 0) return status;
@@ -244,7 +246,9 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
   RLT_REQUIRE(q_stride >= static_cast<int64_t>(q_heads) * key_dim && out_stride >= static_cast<int64_t>(q_heads) * value_dim,
               "scored_attention: row strides smaller than a row");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (max_new > 16) {
+  if (window > 0) {
+    // the page kernels walk whole contexts: windowed rows go to the tile or generic kernel
+  } else if (max_new > 16) {
     if (prefill_sm100_supported(a)) {
       status = launch_prefill_sm100(a, workspace, workspace_bytes, s);
       if (status != RLT_ERR_UNSUPPORTED) return status;

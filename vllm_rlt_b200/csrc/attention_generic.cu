@@ -1,10 +1,10 @@
-// Shape-generic paged attention: any head_dim <= 256 (keys and values may differ), any block size,
+// Shape-generic paged attention: any head_dim <= 640 (keys and values may differ), any block size,
 // any GQA ratio, fp32 / fp16 / bf16, with the score terms of attention.cuh.  One CTA per (query row, query head); four warps stride over the
 // row's tokens with an fp32 online softmax each and are merged in warp order, so a row's
 // result depends on nothing but its own query, length and K/V.  This is the path for
 // shapes the tiled sm_100a kernel (attention_sm100.cu) does not cover — the fp32 tiny
 // model and the odd head sizes the reference's tests use; it reads K/V once per row.
-// With window > 0 a row attends only its last `window` keys (sliding-window layers).
+// With terms.window > 0 a row attends only its last `window` keys (sliding-window layers).
 #include <math.h>
 
 #include "attention.cuh"
@@ -14,11 +14,10 @@ namespace {
 
 constexpr int kWarps = 4;
 constexpr int kThreads = kWarps * 32;
-constexpr int kMaxPerLane = 8;  // head_dim <= 256
-
-template <typename T>
+template <typename T, int kMaxPerLane>   // head_dim <= 32 * kMaxPerLane
 __global__ void __launch_bounds__(kThreads)
-attention_generic_kernel(AttentionArgs a, float scale, int window) {
+attention_generic_kernel(AttentionArgs a, float scale) {
+  const int window = a.terms.window;
   const int row = blockIdx.x / a.q_heads;
   const int head = blockIdx.x % a.q_heads;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -99,9 +98,10 @@ attention_generic_kernel(AttentionArgs a, float scale, int window) {
 
 }  // namespace
 
-int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream, int window) {
-  if (a.head_dim > 32 * kMaxPerLane || a.value_dim > 32 * kMaxPerLane) {
-    set_last_error_text("verify_attention supports head_dim <= 256");
+int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream) {
+  const int widest = a.head_dim > a.value_dim ? a.head_dim : a.value_dim;
+  if (widest > 640) {
+    set_last_error_text("attention supports head_dim <= 640");
     return RLT_ERR_UNSUPPORTED;
   }
   const int64_t ctas = static_cast<int64_t>(a.rows) * a.q_heads;
@@ -110,8 +110,10 @@ int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream, int wi
     return RLT_ERR_INVALID;
   }
   const float scale = score_scale(a);
-  RLT_DISPATCH_DTYPE(a.dtype, T,
-                     (attention_generic_kernel<T><<<static_cast<unsigned>(ctas), kThreads, 0, stream>>>(a, scale, window)));
+  RLT_DISPATCH_DTYPE(a.dtype, T, {
+    if (widest <= 256) attention_generic_kernel<T, 8><<<static_cast<unsigned>(ctas), kThreads, 0, stream>>>(a, scale);
+    else attention_generic_kernel<T, 20><<<static_cast<unsigned>(ctas), kThreads, 0, stream>>>(a, scale);
+  });
   return launch_status("attention_generic_kernel");
 }
 

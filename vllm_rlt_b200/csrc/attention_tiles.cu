@@ -1,5 +1,5 @@
 // Tensor-core paged attention for head sizes the sm_100a page kernels do not cover: bf16, key and value sizes of
-// their own (multiples of 8, up to 256), any page size and GQA ratio, with the score terms of attention.cuh.
+// their own (multiples of 8, up to 256), any page size and GQA ratio, with the score terms of attention.cuh (windows included).
 //
 // The query rows of one KV head are the (token, query head of the group) pairs of a sequence's portion, token
 // major, so a K / V stage serves every head of the group.  Keys come in stages of 64, gathered row by row with
@@ -59,10 +59,12 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
   const int base_len = context - tokens + 1;           // keys the portion's first token sees (<= 0: padding)
   auto row_len = [&](int r) { return r < all_rows ? max(base_len + r / gqa, 0) : 0; };
   const int kv_end = row_len(min(all_rows - 1, r_base + kRows - 1));
-  int key_begin = 0, key_end = kv_end;
+  const int window = a.terms.window > 0 ? a.terms.window : 0x40000000;
+  const int kv_begin = max(row_len(r_base) - window, 0) / kKeys * kKeys;   // stages before it hold no key any row sees
+  int key_begin = kv_begin, key_end = kv_end;
   if (kSplit) {
-    const int per = ((kv_end + splits - 1) / splits + kKeys - 1) / kKeys * kKeys;
-    key_begin = min(split * per, kv_end);
+    const int per = ((kv_end - kv_begin + splits - 1) / splits + kKeys - 1) / kKeys * kKeys;
+    key_begin = min(kv_begin + split * per, kv_end);
     key_end = min(kv_end, key_begin + per);
   }
   const int stages = (key_end - key_begin + kKeys - 1) / kKeys;
@@ -102,6 +104,7 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
   const float slope0 = kLog2e * distance_slope(a.terms, head0, a.q_heads), slope1 = kLog2e * distance_slope(a.terms, head1, a.q_heads);
   const int warp_end = kSplit ? key_end : row_len(min(all_rows - 1, r_base + warp * 16 + 15));   // keys any row of the warp sees
   const int unmasked_end = min(row_len(r_base + (kSplit ? 0 : warp * 16)), key_end);   // keys every row of the warp sees
+  const int masked_before = row_len(min(all_rows - 1, r_base + (kSplit ? 15 : warp * 16 + 15))) - window;   // from here on no row's window ends
   float o[kD / 8][4];
 #pragma unroll
   for (int j = 0; j < kD / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
@@ -137,6 +140,17 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
           const float at = static_cast<float>(n * 8 + e);
           s[n][e] = fmaf(s[n][e], rs0, fmaf(slope0, at, first0));
           s[n][2 + e] = fmaf(s[n][2 + e], rs1, fmaf(slope1, at, first1));
+        }
+      }
+      if (first_key < masked_before) {                  // the window's lower edge crosses the stage
+        const int skip0 = len0 - window - first_key - 2 * t, skip1 = len1 - window - first_key - 2 * t;
+#pragma unroll
+        for (int n = 0; n < kMine / 8; ++n) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            if (n * 8 + e < skip0) s[n][e] = -INFINITY;
+            if (n * 8 + e < skip1) s[n][2 + e] = -INFINITY;
+          }
         }
       }
       if (first_key + kMine > unmasked_end) {

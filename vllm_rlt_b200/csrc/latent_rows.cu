@@ -1,0 +1,227 @@
+// Rows of latent attention: a token's keys and values are kept as one latent vector c (normed) and one rotated key part
+// shared by all heads, side by side in one cache row [c | r].
+//
+//   latent_write_kernel   the stacked down projections of a row: the query latent normed into the next GEMM's operand,
+//                         the key/value latent normed and the key part rotated into the row's page
+//   rotate_heads_kernel   the rotated part of every query head, in place or into another operand
+//   latent_gather_kernel  the cache rows of a range of positions of every sequence, side by side: what a prompt expands
+//                         into keys and values
+//
+// Rotation: dimensions 2i and 2i + 1 are a pair, turned by position * frequency_i.  The product is formed and reduced to one
+// turn in double, so that angles far into a sequence keep 32-bit precision.
+#include <math.h>
+
+#include "layer_math.cuh"
+
+namespace rlt {
+namespace {
+
+constexpr int kThreads = 256;
+
+__device__ __forceinline__ void rotation(int position, double frequency, float* cosine, float* sine) {
+  constexpr double kTurn = 6.283185307179586476925286766559;
+  double angle = static_cast<double>(position) * frequency;
+  angle -= rint(angle * (1.0 / kTurn)) * kTurn;
+  sincosf(static_cast<float>(angle), sine, cosine);
+}
+
+__device__ __forceinline__ float block_sum(float v, float* scratch) {
+#pragma unroll
+  for (int x = 16; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  v = (threadIdx.x & 31) < kThreads / 32 ? scratch[threadIdx.x & 31] : 0.0f;
+#pragma unroll
+  for (int x = 4; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
+  return __shfl_sync(0xffffffffu, v, 0);
+}
+
+struct LatentArgs {
+  const void* proj; int64_t proj_stride;
+  int q_col, q_rank, kv_col, kv_rank, rot_dim, rot_dims;   // rot_dims of the rot_dim are turned
+  const float* q_weight; const float* kv_weight; float eps;
+  const double* frequencies;
+  void* q_out; int64_t q_out_stride;
+  void* cache; int64_t block_stride, token_stride, num_blocks; int block_size;
+  const int32_t* tables; int table_width; const int32_t* row_seq; const int32_t* positions;
+};
+
+// blockIdx.y 0: the cache row, 1: the query latent.
+template <typename T, int kVec>
+__global__ void __launch_bounds__(kThreads)
+latent_write_kernel(LatentArgs a) {
+  __shared__ float scratch[kThreads / 32];
+  const int row = blockIdx.x;
+  const bool query = blockIdx.y == 1;
+  const T* proj = static_cast<const T*>(a.proj) + row * a.proj_stride + (query ? a.q_col : a.kv_col);
+  const float* weight = query ? a.q_weight : a.kv_weight;
+  const int width = query ? a.q_rank : a.kv_rank;
+  T* dst;
+  int position = 0;
+  if (query) {
+    dst = static_cast<T*>(a.q_out) + row * a.q_out_stride;
+  } else {
+    const int seq = a.row_seq[row];
+    if (seq < 0) return;                      // a padding row of a captured step
+    position = a.positions[row];
+    const int page_index = position / a.block_size;
+    if (position < 0 || page_index >= a.table_width) return;
+    const int64_t page = a.tables[static_cast<int64_t>(seq) * a.table_width + page_index];
+    if (page < 0 || page >= a.num_blocks) return;
+    dst = static_cast<T*>(a.cache) + page * a.block_stride + (position % a.block_size) * a.token_stride;
+  }
+  float ss = 0.0f;
+  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
+    float v[kVec];
+    load_floats<T, kVec>(proj + i, v);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) ss = fmaf(v[e], v[e], ss);
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + a.eps);
+  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
+    float v[kVec], w[kVec];
+    load_floats<T, kVec>(proj + i, v);
+    load_floats<float, kVec>(weight + i, w);
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) v[e] *= r * w[e];
+    store_floats<T, kVec>(dst + i, v);
+  }
+  if (query) return;
+  const T* part = proj + a.kv_rank;
+  for (int i = threadIdx.x; 2 * i < a.rot_dim; i += kThreads) {
+    const int d = 2 * i;
+    float u = Elem<T>::to_float(part[d]), v = d + 1 < a.rot_dim ? Elem<T>::to_float(part[d + 1]) : 0.0f;
+    if (d < a.rot_dims) {
+      float c, s;
+      rotation(position, a.frequencies[i], &c, &s);
+      const float u0 = u;
+      u = u0 * c - v * s;
+      v = v * c + u0 * s;
+    }
+    dst[a.kv_rank + d] = Elem<T>::from_float(u);
+    if (d + 1 < a.rot_dim) dst[a.kv_rank + d + 1] = Elem<T>::from_float(v);
+  }
+}
+
+// One CTA per row: the row's angles once, then every head's pairs.
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+rotate_heads_kernel(const T* src, int64_t src_row, int64_t src_head, T* dst, int64_t dst_row, int64_t dst_head, int heads, int dim,
+                    int rot_dims, const double* __restrict__ frequencies, const int32_t* __restrict__ positions) {
+  extern __shared__ float2 turns[];
+  const int64_t row = blockIdx.x;
+  for (int i = threadIdx.x; i < rot_dims / 2; i += kThreads) rotation(positions[row], frequencies[i], &turns[i].x, &turns[i].y);
+  __syncthreads();
+  const int pairs = (dim + 1) / 2;
+  for (int i = threadIdx.x; i < heads * pairs; i += kThreads) {
+    const int head = i / pairs, d = 2 * (i % pairs);
+    const T* from = src + row * src_row + head * src_head + d;
+    T* to = dst + row * dst_row + head * dst_head + d;
+    float u = Elem<T>::to_float(from[0]), v = d + 1 < dim ? Elem<T>::to_float(from[1]) : 0.0f;
+    if (d < rot_dims) {
+      const float2 t = turns[d / 2];
+      const float u0 = u;
+      u = u0 * t.x - v * t.y;
+      v = v * t.x + u0 * t.y;
+    }
+    to[0] = Elem<T>::from_float(u);
+    if (d + 1 < dim) to[1] = Elem<T>::from_float(v);
+  }
+}
+
+// One warp per gathered row, kBytes per lane and access.
+template <typename V>
+__global__ void __launch_bounds__(kThreads)
+latent_gather_kernel(const unsigned char* __restrict__ cache, int64_t block_bytes, int64_t token_bytes, int64_t num_blocks, int block_size,
+                     int row_bytes, const int32_t* __restrict__ tables, int table_width, const int32_t* __restrict__ first,
+                     const int32_t* __restrict__ cu, int sequences, int rows, unsigned char* __restrict__ out) {
+  const int row = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  int lo = 0, hi = sequences - 1;             // last sequence with cu <= row
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu[mid] <= row) lo = mid; else hi = mid - 1;
+  }
+  const int position = first[lo] + row - cu[lo];
+  const int page_index = position / block_size;
+  int64_t page = -1;
+  if (position >= 0 && page_index < table_width) page = tables[static_cast<int64_t>(lo) * table_width + page_index];
+  const bool live = page >= 0 && page < num_blocks;
+  const V* src = reinterpret_cast<const V*>(cache + (live ? page * block_bytes + (position % block_size) * token_bytes : 0));
+  V* dst = reinterpret_cast<V*>(out + static_cast<int64_t>(row) * row_bytes);
+  const int count = row_bytes / static_cast<int>(sizeof(V));
+  for (int i = lane; i < count; i += 32) dst[i] = live ? src[i] : V{};
+}
+
+}  // namespace
+}  // namespace rlt
+
+extern "C" RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, int q_col, int q_rank, int kv_col, int kv_rank,
+                                        int rot_dim, int rot_dims, const float* q_weight, const float* kv_weight, float eps,
+                                        const double* frequencies, void* q_out, int64_t q_out_stride, void* cache, int64_t block_stride,
+                                        int64_t token_stride, int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
+                                        const int32_t* row_seq, const int32_t* positions, int rows, int dtype, rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype_valid(dtype), "latent_write: dtype must be float32, float16 or bfloat16");
+  RLT_REQUIRE(rows >= 0 && q_rank >= 0 && kv_rank > 0 && rot_dim >= 0 && rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0 && eps >= 0.0f,
+              "latent_write: invalid shape");
+  if (rows == 0) return RLT_OK;
+  RLT_REQUIRE(proj && kv_weight && cache && tables && row_seq && positions && block_size > 0 && table_width > 0 && num_blocks > 0,
+              "latent_write: null pointer or empty cache");
+  RLT_REQUIRE(q_rank == 0 || (q_weight && q_out), "latent_write: the query latent needs a weight and an output");
+  RLT_REQUIRE(rot_dims == 0 || frequencies, "latent_write: rotation needs frequencies");
+  RLT_REQUIRE(token_stride >= kv_rank + rot_dim && block_stride >= token_stride * block_size, "latent_write: cache rows overlap");
+  LatentArgs a;
+  a.proj = proj; a.proj_stride = proj_stride; a.q_col = q_col; a.q_rank = q_rank; a.kv_col = kv_col; a.kv_rank = kv_rank;
+  a.rot_dim = rot_dim; a.rot_dims = rot_dims; a.q_weight = q_weight; a.kv_weight = kv_weight; a.eps = eps; a.frequencies = frequencies;
+  a.q_out = q_out; a.q_out_stride = q_out_stride; a.cache = cache; a.block_stride = block_stride; a.token_stride = token_stride;
+  a.num_blocks = num_blocks; a.block_size = block_size; a.tables = tables; a.table_width = table_width; a.row_seq = row_seq; a.positions = positions;
+  const dim3 grid(static_cast<unsigned>(rows), q_rank > 0 ? 2u : 1u);
+  const size_t bytes = 4 * dtype_size(dtype);
+  auto aligned = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
+  bool wide = proj_stride % 4 == 0 && q_col % 4 == 0 && q_rank % 4 == 0 && kv_col % 4 == 0 && kv_rank % 4 == 0 && block_stride % 4 == 0 &&
+              token_stride % 4 == 0 && q_out_stride % 4 == 0 && aligned(proj) && aligned(q_out) && aligned(cache) && aligned16(q_weight) && aligned16(kv_weight);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  RLT_DISPATCH_DTYPE(dtype, T, {
+    if (wide) latent_write_kernel<T, 4><<<grid, kThreads, 0, s>>>(a);
+    else latent_write_kernel<T, 1><<<grid, kThreads, 0, s>>>(a);
+  });
+  return launch_status("latent_write_kernel");
+}
+
+extern "C" RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head, void* dst, int64_t dst_row, int64_t dst_head,
+                                        int heads, int dim, int rot_dims, const double* frequencies, const int32_t* positions, int rows,
+                                        int dtype, rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype_valid(dtype), "rotate_heads: dtype must be float32, float16 or bfloat16");
+  RLT_REQUIRE(rows >= 0 && heads > 0 && dim >= 0 && rot_dims >= 0 && rot_dims <= dim && rot_dims % 2 == 0 && rot_dims <= 4096, "rotate_heads: invalid shape");
+  if (rows == 0 || dim == 0) return RLT_OK;
+  RLT_REQUIRE(src && dst && positions && (frequencies || rot_dims == 0), "rotate_heads: null pointer");
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const size_t smem = static_cast<size_t>(rot_dims / 2) * sizeof(float2);
+  RLT_DISPATCH_DTYPE(dtype, T, (rotate_heads_kernel<T><<<rows, kThreads, smem, s>>>(static_cast<const T*>(src), src_row, src_head, static_cast<T*>(dst),
+                                dst_row, dst_head, heads, dim, rot_dims, frequencies, positions)));
+  return launch_status("rotate_heads_kernel");
+}
+
+extern "C" RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks, int block_size,
+                                         int row_width, const int32_t* tables, int table_width, const int32_t* first, const int32_t* cu,
+                                         int sequences, int rows, void* out, int dtype, rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype_valid(dtype), "latent_gather: dtype must be float32, float16 or bfloat16");
+  RLT_REQUIRE(rows >= 0 && row_width > 0 && block_size > 0 && num_blocks > 0 && sequences >= 0 && table_width > 0, "latent_gather: invalid shape");
+  if (rows == 0) return RLT_OK;
+  RLT_REQUIRE(cache && tables && first && cu && out && sequences > 0, "latent_gather: null pointer");
+  const int64_t size = static_cast<int64_t>(dtype_size(dtype));
+  const int64_t block_bytes = block_stride * size, token_bytes = token_stride * size;
+  const int row_bytes = static_cast<int>(row_width * size);
+  const unsigned grid = static_cast<unsigned>((rows + kThreads / 32 - 1) / (kThreads / 32));
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const unsigned char* from = static_cast<const unsigned char*>(cache);
+  unsigned char* to = static_cast<unsigned char*>(out);
+  if (row_bytes % 16 == 0 && block_bytes % 16 == 0 && token_bytes % 16 == 0 && aligned16(cache) && aligned16(out))
+    latent_gather_kernel<uint4><<<grid, kThreads, 0, s>>>(from, block_bytes, token_bytes, num_blocks, block_size, row_bytes, tables, table_width, first, cu, sequences, rows, to);
+  else
+    latent_gather_kernel<uint16_t><<<grid, kThreads, 0, s>>>(from, block_bytes, token_bytes, num_blocks, block_size, row_bytes, tables, table_width, first, cu, sequences, rows, to);
+  return launch_status("latent_gather_kernel");
+}

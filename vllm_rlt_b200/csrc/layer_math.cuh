@@ -7,8 +7,8 @@
 
 namespace rlt {
 
-enum Activation { kActGeluErf = 1, kActGeluTanh = 2 };
-inline bool act_valid(int act) { return act == kActGeluErf || act == kActGeluTanh; }
+enum Activation { kActGeluErf = 1, kActGeluTanh = 2, kActSilu = 3, kActSquaredRelu = 4 };
+inline bool act_valid(int act) { return act >= kActGeluErf && act <= kActSquaredRelu; }
 
 __device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }   // a few ulp; 0 far on the left
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
@@ -19,6 +19,12 @@ __device__ __forceinline__ float erf_approx(float x) {
   return copysignf(fmaf(-p, __expf(-z * z), 1.0f), x);
 }
 
+// 32-bit results take the full exponential, 16-bit ones the fast one.
+template <typename T>
+__device__ __forceinline__ float sigmoid(float x) {
+  return sizeof(T) == 4 ? 1.0f / (1.0f + expf(-x)) : __fdividef(1.0f, 1.0f + __expf(-x));
+}
+
 // The activation of a value stored as T: 16-bit results do not show erf's last digits, 32-bit ones take erff.
 template <typename T>
 __device__ __forceinline__ float activate(float x, int act) {
@@ -26,6 +32,8 @@ __device__ __forceinline__ float activate(float x, int act) {
     const float u = x * 0.70710678118654752f;
     return 0.5f * x * (1.0f + (sizeof(T) == 4 ? erff(u) : erf_approx(u)));
   }
+  if (act == kActSilu) return x * sigmoid<T>(x);
+  if (act == kActSquaredRelu) { const float r = fmaxf(x, 0.0f); return r * r; }
   return 0.5f * x * (1.0f + tanhf(0.79788456080286536f * (x + 0.044715f * x * x * x)));
 }
 

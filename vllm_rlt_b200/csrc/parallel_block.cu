@@ -6,7 +6,8 @@
 //                          the tail of one layer and the head of the next in one pass over the row
 //   block_epilogue_kernel  columns of the stacked input projection: keys and values to their pages,
 //                          the feed-forward columns through their activation into the stacked output operand
-//   gated_norm_kernel      y * silu(z), RMS-normed in equal parts, into the stacked output operand
+//   gated_norm_kernel      y * silu(z), RMS-normed in equal parts, into the stacked output operand; or y RMS-normed first
+//                          and gated by sigmoid(z) behind the norm
 //
 // All three are streaming kernels: every input is read once and every output written once.  Sums, norms
 // and activations are fp32; only the stored operand of the next GEMM is rounded to the model dtype.
@@ -119,7 +120,7 @@ block_epilogue_kernel(EpilogueArgs a) {
   }
 }
 
-template <typename T, int kVec>
+template <typename T, int kVec, bool kGateBehind>
 __global__ void __launch_bounds__(kThreads)
 gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z, int64_t z_stride,
                   const float* __restrict__ weight, T* __restrict__ out, int64_t out_stride, int part, float eps) {
@@ -133,10 +134,10 @@ gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict
   for (int i = threadIdx.x * kVec; i < part; i += kThreads * kVec) {
     float v[kVec], g[kVec];
     load_floats<T, kVec>(yr + i, v);
-    load_floats<T, kVec>(zr + i, g);
+    if (!kGateBehind) load_floats<T, kVec>(zr + i, g);
 #pragma unroll
     for (int e = 0; e < kVec; ++e) {
-      v[e] *= silu(g[e]);
+      if (!kGateBehind) v[e] *= silu(g[e]);
       ss = fmaf(v[e], v[e], ss);
     }
     store_floats<float, kVec>(row_values + i, v);
@@ -149,6 +150,12 @@ gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict
     load_floats<float, kVec>(weight + first + i, w);
 #pragma unroll
     for (int e = 0; e < kVec; ++e) v[e] *= r * w[e];
+    if (kGateBehind) {
+      float g[kVec];
+      load_floats<T, kVec>(zr + i, g);
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) v[e] *= sigmoid<T>(g[e]);
+    }
     store_floats<T, kVec>(dst + i, v);
   }
 }
@@ -231,8 +238,8 @@ extern "C" RLT_API int rlt_block_epilogue(const void* proj, int64_t proj_stride,
 }
 
 extern "C" RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight,
-                                      void* out, int64_t out_stride, int rows, int width, int parts, float eps, int dtype,
-                                      rlt_stream_t stream) {
+                                      void* out, int64_t out_stride, int rows, int width, int parts, float eps, int gate_behind,
+                                      int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "gated_norm: dtype must be float32, float16 or bfloat16");
   RLT_REQUIRE(rows >= 0 && width > 0 && parts > 0 && width % parts == 0 && eps >= 0.0f, "gated_norm: the width must be a whole number of parts");
@@ -249,10 +256,13 @@ extern "C" RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const voi
   const size_t bytes = 4 * dtype_size(dtype);
   auto aligned = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
   const bool wide = part % 4 == 0 && y_stride % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 && aligned(y) && aligned(z) && aligned(out) && aligned16(weight);
-#define RLT_LAUNCH(T, V)                                                                                                  \
-  gated_norm_kernel<T, V><<<grid, kThreads, smem, s>>>(static_cast<const T*>(y), y_stride, static_cast<const T*>(z),       \
+#define RLT_LAUNCH(T, V, G)                                                                                               \
+  gated_norm_kernel<T, V, G><<<grid, kThreads, smem, s>>>(static_cast<const T*>(y), y_stride, static_cast<const T*>(z),    \
       z_stride, weight, static_cast<T*>(out), out_stride, part, eps)
-  RLT_DISPATCH_DTYPE(dtype, T, { if (wide) RLT_LAUNCH(T, 4); else RLT_LAUNCH(T, 1); });
+  RLT_DISPATCH_DTYPE(dtype, T, {
+    if (gate_behind) { if (wide) RLT_LAUNCH(T, 4, true); else RLT_LAUNCH(T, 1, true); }
+    else { if (wide) RLT_LAUNCH(T, 4, false); else RLT_LAUNCH(T, 1, false); }
+  });
 #undef RLT_LAUNCH
   return launch_status("gated_norm_kernel");
 }

@@ -115,7 +115,9 @@ scan_chunk_kernel(ScanArgs a) {
   };
   if (kOutput) publish_state();
 
-  const float rate = -kLog2e * expf(a.a_log[head]), dt_bias = a.dt_bias[head], skip = a.d[head];
+  const bool constant = a.decay != nullptr;        // dt = 1 and one decay per head
+  const float rate = constant ? a.decay[a.heads + head] : -kLog2e * expf(a.a_log[head]);
+  const float dt_bias = constant ? 0.0f : a.dt_bias[head], skip = constant ? 0.0f : a.d[head];
   const uint16_t* xg = static_cast<const uint16_t*>(a.x) + static_cast<int64_t>(head) * a.p + p0;
   const uint16_t* bg = static_cast<const uint16_t*>(a.b) + static_cast<int64_t>(group) * a.n;
   const uint16_t* cg = static_cast<const uint16_t*>(a.c) + static_cast<int64_t>(group) * a.n;
@@ -147,8 +149,9 @@ scan_chunk_kernel(ScanArgs a) {
     load_tile(&sm.x[0][0], kP + 8, kP, xg + row * a.xbc_stride, min(kP, a.p - p0), count);
     if (warp == 0) {   // step sizes and their running log-decay: two tokens per lane
       float d0 = 0.0f, d1 = 0.0f;
-      if (2 * lane < count) d0 = softplus(Elem<T>::to_float(dtg[(row + 2 * lane) * a.dt_stride]) + dt_bias);
-      if (2 * lane + 1 < count) d1 = softplus(Elem<T>::to_float(dtg[(row + 2 * lane + 1) * a.dt_stride]) + dt_bias);
+      if (constant) { d0 = 2 * lane < count ? 1.0f : 0.0f; d1 = 2 * lane + 1 < count ? 1.0f : 0.0f; }
+      else if (2 * lane < count) d0 = softplus(Elem<T>::to_float(dtg[(row + 2 * lane) * a.dt_stride]) + dt_bias);
+      if (!constant && 2 * lane + 1 < count) d1 = softplus(Elem<T>::to_float(dtg[(row + 2 * lane + 1) * a.dt_stride]) + dt_bias);
       const float l0 = rate * d0, l1 = rate * d1;
       float sum = l0 + l1;
 #pragma unroll

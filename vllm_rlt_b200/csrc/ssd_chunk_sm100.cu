@@ -127,7 +127,9 @@ scan_umma_kernel(ScanArgs a) {
   };
   if (kOutput) publish_state();
 
-  const float rate = -kLog2e * expf(a.a_log[head]), dt_bias = a.dt_bias[head], skip = a.d[head];
+  const bool constant = a.decay != nullptr;          // dt = 1 and one decay per head
+  const float rate = constant ? a.decay[a.heads + head] : -kLog2e * expf(a.a_log[head]);
+  const float dt_bias = constant ? 0.0f : a.dt_bias[head], skip = constant ? 0.0f : a.d[head];
   const T* xg = static_cast<const T*>(a.x) + static_cast<int64_t>(head) * a.p + p0;
   const T* bg = static_cast<const T*>(a.b) + static_cast<int64_t>(group) * a.n;
   const T* cg = static_cast<const T*>(a.c) + static_cast<int64_t>(group) * a.n;
@@ -167,7 +169,8 @@ scan_umma_kernel(ScanArgs a) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int token = 4 * lane + i;
-        dt[i] = token < count ? softplus(Elem<T>::to_float(dtg[(first_row + token) * a.dt_stride]) + dt_bias) : 0.0f;
+        if (constant) dt[i] = token < count ? 1.0f : 0.0f;
+        else dt[i] = token < count ? softplus(Elem<T>::to_float(dtg[(first_row + token) * a.dt_stride]) + dt_bias) : 0.0f;
         sum += rate * dt[i];
         l[i] = sum;
       }

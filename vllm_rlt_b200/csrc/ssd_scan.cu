@@ -17,6 +17,9 @@
 //                 A long sequence is also cut into segments that run side by side: a first launch computes what
 //                 every segment adds to the state (and its total decay), the second one starts each segment
 //                 from the folded contributions of those before it.
+//
+// Linear attention with a constant decay per head (S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t) is the same recurrence
+// with dt = 1, D = 0, B = k, C = q, x = v and one group per head: `decay` replaces what dt drives.
 #include "ssd_scan.cuh"
 
 namespace rlt {
@@ -67,12 +70,14 @@ scan_step_kernel(ScanArgs a, int tile_p, int lanes) {
       dst[i] = Elem<T>::to_float(i < a.n ? bp[(row0 + t) * a.xbc_stride + i] : cp[(row0 + t) * a.xbc_stride + i - a.n]);
   };
   stage(0);
-  const float rate = -expf(a.a_log[head]), dt_bias = a.dt_bias[head], skip = a.d[head];
+  const bool constant = a.decay != nullptr;
+  const float rate = constant ? 0.0f : -expf(a.a_log[head]), dt_bias = constant ? 0.0f : a.dt_bias[head], skip = constant ? 0.0f : a.d[head];
+  const float constant_decay = constant ? a.decay[head] : 0.0f;
   __syncthreads();
   for (int t = 0; t < count; ++t) {
     const int64_t row = row0 + t;
-    const float dt = softplus(Elem<T>::to_float(dtp[row * a.dt_stride]) + dt_bias);
-    const float decay = expf(rate * dt);
+    const float dt = constant ? 1.0f : softplus(Elem<T>::to_float(dtp[row * a.dt_stride]) + dt_bias);
+    const float decay = constant ? constant_decay : expf(rate * dt);
     const float* bt = staged + (t & 1) * 2 * a.n;
     const float* ct = bt + a.n;
     float* buffer = partial + (t & 1) * slices * tile_p;   // two buffers each: one barrier per token
@@ -166,6 +171,41 @@ extern "C" RLT_API size_t rlt_ssd_scan_workspace_bytes(int sequences, int max_to
   return static_cast<size_t>(sequences) * ((kMaxSegments + 1) * per_entry + kMaxSegments * heads * sizeof(float)) + 256;
 }
 
+namespace rlt {
+namespace {
+
+// The scan of checked arguments, on the kernels that its shape calls for.
+int run_scan(ScanArgs& a, int sequences, int max_tokens, int dtype, void* workspace, size_t workspace_bytes, cudaStream_t s) {
+  // workspace: an error word (256 bytes), then the segments'
+  a.error = (reinterpret_cast<uintptr_t>(workspace) & 15u) == 0 && workspace_bytes >= 256 ? static_cast<unsigned*>(workspace) : nullptr;
+  a.segments = nullptr; a.segment_decay = nullptr; a.segment_tokens = 1 << 30; a.segment_count = 1;
+  if (!chunked(max_tokens, a.n, dtype)) {
+    if (dtype == RLT_F32) return launch_step<float>(a, sequences, s);
+    return launch_step<__nv_bfloat16>(a, sequences, s);
+  }
+  DeviceInfo info;
+  const int status = current_device_info(&info);
+  if (status != RLT_OK) return status;
+  int count = segments_for(sequences, max_tokens, a.heads, a.p, info.sm_count);
+  if (max_tokens < 512) count = 1;
+  if (count > 1) {
+    if (workspace == nullptr || workspace_bytes < rlt_ssd_scan_workspace_bytes(sequences, max_tokens, a.heads, a.n, a.p, dtype) ||
+        (reinterpret_cast<uintptr_t>(workspace) & 15u) != 0) {
+      set_last_error_text("ssd_scan: workspace missing, misaligned or too small");
+      return RLT_ERR_WORKSPACE;
+    }
+    a.segment_count = count;
+    a.segment_tokens = ((max_tokens + count - 1) / count + 127) / 128 * 128;
+    a.segments = reinterpret_cast<float*>(static_cast<unsigned char*>(workspace) + 256);
+    a.segment_decay = a.segments + static_cast<size_t>(sequences) * (kMaxSegments + 1) * a.heads * a.n * a.p;
+  }
+  if (scan_umma_supported(a)) return launch_scan_umma(a, sequences, s);
+  return launch_scan_chunks(a, sequences, s);
+}
+
+}  // namespace
+}  // namespace rlt
+
 extern "C" RLT_API int rlt_ssd_scan(const void* x, const void* b, const void* c, int64_t xbc_stride, const void* dt,
                                     int64_t dt_stride, const float* dt_bias, const float* a_log, const float* d, void* y,
                                     int64_t y_stride, float* state, int64_t slots, const int32_t* cu_seqlens,
@@ -181,33 +221,26 @@ extern "C" RLT_API int rlt_ssd_scan(const void* x, const void* b, const void* c,
   RLT_REQUIRE(sequences <= 16384 && head_dim <= 256, "ssd_scan: batch or head size exceeds the grid limits");
   ScanArgs a;
   a.x = x; a.b = b; a.c = c; a.xbc_stride = xbc_stride; a.dt = dt; a.dt_stride = dt_stride;
-  a.dt_bias = dt_bias; a.a_log = a_log; a.d = d; a.y = y; a.y_stride = y_stride; a.state = state; a.slots = slots;
+  a.dt_bias = dt_bias; a.a_log = a_log; a.d = d; a.decay = nullptr; a.y = y; a.y_stride = y_stride; a.state = state; a.slots = slots;
   a.cu = cu_seqlens; a.starts = starts; a.slot_of = slot_of;
   a.heads = heads; a.groups = groups; a.n = state_size; a.p = head_dim;
-  // workspace: an error word (256 bytes), then the segments'
-  a.error = (reinterpret_cast<uintptr_t>(workspace) & 15u) == 0 && workspace_bytes >= 256 ? static_cast<unsigned*>(workspace) : nullptr;
-  a.segments = nullptr; a.segment_decay = nullptr; a.segment_tokens = 1 << 30; a.segment_count = 1;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (!chunked(max_tokens, state_size, dtype)) {
-    if (dtype == RLT_F32) return launch_step<float>(a, sequences, s);
-    return launch_step<__nv_bfloat16>(a, sequences, s);
-  }
-  DeviceInfo info;
-  const int status = current_device_info(&info);
-  if (status != RLT_OK) return status;
-  int count = segments_for(sequences, max_tokens, heads, head_dim, info.sm_count);
-  if (max_tokens < 512) count = 1;
-  if (count > 1) {
-    if (workspace == nullptr || workspace_bytes < rlt_ssd_scan_workspace_bytes(sequences, max_tokens, heads, state_size, head_dim, dtype) ||
-        (reinterpret_cast<uintptr_t>(workspace) & 15u) != 0) {
-      set_last_error_text("ssd_scan: workspace missing, misaligned or too small");
-      return RLT_ERR_WORKSPACE;
-    }
-    a.segment_count = count;
-    a.segment_tokens = ((max_tokens + count - 1) / count + 127) / 128 * 128;
-    a.segments = reinterpret_cast<float*>(static_cast<unsigned char*>(workspace) + 256);
-    a.segment_decay = a.segments + static_cast<size_t>(sequences) * (kMaxSegments + 1) * heads * state_size * head_dim;
-  }
-  if (scan_umma_supported(a)) return launch_scan_umma(a, sequences, s);
-  return launch_scan_chunks(a, sequences, s);
+  return run_scan(a, sequences, max_tokens, dtype, workspace, workspace_bytes, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" RLT_API int rlt_decay_scan(const void* q, const void* k, const void* v, int64_t qkv_stride, const float* decay, void* out,
+                                      int64_t out_stride, float* state, int64_t slots, const int32_t* cu_seqlens, const int32_t* starts,
+                                      const int32_t* slot_of, int sequences, int max_tokens, int heads, int key_dim, int value_dim,
+                                      int dtype, void* workspace, size_t workspace_bytes, rlt_stream_t stream) {
+  using namespace rlt;
+  RLT_REQUIRE(dtype == RLT_F32 || dtype == RLT_BF16, "decay_scan: dtype must be float32 or bfloat16");
+  RLT_REQUIRE(sequences >= 0 && max_tokens >= 0 && heads > 0 && key_dim > 0 && value_dim > 0 && slots > 0, "decay_scan: sizes must be positive");
+  if (sequences == 0 || max_tokens == 0) return RLT_OK;
+  RLT_REQUIRE(q && k && v && decay && out && state && cu_seqlens && starts && slot_of, "decay_scan: null pointer");
+  RLT_REQUIRE(sequences <= 16384 && value_dim <= 256, "decay_scan: batch or head size exceeds the grid limits");
+  ScanArgs a;
+  a.x = v; a.b = k; a.c = q; a.xbc_stride = qkv_stride; a.dt = nullptr; a.dt_stride = 0;
+  a.dt_bias = nullptr; a.a_log = nullptr; a.d = nullptr; a.decay = decay;
+  a.y = out; a.y_stride = out_stride; a.state = state; a.slots = slots; a.cu = cu_seqlens; a.starts = starts; a.slot_of = slot_of;
+  a.heads = heads; a.groups = heads; a.n = key_dim; a.p = value_dim;
+  return run_scan(a, sequences, max_tokens, dtype, workspace, workspace_bytes, static_cast<cudaStream_t>(stream));
 }

@@ -12,6 +12,7 @@ struct ScanArgs {
   int64_t xbc_stride;
   const void* dt; int64_t dt_stride;             // raw step sizes [rows, heads]
   const float* dt_bias; const float* a_log; const float* d;
+  const float* decay;                            // [2][heads]: constant decays and their log2; dt and the four above are null then
   void* y; int64_t y_stride;                     // [rows, heads * P]
   float* state; int64_t slots;                   // [slots][heads][N][P]
   const int32_t* cu; const int32_t* starts; const int32_t* slot_of;

@@ -31,6 +31,27 @@ class StepEntry:
 
 
 @dataclass
+class KeyRanges:
+    """Positions `first[s]` .. of every sequence, packed: those of sequence s are rows cu[s] .. cu[s + 1] - 1."""
+
+    first: torch.Tensor      # int32 [n]
+    cu: torch.Tensor         # int32 [n + 1]
+    rows: int
+
+    @classmethod
+    def of(cls, portions, window: int, device) -> "KeyRanges":
+        first = [max(start - window + 1, 0) if window else 0 for start, _ in portions]
+        cu = [0]
+        for f, (start, n) in zip(first, portions):
+            cu.append(cu[-1] + start + n - f)
+        host = torch.tensor(first + cu, dtype=torch.int32)
+        if device.type == "cuda":
+            host = host.pin_memory()
+        both = host.to(device, non_blocking=True)
+        return cls(both[:len(first)], both[len(first):], cu[-1])
+
+
+@dataclass
 class StepGroup:
     """Consecutive sequences of a step that take the same kernels."""
 
@@ -43,6 +64,14 @@ class StepGroup:
     lengths: torch.Tensor    # int32 [n], tokens of the sequence after the step (0: padding)
     slots: torch.Tensor      # int32 [n]
     tables: torch.Tensor     # int32 [n, pages] of plane 0
+    portions: list | None = None   # host side: (start, tokens) of every sequence; None in a captured step
+    _ranges: dict = field(default_factory=dict)
+
+    def key_ranges(self, window: int) -> "KeyRanges":
+        """The positions the group's rows see in a layer with this window (0: all), for kernels that want them packed."""
+        if window not in self._ranges:
+            self._ranges[window] = KeyRanges.of(self.portions, window, self.cu.device)
+        return self._ranges[window]
 
 
 @dataclass
@@ -55,6 +84,7 @@ class StepBatch:
     tokens: torch.Tensor     # int64 [rows]
     positions: torch.Tensor  # int32 [rows]
     row_seq: torch.Tensor    # int32 [rows], -1 for padding rows
+    previous: torch.Tensor   # int32 [rows], the token before each row's, -1 for the first of a sequence
     cu: torch.Tensor
     starts: torch.Tensor
     lengths: torch.Tensor
@@ -70,7 +100,7 @@ class _Layout:
         self.rows, self.sequences, self.planes, self.width, self.short = rows, sequences, planes, width, short
         at = 0
         self.at = {}
-        for name, size in (("tokens", 2 * rows), ("positions", rows), ("row_seq", rows), ("cu", sequences + 1),
+        for name, size in (("tokens", 2 * rows), ("positions", rows), ("row_seq", rows), ("previous", rows), ("cu", sequences + 1),
                            ("long_cu", sequences - short + 1), ("starts", sequences), ("lengths", sequences),
                            ("slots", sequences), ("tables", planes * sequences * width)):
             self.at[name] = slice(at, at + size)
@@ -92,8 +122,8 @@ class _Layout:
         if self.sequences > n:
             groups.append(StepGroup(self.sequences - n, long_max, slice(short_rows, self.rows), v["cu"][n:], v["long_cu"],
                                     v["starts"][n:], v["lengths"][n:], v["slots"][n:], v["tables"][0, n:]))
-        return StepBatch(self.rows, self.sequences, max(short_max, long_max), v["tokens"], v["positions"], v["row_seq"], v["cu"],
-                         v["starts"], v["lengths"], v["slots"], v["tables"], groups)
+        return StepBatch(self.rows, self.sequences, max(short_max, long_max), v["tokens"], v["positions"], v["row_seq"], v["previous"],
+                         v["cu"], v["starts"], v["lengths"], v["slots"], v["tables"], groups)
 
 
 class Engine:
@@ -147,7 +177,7 @@ class Engine:
         decode = self.cuda_graphs and all(len(e.tokens) == 1 for e in ordered)
         logits = self._decode_step(ordered) if decode else self._eager_step(ordered, entries)
         for e in entries:
-            self.cache.advance(e.name, len(e.tokens))
+            self.cache.advance(e.name, len(e.tokens), e.tokens[-1])
         self.steps += 1
         if decode:
             picked = [i for i, e in enumerate(entries) for _ in e.want]
@@ -176,12 +206,13 @@ class Engine:
 
     def _fill(self, layout: _Layout, host: torch.Tensor, entries) -> None:
         cache, v = self.cache, layout.views(host)
-        rows, tokens, positions, row_seq, cu, starts, lengths, slots = 0, [], [], [], [0], [], [], []
+        rows, tokens, positions, row_seq, previous, cu, starts, lengths, slots = 0, [], [], [], [], [0], [], [], []
         for i, e in enumerate(entries):
             n, start = len(e.tokens), cache.length(e.name)
             tokens += e.tokens
             positions += range(start, start + n)
             row_seq += [i] * n
+            previous += [cache.last_token(e.name), *e.tokens[:-1]]
             rows += n
             cu.append(rows)
             starts.append(start)
@@ -191,10 +222,10 @@ class Engine:
                 pages = cache.pages(e.name, plane)[:layout.width]
                 v["tables"][plane, i, :len(pages)] = torch.tensor(pages, dtype=torch.int32)
         for _ in range(layout.sequences - len(entries)):     # padding sequences of one row
-            tokens.append(0); positions.append(0); row_seq.append(-1); starts.append(0); lengths.append(0)
+            tokens.append(0); positions.append(0); row_seq.append(-1); previous.append(-1); starts.append(0); lengths.append(0)
             slots.append(cache.dummy_slot)
             cu.append(cu[-1] + 1)
-        for name, values in (("tokens", tokens), ("positions", positions), ("row_seq", row_seq), ("cu", cu), ("starts", starts),
+        for name, values in (("tokens", tokens), ("positions", positions), ("row_seq", row_seq), ("previous", previous), ("cu", cu), ("starts", starts),
                              ("lengths", lengths), ("slots", slots)):
             v[name].copy_(torch.tensor(values))
         base = cu[layout.short]
@@ -213,8 +244,12 @@ class Engine:
         layout = _Layout(sum(counts), len(ordered), cache.spec.planes, width, short)
         host = self._host_buffer(layout.size)
         self._fill(layout, host, ordered)
-        return layout.batch(host.to(self.device, non_blocking=True), sum(counts[:short]), max(counts[:short], default=0),
-                            max(counts[short:], default=0))
+        batch = layout.batch(host.to(self.device, non_blocking=True), sum(counts[:short]), max(counts[:short], default=0),
+                             max(counts[short:], default=0))
+        portions = [(cache.length(e.name), n) for e, n in zip(ordered, counts)]
+        for group in batch.groups:
+            group.portions, portions = portions[:group.sequences], portions[group.sequences:]
+        return batch
 
     def _eager_step(self, ordered, entries):
         hidden = self.model.forward_step(self._batch(ordered), self.cache)

@@ -18,7 +18,6 @@ softmax, recurrent state and everything that drives it are fp32; in float32 ever
 
 from __future__ import annotations
 
-from contextlib import contextmanager
 from dataclasses import dataclass
 
 import torch
@@ -26,28 +25,12 @@ import torch.nn.functional as F
 
 from .attention import B200PagedAttention, ScoreTerms
 from .layers import block_epilogue, residual_norm
+from .model_parts import check_positive, check_shapes, full_accumulation, stack_blocks, take_keys
 from .recurrent import causal_conv, gated_norm, ssd_scan
 from .sequence_cache import CacheSpec, KVSpec, StateSpec
 
 
 # ---- configuration -----------------------------------------------------------------------------
-def _take(entry: dict, what: str, required, optional=()) -> dict:
-    """The named keys of a config entry; a key nobody knows, unless it is off, is an error and not a guess."""
-    missing = [k for k in required if k not in entry]
-    if missing:
-        raise ValueError(f"{what}: config lacks {missing}")
-    unknown = [k for k, v in entry.items() if k not in required and k not in optional and v not in (None, False)]
-    if unknown:
-        raise ValueError(f"{what}: unknown config keys {unknown}")
-    return {k: entry.get(k) for k in (*required, *optional)}
-
-
-def _positive(what: str, **sizes) -> None:
-    for name, value in sizes.items():
-        if isinstance(value, bool) or not isinstance(value, int) or value < 1:
-            raise ValueError(f"{what}: {name} must be a positive integer")
-
-
 @dataclass(frozen=True)
 class AttentionConfig:
     heads: int
@@ -61,11 +44,11 @@ class AttentionConfig:
 
     @classmethod
     def from_json(cls, entry: dict, what: str) -> "AttentionConfig":
-        m = _take(entry, what, ("heads", "kv_heads", "dim", "vdim", "scale"), ("q_temp", "kv_from"))
-        _positive(what, heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"])
+        m = take_keys(entry, what, ("heads", "kv_heads", "dim", "vdim", "scale"), ("q_temp", "kv_from"))
+        check_positive(what, heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"])
         if m["heads"] % m["kv_heads"]:
             raise ValueError(f"{what}: heads must be a multiple of kv_heads")
-        temp = _take(m["q_temp"], what + " q_temp", ("coef", "every")) if m["q_temp"] else {"coef": 0.0, "every": 1}
+        temp = take_keys(m["q_temp"], what + " q_temp", ("coef", "every")) if m["q_temp"] else {"coef": 0.0, "every": 1}
         if int(temp["every"]) != temp["every"] or temp["every"] < 1:
             raise ValueError(f"{what}: q_temp.every must be a positive integer")
         return cls(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), float(temp["coef"]), int(temp["every"]),
@@ -87,8 +70,8 @@ class Mamba2Config:
 
     @classmethod
     def from_json(cls, entry: dict, what: str) -> "Mamba2Config":
-        m = _take(entry, what, ("heads", "vdim", "state", "groups", "conv", "norm_groups"))
-        _positive(what, **m)
+        m = take_keys(entry, what, ("heads", "vdim", "state", "groups", "conv", "norm_groups"))
+        check_positive(what, **m)
         if m["heads"] % m["groups"] or m["heads"] * m["vdim"] % m["norm_groups"]:
             raise ValueError(f"{what}: heads must be a multiple of groups, and heads * vdim of norm_groups")
         return cls(**m)
@@ -120,20 +103,20 @@ class HybridLMConfig:
 
     @classmethod
     def from_json(cls, config: dict) -> "HybridLMConfig":
-        _positive("config", vocab=config.get("vocab"), width=config.get("width"))
+        check_positive("config", vocab=config.get("vocab"), width=config.get("width"))
         layers = []
         for i, entry in enumerate(config["layers"]):
             what = f"layer {i}"
-            entry = _take(entry, what, ("type", "mixer"), ("mlp",))
+            entry = take_keys(entry, what, ("type", "mixer"), ("mlp",))
             if entry["type"] not in MIXERS:
                 raise ValueError(f"{what}: unknown mixer type {entry['type']!r}; known: {', '.join(MIXERS)}")
             mixer = MIXERS[entry["type"]].from_json(entry["mixer"], what)
             ff = 0
             if entry["mlp"]:
-                mlp = _take(entry["mlp"], what + " mlp", ("ff",), ("kind",))
+                mlp = take_keys(entry["mlp"], what + " mlp", ("ff",), ("kind",))
                 if mlp["kind"] not in (None, "dense"):
                     raise ValueError(f"{what}: unknown feed-forward kind {mlp['kind']!r}")
-                _positive(what + " mlp", ff=mlp["ff"])
+                check_positive(what + " mlp", ff=mlp["ff"])
                 ff = mlp["ff"]
             layers.append(HybridLayerConfig(mixer, ff))
         built = cls(config["vocab"], config["width"], float(config["norm"]["eps"]), tuple(layers))
@@ -173,34 +156,6 @@ def parameter_shapes(config: HybridLMConfig) -> dict[str, tuple]:
 
 
 # ---- the model ---------------------------------------------------------------------------------
-def _aligned(columns: int) -> int:
-    """Column blocks of a stacked projection start at multiples of 8 elements (16 bytes in 16-bit types)."""
-    return -(-columns // 8) * 8
-
-
-def _stack(blocks, dim: int):
-    """Weights side by side along `dim`, each block padded with zeros to a multiple of 8; the blocks' offsets, and the total."""
-    parts, offsets, at = [], [], 0
-    for block in blocks:
-        pad = _aligned(block.shape[dim]) - block.shape[dim]
-        parts.append(block if not pad else F.pad(block, (0, pad) if dim == 1 else (0, 0, 0, pad)))
-        offsets.append(at)
-        at += block.shape[dim] + pad
-    return torch.cat(parts, dim).contiguous(), offsets, at
-
-
-@contextmanager
-def _full_accumulation():
-    """fp32 accumulation in every GEMM: no TF32 for 32-bit inputs, no 16-bit partial sums for 16-bit ones."""
-    m = torch.backends.cuda.matmul
-    saved = m.allow_tf32, m.allow_bf16_reduced_precision_reduction
-    m.allow_tf32, m.allow_bf16_reduced_precision_reduction = False, False
-    try:
-        yield
-    finally:
-        m.allow_tf32, m.allow_bf16_reduced_precision_reduction = saved
-
-
 class _Layer:
     """Stacked weights of one layer and where their columns lie."""
 
@@ -217,17 +172,17 @@ class _Layer:
             own = m.kv_from is None
             blocks = [take(p + "mix.q")] + ([take(p + "mix.k"), take(p + "mix.v")] if own else [])
             self.inner = m.heads * m.vdim
-            self.w_in, offsets, _ = _stack(blocks + up, 0)
+            self.w_in, offsets, _ = stack_blocks(blocks + up, 0)
             self.k_col, self.v_col = (offsets[1], offsets[2]) if own else (0, 0)
             self.terms = m.terms
         else:
             self.inner = m.inner
-            self.w_in, offsets, _ = _stack([take(p + "mix.in")] + up, 0)
+            self.w_in, offsets, _ = stack_blocks([take(p + "mix.in")] + up, 0)
             self.conv, self.conv_bias = take(p + "mix.conv", torch.float32), take(p + "mix.conv.b", torch.float32)
             self.dt_bias, self.a_log, self.d = (take(p + "mix." + n, torch.float32) for n in ("dt_bias", "A_log", "D"))
             self.gate_norm = take(p + "mix.norm", torch.float32)
         self.up_col = offsets[-1] if self.ff else 0
-        self.w_out, offsets, self.operand_width = _stack([take(p + "mix.o")] + down, 1)
+        self.w_out, offsets, self.operand_width = stack_blocks([take(p + "mix.o")] + down, 1)
         self.act_col = offsets[-1] if self.ff else 0
         self.padded = self.operand_width != self.inner + self.ff
 
@@ -243,13 +198,7 @@ class HybridLM:
         if dtype not in (torch.float32, torch.bfloat16):
             raise ValueError("HybridLM runs in float32 or bfloat16")
         self.config, self.device, self.dtype = config, torch.device(device), dtype
-        shapes = parameter_shapes(config)
-        missing = sorted(set(shapes) - set(state_dict))
-        if missing:
-            raise ValueError(f"state dict lacks {missing[:3]}{'...' if len(missing) > 3 else ''}")
-        for name, shape in shapes.items():
-            if tuple(state_dict[name].shape) != shape:
-                raise ValueError(f"{name} has shape {tuple(state_dict[name].shape)}, the configuration needs {shape}")
+        check_shapes(parameter_shapes(config), state_dict)
 
         def take(name, as_type=None):
             return state_dict[name].to(device=self.device, dtype=as_type or dtype).contiguous()
@@ -281,7 +230,7 @@ class HybridLM:
         the complete 32-bit residual after every layer (tests and debugging: it costs an addition per layer)."""
         residual = torch.empty(batch.rows, self.config.width, dtype=torch.float32, device=self.device)
         eps, delta = self.config.eps, None
-        with _full_accumulation(), self.attention.shared_plan():
+        with full_accumulation(), self.attention.shared_plan():
             for i, layer in enumerate(self.layers):
                 first = i == 0
                 h = residual_norm(residual, layer.norm, eps, self.dtype, delta=delta, tokens=batch.tokens if first else None,
@@ -327,7 +276,7 @@ class HybridLM:
     def step_logits(self, hidden, rows=None):
         """fp32 logits of the given rows (int64 indices; None: all)."""
         residual, delta = hidden
-        with _full_accumulation():
+        with full_accumulation():
             h = residual_norm(residual, self.final_norm, self.config.eps, self.dtype, delta=delta, row_index=rows,
                               weight_offset=self.norm_offset, store=False)
             if self.dtype == torch.float32:

@@ -101,7 +101,7 @@ def sandwich_norm(x, weight, eps: float, residual=None, weight2=None, *, in_plac
     return total, norm
 
 
-ACTIVATIONS = {"gelu": 1, "gelu_tanh": 2}      # the erf form and the tanh form
+ACTIVATIONS = {"gelu": 1, "gelu_tanh": 2, "silu": 3, "squared_relu": 4}      # gelu: the erf form
 
 
 def residual_norm(residual, weight, eps: float, dtype, *, delta=None, tokens=None, embed=None, row_index=None,
@@ -193,3 +193,81 @@ def block_epilogue(proj, batch, *, kv=None, act=None):
             _capi.ptr(None if kv is None else batch.positions), act_col, act_width, kind, _capi.ptr(out), out_stride, out_col,
             rows, _capi.DTYPE_CODES[proj.dtype], _capi.stream_of(proj))
     _capi.check(code, "block_epilogue")
+
+
+def stream_mix(streams, weight, eps: float, dtype, *, delta=None, parts=None, ran=None, follows=None, tokens=None, previous=None,
+               embed=None, bigram=None, embed_weight=None, row_index=None, weight_offset: float = 0.0, store: bool = True):
+    """Hyper-connected residual streams (float32 `[rows, S, width]`, updated in place) between two sublayers:
+
+        x_t <- sum_s mix[s, t] x_s + out[t] * y        ran = (out [S], mix [S, S]) of the sublayer whose output y is
+        u = sum_t in[t] x_t                            follows = in [S] of the next one (None: the plain sum)
+        returns rmsnorm(u) * (weight_offset + weight), in `dtype`
+
+    y is `delta` `[rows, width]`, or with parts = (rows, weights), both `[rows, k]`, the weighted sum of rows of `delta`.
+    With `tokens` the streams start: all of them `rmsnorm(embed[token] + table[bucket]) * embed_weight`, where
+    bigram = (table, mul_prev, mul_cur), the table's last row serves first tokens (`previous` < 0, int32 [rows]) and the
+    other rows are the buckets of `previous * mul_prev + token * mul_cur`.  `row_index` as in `residual_norm`."""
+    _capi.require_cuda(streams, weight, delta, tokens, previous, embed, embed_weight, row_index)
+    if streams.dim() != 3 or streams.dtype != torch.float32 or not streams.is_contiguous():
+        raise ValueError("streams must be contiguous float32 [rows, streams, width]")
+    rows, count, width = streams.shape
+    for name, w, shape in (("weight", weight, (width,)), ("embed_weight", embed_weight, (width,)), ("follows", follows, (count,)),
+                           ("out", ran[0] if ran else None, (count,)), ("mix", ran[1] if ran else None, (count, count))):
+        if w is not None and (w.dtype != torch.float32 or w.shape != shape or not w.is_contiguous()):
+            raise ValueError(f"{name} must be contiguous float32 {list(shape)}")
+    if dtype not in _capi.DTYPE_CODES or (ran is None) != (delta is None):
+        raise ValueError("dtype must be float32 / float16 / bfloat16; delta and ran go together")
+    k, part_rows, part_weights = 0, None, None
+    if delta is not None:
+        if delta.dtype != dtype or delta.dim() != 2 or delta.shape[1] != width or not delta.is_contiguous():
+            raise ValueError("delta must be contiguous [rows, width] of the model dtype")
+        if parts is not None:
+            part_rows, part_weights = parts
+            k = part_rows.shape[1]
+            if part_rows.dtype != torch.int32 or part_weights.dtype != torch.float32 or part_rows.shape != (rows, k) \
+                    or part_weights.shape != (rows, k) or not part_rows.is_contiguous() or not part_weights.is_contiguous():
+                raise ValueError("parts must be int32 rows and float32 weights, both contiguous [rows, k]")
+        elif delta.shape[0] != rows:
+            raise ValueError("delta needs one row per row of the streams")
+    table, buckets, mul_prev, mul_cur = None, 0, 0, 0
+    if tokens is not None:
+        if tokens.dtype != torch.int64 or tokens.shape != (rows,) or embed is None or embed.dtype != dtype or embed.dim() != 2 \
+                or embed.shape[1] != width or not embed.is_contiguous() or embed_weight is None:
+            raise ValueError("tokens must be int64 [rows], embed contiguous [vocab, width] of the model dtype, with a norm weight")
+        if bigram is not None:
+            table, mul_prev, mul_cur = bigram
+            buckets = table.shape[0] - 1
+            if table.dtype != dtype or table.dim() != 2 or table.shape[1] != width or not table.is_contiguous() or buckets < 1 \
+                    or previous is None or previous.dtype != torch.int32 or previous.shape != (rows,):
+                raise ValueError("the bigram table must be contiguous [buckets + 1, width] of the model dtype, previous int32 [rows]")
+    if row_index is not None:
+        if row_index.dtype != torch.int64 or row_index.dim() != 1 or store:
+            raise ValueError("row_index must be int64, and selected rows are not stored: pass store=False")
+        row_index = row_index.contiguous()
+    n = rows if row_index is None else row_index.numel()
+    out = torch.empty(n, width, dtype=dtype, device=streams.device)
+    if n == 0:
+        return out
+    with torch.cuda.device(streams.device):
+        code = _capi.load().rlt_stream_mix(
+            _capi.ptr(streams), count, _capi.ptr(delta), k, _capi.ptr(part_rows), _capi.ptr(part_weights),
+            _capi.ptr(ran[0] if ran else None), _capi.ptr(ran[1] if ran else None), _capi.ptr(tokens), _capi.ptr(previous),
+            _capi.ptr(embed), 0 if embed is None else embed.shape[0], _capi.ptr(table), buckets, int(mul_prev), int(mul_cur),
+            _capi.ptr(embed_weight), _capi.ptr(follows), _capi.ptr(row_index), int(store), _capi.ptr(weight), float(weight_offset),
+            _capi.ptr(out), n, width, float(eps), _capi.DTYPE_CODES[dtype], _capi.stream_of(streams))
+    _capi.check(code, "stream_mix")
+    return out
+
+
+def clamped_glu(gate_up, up_col: int, cols: int, limit: float, slope: float):
+    """`g * sigmoid(slope * g) * (u + 1)` with g = min(gate, limit), u = clamp(up, -limit, limit), over columns 0 .. and
+    `up_col` .. of one projection output; returns contiguous `[rows, cols]`."""
+    _capi.require_cuda(gate_up)
+    if gate_up.dim() != 2 or gate_up.stride(1) != 1 or gate_up.dtype not in _capi.DTYPE_CODES or up_col + cols > gate_up.shape[1]:
+        raise ValueError("gate_up must be [rows, columns] with unit inner stride that holds both halves")
+    out = torch.empty(gate_up.shape[0], cols, dtype=gate_up.dtype, device=gate_up.device)
+    with torch.cuda.device(gate_up.device):
+        code = _capi.load().rlt_clamped_glu(_capi.ptr(gate_up), gate_up.stride(0), up_col, _capi.ptr(out), out.stride(0), out.shape[0],
+                                            cols, float(limit), float(slope), _capi.DTYPE_CODES[gate_up.dtype], _capi.stream_of(gate_up))
+    _capi.check(code, "clamped_glu")
+    return out

@@ -1,5 +1,5 @@
 """Recurrent layers over packed sequences with per-sequence state slots: short causal convolution, the Mamba-2
-state-space recurrence, and the gated norm behind it.
+state-space recurrence, linear attention with constant decays, and the gated norm behind them.
 
 `group` arguments are a step's sequence group (`StepGroup`): `cu` (int32 [n + 1], row offsets into the step's
 rows), `starts` (position of each portion's first token), `slots`, and the host-side bound `max_new`.
@@ -81,8 +81,47 @@ def ssd_scan(x, b, c, dt, dt_bias, a_log, d, state, out, group):
     return out
 
 
-def gated_norm(y, z, weight, out, parts: int, eps: float):
-    """`out = rmsnorm(y * silu(z)) * weight`, the row normed in `parts` equal parts; all `[rows, width]`, any row stride."""
+def decay_scan(q, k, v, decay, state, out, group):
+    """Linear attention with a constant decay per head (`rlt_decay_scan`): `S_t = decay S_(t-1) + k_t v_t^T`, `out_t = S_t^T q_t`.
+
+    q, k `[rows, heads * key_dim]`, v, out `[rows, heads * value_dim]` (q, k and v slices of rows of one stride), decay float32
+    `[2, heads]` (`decay_table`), state float32 `[slots, heads, key_dim, value_dim]`, updated in place."""
+    device = _capi.require_cuda(q, k, v, decay, state, out, group.cu, group.starts, group.slots)
+    if state.dim() != 4 or state.dtype != torch.float32 or not state.is_contiguous():
+        raise ValueError("state must be contiguous float32 [slots, heads, key_dim, value_dim]")
+    slots, heads, key_dim, value_dim = state.shape
+    rows = q.shape[0]
+    if q.shape != (rows, heads * key_dim) or k.shape != q.shape or v.shape != (rows, heads * value_dim) or out.shape != v.shape:
+        raise ValueError("q / k [rows, heads * key_dim], v / out [rows, heads * value_dim]")
+    if q.stride(0) != k.stride(0) or k.stride(0) != v.stride(0) or any(t.stride(1) != 1 for t in (q, k, v, out)):
+        raise ValueError("q, k and v must be column slices of the same rows")
+    if q.dtype not in (torch.float32, torch.bfloat16) or any(t.dtype != q.dtype for t in (k, v, out)):
+        raise ValueError("q, k, v and out must share float32 or bfloat16")
+    if decay.dtype != torch.float32 or decay.shape != (2, heads) or not decay.is_contiguous():
+        raise ValueError("decay must be contiguous float32 [2, heads]")
+    if group.sequences == 0:
+        return out
+    lib, dtype = _capi.load(), _capi.DTYPE_CODES[q.dtype]
+    with torch.cuda.device(device):
+        nbytes = lib.rlt_ssd_scan_workspace_bytes(group.sequences, group.max_new, heads, key_dim, value_dim, dtype)
+        workspace = torch.empty(nbytes, dtype=torch.uint8, device=device)
+        code = lib.rlt_decay_scan(
+            _capi.ptr(q), _capi.ptr(k), _capi.ptr(v), q.stride(0), _capi.ptr(decay), _capi.ptr(out), out.stride(0), _capi.ptr(state),
+            slots, _capi.ptr(group.cu), _capi.ptr(group.starts), _capi.ptr(group.slots), group.sequences, group.max_new, heads, key_dim,
+            value_dim, dtype, _capi.ptr(workspace), nbytes, _capi.stream_of(q))
+    _capi.check(code, "decay_scan")
+    return out
+
+
+def decay_table(decays, device) -> torch.Tensor:
+    """The `[2, heads]` argument of `decay_scan`: decays and their base-2 logarithms (bounded below: a decay of zero forgets)."""
+    d = torch.tensor(decays, dtype=torch.float64)
+    return torch.stack([d, torch.log2(d.clamp_min(2.0 ** -100))]).to(device=device, dtype=torch.float32)
+
+
+def gated_norm(y, z, weight, out, parts: int, eps: float, *, gate_behind: bool = False):
+    """`out = rmsnorm(y * silu(z)) * weight`, or with `gate_behind` `rmsnorm(y) * weight * sigmoid(z)`; the row normed in
+    `parts` equal parts; all `[rows, width]`, any row stride."""
     device = _capi.require_cuda(y, z, weight, out)
     rows, width = y.shape
     if z.shape != y.shape or out.shape != y.shape or weight.shape != (width,) or weight.dtype != torch.float32 \
@@ -92,7 +131,7 @@ def gated_norm(y, z, weight, out, parts: int, eps: float):
         return out
     with torch.cuda.device(device):
         code = _capi.load().rlt_gated_norm(_capi.ptr(y), y.stride(0), _capi.ptr(z), z.stride(0), _capi.ptr(weight), _capi.ptr(out),
-                                           out.stride(0), rows, width, parts, float(eps), _capi.DTYPE_CODES[y.dtype],
+                                           out.stride(0), rows, width, parts, float(eps), int(gate_behind), _capi.DTYPE_CODES[y.dtype],
                                            _capi.stream_of(y))
     _capi.check(code, "gated_norm")
     return out

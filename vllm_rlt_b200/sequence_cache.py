@@ -17,7 +17,8 @@ import torch
 
 @dataclass(frozen=True)
 class KVSpec:
-    """One layer's pages: head count and the sizes of a key and of a value head."""
+    """One layer's pages: head count and the sizes of a key and of a value head (0: values are a part of the key row, as in
+    latent attention, and have no pages of their own)."""
 
     kv_heads: int
     key_dim: int
@@ -49,6 +50,7 @@ class _Sequence:
     slot: int
     pages: list            # one list of page ids per plane
     length: int = 0        # tokens stored
+    last: int = -1         # the last of them
 
 
 class SequenceCache:
@@ -75,7 +77,9 @@ class SequenceCache:
         else:
             for layer, kind in spec.layers.items():
                 shape = (self.num_pages, block, kind.kv_heads)
-                if kind.key_dim == kind.value_dim:      # one allocation: a page of both caches is one TMA copy
+                if kind.value_dim == 0:
+                    self.key[layer] = torch.zeros(*shape, kind.key_dim, device=device, dtype=dtype)
+                elif kind.key_dim == kind.value_dim:      # one allocation: a page of both caches is one TMA copy
                     both = torch.zeros(2, *shape, kind.key_dim, device=device, dtype=dtype)
                     self.key[layer], self.value[layer] = both[0], both[1]
                 else:
@@ -129,8 +133,13 @@ class SequenceCache:
         for pages in sequence.pages:
             pages.extend(self._free_pages.pop() for _ in range(need))
 
-    def advance(self, name, tokens: int) -> None:
+    def last_token(self, name) -> int:
+        """The last stored token, -1 before the first (-1 too when `advance` was not told)."""
+        return self._sequences[name].last
+
+    def advance(self, name, tokens: int, last: int = -1) -> None:
         self._sequences[name].length += tokens
+        self._sequences[name].last = last
 
     def release(self, name) -> None:
         """Give the sequence's pages and slot back.  Steps already queued on the stream run first: whoever gets
