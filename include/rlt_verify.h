@@ -530,6 +530,8 @@ RLT_API int rlt_sandwich_norm(const void* x, const void* weight, const void* res
  *             - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
  * softmax over the visible keys, weighted sum of the values.  Keys and values may have different head
  * sizes and cache strides; query and output rows may be column slices (strides in elements).
+ * window > 0: only keys with p - j < window.  value_cache may be key_cache with one KV head: a value is then the first value_dim
+ * elements of its key row.
  * context_lengths[s]: tokens of sequence s after this portion.  planned != 0: the workspace holds the
  * plan of rlt_verify_attention_plan for the same tables, lengths and packing (max_new <= 16 only). */
 RLT_API size_t rlt_scored_attention_workspace_bytes(int rows, int sequences, int max_new, int q_heads, int kv_heads,
@@ -626,6 +628,18 @@ RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head,
 RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks,
                       int block_size, int row_width, const int32_t* tables, int table_width, const int32_t* first,
                       const int32_t* cu, int sequences, int rows, void* out, int dtype, rlt_stream_t stream);
+
+/* Prompt attention of latent layers (bf16).  q [rows][heads][dim + rot_dim]; kv [key_rows][heads * dim | heads * vdim]: keys and
+ * values expanded from the latents; shared_keys [key_rows][rot_dim]: the rotated key part of all heads; out [rows][heads * vdim].
+ * Query position p sees positions p - window + 1 .. p (window 0: all before it).  tiles: eight int32 words per tile of up to 256
+ * consecutive query rows of a sequence: first query row, rows, position of the first row, packed key row of position f, f, 0, 0, 0
+ * (f: first position of the sequence among the packed keys).  workspace: 256 bytes; its first word is set when a bounded wait
+ * gave up.  Supported: bf16, dim and vdim up to 128, rot_dim up to 64, multiples of 8. */
+RLT_API int rlt_latent_prompt_supported(int dim, int rot_dim, int vdim, int dtype);
+RLT_API int rlt_latent_prompt_attention(const void* q, int64_t q_stride, const void* kv, int64_t kv_stride,
+                                const void* shared_keys, int64_t shared_stride, void* out, int64_t out_stride, int rows,
+                                int key_rows, int heads, int dim, int rot_dim, int vdim, const int32_t* tiles, int tile_count,
+                                float scale, int window, int dtype, void* workspace, rlt_stream_t stream);
 
 /* Mixture of experts.  route: s = softmax(logits) in fp32, the `top` largest of s + correction (null: none), weights =
  * chosen s / (their sum + floor_sum); counts [experts] must be zero before.  gather: rows sorted by expert, and every

@@ -207,6 +207,62 @@ def test_a_key_just_inside_a_window_is_found_and_one_just_outside_is_not(dtype, 
                 assert missed < 0.05 if distance < window else missed > 0.5
 
 
+PROMPTS = [([300], [300]), ([17, 64, 129], [17, 200, 129]), ([256, 257, 128], [300, 900, 128]), ([70], [700]), ([40, 600], [41, 600])]
+
+
+def expanded_case(portions, contexts, heads, dim, rot, vdim, window, seed, peak=None):
+    """Packed keys and values of what the portions see.  peak = distance: the last row of every portion finds the key that far back."""
+    g = torch.Generator().manual_seed(seed)
+    ranges = KeyRanges.of([(c - n, n) for c, n in zip(contexts, portions)], window, torch.device("cuda"))
+    q = [torch.randn(n, heads, dim + rot, generator=g).bfloat16() for n in portions]
+    k = [torch.randn(c, heads, dim, generator=g).bfloat16() for c in contexts]
+    r = [torch.randn(c, rot, generator=g).bfloat16() for c in contexts]
+    v = [torch.randn(c, heads, vdim, generator=g).bfloat16() for c in contexts]
+    if peak is not None:
+        for s, c in enumerate(contexts):
+            if c - 1 - peak >= 0:
+                direction = torch.randn(dim, generator=g)
+                direction /= direction.norm()
+                q[s][-1, :, :dim] = (12 * direction).bfloat16()
+                k[s][c - 1 - peak] = (12 * (dim + rot) ** 0.5 * direction).bfloat16()
+    first = ranges.first.tolist()
+    kv = torch.cat([torch.cat([k[s][first[s]:].flatten(1), v[s][first[s]:].flatten(1)], 1) for s in range(len(contexts))])
+    shared = torch.cat([torch.cat([torch.full((contexts[s] - first[s], 8), float("nan")).bfloat16(), r[s][first[s]:]], 1) for s in range(len(contexts))])
+    out = torch.full((sum(portions), heads, vdim), 7.0, dtype=torch.bfloat16, device="cuda")
+    rlt.latent_prompt_attention(torch.cat(q).cuda(), kv.cuda(), shared.cuda()[:, 8:], out, dim, ranges, (dim + rot) ** -0.5, window)
+    return q, [torch.cat([k[s], r[s][:, None].expand(-1, heads, -1)], -1) for s in range(len(contexts))], v, out
+
+
+@pytest.mark.parametrize("heads,dim,rot,vdim", [(3, 128, 64, 128), (2, 64, 32, 80), (5, 40, 8, 64), (2, 72, 64, 24), (1, 8, 16, 128)])
+@pytest.mark.parametrize("window", [0, 1, 40, 64, 127, 128, 129, 300])
+@pytest.mark.parametrize("portions,contexts", PROMPTS, ids=str)
+def test_prompt_attention_over_expanded_latents(heads, dim, rot, vdim, window, portions, contexts):
+    assert rlt.latent_prompt_supported(dim, rot, vdim, torch.bfloat16)
+    q, k, v, got = expanded_case(portions, contexts, heads, dim, rot, vdim, window, 3)
+    want = torch.cat([plain.windowed_attention(q[s].double(), k[s].double(), v[s].double(), (dim + rot) ** -0.5, window, contexts[s] - portions[s])
+                      for s in range(len(portions))])
+    close(got, want, torch.bfloat16, 2.0)
+
+
+@pytest.mark.parametrize("heads,dim,rot,vdim", [(2, 128, 64, 128), (2, 64, 32, 80)])
+@pytest.mark.parametrize("window", [16, 64, 130, 200])
+def test_prompt_rows_find_a_key_just_inside_the_window_and_none_outside(heads, dim, rot, vdim, window):
+    portions, contexts = [20, 150, 257, 129], [320, 333, 300, 400]
+    for distance in (window - 1, window):
+        _, _, v, got = expanded_case(portions, contexts, heads, dim, rot, vdim, window, 5, peak=distance)
+        at = 0
+        for s, n in enumerate(portions):
+            at += n
+            value = v[s][contexts[s] - 1 - distance].double()
+            missed = float((got[at - 1].double().cpu() - value).norm() / value.norm())
+            assert missed < 0.05 if distance < window else missed > 0.5
+
+
+def test_other_head_sizes_are_left_to_the_general_kernels():
+    assert not rlt.latent_prompt_supported(128, 64, 128, torch.float32)
+    assert not any(rlt.latent_prompt_supported(*sizes, torch.bfloat16) for sizes in ((136, 64, 128), (128, 72, 128), (128, 64, 136), (60, 32, 64), (64, 30, 64)))
+
+
 # ---- linear attention ----------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,dim,vdim", [(5, 24, 40), (3, 10, 7), (2, 128, 128), (2, 96, 64), (3, 64, 32), (1, 160, 80)])

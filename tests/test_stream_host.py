@@ -113,6 +113,8 @@ def test_the_previous_token_crosses_portions_and_ends_with_its_sequence(monkeypa
 def test_key_ranges_hold_what_the_rows_see():
     ranges = KeyRanges.of([(0, 5), (10, 3), (2, 1), (40, 20)], 4, torch.device("cpu"))
     assert ranges.first.tolist() == [0, 7, 0, 37] and ranges.cu.tolist() == [0, 5, 11, 14, 37] and ranges.rows == 37
+    assert KeyRanges.of([(10, 300), (2, 20)], 4, torch.device("cpu")).tiles.tolist() == [
+        [0, 256, 10, 0, 7, 0, 0, 0], [256, 44, 266, 0, 7, 0, 0, 0], [300, 20, 2, 303, 0, 0, 0, 0]]
     assert KeyRanges.of([(3, 5)], 0, torch.device("cpu")).first.tolist() == [0]
     assert KeyRanges.of([(3, 5)], 1, torch.device("cpu")).cu.tolist() == [0, 5]
 

@@ -18,7 +18,7 @@ from .engine import Engine, StepEntry
 from .hybrid_lm import HybridLM, HybridLMConfig
 from .kv_cache import RollbackResult, finalize_tokens, kv_write, rollback
 from .experts import expert_gather, expert_gemm, expert_route
-from .latent import latent_gather, latent_write, rotate_heads, rotation_frequencies
+from .latent import latent_gather, latent_prompt_attention, latent_prompt_supported, latent_write, rotate_heads, rotation_frequencies
 from .layers import block_epilogue, clamped_glu, residual_norm, rope_kv_write, sandwich_norm, stream_mix
 from .looped_lm import LoopedLM, LoopedLMConfig, seeded_state_dict
 from .recurrent import causal_conv, decay_scan, decay_table, gated_norm, ssd_scan
@@ -43,5 +43,5 @@ __all__ = [
     "SequenceCache", "StateSpec", "StepEntry", "block_epilogue", "causal_conv", "gated_norm", "load_model", "read_safetensors",
     "read_weights", "register_model", "registered_architectures", "residual_norm", "ssd_scan",
     "StreamLM", "StreamLMConfig", "clamped_glu", "decay_scan", "decay_table", "expert_gather", "expert_gemm", "expert_route",
-    "latent_gather", "latent_write", "rotate_heads", "rotation_frequencies", "stream_mix",
+    "latent_gather", "latent_prompt_attention", "latent_prompt_supported", "latent_write", "rotate_heads", "rotation_frequencies", "stream_mix",
 ]

@@ -68,6 +68,8 @@ SIGNATURES = {
     "rlt_latent_write": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _L, _P, _L, _L, _L, _I, _P, _I, _P, _P, _I, _I, _P]),
     "rlt_rotate_heads": (_I, [_P, _L, _L, _P, _L, _L, _I, _I, _I, _P, _P, _I, _I, _P]),
     "rlt_latent_gather": (_I, [_P, _L, _L, _L, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _P]),
+    "rlt_latent_prompt_supported": (_I, [_I, _I, _I, _I]),
+    "rlt_latent_prompt_attention": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P, _I, _F, _I, _I, _P, _P]),
     "rlt_expert_route": (_I, [_P, _L, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P]),
     "rlt_expert_gather": (_I, [_P, _L, _P, _P, _P, _I, _I, _I, _P, _P, _I, _P]),
     "rlt_expert_gemm": (_I, [_P, _L, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _P, _P]),

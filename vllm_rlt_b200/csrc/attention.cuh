@@ -112,6 +112,14 @@ bool attention_tiles_supported(const AttentionArgs& a);
 size_t attention_tiles_workspace_bytes(int rows, int sequences, int max_new, int q_heads, int kv_heads, int value_dim, int64_t capacity);
 int launch_attention_tiles(const AttentionArgs& a, int max_new, void* workspace, size_t workspace_bytes, cudaStream_t stream);
 
+// Folds partial results [row][query head][split][value_dim + 2] (fp32: O, maximum in log2 units, sum) of up to 32 splits into a.out (bf16).
+int launch_merge_splits(const AttentionArgs& a, int splits, const float* partials, cudaStream_t stream);
+
+// attention_latent.cu: one cache row per key for all heads, whose first part is the value (bf16, short portions).
+bool attention_latent_supported(const AttentionArgs& a, int max_new);
+size_t attention_latent_workspace_bytes(int rows, int q_heads, int value_dim);
+int launch_attention_latent(const AttentionArgs& a, int max_new, void* workspace, size_t workspace_bytes, cudaStream_t stream);
+
 // attention_sm100.cu: head_dim 128, 16-token pages, fp16/bf16 — TMA page streaming,
 // request-grouped rows on tensor cores, split-KV with a deterministic merge.
 bool attention_sm100_supported(const AttentionArgs& a);        // shape and cache view

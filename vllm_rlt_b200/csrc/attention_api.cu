@@ -210,6 +210,10 @@ extern "C" RLT_API size_t rlt_scored_attention_workspace_bytes(int rows, int seq
   // the tile kernel's own scratch also where the page kernels are expected: they may refuse a cache's placement
   const size_t tiles = rlt::attention_tiles_workspace_bytes(rows, sequences, max_new, q_heads, kv_heads, value_dim,
                                                             static_cast<int64_t>(table_width) * block_size);
+  if (kv_heads == 1 && value_dim < key_dim && max_new <= 16) {     // values may turn out to be a part of the key rows
+    const size_t latent = rlt::attention_latent_workspace_bytes(rows, q_heads, value_dim);
+    return tiles > latent ? tiles : latent;
+  }
   const bool pages_kernel = key_dim == value_dim && block_size == 16 && (key_dim == 128 || (key_dim == 64 && max_new > 16));
   if (!pages_kernel) return tiles;
   const size_t pages = max_new > 16 ? rlt::prefill_sm100_workspace_bytes(rows, sequences)
@@ -246,6 +250,7 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
   RLT_REQUIRE(q_stride >= static_cast<int64_t>(q_heads) * key_dim && out_stride >= static_cast<int64_t>(q_heads) * value_dim,
               "scored_attention: row strides smaller than a row");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (attention_latent_supported(a, max_new)) return launch_attention_latent(a, max_new, workspace, workspace_bytes, s);
   if (window > 0) {
     // the page kernels walk whole contexts: windowed rows go to the tile or generic kernel
   } else if (max_new > 16) {

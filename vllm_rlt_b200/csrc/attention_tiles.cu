@@ -325,12 +325,16 @@ int launch(const AttentionArgs& a, int max_new, int splits, float* partials, cud
   kernel<<<grid, kThreads, smem, stream>>>(a, scale_log2, splits, partials);
   const int status = launch_status("attention_tiles_kernel (split)");
   if (status != RLT_OK || splits == 1) return status;
+  return launch_merge_splits(a, splits, partials, stream);
+}
+
+}  // namespace
+
+int launch_merge_splits(const AttentionArgs& a, int splits, const float* partials, cudaStream_t stream) {
   const int64_t pairs = static_cast<int64_t>(a.rows) * a.q_heads;
   merge_splits_kernel<<<static_cast<unsigned>((pairs + kWarps - 1) / kWarps), kThreads, 0, stream>>>(a, splits, partials);
   return launch_status("merge_splits_kernel");
 }
-
-}  // namespace
 
 bool attention_tiles_supported(const AttentionArgs& a) {
   if (a.dtype != RLT_BF16 || a.cu_seqlens_q == nullptr) return false;

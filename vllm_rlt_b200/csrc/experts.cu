@@ -212,6 +212,10 @@ extern "C" RLT_API int rlt_expert_gemm(const void* x, int64_t x_stride, const vo
   g.x = x; g.x_stride = x_stride; g.w = w; g.y = y; g.y_stride = y_stride; g.counts = counts; g.rows = rows; g.experts = experts;
   g.in = in; g.out = out; g.act = act; g.dtype = dtype; g.error = static_cast<unsigned*>(workspace);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (expert_gemm_sm100_supported(g)) {
+    const int status = launch_expert_gemm_sm100(g, s);
+    if (status != RLT_ERR_UNSUPPORTED) return status;
+  }
   const int64_t tiles = rows / kTile + (rows < experts ? rows : experts);   // every expert with rows adds at most one partial tile
   RLT_REQUIRE(tiles <= 65535, "expert_gemm: too many rows for one launch");
   const dim3 grid(static_cast<unsigned>((out + kTile - 1) / kTile), static_cast<unsigned>(tiles));

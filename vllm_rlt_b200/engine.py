@@ -32,11 +32,17 @@ class StepEntry:
 
 @dataclass
 class KeyRanges:
-    """Positions `first[s]` .. of every sequence, packed: those of sequence s are rows cu[s] .. cu[s + 1] - 1."""
+    """Positions `first[s]` .. of every sequence, packed: those of sequence s are rows cu[s] .. cu[s + 1] - 1.
+
+    tiles: the portions in runs of up to TILE_ROWS query rows, those with the most keys first, as records (first query row, rows,
+    position of the first row, packed row of position first[s], first[s], 0, 0, 0)."""
 
     first: torch.Tensor      # int32 [n]
     cu: torch.Tensor         # int32 [n + 1]
     rows: int
+    tiles: torch.Tensor      # int32 [tiles, 8]
+
+    TILE_ROWS = 256
 
     @classmethod
     def of(cls, portions, window: int, device) -> "KeyRanges":
@@ -44,11 +50,17 @@ class KeyRanges:
         cu = [0]
         for f, (start, n) in zip(first, portions):
             cu.append(cu[-1] + start + n - f)
-        host = torch.tensor(first + cu, dtype=torch.int32)
+        tiles, row = [], 0
+        for s, (start, n) in enumerate(portions):
+            for at in range(0, n, cls.TILE_ROWS):
+                tiles.append((row + at, min(n - at, cls.TILE_ROWS), start + at, cu[s], first[s], 0, 0, 0))
+            row += n
+        tiles.sort(key=lambda t: min(t[2] + t[1], window + t[1]) if window else t[2] + t[1], reverse=True)
+        host = torch.tensor([x for t in tiles for x in t] + first + cu, dtype=torch.int32)
         if device.type == "cuda":
             host = host.pin_memory()
-        both = host.to(device, non_blocking=True)
-        return cls(both[:len(first)], both[len(first):], cu[-1])
+        tile_words, rest = host.to(device, non_blocking=True).split((8 * len(tiles), len(first) + len(cu)))
+        return cls(rest[:len(first)], rest[len(first):], cu[-1], tile_words.view(-1, 8))
 
 
 @dataclass

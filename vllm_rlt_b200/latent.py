@@ -71,3 +71,33 @@ def latent_gather(cache, tables, ranges):
                                               _capi.stream_of(cache))
     _capi.check(code, "latent_gather")
     return out
+
+
+def latent_prompt_supported(dim: int, rot_dim: int, vdim: int, dtype) -> bool:
+    """Whether `latent_prompt_attention` takes heads of these sizes."""
+    return bool(_capi.load().rlt_latent_prompt_supported(dim, rot_dim, vdim, _capi.DTYPE_CODES[dtype]))
+
+
+def latent_prompt_attention(q, kv, shared_keys, out, dim: int, ranges, scale: float, window: int):
+    """Attention of portions over packed keys and values expanded from latents, into `out`.
+
+    q `[rows, heads, dim + rot_dim]`, kv `[ranges.rows, heads * dim + heads * vdim]` (keys, then values, head by head),
+    shared_keys `[ranges.rows, rot_dim]` (any row stride), out `[rows, heads, vdim]`; `ranges` (KeyRanges) of the same window."""
+    _capi.require_cuda(q, kv, shared_keys, out, ranges.tiles)
+    rows, heads, key_dim = q.shape
+    vdim, rot_dim = out.shape[2], key_dim - dim
+    if out.shape[:2] != (rows, heads) or kv.shape != (ranges.rows, heads * (dim + vdim)) or shared_keys.shape != (ranges.rows, rot_dim):
+        raise ValueError("q [rows, heads, dim + rot_dim], out [rows, heads, vdim], kv and shared_keys one row per packed key")
+    if any(t.dtype != q.dtype for t in (kv, shared_keys, out)) or any(t.stride(-1) != 1 for t in (q, kv, shared_keys, out)) \
+            or q.stride(1) != key_dim or out.stride(1) != vdim:
+        raise ValueError("one dtype, unit inner strides, heads side by side")
+    if rows == 0:
+        return out
+    workspace = torch.empty(256, dtype=torch.uint8, device=q.device)
+    with torch.cuda.device(q.device):
+        code = _capi.load().rlt_latent_prompt_attention(
+            _capi.ptr(q), q.stride(0), _capi.ptr(kv), kv.stride(0), _capi.ptr(shared_keys), shared_keys.stride(0), _capi.ptr(out), out.stride(0),
+            rows, ranges.rows, heads, dim, rot_dim, vdim, _capi.ptr(ranges.tiles), ranges.tiles.shape[0], float(scale), int(window),
+            _capi.DTYPE_CODES[q.dtype], _capi.ptr(workspace), _capi.stream_of(q))
+    _capi.check(code, "latent_prompt_attention")
+    return out

@@ -28,11 +28,13 @@ import torch.nn.functional as F
 
 from .attention import B200PagedAttention, ScoreTerms
 from .experts import expert_gather, expert_gemm, expert_route
-from .latent import latent_write, rotate_heads, rotation_frequencies
+from .latent import latent_gather, latent_prompt_attention, latent_prompt_supported, latent_write, rotate_heads, rotation_frequencies
 from .layers import block_epilogue, clamped_glu, stream_mix
 from .model_parts import check_positive, check_shapes, full_accumulation, stack_blocks, take_keys
 from .recurrent import decay_scan, decay_table, gated_norm
 from .sequence_cache import CacheSpec, KVSpec, StateSpec
+
+SHORT_PORTION = 16      # groups of portions up to this long attend over the cache rows, longer ones over expanded keys and values
 
 
 # ---- configuration -----------------------------------------------------------------------------
@@ -247,8 +249,9 @@ class _Layer:
             self.w_down, (self.q_col, self.kv_col), _ = stack_blocks([take(p + "mix.dq"), take(p + "mix.dkv")], 0)
             self.q_norm, self.kv_norm = fp32("mix.dq.norm"), fp32("mix.dkv.norm")
             self.w_q = take(p + "mix.uq")
-            self.w_uk = take(p + "mix.uk").view(m.heads, m.dim, m.kv_rank)
-            self.w_uv = take(p + "mix.uv").view(m.heads, m.vdim, m.kv_rank)
+            keys = m.heads * m.dim
+            self.w_kv = torch.cat([take(p + "mix.uk"), take(p + "mix.uv")])       # all heads' keys, then all values
+            self.w_uk, self.w_uv = self.w_kv[:keys].view(m.heads, m.dim, m.kv_rank), self.w_kv[keys:].view(m.heads, m.vdim, m.kv_rank)
             self.frequencies = rotation_frequencies(m.rot_base, m.rot_dims, model.device)
         else:
             self.w_in, (self.q_at, self.k_at, self.v_at, self.g_at), _ = stack_blocks([take(p + "mix." + n) for n in "qkvg"], 0)
@@ -346,8 +349,19 @@ class StreamLM:
         q = F.linear(latent, layer.w_q).view(rows, m.heads, m.dim + m.rot_dim)
         out = torch.empty(rows, m.heads, m.vdim, dtype=self.dtype, device=self.device)
         for group in batch.groups:
-            self._attend_latents(layer, q[group.rows], out[group.rows], pages, batch.positions[group.rows], group)
+            expand = group.max_new > SHORT_PORTION and group.portions is not None and \
+                latent_prompt_supported(m.dim, m.rot_dim, m.vdim, self.dtype)
+            attend = self._attend_expanded if expand else self._attend_latents
+            attend(layer, q[group.rows], out[group.rows], pages, batch.positions[group.rows], group)
         return F.linear(out.view(rows, -1), layer.w_o)
+
+    def _attend_expanded(self, layer, q, out, pages, positions, group):
+        """Over keys and values expanded from the latents of every position the portions see."""
+        m = layer.mixer
+        ranges = group.key_ranges(m.window)
+        rows = latent_gather(pages, group.tables, ranges)
+        rotate_heads(q[:, :, m.dim:], q[:, :, m.dim:], layer.frequencies, positions)
+        latent_prompt_attention(q, F.linear(rows[:, :m.kv_rank], layer.w_kv), rows[:, m.kv_rank:], out, m.dim, ranges, m.scale, m.window)
 
     def _attend_latents(self, layer, q, out, pages, positions, group):
         """Over the cache rows themselves: a head's query is taken into the latent's space (q . W_uk c = W_uk^T q . c), so all
