@@ -43,6 +43,9 @@ Other entry points (each prints its own JSON line; none is the contract line abo
                       prefill and decode of Sobipel-shaped models (parallel attention / Mamba-2 blocks, random weights)
                       beside the looped model at equal size with one loop, through the same engine, and every kernel
                       of a layer against its roofline beside the like kernel of the looped model
+    --workload stream [--steps K --warmup W]
+                      the same for Sugosun-shaped models (hyper-connected streams, latent / lightning attention, dense and
+                      mixture-of-experts feed-forwards)
     --only attention  [--requests --layers --tokens --depths --kv-heads --context-min --context-max --shared-plan]
     --only prefill    [--requests --tokens --kv-heads --eager]   packed causal prefill, TFLOP/s
     --only accept | --only silu                                  the small kernels at the step's shapes
@@ -952,7 +955,7 @@ def hybrid_model_rows(name, model, steps, warmup):
 
     rows = []
     for requests, tokens in ((8, 2048), (1, 16384)):
-        engine = rlt.Engine(model, max_tokens=requests * (tokens + BLOCK), max_sequences=requests, cuda_graphs=False)
+        engine = rlt.Engine(model, max_tokens=requests * (tokens + 4 * BLOCK), max_sequences=requests, cuda_graphs=False)
         entries = [rlt.StepEntry(i, torch.randint(0, model.vocab_size, (tokens,)).tolist(), [tokens - 1]) for i in range(requests)]
         engine._claim(entries)
         batch = engine._batch(entries)
@@ -961,7 +964,7 @@ def hybrid_model_rows(name, model, steps, warmup):
         rows.append({"model": name, "phase": "prefill", "requests": requests, "tokens": tokens, "ms": ms, "tokens_per_s": requests * tokens / ms * 1e3})
         del engine, batch
     for requests, context in ((1, 4096), (16, 4096), (64, 2048)):
-        engine = rlt.Engine(model, max_tokens=requests * (context + BLOCK), max_sequences=requests, max_sequence_tokens=context + BLOCK,
+        engine = rlt.Engine(model, max_tokens=requests * (context + 4 * BLOCK), max_sequences=requests, max_sequence_tokens=context + BLOCK,
                             capture_sizes=[requests])
         for i in range(requests):
             engine.step([rlt.StepEntry(i, torch.randint(0, model.vocab_size, (context,)).tolist())])
@@ -1149,6 +1152,223 @@ def run_hybrid_workload(args):
             del model
             torch.cuda.empty_cache()
             report["sizes"][name] = {"shape": {k: v for k, v in size.items()}, "throughput": rows, "kernels": hybrid_kernel_rows(size, args.steps)}
+            torch.cuda.empty_cache()
+    report["clocks"] = clocks.summary()
+    print(json.dumps(report))
+
+
+# Layer shapes of the stream workload: a Sugosun layer has the parameters of a looped layer of the same width (of the experts, those
+# that a token uses).
+STREAM_SIZES = {
+    "2048": dict(width=2048, heads=16, q_rank=1536, kv_rank=512, rot_dim=64, window=1024, streams=4, experts=64, top=8, expert_ff=1024,
+                 ff=5632, layers=8, vocab=49152),
+    "4096": dict(width=4096, heads=32, q_rank=1536, kv_rank=512, rot_dim=64, window=1024, streams=4, experts=32, top=4, expert_ff=3584,
+                 ff=9600, layers=6, vocab=49152),
+}
+
+
+def stream_config(size, pattern):
+    """config.json of a Sugosun model whose layers repeat `pattern`: pairs of a mixer ('a' latent attention, 'l' lightning) and a
+    feed-forward ('d' dense, 'e' experts)."""
+    heads = size["heads"]
+    mixers = {"a": ("latent_attention", {"heads": heads, "dim": HEAD_DIM, "rot_dim": size["rot_dim"], "vdim": HEAD_DIM, "q_rank": size["q_rank"],
+                                         "kv_rank": size["kv_rank"], "scale": (HEAD_DIM + size["rot_dim"]) ** -0.5,
+                                         "mask": {"size": size["window"]}, "rot": {"base": 10000.0, "dims": size["rot_dim"]}}),
+              "l": ("lightning", {"heads": heads, "dim": HEAD_DIM, "vdim": HEAD_DIM, "decay": [1 - 2.0 ** -(2 + 8 * h / heads) for h in range(heads)]})}
+    feeds = {"d": {"kind": "dense", "ff": size["ff"], "limit": 7.0},
+             "e": {"kind": "moe", "router": {"experts": size["experts"], "top": size["top"]}, "expert": {"ff": size["expert_ff"]}}}
+    layers = []
+    for i in range(size["layers"]):
+        mixer, feed = pattern[i % len(pattern)]
+        layers.append({"type": mixers[mixer][0], "mixer": mixers[mixer][1], "mlp": feeds[feed]})
+    return {"architecture": "Sugosun", "vocab": size["vocab"], "width": size["width"], "streams": size["streams"], "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 131}}, "layers": layers}
+
+
+@torch.no_grad()
+def stream_kernel_rows(size, steps):
+    """Every kernel of a Sugosun layer at prefill (16384 rows: 8 x 2048) and decode (64 rows, context 2048), with its algorithmic bytes
+    or flops against the measured peak, beside the like kernel of the looped model."""
+    from types import SimpleNamespace
+
+    import vllm_rlt_b200 as rlt
+    from vllm_rlt_b200.engine import KeyRanges
+
+    device = torch.device("cuda", 0)
+    peak_gbs, _ = measured_peaks()
+    peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+    peak_tflops = float(peaks.get("bf16_tflops", 1590.0))
+    width, heads, rank, rot, q_rank = size["width"], size["heads"], size["kv_rank"], size["rot_dim"], size["q_rank"]
+    ff, experts, top, expert_ff, s_count = size["ff"], size["experts"], size["top"], size["expert_ff"], size["streams"]
+    row_dim, inner, key_dim = rank + rot, heads * HEAD_DIM, HEAD_DIM + rot
+    bf16 = lambda *shape: torch.randn(*shape, device=device).to(torch.bfloat16)
+    f32 = lambda *shape: torch.randn(*shape, device=device)
+    rows_out = []
+
+    def add(kernel, phase, like, make, nbytes=0.0, flops=0.0, copies=None):
+        """make(i) -> a call on the i-th set of tensors.  The roofline is the later of the two bounds."""
+        copies = copies or max(2, min(48, int(400e6 // max(nbytes, 1)) + 1))
+        us = ring_us([make(i) for i in range(copies)], steps)
+        tensor = flops / peak_tflops / 1e6 > nbytes / peak_gbs / 1e3
+        frac = flops / us / 1e6 / peak_tflops if tensor else nbytes / us / 1e3 / peak_gbs
+        rows_out.append({"kernel": kernel, "phase": phase, "like": like, "us": us, "bound": "tensor" if tensor else "hbm", "roofline_frac": frac})
+        torch.cuda.empty_cache()
+
+    for phase, seqs, new, context in (("prefill", 8, 2048, 2048), ("decode", 64, 1, 2048)):
+        rows, page = seqs * new, 64
+        pages = context // page
+        tables = torch.randperm(seqs * pages, device=device).int().view(seqs, pages)
+        lengths = torch.full((seqs,), context, dtype=torch.int32, device=device)
+        cu = (torch.arange(seqs + 1, device=device) * new).int()
+        positions = (torch.arange(rows, device=device) % new).int() + (context - new)
+        row_seq = torch.arange(seqs, device=device, dtype=torch.int32).repeat_interleave(new)
+        batch = SimpleNamespace(tables=tables[None], row_seq=row_seq, positions=positions)
+        group = SimpleNamespace(sequences=seqs, max_new=new, cu=cu, starts=lengths - new, slots=torch.arange(seqs, device=device, dtype=torch.int32))
+        kernels = rlt.B200PagedAttention()
+        small = lambda nbytes: max(2, min(48, int(400e6 // nbytes) + 1))
+
+        # attention: pairs that are scored, with and without the window, and the looped model's of the same head count
+        for window in (0, size["window"]):
+            seen = [min(p + 1, window or context) for p in range(context - new, context)]
+            name = f"latent attention, window {window}" if window else "latent attention, all keys"
+            if new > 1:
+                ranges = KeyRanges.of([(0, new)] * seqs, window, device)
+                q, kv, latent, out = [bf16(rows, heads, key_dim) for _ in range(2)], [bf16(rows, 2 * inner) for _ in range(2)], bf16(rows, row_dim), bf16(rows, heads, HEAD_DIM)
+                add(name, phase, "attention of the looped model",
+                    lambda i: (lambda: rlt.latent_prompt_attention(q[i % 2], kv[i % 2], latent[:, rank:], out, HEAD_DIM, ranges, key_dim ** -0.5, window)),
+                    rows * (heads * key_dim + 3 * inner + row_dim) * 2.0, 2.0 * sum(seen) * seqs * heads * (key_dim + HEAD_DIM), copies=4)
+                del q, kv, latent, out
+            else:
+                copies = small(seqs * seen[0] * row_dim * 2)
+                pools = [bf16(seqs * pages, page, 1, row_dim) for _ in range(copies)]
+                q, out = bf16(rows, heads, row_dim), bf16(rows, heads, rank)
+                add(name, phase, "attention of the looped model",
+                    lambda i: (lambda: kernels.scored(q, out, pools[i], pools[i][..., :rank], tables, lengths, cu, 1, rlt.ScoreTerms(key_dim ** -0.5, window=window))),
+                    seqs * seen[0] * row_dim * 2.0 + rows * heads * (row_dim + rank) * 2.0, 2.0 * seqs * seen[0] * heads * (row_dim + rank), copies=copies)
+                del pools
+        small_pages = context // BLOCK
+        looped_tables = torch.randperm(seqs * small_pages, device=device).int().view(seqs, small_pages)
+        pools = [bf16(2, seqs * small_pages, BLOCK, heads, HEAD_DIM) for _ in range(2)]
+        q = [bf16(rows, heads, HEAD_DIM) for _ in range(2)]
+        pairs = sum(range(context - new + 1, context + 1)) * seqs
+        add("attention of the looped model", phase, None,
+            lambda i: (lambda: kernels.prefill(q[i % 2], pools[i % 2][0], pools[i % 2][1], looped_tables, lengths, cu, new)),
+            seqs * context * heads * HEAD_DIM * 4.0 + rows * inner * 4.0, 4.0 * pairs * inner, copies=4)
+        del pools, q
+
+        # between the sublayers
+        nbytes = rows * width * (s_count * 8.0 + 4)
+        copies = small(nbytes)
+        streams, delta = [f32(rows, s_count, width) for _ in range(copies)], [bf16(rows, width) for _ in range(copies)]
+        out_c, mix, reads, weight = f32(s_count), 0.3 * f32(s_count, s_count), f32(s_count), f32(width)
+        add("stream_mix", phase, "sandwich_norm", lambda i: (lambda: rlt.stream_mix(streams[i], weight, 1e-6, torch.bfloat16, delta=delta[i], ran=(out_c, mix), follows=reads)),
+            nbytes, copies=copies)
+        parts = bf16(rows * top, width)
+        places, shares = torch.randperm(rows * top, device=device).int().view(rows, top), torch.rand(rows, top, device=device)
+        add("stream_mix, weighted parts", phase, "sandwich_norm", lambda i: (lambda: rlt.stream_mix(
+            streams[i], weight, 1e-6, torch.bfloat16, delta=parts, parts=(places, shares), ran=(out_c, mix), follows=reads)),
+            nbytes + rows * width * 2.0 * (top - 1), copies=copies)
+        w16, res16 = bf16(width), [bf16(rows, width) for _ in range(copies)]
+        add("sandwich_norm", phase, None, lambda i: (lambda: rlt.sandwich_norm(delta[i], w16, 1e-6, res16[i], w16, in_place=True)), rows * width * 8.0, copies=copies)
+        del streams, delta, parts, res16
+
+        # latent rows
+        down = q_rank + row_dim
+        nbytes = rows * down * 4.0
+        copies = small(nbytes)
+        proj, cache = [bf16(rows, down) for _ in range(copies)], bf16(seqs * pages, page, 1, row_dim)
+        frequencies = rlt.rotation_frequencies(10000.0, rot, device)
+        q_norm, kv_norm = f32(q_rank), f32(rank)
+        add("latent_write", phase, "rope_kv_write", lambda i: (lambda: rlt.latent_write(proj[i], 0, q_rank, q_norm, kv_norm, 1e-6, frequencies, cache, batch)),
+            nbytes, copies=copies)
+        nbytes = rows * heads * rot * 4.0
+        copies = small(rows * heads * key_dim * 2)
+        q = [bf16(rows, heads, key_dim) for _ in range(copies)]
+        add("rotate_heads", phase, "rope_kv_write", lambda i: (lambda: rlt.rotate_heads(q[i][:, :, HEAD_DIM:], q[i][:, :, HEAD_DIM:], frequencies, positions)), nbytes, copies=copies)
+        del proj, q
+        if new > 1:
+            ranges = KeyRanges.of([(0, new)] * seqs, size["window"], device)
+            caches = [bf16(seqs * pages, page, 1, row_dim) for _ in range(12)]
+            add("latent_gather", phase, "rope_kv_write", lambda i: (lambda: rlt.latent_gather(caches[i], tables, ranges)), ranges.rows * row_dim * 4.0, copies=12)
+            del caches
+        copies = small(rows * inner * 8)
+        k_cache = bf16(2, seqs * small_pages, BLOCK, heads, HEAD_DIM)
+        qkv = [bf16(rows, 3 * inner) for _ in range(copies)]
+        cos = bf16(rows, HEAD_DIM)
+        blocks, offsets = looped_tables[row_seq.long(), (positions // BLOCK).long()].long(), (positions % BLOCK).long()
+        cut = lambda p, a: p[:, a * inner:(a + 1) * inner].view(rows, heads, HEAD_DIM)
+        add("rope_kv_write", phase, None, lambda i: (lambda: rlt.rope_kv_write(cut(qkv[i], 0), cut(qkv[i], 1), cut(qkv[i], 2), cos, cos, k_cache[0], k_cache[1], blocks, offsets)),
+            rows * (3 * inner * 4.0 + HEAD_DIM * 4), copies=copies)
+        del k_cache, qkv
+
+        # lightning attention
+        copies = small(rows * inner * 8)
+        proj = [bf16(rows, 4 * inner) for _ in range(copies)]
+        mixed = [bf16(rows, 3 * inner) for _ in range(min(copies, 4))]
+        add("block_epilogue (silu)", phase, "silu_and_mul", lambda i: (lambda: rlt.block_epilogue(proj[i], batch, act=(0, 3 * inner, "silu", mixed[i % len(mixed)], 0))),
+            rows * 3 * inner * 4.0, copies=copies)
+        y, table = bf16(rows, inner), rlt.decay_table([1 - 2.0 ** -(2 + 8 * h / heads) for h in range(heads)], device)
+        states = [torch.zeros(seqs, heads, HEAD_DIM, HEAD_DIM, device=device) for _ in range(4)]
+        add("decay_scan", phase, None, lambda i: (lambda: rlt.decay_scan(
+            *(mixed[i % len(mixed)][:, a * inner:(a + 1) * inner] for a in range(3)), table, states[i % 4], y, group)),
+            rows * 4 * inner * 2.0 + 2 * states[0].numel() * 4.0, copies=4)
+        norm_w, gated = f32(inner), bf16(rows, inner)
+        add("gated_norm (gate behind)", phase, "sandwich_norm", lambda i: (lambda: rlt.gated_norm(y, proj[i][:, 3 * inner:], norm_w, gated, 1, 1e-6, gate_behind=True)),
+            rows * inner * 6.0, copies=copies)
+        del proj, mixed, y, states, gated
+
+        # feed-forwards
+        copies = small(rows * ff * 6)
+        gate_up = [bf16(rows, 2 * ff) for _ in range(copies)]
+        add("clamped_glu", phase, "silu_and_mul", lambda i: (lambda: rlt.clamped_glu(gate_up[i], ff, ff, 7.0, 1.702)), rows * ff * 6.0, copies=copies)
+        add("silu_and_mul", phase, None, lambda i: (lambda: rlt.silu_and_mul_packed(gate_up[i])), rows * ff * 6.0, copies=copies)
+        del gate_up
+        logits, correction = [f32(rows, experts) for _ in range(4)], 0.01 * f32(experts)
+        routing = rlt.expert_route(logits[0], correction, top)
+        add("expert_route (with its zeroing)", phase, "sandwich_norm", lambda i: (lambda: rlt.expert_route(logits[i % 4], correction, top)), rows * (experts * 4.0 + top * 12), copies=8)
+        h = [bf16(rows, width) for _ in range(4)]
+        add("expert_gather", phase, "rope_kv_write", lambda i: (lambda: rlt.expert_gather(h[i % 4], routing)), rows * (1 + top) * width * 2.0, copies=4)
+        used = int((routing.counts > 0).sum())
+        up, downs = [bf16(experts, expert_ff, width) for _ in range(2)], [bf16(experts, width, expert_ff) for _ in range(2)]
+        x, act = rlt.expert_gather(h[0], routing), bf16(rows * top, expert_ff)
+        nbytes, flops = used * width * expert_ff * 2.0 + rows * top * (width + expert_ff) * 2.0, 2.0 * rows * top * width * expert_ff
+        add("expert_gemm, up and squared relu", phase, "cuBLAS GEMM", lambda i: (lambda: rlt.expert_gemm(x, up[i % 2], routing.counts, "squared_relu")), nbytes, flops, copies=4)
+        add("expert_gemm, down", phase, "cuBLAS GEMM", lambda i: (lambda: rlt.expert_gemm(act, downs[i % 2], routing.counts)), nbytes, flops, copies=4)
+        del up, downs, x, act, h
+        dense, inputs = [bf16(2 * ff, width) for _ in range(8)], bf16(rows, width)
+        add("cuBLAS GEMM (gate and up)", phase, None, lambda i: (lambda: torch.nn.functional.linear(inputs, dense[i])),
+            (2 * ff * width + rows * (width + 2 * ff)) * 2.0, 2.0 * rows * width * 2 * ff, copies=8)
+        del dense, inputs
+    return rows_out
+
+
+def run_stream_workload(args):
+    """`--workload stream`: one JSON line with throughput rows, kernel rows and the clocks under them."""
+    import vllm_rlt_b200 as rlt
+    from vllm_rlt_b200.looped_lm import parameter_shapes as looped_shapes
+    from vllm_rlt_b200.stream_lm import parameter_shapes as stream_shapes
+
+    torch.cuda.set_device(0)
+    device = torch.device("cuda", 0)
+    report = {"workload": "stream", "data": "synthetic, random weights", "dtype": "bf16", "steps": args.steps, "sizes": {}}
+    with ClockSampler(0) as clocks:
+        for name, size in STREAM_SIZES.items():
+            rows = []
+            for label, pattern in (("Sugosun, latent attention and dense", ["ad"]), ("Sugosun, lightning and dense", ["ld"]),
+                                   ("Sugosun, latent attention and experts", ["ae"]), ("Sugosun, 1 latent : 3 lightning, experts", ["ae", "le", "le", "le"])):
+                config = rlt.StreamLMConfig.from_json(stream_config(size, pattern))
+                model = rlt.StreamLM(config, device_weights(stream_shapes(config), device), device)
+                rows += hybrid_model_rows(label, model, args.steps, args.warmup)
+                del model
+                torch.cuda.empty_cache()
+            looped = rlt.LoopedLMConfig(vocab_size=size["vocab"], hidden_size=size["width"], intermediate_size=size["ff"],
+                                        num_hidden_layers=size["layers"], num_attention_heads=size["heads"],
+                                        num_key_value_heads=size["heads"], head_dim=HEAD_DIM, total_ut_steps=1)
+            model = rlt.LoopedLM(looped, device_weights(looped_shapes(looped), device), device, torch.bfloat16)
+            rows += hybrid_model_rows("looped model, one loop", model, args.steps, args.warmup)
+            del model
+            torch.cuda.empty_cache()
+            report["sizes"][name] = {"shape": dict(size), "throughput": rows, "kernels": stream_kernel_rows(size, args.steps)}
             torch.cuda.empty_cache()
     report["clocks"] = clocks.summary()
     print(json.dumps(report))
@@ -1446,7 +1666,7 @@ def main():
     parser.add_argument("--no-cpu-baseline", action="store_true")
     parser.add_argument("--only", default=None, choices=["attention", "accept", "silu", "prefill"],
                         help="profiling aid: run only this kernel family (not a bench line)")
-    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded", "hybrid"],
+    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded", "hybrid", "stream"],
                         help="rounds: timed speculative rounds (the bench line); decode: one complete generation; "
                              "sharded: a fixed request set shared out over the ranks, decoded to completion")
     parser.add_argument("--engine", default="b200", choices=["b200", "reference"],
@@ -1494,6 +1714,9 @@ def main():
             setattr(args, name, sharded_default if sharded else decode_default)
     if sharded:
         run_sharded_workload(args)
+        return
+    if args.workload == "stream":
+        run_stream_workload(args)
         return
     if args.workload == "hybrid":
         run_hybrid_workload(args)

@@ -171,18 +171,34 @@ def run_latent(q, key, tables, contexts, portions, rank, terms):
     return out
 
 
+def larger_pages(key, tables, size):
+    """The same rows over pages of `size` tokens (in an order of their own), unwritten slots NaN."""
+    n, width = tables.shape
+    per = size // BLOCK
+    order = torch.randperm(n * -(-width // per), generator=torch.Generator().manual_seed(size)).view(n, -1)
+    pages = torch.full((order.numel(), size, *key.shape[2:]), float("nan"), dtype=key.dtype)
+    for s in range(n):
+        for i, page in enumerate(tables[s].tolist()):
+            if page >= 0:
+                pages[order[s, i // per], i % per * BLOCK:(i % per + 1) * BLOCK] = key[page]
+    return pages, order.int()
+
+
 LATENTS = [(6, 48, 16), (16, 512, 64), (20, 72, 24), (1, 4, 2), (5, 11, 6), (32, 256, 32), (40, 128, 64), (3, 64, 8)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,rank,rot", LATENTS)
 @pytest.mark.parametrize("window", [0, 1, 40, 64, 129])
-def test_attention_over_cache_rows(dtype, heads, rank, rot, window):
+@pytest.mark.parametrize("page", [16, 64])
+def test_attention_over_cache_rows(dtype, heads, rank, rot, window, page):
     """Every head scores one row per key, and the row's first part is its value: decoded tokens and short portions."""
     row = rank + rot
     terms = rlt.ScoreTerms(0.7 * row ** -0.5, window=window)
     for portions, contexts in (([1, 1, 1], [1, 17, 530]), ([2, 16, 5], [2, 33, 300]), ([1] * 5, [64, 65, 128, 129, 40])):
         q, k, key, tables = latent_case(portions, contexts, heads, row, dtype, 7)
+        if page > BLOCK:
+            key, tables = larger_pages(key, tables, page)
         got = run_latent(q, key, tables, contexts, portions, rank, terms)
         want = torch.cat([plain.windowed_attention(q[s].double(), k[s].double()[:, None].expand(-1, heads, -1), k[s].double()[:, None, :rank].expand(-1, heads, -1),
                                                    terms.scale, window, contexts[s] - portions[s]) for s in range(len(portions))])
@@ -198,6 +214,8 @@ def test_a_key_just_inside_a_window_is_found_and_one_just_outside_is_not(dtype, 
     for portions in ([1, 1, 1], [2, 9, 16]):
         for distance in (window - 1, window):
             q, k, key, tables = latent_case(portions, contexts, heads, row, dtype, 11, peak=(distance, 12.0))
+            if portions[0] == 1:
+                key, tables = larger_pages(key, tables, 64)
             got = run_latent(q, key, tables, contexts, portions, rank, terms).double().cpu()
             at = 0
             for s, n in enumerate(portions):

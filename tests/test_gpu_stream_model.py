@@ -75,11 +75,12 @@ def test_residual_after_every_layer_run(name, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", sorted(CONFIGS))
+@pytest.mark.parametrize("block", [16, 64])
 @pytest.mark.parametrize("cuts", [[200], [1], [2], [3, 17, 40, 5, 16, 2], [64, 1], [33], [150, 20, 2]], ids=str)
-def test_logits_do_not_depend_on_the_cut(name, dtype, cuts):
+def test_logits_do_not_depend_on_the_cut(name, dtype, cuts, block):
     model, _ = build(name, dtype)
     tokens = prompt(1, 200, model.vocab_size)
-    engine = rlt.Engine(model, max_tokens=208, max_sequences=2)
+    engine = rlt.Engine(model, max_tokens=256, max_sequences=2, block=block)
     check_logits(feed(engine, "s", tokens, cuts), name, tokens, dtype)
 
 
@@ -90,7 +91,7 @@ def test_unequal_requests_in_mixed_batches_over_reused_pages(name, graphs, dtype
     """Six requests over room for three: portions of some beside single tokens of others, in a pool that is handed on again and
     again; requests pause and go on."""
     model, _ = build(name, dtype)
-    engine = rlt.Engine(model, max_tokens=160, max_sequences=3, cuda_graphs=graphs)
+    engine = rlt.Engine(model, max_tokens=160, max_sequences=3, block=16, cuda_graphs=graphs)
     lengths = [70, 1, 33, 5, 48, 90]
     texts = [prompt(10 + i, n, model.vocab_size) for i, n in enumerate(lengths)]
     portions = [1, 7, 20, 1, 1, 16, 2, 40, 1, 3, 17, 1]
@@ -145,7 +146,7 @@ def test_long_decoding(dtype):
     """Hundreds of decoded tokens behind a short prompt: across pages and past every window."""
     model, _ = build("mixed", dtype)
     tokens = prompt(8, 420, model.vocab_size)
-    engine = rlt.Engine(model, max_tokens=432, max_sequences=1)
+    engine = rlt.Engine(model, max_tokens=448, max_sequences=1)
     check_logits(feed(engine, "s", tokens, [9, 1]), "mixed", tokens, dtype)
     engine.release("s")
     check_logits(feed(engine, "s", tokens, [420]), "mixed", tokens, dtype)
@@ -184,7 +185,7 @@ def test_a_token_outside_the_window_changes_nothing(window, dtype):
 def test_greedy_generation_follows_the_plain_model(name):
     model, _ = build(name, torch.float32)
     prompts = [prompt(20 + i, n, model.vocab_size) for i, n in enumerate([30, 4, 1, 50, 17])]
-    engine = rlt.Engine(model, max_tokens=144, max_sequences=2, max_step_tokens=24)
+    engine = rlt.Engine(model, max_tokens=144, max_sequences=2, block=16, max_step_tokens=24)
     got = engine.generate(prompts, SamplingParams(max_tokens=12))
     for p, out in zip(prompts, got):
         assert plain_run(name, torch.float32, p + out[:-1])[0][len(p) - 1:].argmax(-1).tolist() == out

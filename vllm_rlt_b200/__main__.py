@@ -32,9 +32,9 @@ def _generate(args) -> int:
     if not prompts or not all(prompts):
         raise SystemExit("generate: give at least one nonempty --prompt or a --prompts-file")
     model = load_model(args.model, device="cuda", dtype={"bfloat16": torch.bfloat16, "float32": torch.float32}[args.dtype])
-    page = 16
+    page = model.cache_spec().block
     pool = args.pool_tokens or sum(-(-(len(p) + args.max_tokens) // page) * page for p in prompts)
-    engine = Engine(model, max_tokens=pool, max_sequences=min(args.max_sequences, len(prompts)), block=page,
+    engine = Engine(model, max_tokens=pool, max_sequences=min(args.max_sequences, len(prompts)),
                     max_step_tokens=args.max_step_tokens, cuda_graphs=not args.eager)
     params = SamplingParams(args.max_tokens, args.temperature, args.top_p, args.top_k, args.seed)
     for tokens in engine.generate(prompts, params):

@@ -115,7 +115,7 @@ int launch_attention_tiles(const AttentionArgs& a, int max_new, void* workspace,
 // Folds partial results [row][query head][split][value_dim + 2] (fp32: O, maximum in log2 units, sum) of up to 32 splits into a.out (bf16).
 int launch_merge_splits(const AttentionArgs& a, int splits, const float* partials, cudaStream_t stream);
 
-// attention_latent.cu: one cache row per key for all heads, whose first part is the value (bf16, short portions).
+// attention_latent_sm100.cu: one cache row per key for all heads, whose first part is the value (bf16, short portions).
 bool attention_latent_supported(const AttentionArgs& a, int max_new);
 size_t attention_latent_workspace_bytes(int rows, int q_heads, int value_dim);
 int launch_attention_latent(const AttentionArgs& a, int max_new, void* workspace, size_t workspace_bytes, cudaStream_t stream);

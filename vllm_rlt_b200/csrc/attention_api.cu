@@ -250,7 +250,10 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
   RLT_REQUIRE(q_stride >= static_cast<int64_t>(q_heads) * key_dim && out_stride >= static_cast<int64_t>(q_heads) * value_dim,
               "scored_attention: row strides smaller than a row");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (attention_latent_supported(a, max_new)) return launch_attention_latent(a, max_new, workspace, workspace_bytes, s);
+  if (attention_latent_supported(a, max_new)) {
+    status = launch_attention_latent(a, max_new, workspace, workspace_bytes, s);
+    if (status != RLT_ERR_UNSUPPORTED) return status;
+  }
   if (window > 0) {
     // the page kernels walk whole contexts: windowed rows go to the tile or generic kernel
   } else if (max_new > 16) {

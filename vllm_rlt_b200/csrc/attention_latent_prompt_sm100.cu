@@ -121,6 +121,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   const Span span0 = span(0), span1 = span(1);
   const int all_stages = max(span0.end, span1.end);
 
+  if ((blockIdx.x | blockIdx.y) == 0 && threadIdx.x == 0) *a.error = 0;   // a wait gives up seconds later
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(&sm.full_q), 1);
     for (int s = 0; s < kStages; ++s) {
@@ -366,7 +367,6 @@ extern "C" RLT_API int rlt_latent_prompt_attention(const void* q, int64_t q_stri
     return RLT_ERR_UNSUPPORTED;
   }
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  RLT_CUDA_TRY(cudaMemsetAsync(a.error, 0, sizeof(unsigned), s));
   if (dim <= 64) return vdim <= 64 ? launch<1, 1>(a, maps, s) : launch<1, 2>(a, maps, s);
   return vdim <= 64 ? launch<2, 1>(a, maps, s) : launch<2, 2>(a, maps, s);
 }

@@ -274,7 +274,7 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
   }
 }
 
-// One warp per (row, query head): the splits' partials in order.
+// One warp per (row, query head) and 64 output columns (blockIdx.y): the splits' partials in order.
 __global__ void __launch_bounds__(kThreads)
 merge_splits_kernel(AttentionArgs a, int splits, const float* __restrict__ partials) {
   const int lane = threadIdx.x & 31;
@@ -283,25 +283,35 @@ merge_splits_kernel(AttentionArgs a, int splits, const float* __restrict__ parti
   const int64_t row = pair / a.q_heads;
   const int stride = a.value_dim + 2;
   const float* part = partials + pair * splits * stride;
+  const int d = blockIdx.y * 64 + 2 * lane;              // value_dim is even: a pair of columns is inside or outside as one
+  const bool live = d < a.value_dim;
   const float m = lane < splits ? part[lane * stride + a.value_dim] : -INFINITY;   // at most 32 splits: one per lane
+  const float sum = lane < splits ? part[lane * stride + a.value_dim + 1] : 0.f;
+  float2 first[4];
+#pragma unroll
+  for (int s = 0; s < 4; ++s) first[s] = live && s < splits ? *reinterpret_cast<const float2*>(part + s * stride + d) : make_float2(0.f, 0.f);
   float big = m;
 #pragma unroll
   for (int x = 16; x > 0; x >>= 1) big = fmaxf(big, __shfl_xor_sync(0xffffffffu, big, x));
   const float f = m == -INFINITY ? 0.f : fast_exp2(m - big);
-  float total = lane < splits ? part[lane * stride + a.value_dim + 1] * f : 0.f;
+  float total = sum * f;
 #pragma unroll
   for (int x = 16; x > 0; x >>= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
   const float inv = total > 0.f ? 1.f / total : 0.f;
-  T* out = static_cast<T*>(a.out) + row * a.out_stride + (pair - row * a.q_heads) * a.value_dim;
-  for (int base = 0; base < a.value_dim; base += 32) {   // whole warps: every lane takes part in the shuffles
-    const int d = base + lane;
-    float acc = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float fs = __shfl_sync(0xffffffffu, f, s);
-      if (fs != 0.f && d < a.value_dim) acc = fmaf(part[s * stride + d], fs, acc);
-    }
-    if (d < a.value_dim) out[d] = __float2bfloat16_rn(acc * inv);
+  float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int s = 0; s < 4; ++s) {
+    const float fs = __shfl_sync(0xffffffffu, f, s);
+    if (fs != 0.f) acc = make_float2(fmaf(first[s].x, fs, acc.x), fmaf(first[s].y, fs, acc.y));
   }
+#pragma unroll 4
+  for (int s = 4; s < splits; ++s) {
+    const float fs = __shfl_sync(0xffffffffu, f, s);
+    const float2 v = live && fs != 0.f ? *reinterpret_cast<const float2*>(part + s * stride + d) : make_float2(0.f, 0.f);
+    acc = make_float2(fmaf(v.x, fs, acc.x), fmaf(v.y, fs, acc.y));
+  }
+  T* out = static_cast<T*>(a.out) + row * a.out_stride + (pair - row * a.q_heads) * a.value_dim;
+  if (live) *reinterpret_cast<uint32_t*>(out + d) = pack2<true>(acc.x * inv, acc.y * inv);
 }
 
 constexpr int kMaxSplits = 32;
@@ -332,7 +342,8 @@ int launch(const AttentionArgs& a, int max_new, int splits, float* partials, cud
 
 int launch_merge_splits(const AttentionArgs& a, int splits, const float* partials, cudaStream_t stream) {
   const int64_t pairs = static_cast<int64_t>(a.rows) * a.q_heads;
-  merge_splits_kernel<<<static_cast<unsigned>((pairs + kWarps - 1) / kWarps), kThreads, 0, stream>>>(a, splits, partials);
+  const dim3 grid(static_cast<unsigned>((pairs + kWarps - 1) / kWarps), static_cast<unsigned>((a.value_dim + 63) / 64));
+  merge_splits_kernel<<<grid, kThreads, 0, stream>>>(a, splits, partials);
   return launch_status("merge_splits_kernel");
 }
 

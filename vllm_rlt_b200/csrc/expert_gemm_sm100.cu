@@ -49,6 +49,7 @@ expert_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
   extern __shared__ unsigned char smem_raw[];
   Shared& sm = *reinterpret_cast<Shared*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const int lane = threadIdx.x & 31, warp = __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0);
+  if (blockIdx.x == 0 && threadIdx.x == 0) *g.error = 0;   // a wait gives up seconds later
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
       mbar_init(smem_u32(&sm.full[s]), 1);
@@ -185,7 +186,7 @@ expert_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
       if (buffer == 0) parity ^= 1u;
     }
   }
-  if (failed && lane == 0 && g.error != nullptr) atomicOr(g.error, 1u);
+  if (failed && lane == 0) atomicOr(g.error, 1u);
   tcgen05_before_sync();
   __syncthreads();
   if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kColumns) : "memory");

@@ -143,12 +143,15 @@ class Engine:
 
     max_tokens: tokens the live sequences may hold together (each rounded up to whole pages); max_sequences: live
     sequences (state slots).  `max_step_tokens` bounds the rows of one step of `generate`; `max_sequence_tokens` the
-    length of one sequence (default: the pool), which sizes the page tables of captured steps."""
+    length of one sequence (default: the pool), which sizes the page tables of captured steps; `block` the tokens of a
+    page (default: the model's choice)."""
 
-    def __init__(self, model, *, max_tokens: int, max_sequences: int, block: int = 16, max_step_tokens: int = 8192,
+    def __init__(self, model, *, max_tokens: int, max_sequences: int, block: int | None = None, max_step_tokens: int = 8192,
                  max_sequence_tokens: int | None = None, cuda_graphs: bool = True, capture_sizes=None):
         self.model, self.device = model, model.device
-        self.cache = SequenceCache(model.cache_spec(), max_tokens=max_tokens, max_sequences=max_sequences, block=block,
+        spec = model.cache_spec()
+        block = block or spec.block
+        self.cache = SequenceCache(spec, max_tokens=max_tokens, max_sequences=max_sequences, block=block,
                                    device=model.device, dtype=model.dtype)
         self.max_step_tokens = max_step_tokens
         self.max_sequence_tokens = min(max_sequence_tokens or max_tokens, self.cache.plane_pages * block)

@@ -1,6 +1,6 @@
 """What live sequences keep between steps: paged keys and values, and recurrent state slots.
 
-Pages: the pool has a fixed number of `block`-token pages.  A model asks for `planes` tables per sequence
+Pages: the pool has a fixed number of `block`-token pages (the model's choice unless the engine is told).  A model asks for `planes` tables per sequence
 (one per loop depth of a looped model, one otherwise); page i of a plane holds tokens i * block .. of every
 layer that writes keys and values.  Slots: a sequence owns one slot in every recurrent state tensor; one more
 slot at the end takes what the padding sequences of a captured step write.  Nothing is cleared when pages and
@@ -39,6 +39,7 @@ class CacheSpec:
     layers: dict = field(default_factory=dict)    # layer -> KVSpec
     states: dict = field(default_factory=dict)    # name -> StateSpec
     pooled: bool = False                          # one [pages, layers, block, heads, dim] pool for all layers
+    block: int = 16                               # tokens per page the model's kernels like best
 
 
 class CacheFull(RuntimeError):

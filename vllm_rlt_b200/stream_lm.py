@@ -301,7 +301,7 @@ class StreamLM:
                 layers[run] = KVSpec(1, m.row, 0)
             else:
                 states[f"r{run}.state"] = StateSpec((m.heads, m.dim, m.vdim), torch.float32)
-        return CacheSpec(layers=layers, states=states)
+        return CacheSpec(layers=layers, states=states, block=64)      # a page is a stage of the attention over cache rows
 
     # ---- one step ------------------------------------------------------------------------------
     def _mix(self, streams, pending, norm, reads, **kw):
