@@ -37,7 +37,7 @@ def make_config(layers, *, streams, vocab, width, loop=None, bigram=(61, 31, 7),
 CONFIGS = {
     "mixed": make_config([latent_layer(6, 24, 16, 40, 56, 48, 21, mlp=moe(9, 3, 40)),
                           lightning_layer([0.3, 0.7, 0.9, 0.97, 1.0], 24, 40, mlp=dense(88, 1.5)),
-                          latent_layer(3, 32, 8, 16, 24, 32, 0, base=1e4),
+                          latent_layer(3, 32, 8, 16, 24, 36, 0, base=1e4),       # sizes the prompt kernel takes over a row it does not
                           lightning_layer([0.95, 0.5], 8, 16, mlp=moe(5, 1, 24))],
                          streams=3, vocab=131, width=96, loop=(1, 3, 2)),
     "odd": make_config([latent_layer(5, 9, 6, 7, 13, 11, 1, mlp=dense(33, 0.8)),

@@ -40,7 +40,7 @@ def test_looped_layers_have_a_cache_for_every_pass():
     config = rlt.StreamLMConfig.from_json(CONFIGS["mixed"])
     assert config.runs == [0, 1, 2, 1, 2, 3]
     spec = rlt.StreamLM(config, random_weights(stream_lm.parameter_shapes(config), 0), "cpu").cache_spec()
-    assert sorted(spec.layers) == [0, 2, 4] and spec.layers[4] == rlt.KVSpec(1, 32 + 8, 0)
+    assert sorted(spec.layers) == [0, 2, 4] and spec.layers[4] == rlt.KVSpec(1, 36 + 8, 0)
     assert {k: v.shape for k, v in spec.states.items()} == {"r1.state": (5, 24, 40), "r3.state": (5, 24, 40), "r5.state": (2, 8, 16)}
     cache = rlt.SequenceCache(spec, max_tokens=64, max_sequences=2, device="cpu")
     assert spec.block == 64 and cache.key[0].shape == (4, 16, 1, 64) and not cache.value and cache.state["r5.state"].dtype == torch.float32

@@ -191,7 +191,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
     const int seen_end = live ? position + 1 : 0, seen_begin = position - window + 1;   // keys seen_begin .. seen_end - 1
     const uint32_t tmem_row = tmem + (static_cast<uint32_t>(warp_row) << 16);
     const uint32_t s_col = tmem_row + t * kTileCols, p_col = s_col + kColP, o_col = tmem_row + kColO + t * kRows;
-    constexpr float kRaise = 8.0f;       // the running maximum is raised, and the output row rescaled, only when it is exceeded by this much
+    constexpr float kRaise = 40.0f;      // the running maximum is raised, and the output row rescaled, only when it is exceeded by this much
     float m = -INFINITY, l = 0.f;
     for (int i = 0; i < stages; ++i) {
       if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&sm.s_ready[t]), i & 1))) { failed = true; break; }

@@ -10,7 +10,7 @@
 // stages, as TMA boxes of 64 columns with 128-byte swizzle: 64 tokens high where pages are (one copy per 64 columns of a stage),
 // else 16 (the copies' issue is then what bounds the kernel).  Seven warps:
 //   warps 0..3   16 keys each: scores out of tensor memory as 16 x 8 fragments, mask, exponentials, P^T into shared memory (transposed
-//                by stmatrix); sums stay per thread.  Running maxima are raised, and O^T rescaled, only when one is exceeded by 2^8
+//                by stmatrix); sums stay per thread.  Running maxima are raised, and O^T rescaled, only when one is exceeded by 2^40
 //   warp 4 / 5   issue S^T / O^T products,   warp 6 the copies
 // Splits are folded by the merge kernel of attention_tiles.cu.
 #include <math.h>
@@ -27,7 +27,7 @@ constexpr int kThreads = 224;
 constexpr int kRowThreads = 128;              // warps 0 .. 3
 constexpr int kMaxSplits = 32;
 constexpr int kBlockBytes = kKeys * 128;      // 64 columns of a stage's keys
-constexpr float kRaise = 8.0f;
+constexpr float kRaise = 40.0f;               // P and its sums stay far inside the range of their formats, and nothing is lost: all are floating point
 
 template <int kN>
 struct LatentShared {                         // behind the stages and the queries
@@ -93,27 +93,15 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
   constexpr uint32_t kColO = 2 * kN;          // S^T of two stages, then O^T of up to four blocks of 128 value columns
   constexpr uint32_t kColumns = kN == 16 ? 128 : (kN == 32 ? 256 : 512);
   extern __shared__ unsigned char smem_raw[];
-  if ((blockIdx.x | blockIdx.y | blockIdx.z) == 0 && threadIdx.x == 0) *error = 0;   // a wait gives up seconds later
   const int row_dim = a.head_dim, blocks = (row_dim + 63) / 64, value_tiles = (a.value_dim + 127) / 128;
   unsigned char* const keys = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));   // [2][block][key][64]
   unsigned char* const queries = keys + 2 * blocks * kBlockBytes;                                                                                // [block][row][64]
   LatentShared<kN>& sm = *reinterpret_cast<LatentShared<kN>*>(queries + blocks * kN * 128);
   const int lane = threadIdx.x & 31, warp = __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0);
-  const int heads = a.q_heads, seq = blockIdx.z, split = blockIdx.y;
-  const int first_row = a.cu_seqlens_q[seq], tokens = a.cu_seqlens_q[seq + 1] - first_row;
-  const int all_rows = tokens * heads, r_base = blockIdx.x * kN;
-  if (r_base >= all_rows) return;
-  const int64_t capacity = static_cast<int64_t>(a.table_width) * a.block_size;
-  const int context = static_cast<int>(a.context_lengths[seq] < capacity ? a.context_lengths[seq] : capacity);
-  const int base_len = context - tokens + 1;                    // keys the portion's first token sees (<= 0: padding)
-  auto row_len = [&](int r) { return max(base_len + min(r, all_rows - 1) / heads, 0); };   // rows behind the last are computed like it and not stored
-  const int window = a.terms.window > 0 ? a.terms.window : 0x40000000;
-  const int kv_end = row_len(r_base + kN - 1), shortest = row_len(r_base);
-  const int kv_begin = max(shortest - window, 0) / box_tokens * box_tokens;
-  const int per = ((kv_end - kv_begin + splits - 1) / splits + kKeys - 1) / kKeys * kKeys;
-  const int key_begin = min(kv_begin + split * per, kv_end), key_end = min(kv_end, key_begin + per);
-  const int stages = (key_end - key_begin + kKeys - 1) / kKeys;
-
+  if (warp == 4) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&sm.tmem_base)), "r"(kColumns) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(&sm.full_q), 1);
     for (int s = 0; s < 2; ++s) {
@@ -124,10 +112,24 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
     }
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
-  if (warp == 4) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&sm.tmem_base)), "r"(kColumns) : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-  }
+  grid_dependency_wait();                     // the queries, the newest cache row and the scratch belong to the kernels before until here
+  grid_dependency_release();
+  if ((blockIdx.x | blockIdx.y | blockIdx.z) == 0 && threadIdx.x == 0) *error = 0;   // a wait gives up seconds later
+  const int heads = a.q_heads, seq = blockIdx.z, split = blockIdx.y;
+  const int first_row = a.cu_seqlens_q[seq], tokens = a.cu_seqlens_q[seq + 1] - first_row;
+  const int all_rows = tokens * heads, r_base = blockIdx.x * kN;
+  const bool idle = r_base >= all_rows;      // a shorter portion than the longest: this CTA only gives its tensor memory back
+  const int64_t capacity = static_cast<int64_t>(a.table_width) * a.block_size;
+  const int context = static_cast<int>(a.context_lengths[seq] < capacity ? a.context_lengths[seq] : capacity);
+  const int base_len = context - tokens + 1;                    // keys the portion's first token sees (<= 0: padding)
+  auto row_len = [&](int r) { return max(base_len + min(r, all_rows - 1) / heads, 0); };   // rows behind the last are computed like it and not stored
+  const int window = a.terms.window > 0 ? a.terms.window : 0x40000000;
+  const int kv_end = idle ? 0 : row_len(r_base + kN - 1), shortest = idle ? 0 : row_len(r_base);
+  const int kv_begin = max(shortest - window, 0) / box_tokens * box_tokens;
+  const int per = ((kv_end - kv_begin + splits - 1) / splits + kKeys - 1) / kKeys * kKeys;
+  const int key_begin = min(kv_begin + split * per, kv_end), key_end = min(kv_end, key_begin + per);
+  const int stages = (key_end - key_begin + kKeys - 1) / kKeys;
+
   for (int i = threadIdx.x; i < kN; i += kThreads) {
     sm.m[i] = -INFINITY;
     sm.alpha[i] = 1.0f;
@@ -424,8 +426,8 @@ int launch(const AttentionArgs& a, int max_new, int sm_count, float* partials, u
   const int row_tiles = (max_new * a.q_heads + kN - 1) / kN;
   const int splits = choose_splits(static_cast<int64_t>(row_tiles) * a.table_rows, visible_keys(a, max_new), sm_count);
   const dim3 grid(static_cast<unsigned>(row_tiles), static_cast<unsigned>(splits), static_cast<unsigned>(a.table_rows));
-  kernel<<<grid, kThreads, smem, stream>>>(map, q_map, a, box_tokens, static_cast<float>(1.4426950408889634 * static_cast<double>(score_scale(a))), splits, partials, error);
-  const int status = launch_status("attention_latent_kernel");
+  const int status = launch_dependent("attention_latent_kernel", kernel, grid, dim3(kThreads), smem, stream, map, q_map, a, box_tokens,
+                                      static_cast<float>(1.4426950408889634 * static_cast<double>(score_scale(a))), splits, partials, error);
   if (status != RLT_OK || splits == 1) return status;
   return launch_merge_splits(a, splits, partials, stream);
 }

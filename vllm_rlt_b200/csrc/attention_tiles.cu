@@ -276,7 +276,8 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
 
 // One warp per (row, query head) and 64 output columns (blockIdx.y): the splits' partials in order.
 __global__ void __launch_bounds__(kThreads)
-merge_splits_kernel(AttentionArgs a, int splits, const float* __restrict__ partials) {
+merge_splits_kernel(AttentionArgs a, int splits, const float* partials) {
+  grid_dependency_wait();
   const int lane = threadIdx.x & 31;
   const int64_t pair = static_cast<int64_t>(blockIdx.x) * kWarps + (threadIdx.x >> 5);
   if (pair >= static_cast<int64_t>(a.rows) * a.q_heads) return;
@@ -343,8 +344,7 @@ int launch(const AttentionArgs& a, int max_new, int splits, float* partials, cud
 int launch_merge_splits(const AttentionArgs& a, int splits, const float* partials, cudaStream_t stream) {
   const int64_t pairs = static_cast<int64_t>(a.rows) * a.q_heads;
   const dim3 grid(static_cast<unsigned>((pairs + kWarps - 1) / kWarps), static_cast<unsigned>((a.value_dim + 63) / 64));
-  merge_splits_kernel<<<grid, kThreads, 0, stream>>>(a, splits, partials);
-  return launch_status("merge_splits_kernel");
+  return launch_dependent("merge_splits_kernel", merge_splits_kernel, grid, dim3(kThreads), 0, stream, a, splits, partials);
 }
 
 bool attention_tiles_supported(const AttentionArgs& a) {

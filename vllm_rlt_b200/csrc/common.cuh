@@ -43,6 +43,27 @@ inline int launch_status(const char* what) {
   return RLT_OK;
 }
 
+// Programmatic dependent launch: the kernel may be brought onto the GPU while its predecessor in the stream still runs, and waits
+// for it (grid_dependency_wait) before it touches what that one writes.
+template <typename... Params, typename... Args>
+inline int launch_dependent(const char* what, void (*kernel)(Params...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
+  cudaLaunchConfig_t config = {};
+  config.gridDim = grid; config.blockDim = block; config.dynamicSmemBytes = smem; config.stream = stream;
+  cudaLaunchAttribute attribute;
+  attribute.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attribute.val.programmaticStreamSerializationAllowed = 1;
+  config.attrs = &attribute; config.numAttrs = 1;
+  const cudaError_t err = cudaLaunchKernelEx(&config, kernel, Params(args)...);
+  if (err != cudaSuccess) {
+    cudaGetLastError();
+    set_last_error(what, err);
+    return RLT_ERR_CUDA;
+  }
+  return RLT_OK;
+}
+__device__ __forceinline__ void grid_dependency_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void grid_dependency_release() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+
 struct DeviceInfo {
   int device = -1;
   int sm_count = 0;

@@ -2,7 +2,7 @@
 //
 //   expert_route_kernel   one warp per token: softmax of the router's fp32 logits, the `top` largest of score +
 //                         correction, weights = the chosen scores over their sum, and the token's place in each chosen
-//                         expert's queue (an atomic count: the order inside an expert is arbitrary, and no result depends on it)
+//                         expert's queue (atomic counts, a CTA's rows together: the order inside an expert is arbitrary, and no result depends on it)
 //   expert_gather_kernel  copies each token's row behind the others of its experts: rows sorted by expert, expert e from
 //                         counts[0] + .. + counts[e - 1] on
 //   expert_gemm_*         y = act(x W_e^T) over the sorted rows, every expert its own weights; tcgen05 in 16 bits
@@ -19,68 +19,86 @@ namespace {
 constexpr int kThreads = 256;
 constexpr int kWarps = kThreads / 32;
 constexpr int kMaxPerLane = 32;         // experts <= 1024
+constexpr int kRowsPerWarp = 8;         // at most: a CTA counts its rows in shared memory and reserves their places at once
 
 template <int kPerLane>
 __global__ void __launch_bounds__(kThreads)
 expert_route_kernel(const float* __restrict__ logits, int64_t logit_stride, const float* __restrict__ correction, int rows, int experts,
-                    int top, float floor_sum, int32_t* __restrict__ counts, int32_t* __restrict__ chosen, int32_t* __restrict__ rank,
+                    int top, float floor_sum, int per_warp, int32_t* __restrict__ counts, int32_t* __restrict__ chosen, int32_t* __restrict__ rank,
                     float* __restrict__ weights) {
-  const int row = blockIdx.x * kWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= rows) return;
-  const float* z = logits + row * logit_stride;
-  float s[kPerLane], choice[kPerLane];
-  float m = -INFINITY;
+  __shared__ int queued[32 * kMaxPerLane];    // rows of this CTA per expert, then where they start in the expert's queue
+  const int lane = threadIdx.x & 31, first = (blockIdx.x * kWarps + (threadIdx.x >> 5)) * per_warp;
+  for (int e = threadIdx.x; e < experts; e += kThreads) queued[e] = 0;
+  __syncthreads();
+  int place[kRowsPerWarp], expert[kRowsPerWarp];
 #pragma unroll
-  for (int j = 0; j < kPerLane; ++j) {
-    const int e = lane + 32 * j;
-    s[j] = e < experts ? z[e] : -INFINITY;
-    m = fmaxf(m, s[j]);
-  }
+  for (int n = 0; n < kRowsPerWarp; ++n) {
+    const int row = first + n;
+    expert[n] = -1;
+    if (n >= per_warp || row >= rows) continue;
+    const float* z = logits + row * logit_stride;
+    float s[kPerLane], choice[kPerLane];
+    float m = -INFINITY;
 #pragma unroll
-  for (int x = 16; x > 0; x >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, x));
-  float total = 0.0f;
-#pragma unroll
-  for (int j = 0; j < kPerLane; ++j) {
-    s[j] = expf(s[j] - m);
-    total += s[j];
-  }
-#pragma unroll
-  for (int x = 16; x > 0; x >>= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
-#pragma unroll
-  for (int j = 0; j < kPerLane; ++j) {
-    const int e = lane + 32 * j;
-    s[j] /= total;
-    choice[j] = e < experts ? s[j] + (correction != nullptr ? correction[e] : 0.0f) : -INFINITY;
-  }
-  float mine = 0.0f, sum = 0.0f;        // the weight of choice `lane`, and of all
-  int mine_expert = 0;
-  for (int k = 0; k < top; ++k) {
-    float best = -INFINITY;
-    int at = 0x7fffffff;
-#pragma unroll
-    for (int j = 0; j < kPerLane; ++j)
-      if (choice[j] > best) { best = choice[j]; at = lane + 32 * j; }
-#pragma unroll
-    for (int x = 16; x > 0; x >>= 1) {  // the largest, the lower index of equal ones
-      const float other = __shfl_xor_sync(0xffffffffu, best, x);
-      const int other_at = __shfl_xor_sync(0xffffffffu, at, x);
-      if (other > best || (other == best && other_at < at)) { best = other; at = other_at; }
+    for (int j = 0; j < kPerLane; ++j) {
+      const int e = lane + 32 * j;
+      s[j] = e < experts ? z[e] : -INFINITY;
+      m = fmaxf(m, s[j]);
     }
-    if (at >= experts) at = 0;          // nothing comparable (NaN logits): some expert inside the table
-    float score = 0.0f;
 #pragma unroll
-    for (int j = 0; j < kPerLane; ++j)
-      if (lane + 32 * j == at) { score = s[j]; choice[j] = -INFINITY; }
-    score = __shfl_sync(0xffffffffu, score, at & 31);
-    sum += score;
-    if (lane == k) { mine = score; mine_expert = at; }
+    for (int x = 16; x > 0; x >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, x));
+    float total = 0.0f;
+#pragma unroll
+    for (int j = 0; j < kPerLane; ++j) {
+      s[j] = expf(s[j] - m);
+      total += s[j];
+    }
+#pragma unroll
+    for (int x = 16; x > 0; x >>= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
+#pragma unroll
+    for (int j = 0; j < kPerLane; ++j) {
+      const int e = lane + 32 * j;
+      s[j] /= total;
+      choice[j] = e < experts ? s[j] + (correction != nullptr ? correction[e] : 0.0f) : -INFINITY;
+    }
+    float mine = 0.0f, sum = 0.0f;        // the weight of choice `lane`, and of all
+    int mine_expert = 0;
+    for (int k = 0; k < top; ++k) {
+      float best = -INFINITY;
+      int at = 0x7fffffff;
+#pragma unroll
+      for (int j = 0; j < kPerLane; ++j)
+        if (choice[j] > best) { best = choice[j]; at = lane + 32 * j; }
+#pragma unroll
+      for (int x = 16; x > 0; x >>= 1) {  // the largest, the lower index of equal ones
+        const float other = __shfl_xor_sync(0xffffffffu, best, x);
+        const int other_at = __shfl_xor_sync(0xffffffffu, at, x);
+        if (other > best || (other == best && other_at < at)) { best = other; at = other_at; }
+      }
+      if (at >= experts) at = 0;          // nothing comparable (NaN logits): some expert inside the table
+      float score = 0.0f;
+#pragma unroll
+      for (int j = 0; j < kPerLane; ++j)
+        if (lane + 32 * j == at) { score = s[j]; choice[j] = -INFINITY; }
+      score = __shfl_sync(0xffffffffu, score, at & 31);
+      sum += score;
+      if (lane == k) { mine = score; mine_expert = at; }
+    }
+    if (lane < top) {
+      const int64_t at = static_cast<int64_t>(row) * top + lane;
+      chosen[at] = mine_expert;
+      weights[at] = mine / (sum + floor_sum);
+      expert[n] = mine_expert;
+      place[n] = atomicAdd(&queued[mine_expert], 1);
+    }
   }
-  if (lane < top) {
-    const int64_t at = static_cast<int64_t>(row) * top + lane;
-    chosen[at] = mine_expert;
-    weights[at] = mine / (sum + floor_sum);
-    rank[at] = atomicAdd(counts + mine_expert, 1);
-  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < experts; e += kThreads)
+    if (queued[e] > 0) queued[e] = atomicAdd(counts + e, queued[e]);
+  __syncthreads();
+#pragma unroll
+  for (int n = 0; n < kRowsPerWarp; ++n)
+    if (expert[n] >= 0) rank[static_cast<int64_t>(first + n) * top + lane] = queued[expert[n]] + place[n];
 }
 
 // One warp per (token, choice).
@@ -168,8 +186,9 @@ extern "C" RLT_API int rlt_expert_route(const float* logits, int64_t logit_strid
   if (rows == 0) return RLT_OK;
   RLT_REQUIRE(logits && counts && chosen && rank && weights, "expert_route: null pointer");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const unsigned grid = static_cast<unsigned>((rows + kWarps - 1) / kWarps);
-#define RLT_ROUTE(P) expert_route_kernel<P><<<grid, kThreads, 0, s>>>(logits, logit_stride, correction, rows, experts, top, floor_sum, counts, chosen, rank, weights)
+  const int per_warp = rows >= 4096 ? kRowsPerWarp : 1;
+  const unsigned grid = static_cast<unsigned>((rows + kWarps * per_warp - 1) / (kWarps * per_warp));
+#define RLT_ROUTE(P) expert_route_kernel<P><<<grid, kThreads, 0, s>>>(logits, logit_stride, correction, rows, experts, top, floor_sum, per_warp, counts, chosen, rank, weights)
   if (experts <= 32) RLT_ROUTE(1);
   else if (experts <= 64) RLT_ROUTE(2);
   else if (experts <= 128) RLT_ROUTE(4);

@@ -25,17 +25,6 @@ __device__ __forceinline__ void rotation(int position, double frequency, float* 
   sincosf(static_cast<float>(angle), sine, cosine);
 }
 
-__device__ __forceinline__ float block_sum(float v, float* scratch) {
-#pragma unroll
-  for (int x = 16; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
-  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
-  __syncthreads();
-  v = (threadIdx.x & 31) < kThreads / 32 ? scratch[threadIdx.x & 31] : 0.0f;
-#pragma unroll
-  for (int x = 4; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
-  return __shfl_sync(0xffffffffu, v, 0);
-}
-
 struct LatentArgs {
   const void* proj; int64_t proj_stride;
   int q_col, q_rank, kv_col, kv_rank, rot_dim, rot_dims;   // rot_dims of the rot_dim are turned
@@ -46,24 +35,34 @@ struct LatentArgs {
   const int32_t* tables; int table_width; const int32_t* row_seq; const int32_t* positions;
 };
 
-// blockIdx.y 0: the cache row, 1: the query latent.
+// One warp per (row, part): part 0 the cache row, part 1 the query latent.
 template <typename T, int kVec>
-__global__ void __launch_bounds__(kThreads)
-latent_write_kernel(LatentArgs a) {
-  __shared__ float scratch[kThreads / 32];
-  const int row = blockIdx.x;
-  const bool query = blockIdx.y == 1;
+__global__ void __launch_bounds__(kThreads, 4)
+latent_write_kernel(LatentArgs a, int rows, int parts) {
+  struct alignas(sizeof(T) * kVec) Vec { T e[kVec]; };
+  const int item = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (item >= rows * parts) return;
+  const int row = item / parts;
+  const bool query = item - row * parts == 1;
   const T* proj = static_cast<const T*>(a.proj) + row * a.proj_stride + (query ? a.q_col : a.kv_col);
   const float* weight = query ? a.q_weight : a.kv_weight;
   const int width = query ? a.q_rank : a.kv_rank;
-  T* dst;
+  constexpr int kKeep = 8;                    // accesses of a row that stay in registers between the sum and the result
+  Vec kept[kKeep];
+#pragma unroll
+  for (int n = 0; n < kKeep; ++n)
+    if ((n * 32 + lane) * kVec < width) kept[n] = *reinterpret_cast<const Vec*>(proj + (n * 32 + lane) * kVec);
+  T* dst = static_cast<T*>(a.q_out) + row * a.q_out_stride;
   int position = 0;
-  if (query) {
-    dst = static_cast<T*>(a.q_out) + row * a.q_out_stride;
-  } else {
+  float turned[2] = {0.0f, 0.0f};             // the lane's first pair of the rotated part
+  if (!query) {
     const int seq = a.row_seq[row];
     if (seq < 0) return;                      // a padding row of a captured step
     position = a.positions[row];
+    if (2 * lane < a.rot_dim) {
+      turned[0] = Elem<T>::to_float(proj[a.kv_rank + 2 * lane]);
+      if (2 * lane + 1 < a.rot_dim) turned[1] = Elem<T>::to_float(proj[a.kv_rank + 2 * lane + 1]);
+    }
     const int page_index = position / a.block_size;
     if (position < 0 || page_index >= a.table_width) return;
     const int64_t page = a.tables[static_cast<int64_t>(seq) * a.table_width + page_index];
@@ -71,61 +70,96 @@ latent_write_kernel(LatentArgs a) {
     dst = static_cast<T*>(a.cache) + page * a.block_stride + (position % a.block_size) * a.token_stride;
   }
   float ss = 0.0f;
-  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
+#pragma unroll
+  for (int n = 0; n < kKeep; ++n)
+    if ((n * 32 + lane) * kVec < width) {
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) {
+        const float v = Elem<T>::to_float(kept[n].e[e]);
+        ss = fmaf(v, v, ss);
+      }
+    }
+  for (int i = (kKeep * 32 + lane) * kVec; i < width; i += 32 * kVec) {
     float v[kVec];
     load_floats<T, kVec>(proj + i, v);
 #pragma unroll
     for (int e = 0; e < kVec; ++e) ss = fmaf(v[e], v[e], ss);
   }
-  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + a.eps);
-  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
-    float v[kVec], w[kVec];
-    load_floats<T, kVec>(proj + i, v);
-    load_floats<float, kVec>(weight + i, w);
 #pragma unroll
-    for (int e = 0; e < kVec; ++e) v[e] *= r * w[e];
-    store_floats<T, kVec>(dst + i, v);
-  }
+  for (int x = 16; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+  const float r = 1.0f / sqrtf(ss / static_cast<float>(width) + a.eps);
+  auto write = [&](int i, const Vec& x) {
+    constexpr int kQuad = kVec < 4 ? kVec : 4;
+    Vec y;
+#pragma unroll
+    for (int q = 0; q < kVec; q += kQuad) {
+      float w[kQuad];
+      load_floats<float, kQuad>(weight + i + q, w);
+#pragma unroll
+      for (int e = 0; e < kQuad; ++e) y.e[q + e] = Elem<T>::from_float(Elem<T>::to_float(x.e[q + e]) * r * w[e]);
+    }
+    *reinterpret_cast<Vec*>(dst + i) = y;
+  };
+#pragma unroll
+  for (int n = 0; n < kKeep; ++n)
+    if ((n * 32 + lane) * kVec < width) write((n * 32 + lane) * kVec, kept[n]);
+  for (int i = (kKeep * 32 + lane) * kVec; i < width; i += 32 * kVec) write(i, *reinterpret_cast<const Vec*>(proj + i));
   if (query) return;
-  const T* part = proj + a.kv_rank;
-  for (int i = threadIdx.x; 2 * i < a.rot_dim; i += kThreads) {
+  for (int i = lane; 2 * i < a.rot_dim; i += 32) {
     const int d = 2 * i;
-    float u = Elem<T>::to_float(part[d]), v = d + 1 < a.rot_dim ? Elem<T>::to_float(part[d + 1]) : 0.0f;
+    if (i != lane) {
+      turned[0] = Elem<T>::to_float(proj[a.kv_rank + d]);
+      turned[1] = d + 1 < a.rot_dim ? Elem<T>::to_float(proj[a.kv_rank + d + 1]) : 0.0f;
+    }
+    float u = turned[0], v = turned[1];
     if (d < a.rot_dims) {
       float c, s;
       rotation(position, a.frequencies[i], &c, &s);
-      const float u0 = u;
-      u = u0 * c - v * s;
-      v = v * c + u0 * s;
+      u = turned[0] * c - turned[1] * s;
+      v = turned[1] * c + turned[0] * s;
     }
     dst[a.kv_rank + d] = Elem<T>::from_float(u);
     if (d + 1 < a.rot_dim) dst[a.kv_rank + d + 1] = Elem<T>::from_float(v);
   }
 }
 
-// One CTA per row: the row's angles once, then every head's pairs.
-template <typename T>
+// `per_cta` rows: their angles once, then every head's elements, kVec (an even number, or one pair whose second half may lie outside).
+template <typename T, int kVec>
 __global__ void __launch_bounds__(kThreads)
 rotate_heads_kernel(const T* src, int64_t src_row, int64_t src_head, T* dst, int64_t dst_row, int64_t dst_head, int heads, int dim,
-                    int rot_dims, const double* __restrict__ frequencies, const int32_t* __restrict__ positions) {
+                    int rot_dims, const double* __restrict__ frequencies, const int32_t* __restrict__ positions, int rows, int per_cta) {
   extern __shared__ float2 turns[];
-  const int64_t row = blockIdx.x;
-  for (int i = threadIdx.x; i < rot_dims / 2; i += kThreads) rotation(positions[row], frequencies[i], &turns[i].x, &turns[i].y);
+  const int pairs = rot_dims / 2, first = blockIdx.x * per_cta, count = min(per_cta, rows - first);
+  for (int i = threadIdx.x; i < count * pairs; i += kThreads) rotation(positions[first + i / pairs], frequencies[i % pairs], &turns[i].x, &turns[i].y);
   __syncthreads();
-  const int pairs = (dim + 1) / 2;
-  for (int i = threadIdx.x; i < heads * pairs; i += kThreads) {
-    const int head = i / pairs, d = 2 * (i % pairs);
-    const T* from = src + row * src_row + head * src_head + d;
-    T* to = dst + row * dst_row + head * dst_head + d;
-    float u = Elem<T>::to_float(from[0]), v = d + 1 < dim ? Elem<T>::to_float(from[1]) : 0.0f;
-    if (d < rot_dims) {
-      const float2 t = turns[d / 2];
-      const float u0 = u;
-      u = u0 * t.x - v * t.y;
-      v = v * t.x + u0 * t.y;
+  constexpr int kStep = kVec < 2 ? 2 : kVec;
+  const int pieces = (dim + kStep - 1) / kStep, per_row = heads * pieces;
+  for (int i = threadIdx.x; i < count * per_row; i += kThreads) {
+    const int r = i / per_row, rest = i - r * per_row, head = rest / pieces, d = (rest - head * pieces) * kStep;
+    const T* from = src + (first + r) * src_row + head * src_head + d;
+    T* to = dst + (first + r) * dst_row + head * dst_head + d;
+    const float2* turn = turns + r * pairs + d / 2;
+    float v[kStep];
+    if constexpr (kVec > 1) {
+      load_floats<T, kVec>(from, v);
+    } else {
+      v[0] = Elem<T>::to_float(from[0]);
+      v[1] = d + 1 < dim ? Elem<T>::to_float(from[1]) : 0.0f;
     }
-    to[0] = Elem<T>::from_float(u);
-    if (d + 1 < dim) to[1] = Elem<T>::from_float(v);
+#pragma unroll
+    for (int e = 0; e < kStep; e += 2)
+      if (d + e < rot_dims) {
+        const float2 t = turn[e / 2];
+        const float u = v[e];
+        v[e] = u * t.x - v[e + 1] * t.y;
+        v[e + 1] = v[e + 1] * t.x + u * t.y;
+      }
+    if constexpr (kVec > 1) {
+      store_floats<T, kVec>(to, v);
+    } else {
+      to[0] = Elem<T>::from_float(v[0]);
+      if (d + 1 < dim) to[1] = Elem<T>::from_float(v[1]);
+    }
   }
 }
 
@@ -176,15 +210,16 @@ extern "C" RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, i
   a.rot_dim = rot_dim; a.rot_dims = rot_dims; a.q_weight = q_weight; a.kv_weight = kv_weight; a.eps = eps; a.frequencies = frequencies;
   a.q_out = q_out; a.q_out_stride = q_out_stride; a.cache = cache; a.block_stride = block_stride; a.token_stride = token_stride;
   a.num_blocks = num_blocks; a.block_size = block_size; a.tables = tables; a.table_width = table_width; a.row_seq = row_seq; a.positions = positions;
-  const dim3 grid(static_cast<unsigned>(rows), q_rank > 0 ? 2u : 1u);
-  const size_t bytes = 4 * dtype_size(dtype);
-  auto aligned = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
-  bool wide = proj_stride % 4 == 0 && q_col % 4 == 0 && q_rank % 4 == 0 && kv_col % 4 == 0 && kv_rank % 4 == 0 && block_stride % 4 == 0 &&
-              token_stride % 4 == 0 && q_out_stride % 4 == 0 && aligned(proj) && aligned(q_out) && aligned(cache) && aligned16(q_weight) && aligned16(kv_weight);
+  const int parts = q_rank > 0 ? 2 : 1;
+  const int vec = static_cast<int>(16 / dtype_size(dtype));
+  auto whole = [&](int64_t n) { return n % vec == 0; };
+  const bool wide = whole(proj_stride) && whole(q_col) && whole(q_rank) && whole(kv_col) && whole(kv_rank) && whole(block_stride) && whole(token_stride) &&
+                    whole(q_out_stride) && aligned16(proj) && aligned16(q_out) && aligned16(cache) && aligned16(q_weight) && aligned16(kv_weight);
+  const unsigned grid = static_cast<unsigned>((static_cast<int64_t>(rows) * parts + kThreads / 32 - 1) / (kThreads / 32));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   RLT_DISPATCH_DTYPE(dtype, T, {
-    if (wide) latent_write_kernel<T, 4><<<grid, kThreads, 0, s>>>(a);
-    else latent_write_kernel<T, 1><<<grid, kThreads, 0, s>>>(a);
+    if (wide) latent_write_kernel<T, static_cast<int>(16 / sizeof(T))><<<grid, kThreads, 0, s>>>(a, rows, parts);
+    else latent_write_kernel<T, 1><<<grid, kThreads, 0, s>>>(a, rows, parts);
   });
   return launch_status("latent_write_kernel");
 }
@@ -198,9 +233,17 @@ extern "C" RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_
   if (rows == 0 || dim == 0) return RLT_OK;
   RLT_REQUIRE(src && dst && positions && (frequencies || rot_dims == 0), "rotate_heads: null pointer");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const size_t smem = static_cast<size_t>(rot_dims / 2) * sizeof(float2);
-  RLT_DISPATCH_DTYPE(dtype, T, (rotate_heads_kernel<T><<<rows, kThreads, smem, s>>>(static_cast<const T*>(src), src_row, src_head, static_cast<T*>(dst),
-                                dst_row, dst_head, heads, dim, rot_dims, frequencies, positions)));
+  const int vec = static_cast<int>(16 / dtype_size(dtype));
+  auto whole = [&](int64_t n) { return n % vec == 0; };
+  const bool wide = whole(dim) && whole(rot_dims) && whole(src_row) && whole(src_head) && whole(dst_row) && whole(dst_head) && aligned16(src) && aligned16(dst);
+  int per_cta = rows >= 4096 ? 4 : 1;                       // enough CTAs for every SM first
+  if (static_cast<size_t>(per_cta) * (rot_dims / 2) * sizeof(float2) > 40u * 1024u) per_cta = 1;
+  const size_t smem = static_cast<size_t>(per_cta) * (rot_dims / 2) * sizeof(float2);
+  const unsigned grid = static_cast<unsigned>((rows + per_cta - 1) / per_cta);
+#define RLT_LAUNCH(T, V) rotate_heads_kernel<T, V><<<grid, kThreads, smem, s>>>(static_cast<const T*>(src), src_row, src_head, static_cast<T*>(dst), dst_row, \
+                                                                               dst_head, heads, dim, rot_dims, frequencies, positions, rows, per_cta)
+  RLT_DISPATCH_DTYPE(dtype, T, { if (wide) RLT_LAUNCH(T, static_cast<int>(16 / sizeof(T))); else RLT_LAUNCH(T, 1); });
+#undef RLT_LAUNCH
   return launch_status("rotate_heads_kernel");
 }
 

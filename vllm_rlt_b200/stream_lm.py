@@ -349,7 +349,7 @@ class StreamLM:
         q = F.linear(latent, layer.w_q).view(rows, m.heads, m.dim + m.rot_dim)
         out = torch.empty(rows, m.heads, m.vdim, dtype=self.dtype, device=self.device)
         for group in batch.groups:
-            expand = group.max_new > SHORT_PORTION and group.portions is not None and \
+            expand = group.max_new > SHORT_PORTION and group.portions is not None and m.kv_rank % 8 == 0 and \
                 latent_prompt_supported(m.dim, m.rot_dim, m.vdim, self.dtype)
             attend = self._attend_expanded if expand else self._attend_latents
             attend(layer, q[group.rows], out[group.rows], pages, batch.positions[group.rows], group)
