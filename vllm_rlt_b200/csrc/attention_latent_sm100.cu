@@ -182,7 +182,7 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
   } else if (warp == 4) {
     // ---- S^T(j) once the keys are there and the scores of stage j - 2 have been read ----
     const uint64_t q_desc = umma_desc(smem_u32(queries), 16, 1024);
-    const int steps = (row_dim + 15) / 16;
+    const int steps = (row_dim + 15) / 16, whole_blocks = steps / 4;
     for (int j = 0; j < stages; ++j) {
       bool ok = j > 0 || mbar_spin(smem_u32(&sm.full_q), 0);
       ok = ok && (j < 2 || mbar_spin(smem_u32(&sm.p_ready[j & 1]), ((j - 2) >> 1) & 1));
@@ -191,9 +191,19 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
       tcgen05_after_sync();
       const uint64_t k_desc = umma_desc(smem_u32(keys + (j & 1) * blocks * kBlockBytes), 16, 1024);
       if (elect_one()) {
-        for (int ks = 0; ks < steps; ++ks)
-          umma_issue(tmem + (j & 1) * kN, k_desc + static_cast<uint64_t>(((ks >> 2) * kBlockBytes + (ks & 3) * 32) >> 4),
-                     q_desc + static_cast<uint64_t>(((ks >> 2) * kN * 128 + (ks & 3) * 32) >> 4), kIdescS, ks > 0);
+        uint64_t k_at = k_desc, q_at = q_desc;
+        const uint32_t scores = tmem + (j & 1) * kN;
+        for (int block = 0; block < whole_blocks; ++block) {      // the issue of an MMA must not cost more than the MMA: constants only
+#pragma unroll
+          for (int ks = 0; ks < 4; ++ks) umma_issue(scores, k_at + static_cast<uint64_t>(ks * 2), q_at + static_cast<uint64_t>(ks * 2), kIdescS, (block > 0 || ks > 0) ? 1u : 0u);
+          k_at += kBlockBytes >> 4;
+          q_at += kN * 128 >> 4;
+        }
+        for (int ks = whole_blocks * 4; ks < steps; ++ks) {
+          umma_issue(scores, k_at, q_at, kIdescS, ks > 0);
+          k_at += 2;
+          q_at += 2;
+        }
         umma_commit(smem_u32(&sm.s_ready[j & 1]));
       }
       __syncwarp();
@@ -205,11 +215,14 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
       tcgen05_after_sync();
       const uint64_t v_desc = umma_desc(smem_u32(keys + (j & 1) * blocks * kBlockBytes), kBlockBytes, 1024), p_desc = umma_desc(smem_u32(sm.p[j & 1]), 16, 1024);
       if (elect_one()) {
-        for (int tile = 0; tile < value_tiles; ++tile)
+        uint64_t v_at = v_desc;
+        for (int tile = 0; tile < value_tiles; ++tile) {
 #pragma unroll
           for (int ks = 0; ks < kKeys / 16; ++ks)
-            umma_issue(tmem + kColO + tile * kN, v_desc + static_cast<uint64_t>((tile * 2 * kBlockBytes + ks * 2048) >> 4),
-                       p_desc + static_cast<uint64_t>(ks * 2), kIdescO, (j > 0 || ks > 0) ? 1u : 0u);
+            umma_issue(tmem + kColO + tile * kN, v_at + static_cast<uint64_t>(ks * 2048 >> 4), p_desc + static_cast<uint64_t>(ks * 2), kIdescO,
+                       (j > 0 || ks > 0) ? 1u : 0u);
+          v_at += 2 * kBlockBytes >> 4;
+        }
         umma_commit(smem_u32(&sm.pv_done[j & 1]));
       }
       __syncwarp();
