@@ -42,11 +42,6 @@ struct PromptShared {
   uint32_t tmem_base;
 };
 
-__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
-  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-               ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(z), "r"(bar) : "memory");
-}
-
 // Stages [begin, end) of a query tile.
 struct Span { int begin, end; };
 
@@ -304,17 +299,9 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   if (warp == 8) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kColumns) : "memory");
 }
 
-// [rows][heads][width] 16-bit elements in boxes of 64 columns x one head x `box_rows` rows; what lies outside a head reads as zero.
+// [rows][heads][width] elements in boxes of 64 columns x one head x `box_rows` rows.
 int make_head_rows_map(CUtensorMap* map, const void* base, int width, int heads, int64_t rows, int64_t head_stride, int64_t row_stride, int box_rows) {
-  EncodeTiledFn fn = encode_tiled_fn();
-  if (fn == nullptr) return RLT_ERR_UNSUPPORTED;
-  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(width), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(rows)};
-  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(head_stride) * 2, static_cast<cuuint64_t>(row_stride) * 2};
-  const cuuint32_t box[3] = {64, 1, static_cast<cuuint32_t>(box_rows)};
-  const cuuint32_t elem[3] = {1, 1, 1};
-  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? RLT_OK : RLT_ERR_UNSUPPORTED;
+  return make_box_map<3>(map, base, {width, heads, rows}, {1, head_stride, row_stride}, {64, 1, box_rows});
 }
 
 template <int kK, int kV>

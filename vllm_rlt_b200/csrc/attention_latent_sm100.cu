@@ -150,9 +150,7 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
       if (lane == 0) mbar_expect_tx(smem_u32(&sm.full_q), static_cast<uint32_t>(blocks * kN * 128));
       __syncwarp();
       if (lane < blocks)
-        asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-                     ::"r"(smem_u32(queries + lane * kN * 128)), "l"(reinterpret_cast<uint64_t>(&q_map)), "r"(lane * 64), "r"(first_row * heads + r_base),
-                       "r"(smem_u32(&sm.full_q)) : "memory");
+        tma_load_2d(smem_u32(queries + lane * kN * 128), &q_map, lane * 64, first_row * heads + r_base, smem_u32(&sm.full_q));
       __syncwarp();
     }
     const int boxes = kKeys / box_tokens, box = lane % boxes;
@@ -174,9 +172,7 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
       __syncwarp();
       if (from >= 0)
         for (int block = lane / boxes; block < blocks; block += 32 / boxes)
-          asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-                       ::"r"(smem_u32(keys + ((j & 1) * blocks + block) * kBlockBytes + box * box_tokens * 128)), "l"(reinterpret_cast<uint64_t>(&map)),
-                         "r"(block * 64), "r"(at), "r"(from), "r"(bar) : "memory");
+          tma_load_3d(smem_u32(keys + ((j & 1) * blocks + block) * kBlockBytes + box * box_tokens * 128), &map, block * 64, at, from, bar);
       __syncwarp();
     }
   } else if (warp == 4) {
@@ -372,32 +368,6 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
   if (warp == 4) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kColumns) : "memory");
 }
 
-// The cache as [pages][tokens][columns], boxes of 64 columns x `box_tokens` tokens; columns behind a row read as zero.
-int make_latent_map(CUtensorMap* map, const AttentionArgs& a, int box_tokens) {
-  EncodeTiledFn fn = encode_tiled_fn();
-  if (fn == nullptr) return RLT_ERR_UNSUPPORTED;
-  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(a.head_dim), static_cast<cuuint64_t>(a.block_size), static_cast<cuuint64_t>(a.num_blocks)};
-  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(a.token_stride) * 2, static_cast<cuuint64_t>(a.block_stride) * 2};
-  const cuuint32_t box[3] = {64, static_cast<cuuint32_t>(box_tokens), 1};
-  const cuuint32_t elem[3] = {1, 1, 1};
-  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(a.key_cache), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? RLT_OK : RLT_ERR_UNSUPPORTED;
-}
-
-// The queries as [(token, head) pairs][columns], boxes of 64 columns x kN pairs.
-int make_query_map(CUtensorMap* map, const AttentionArgs& a, int box_rows) {
-  EncodeTiledFn fn = encode_tiled_fn();
-  if (fn == nullptr) return RLT_ERR_UNSUPPORTED;
-  const cuuint64_t dims[2] = {static_cast<cuuint64_t>(a.head_dim), static_cast<cuuint64_t>(a.rows) * static_cast<cuuint64_t>(a.q_heads)};
-  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(a.head_dim) * 2};
-  const cuuint32_t box[2] = {64, static_cast<cuuint32_t>(box_rows)};
-  const cuuint32_t elem[2] = {1, 1};
-  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(a.q), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? RLT_OK : RLT_ERR_UNSUPPORTED;
-}
-
 // Keys that a row tile can see: the window and the other tokens of the tile, or the capacity.
 int64_t visible_keys(const AttentionArgs& a, int max_new) {
   const int64_t capacity = static_cast<int64_t>(a.table_width) * a.block_size;
@@ -429,7 +399,9 @@ template <int kN>
 int launch(const AttentionArgs& a, int max_new, int sm_count, float* partials, unsigned* error, cudaStream_t stream) {
   CUtensorMap map, q_map;
   const int box_tokens = a.block_size % kKeys == 0 ? kKeys : 16;
-  if (make_latent_map(&map, a, box_tokens) != RLT_OK || make_query_map(&q_map, a, kN) != RLT_OK) {
+  // the cache as [pages][tokens][columns], the queries as [(token, head) pairs][columns]
+  if (make_box_map<3>(&map, a.key_cache, {a.head_dim, a.block_size, a.num_blocks}, {1, a.token_stride, a.block_stride}, {64, box_tokens, 1}) != RLT_OK ||
+      make_box_map<2>(&q_map, a.q, {a.head_dim, static_cast<int64_t>(a.rows) * a.q_heads}, {1, a.head_dim}, {64, kN}) != RLT_OK) {
     set_last_error_text("scored_attention: cuTensorMapEncodeTiled rejected the latent cache or the queries");
     return RLT_ERR_UNSUPPORTED;
   }

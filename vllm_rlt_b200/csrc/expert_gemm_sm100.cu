@@ -33,11 +33,6 @@ struct ExpertShared {
   uint32_t tmem_base;
 };
 
-__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-               ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(bar) : "memory");
-}
-
 struct Tile { int expert, row, count, output; };   // first sorted row, rows of the tile, first output
 
 template <int kTokens>
@@ -192,17 +187,8 @@ expert_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
   if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kColumns) : "memory");
 }
 
-// A row-major [rows, columns] 16-bit matrix in boxes of 64 columns, 128-byte swizzle; what lies outside reads as zero.
 int make_matrix_map(CUtensorMap* map, const void* base, int64_t rows, int64_t columns, int64_t stride, int box_rows) {
-  EncodeTiledFn fn = encode_tiled_fn();
-  if (fn == nullptr) return RLT_ERR_UNSUPPORTED;
-  const cuuint64_t dims[2] = {static_cast<cuuint64_t>(columns), static_cast<cuuint64_t>(rows)};
-  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(stride) * 2};
-  const cuuint32_t box[2] = {kDepth, static_cast<cuuint32_t>(box_rows)};
-  const cuuint32_t elem[2] = {1, 1};
-  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? RLT_OK : RLT_ERR_UNSUPPORTED;
+  return make_box_map<2>(map, base, {columns, rows}, {1, stride}, {kDepth, box_rows});
 }
 
 template <int kTokens>

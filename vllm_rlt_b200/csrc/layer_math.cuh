@@ -54,4 +54,18 @@ __device__ __forceinline__ void store_floats(T* p, const float (&v)[kVec]) {
   *reinterpret_cast<Vec*>(p) = x;
 }
 
+// Sum over a CTA of kThreads (at most 1024) threads, the same for all of them; scratch: one float per warp, free again at the next call.
+template <int kThreads>
+__device__ __forceinline__ float block_sum(float v, float* scratch) {
+#pragma unroll
+  for (int x = 16; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
+  __syncthreads();                     // an earlier sum has been read
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  v = (threadIdx.x & 31) < kThreads / 32 ? scratch[threadIdx.x & 31] : 0.0f;
+#pragma unroll
+  for (int x = kThreads / 64; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
+  return __shfl_sync(0xffffffffu, v, 0);
+}
+
 }  // namespace rlt

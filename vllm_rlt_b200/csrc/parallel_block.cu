@@ -20,17 +20,6 @@ namespace {
 
 constexpr int kThreads = 256;
 
-__device__ __forceinline__ float block_sum(float v, float* scratch) {
-#pragma unroll
-  for (int x = 16; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
-  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
-  __syncthreads();
-  v = (threadIdx.x & 31) < kThreads / 32 ? scratch[threadIdx.x & 31] : 0.0f;
-#pragma unroll
-  for (int x = 4; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
-  return __shfl_sync(0xffffffffu, v, 0);
-}
-
 template <typename T, int kVec>
 __global__ void __launch_bounds__(kThreads)
 residual_norm_kernel(float* residual, const T* __restrict__ delta, const int64_t* __restrict__ tokens,
@@ -65,7 +54,7 @@ residual_norm_kernel(float* residual, const T* __restrict__ delta, const int64_t
       ss = fmaf(v[e], v[e], ss);
     }
   }
-  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + eps);
+  const float r = 1.0f / sqrtf(block_sum<kThreads>(ss, scratch) / static_cast<float>(width) + eps);
   for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
     float v[kVec], w[kVec];
     load_floats<float, kVec>(weight + i, w);
@@ -142,7 +131,7 @@ gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict
     }
     store_floats<float, kVec>(row_values + i, v);
   }
-  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(part) + eps);
+  const float r = 1.0f / sqrtf(block_sum<kThreads>(ss, scratch) / static_cast<float>(part) + eps);
   T* dst = out + row * out_stride + first;
   for (int i = threadIdx.x * kVec; i < part; i += kThreads * kVec) {   // each thread reads back what it staged itself
     float v[kVec], w[kVec];

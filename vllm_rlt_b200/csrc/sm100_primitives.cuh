@@ -94,6 +94,15 @@ __device__ __forceinline__ void tma_load_page_kv(uint32_t dst, const CUtensorMap
         "l"(policy)
       : "memory");
 }
+// Boxes of bf16 maps made by make_box_map: coordinates innermost first.
+__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
+  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
+               ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(bar) : "memory");
+}
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
+               ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(z), "r"(bar) : "memory");
+}
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -267,6 +276,25 @@ inline EncodeTiledFn encode_tiled_fn() {
       fn = reinterpret_cast<EncodeTiledFn>(p);
   });
   return fn;
+}
+
+// A bf16 tensor of kRank dimensions (innermost first, strides in elements, the innermost one 1) in boxes of 64 x box[1] x .. elements,
+// 128-byte swizzle; what a box holds outside the tensor reads as zero.
+template <int kRank>
+inline int make_box_map(CUtensorMap* map, const void* base, const int64_t (&dims)[kRank], const int64_t (&strides)[kRank], const int (&box)[kRank]) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (fn == nullptr) return RLT_ERR_UNSUPPORTED;
+  cuuint64_t d[kRank], s[kRank];
+  cuuint32_t b[kRank], e[kRank];
+  for (int i = 0; i < kRank; ++i) {
+    d[i] = static_cast<cuuint64_t>(dims[i]);
+    b[i] = static_cast<cuuint32_t>(box[i]);
+    e[i] = 1;
+    if (i > 0) s[i - 1] = static_cast<cuuint64_t>(strides[i]) * 2;
+  }
+  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, kRank, const_cast<void*>(base), d, s, b, e, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? RLT_OK : RLT_ERR_UNSUPPORTED;
 }
 
 // Tensor map over one layer's cache view as [num_blocks][16 tokens][kv_heads * head_dim] elements,

@@ -31,18 +31,6 @@ struct StreamArgs {
   void* out; int width;
 };
 
-__device__ __forceinline__ float block_sum(float v, float* scratch) {
-#pragma unroll
-  for (int x = 16; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
-  __syncthreads();                     // the previous sum has been read
-  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
-  __syncthreads();
-  v = (threadIdx.x & 31) < kThreads / 32 ? scratch[threadIdx.x & 31] : 0.0f;
-#pragma unroll
-  for (int x = 4; x > 0; x >>= 1) v += __shfl_xor_sync(0xffffffffu, v, x);
-  return __shfl_sync(0xffffffffu, v, 0);
-}
-
 template <typename T, int kS, int kVec>
 __global__ void __launch_bounds__(kThreads)
 stream_mix_kernel(StreamArgs a) {
@@ -84,7 +72,7 @@ stream_mix_kernel(StreamArgs a) {
         ss = fmaf(v[e], v[e], ss);
       }
     }
-    const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + a.eps);
+    const float r = 1.0f / sqrtf(block_sum<kThreads>(ss, scratch) / static_cast<float>(width) + a.eps);
     ss = 0.0f;
     for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {   // each thread reads back what it staged itself
       float v[kVec], w[kVec];
@@ -159,7 +147,7 @@ stream_mix_kernel(StreamArgs a) {
       }
     }
   }
-  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + a.eps);
+  const float r = 1.0f / sqrtf(block_sum<kThreads>(ss, scratch) / static_cast<float>(width) + a.eps);
   T* out = static_cast<T*>(a.out) + static_cast<int64_t>(blockIdx.x) * width;
   for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
     float v[kVec], w[kVec];
