@@ -530,7 +530,7 @@ RLT_API int rlt_sandwich_norm(const void* x, const void* weight, const void* res
  *             - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
  * softmax over the visible keys, weighted sum of the values.  Keys and values may have different head
  * sizes and cache strides; query and output rows may be column slices (strides in elements).
- * window > 0: only keys with p - j < window.  value_cache may be key_cache with one KV head: a value is then the first value_dim
+ * window > 0: only keys with p - j < window.  sink (fp32 [q_heads], or null): one more term exp(sink_h) of the denominator.  value_cache may be key_cache with one KV head: a value is then the first value_dim
  * elements of its key row.
  * context_lengths[s]: tokens of sequence s after this portion.  planned != 0: the workspace holds the
  * plan of rlt_verify_attention_plan for the same tables, lengths and packing (max_new <= 16 only). */
@@ -542,16 +542,19 @@ RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, void* out, int
                          int64_t num_blocks, int block_size, int q_heads, int kv_heads, int key_dim,
                          int value_dim, int dtype, const int32_t* block_tables, int sequences, int table_width,
                          const int32_t* context_lengths, const int32_t* cu_seqlens_q, int rows, int max_new,
-                         float scale, float temp_coef, int temp_every, int distance_bias, int window, int planned,
-                         void* workspace, size_t workspace_bytes, rlt_stream_t stream);
+                         float scale, float temp_coef, int temp_every, int distance_bias, int window,
+                         const float* sink, int planned, void* workspace, size_t workspace_bytes, rlt_stream_t stream);
 
 /* The fp32 residual stream and the norm that opens a layer:
  *   r = tokens ? embed[tokens[i]] : residual[i];  r += delta[i];  residual[i] = r (store_residual != 0)
  *   out[row] = r / sqrt(mean(r^2) + eps) * (weight_offset + weight)
- * i = row_index ? row_index[row] : row.  delta, embed, out: `dtype`; residual, weight: fp32. */
+ * i = row_index ? row_index[row] : row.  delta, embed, out: `dtype`; residual, weight, delta_weight: fp32.
+ * delta_weight (may be null): r += delta_scale * norm(delta[i]) * delta_weight instead, a norm of its own behind the sublayer.
+ * centred != 0: both norms subtract the mean first (layer norm), mean(.^2) is then the variance. */
 RLT_API int rlt_residual_norm(float* residual, const void* delta, const int64_t* tokens, const void* embed, int64_t vocab,
                       const int64_t* row_index, int store_residual, const float* weight, float weight_offset,
-                      void* out, int rows, int width, float eps, int dtype, rlt_stream_t stream);
+                      const float* delta_weight, float delta_scale, int centred, void* out, int rows, int width, float eps,
+                      int dtype, rlt_stream_t stream);
 
 /* Columns of a stacked projection to where they are needed: k_width columns from k_col and v_width from v_col into
  * the pages of (row_seq[row], positions[row]) — row_seq -1: a padding row, nothing is written — and act_width
@@ -612,34 +615,40 @@ RLT_API int rlt_stream_mix(float* streams, int stream_count, const void* delta, 
 
 /* The stacked down projections of latent attention: rmsnorm(proj[q_col ..]) * q_weight into q_out, and the cache row
  * [rmsnorm(proj[kv_col .. + kv_rank]) * kv_weight | rotated proj[kv_col + kv_rank .. + rot_dim]] into the row's page.
- * Pairs (2i, 2i + 1) of the first rot_dims dimensions are turned by position * frequencies[i]. */
+ * Pairs (2i, 2i + 1) of the first rot_dims dimensions — with halves != 0 pairs (i, i + rot_dims / 2) — are turned by
+ * position * frequencies[i] and multiplied by amplitude. */
 RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, int q_col, int q_rank, int kv_col, int kv_rank,
                      int rot_dim, int rot_dims, const float* q_weight, const float* kv_weight, float eps,
-                     const double* frequencies, void* q_out, int64_t q_out_stride, void* cache, int64_t block_stride,
-                     int64_t token_stride, int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
+                     const double* frequencies, int halves, float amplitude, void* q_out, int64_t q_out_stride,
+                     void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
                      const int32_t* row_seq, const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
 
 /* The same rotation of `dim` elements of every head, from src to dst (which may be one); strides in elements. */
 RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head, void* dst, int64_t dst_row,
-                     int64_t dst_head, int heads, int dim, int rot_dims, const double* frequencies,
-                     const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
+                     int64_t dst_head, int heads, int dim, int rot_dims, const double* frequencies, int halves,
+                     float amplitude, const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
 
 /* Cache rows of positions first[s] .. of every sequence s, packed: row cu[s] + i holds position first[s] + i. */
 RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks,
                       int block_size, int row_width, const int32_t* tables, int table_width, const int32_t* first,
                       const int32_t* cu, int sequences, int rows, void* out, int dtype, rlt_stream_t stream);
 
-/* Prompt attention of latent layers (bf16).  q [rows][heads][dim + rot_dim]; kv [key_rows][heads * dim | heads * vdim]: keys and
- * values expanded from the latents; shared_keys [key_rows][rot_dim]: the rotated key part of all heads; out [rows][heads * vdim].
- * Query position p sees positions p - window + 1 .. p (window 0: all before it).  tiles: eight int32 words per tile of up to 256
+/* Prompt attention over packed keys and values (bf16): expanded from latents, or gathered from the pages of a windowed layer.
+ * q [rows][heads][dim + rot_dim]; keys [key_rows][kv_heads][dim], values [key_rows][kv_heads][vdim] (strides between rows); shared_keys
+ * [key_rows][rot_dim]: a key part of all heads (null with rot_dim 0); out [rows][heads * vdim].  Query head h reads key/value head
+ * h / (heads / kv_heads).  Query position p sees positions p - window + 1 .. p (window 0: all before it).  sink (fp32 [heads], or null): one
+ * more term exp(sink_h) of the denominator.  gate (or null): the output is multiplied by sigmoid(gate), of one value per element, or with
+ * gate_per_head one per head.  tiles: eight int32 words per tile of up to 256
  * consecutive query rows of a sequence: first query row, rows, position of the first row, packed key row of position f, f, 0, 0, 0
  * (f: first position of the sequence among the packed keys).  workspace: 256 bytes; its first word is set when a bounded wait
  * gave up.  Supported: bf16, dim and vdim up to 128, rot_dim up to 64, multiples of 8. */
 RLT_API int rlt_latent_prompt_supported(int dim, int rot_dim, int vdim, int dtype);
-RLT_API int rlt_latent_prompt_attention(const void* q, int64_t q_stride, const void* kv, int64_t kv_stride,
-                                const void* shared_keys, int64_t shared_stride, void* out, int64_t out_stride, int rows,
-                                int key_rows, int heads, int dim, int rot_dim, int vdim, const int32_t* tiles, int tile_count,
-                                float scale, int window, int dtype, void* workspace, rlt_stream_t stream);
+RLT_API int rlt_latent_prompt_attention(const void* q, int64_t q_stride, const void* keys, int64_t key_stride,
+                                const void* values, int64_t value_stride, const void* shared_keys, int64_t shared_stride,
+                                void* out, int64_t out_stride, int rows, int key_rows, int heads, int kv_heads, int dim,
+                                int rot_dim, int vdim, const int32_t* tiles, int tile_count, float scale, int window,
+                                const float* sink, const void* gate, int64_t gate_stride, int gate_per_head, int dtype,
+                                void* workspace, rlt_stream_t stream);
 
 /* Mixture of experts.  route: s = softmax(logits) in fp32, the `top` largest of s + correction (null: none), weights =
  * chosen s / (their sum + floor_sum); counts [experts] must be zero before.  gather: rows sorted by expert, and every
@@ -656,6 +665,30 @@ RLT_API int rlt_expert_gemm(const void* x, int64_t x_stride, const void* w, void
 /* g = min(gate, limit), u = clamp(up, -limit, limit): out = g * sigmoid(slope * g) * (u + 1); gate at column 0, up at up_col. */
 RLT_API int rlt_clamped_glu(const void* gate_up, int64_t row_stride, int up_col, void* out, int64_t out_stride, int64_t rows,
                     int cols, float limit, float slope, int dtype, rlt_stream_t stream);
+
+/* out = act(gate) * up; gate at column 0, up at up_col; act as in rlt_block_epilogue. */
+RLT_API int rlt_gated_unit(const void* gate_up, int64_t row_stride, int up_col, void* out, int64_t out_stride, int64_t rows,
+                   int cols, int act, int dtype, rlt_stream_t stream);
+
+/* out = y * sigmoid(gate), y and out [rows][heads * dim]; gate [rows][heads * dim], or with per_head != 0 [rows][heads]; out may be y. */
+RLT_API int rlt_head_gate(const void* y, int64_t y_stride, const void* gate, int64_t gate_stride, void* out, int64_t out_stride,
+                  int64_t rows, int heads, int dim, int per_head, int dtype, rlt_stream_t stream);
+
+/* x = cap * tanh(x / cap), fp32, in place. */
+RLT_API int rlt_soft_cap(float* x, int64_t count, float cap, rlt_stream_t stream);
+
+/* What stands between the projections of an attention layer and its scores: a causal convolution over time per channel of q, k and v
+ * (no bias, no activation), then with unit_norm != 0 q and k of every head divided by their root mean square, then k and v into the
+ * pages of the row's position and q into q_out [rows][q_heads * key_dim].  Channels are ordered q, k, v in weight (fp32 [channels][taps])
+ * and in state ([slots][taps - 1][channels] of `dtype`, the last inputs, updated in place); q_col, k_col, v_col: their columns in proj.
+ * Sequences and slots as in rlt_causal_conv; lengths[s]: tokens of sequence s after the portion (0: padding, nothing is written to pages). */
+RLT_API int rlt_conv_heads(const void* proj, int64_t proj_stride, int q_col, int k_col, int v_col, int q_heads, int kv_heads,
+                   int key_dim, int value_dim, const float* weight, int taps, int unit_norm, float eps, void* state,
+                   int64_t slots, void* q_out, int64_t q_out_stride, void* key_cache, int64_t k_block_stride,
+                   int64_t k_token_stride, void* value_cache, int64_t v_block_stride, int64_t v_token_stride,
+                   int64_t num_blocks, int block_size, const int32_t* tables, int table_width, const int32_t* cu_seqlens,
+                   const int32_t* starts, const int32_t* lengths, const int32_t* slot_of, int sequences, int max_tokens,
+                   int dtype, rlt_stream_t stream);
 
 #ifdef __cplusplus
 }

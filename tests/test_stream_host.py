@@ -27,8 +27,8 @@ def test_configurations_parse_and_name_every_tensor(name):
         assert len(layer.sublayers) == (2 if entry["mlp"] else 1)
         assert (f"l{i}.norm2" in shapes) == (f"l{i}.hc2.mix" in shapes) == bool(entry["mlp"])
         if entry["type"] == "latent_attention":
-            assert torch.equal(layer.w_down[layer.kv_col:layer.kv_col + layer.mixer.row], weights[f"l{i}.mix.dkv"])
-            assert torch.equal(layer.w_uk.reshape(-1, layer.mixer.kv_rank), weights[f"l{i}.mix.uk"])
+            assert torch.equal(layer.latent.w_down[layer.latent.kv_col:layer.latent.kv_col + layer.mixer.row], weights[f"l{i}.mix.dkv"])
+            assert torch.equal(layer.latent.w_uk.reshape(-1, layer.mixer.kv_rank), weights[f"l{i}.mix.uk"])
         else:
             for at, n in ((layer.q_at, "q"), (layer.k_at, "k"), (layer.v_at, "v"), (layer.g_at, "g")):
                 assert torch.equal(layer.w_in[at:at + weights[f"l{i}.mix.{n}"].shape[0]], weights[f"l{i}.mix.{n}"])

@@ -18,13 +18,15 @@ from .engine import Engine, StepEntry
 from .hybrid_lm import HybridLM, HybridLMConfig
 from .kv_cache import RollbackResult, finalize_tokens, kv_write, rollback
 from .experts import expert_gather, expert_gemm, expert_route
-from .latent import latent_gather, latent_prompt_attention, latent_prompt_supported, latent_write, rotate_heads, rotation_frequencies
-from .layers import block_epilogue, clamped_glu, residual_norm, rope_kv_write, sandwich_norm, stream_mix
+from .latent import (YarnScaling, latent_gather, latent_prompt_attention, latent_prompt_supported, latent_write, packed_attention,
+                     rotate_heads, rotation_frequencies)
+from .layers import block_epilogue, clamped_glu, gated_unit, head_gate, residual_norm, rope_kv_write, sandwich_norm, soft_cap, stream_mix
 from .looped_lm import LoopedLM, LoopedLMConfig, seeded_state_dict
-from .recurrent import causal_conv, decay_scan, decay_table, gated_norm, ssd_scan
+from .recurrent import causal_conv, conv_heads, decay_scan, decay_table, gated_norm, ssd_scan
 from .registry import load_model, register_model, registered_architectures
 from .runner import (B200SpeculativeRunner, KVCacheManagerView, ModelRunnerOutput, Request, SamplingParams, ScheduledRequest,
                      SchedulerOutput, SpeculativeConfig, SpeculativeRoundTicket, SpeculativeStats)
+from .sandwich_lm import SandwichLM, SandwichLMConfig
 from .stream_lm import StreamLM, StreamLMConfig
 from .sequence_cache import CacheFull, CacheSpec, KVSpec, SequenceCache, StateSpec
 from .speculative import (PipelineState, SpeculativeResult, accept_greedy, accept_rejection, argmax_rows,
@@ -44,4 +46,5 @@ __all__ = [
     "read_weights", "register_model", "registered_architectures", "residual_norm", "ssd_scan",
     "StreamLM", "StreamLMConfig", "clamped_glu", "decay_scan", "decay_table", "expert_gather", "expert_gemm", "expert_route",
     "latent_gather", "latent_prompt_attention", "latent_prompt_supported", "latent_write", "rotate_heads", "rotation_frequencies", "stream_mix",
+    "SandwichLM", "SandwichLMConfig", "YarnScaling", "conv_heads", "gated_unit", "head_gate", "packed_attention", "soft_cap",
 ]

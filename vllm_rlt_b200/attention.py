@@ -48,7 +48,8 @@ class ScoreTerms:
         score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
                 - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
 
-    over the keys j <= p, with `window` > 0 only those with p - j < window.
+    over the keys j <= p, with `window` > 0 only those with p - j < window.  `sink` (float32 [H]): the softmax's denominator
+    has one more term, exp(sink[h]), which is not scaled and has neither key nor value.
     """
 
     scale: float
@@ -56,6 +57,12 @@ class ScoreTerms:
     temp_every: int = 1
     distance_bias: bool = False
     window: int = 0
+    sink: torch.Tensor | None = field(default=None, compare=False)
+
+
+def check_sink(sink, heads: int) -> None:
+    if sink is not None and (sink.dtype != torch.float32 or sink.shape != (heads,) or not sink.is_contiguous()):
+        raise ValueError("sink must be contiguous float32 [heads]")
 
 
 @dataclass
@@ -330,7 +337,7 @@ class B200PagedAttention:
         heads over 16-token pages in 16 bits run on the tiled kernels (portions of at most 16 tokens on the verify
         kernel, whose plan a `shared_plan` block reuses; longer ones on the prompt kernel), everything else on
         the shape-generic ones."""
-        device = _capi.require_cuda(q, out, key_cache, value_cache, block_tables, context_lengths, cu_seqlens_q)
+        device = _capi.require_cuda(q, out, key_cache, value_cache, block_tables, context_lengths, cu_seqlens_q, terms.sink)
         rows, heads, key_dim = q.shape
         if q.dtype not in _capi.DTYPE_CODES or any(t.dtype != q.dtype for t in (out, key_cache, value_cache)):
             raise ValueError("q, out and the caches must share a float32/float16/bfloat16 dtype")
@@ -349,6 +356,7 @@ class B200PagedAttention:
             raise ValueError("tables int32 [sequences, pages], context_lengths int32 [sequences], cu_seqlens_q int32 [sequences + 1]")
         if heads % key_cache.shape[2]:
             raise ValueError("query heads must be a positive multiple of KV heads")
+        check_sink(terms.sink, heads)
         if rows == 0:
             return out
         blocks, block, kv_heads, value_dim = value_cache.shape
@@ -361,7 +369,7 @@ class B200PagedAttention:
             # prompt calls have scratch of their own: a mixed step's plan for its short portions survives them
             workspace = self._workspace(device, stream.value or 0 if max_new <= 16 else ("prompt", stream.value or 0), nbytes)
             planned = False
-            tiled = max_new <= 16 and not terms.window and q.dtype != torch.float32 and key_dim == value_dim == 128 and block == 16
+            tiled = max_new <= 16 and not terms.window and terms.sink is None and q.dtype != torch.float32 and key_dim == value_dim == 128 and block == 16
             versions = self._versions(block_tables, context_lengths, cu_seqlens_q) if self._sharing and tiled else None
             if versions is not None:
                 plan_key = (block_tables.data_ptr(), sequences, width, context_lengths.data_ptr(), cu_seqlens_q.data_ptr(), rows,
@@ -381,7 +389,7 @@ class B200PagedAttention:
                 key_cache.stride(1), _capi.ptr(value_cache), value_cache.stride(0), value_cache.stride(1), blocks, block, heads,
                 kv_heads, key_dim, value_dim, dtype, _capi.ptr(block_tables), sequences, width, _capi.ptr(context_lengths),
                 _capi.ptr(cu_seqlens_q), rows, int(max_new), float(terms.scale), float(terms.temp_coef), int(terms.temp_every),
-                int(terms.distance_bias), int(terms.window), int(planned), _capi.ptr(workspace), workspace.numel(), stream)
+                int(terms.distance_bias), int(terms.window), _capi.ptr(terms.sink), int(planned), _capi.ptr(workspace), workspace.numel(), stream)
         _capi.check(status, "scored_attention")
         return out
 

@@ -11,6 +11,7 @@ namespace rlt {
 // the row's length minus one), query head h of H, key at position j:
 //   score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
 //           - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
+// With a sink the softmax's denominator has one more term, exp(sink[h]), which has no key and no value.
 // The default is the plain 1 / sqrt(head_dim) of the looped models.
 struct ScoreTerms {
   float scale = 0.0f;        // 0: 1 / sqrt(head_dim)
@@ -18,8 +19,9 @@ struct ScoreTerms {
   int temp_every = 1;
   int distance_bias = 0;
   int window = 0;            // 0: all keys before the row, else the last `window` of them (the row's own included)
+  const float* sink = nullptr;   // [q_heads], or none
 
-  __host__ __device__ bool plain() const { return temp_coef == 0.0f && distance_bias == 0 && window == 0; }
+  __host__ __device__ bool plain() const { return temp_coef == 0.0f && distance_bias == 0 && window == 0 && sink == nullptr; }
 };
 
 struct AttentionArgs {
@@ -70,6 +72,17 @@ __device__ __forceinline__ float query_temperature(const ScoreTerms& t, int len)
 // The distance slope of query head `head`, 0 without a distance bias.
 __device__ __forceinline__ float distance_slope(const ScoreTerms& t, int head, int q_heads) {
   return t.distance_bias == 0 ? 0.0f : exp2f(-8.0f * static_cast<float>(head + 1) / static_cast<float>(q_heads));
+}
+
+// The sink of query head `head` in log2 units, -infinity without one.
+__device__ __forceinline__ float sink_log2(const ScoreTerms& t, int head) { return t.sink == nullptr ? -INFINITY : 1.4426950408889634f * t.sink[head]; }
+
+// What an output row accumulated relative to 2^m, with weights that sum to l, is multiplied by in the end (m and sink in log2 units).
+__device__ __forceinline__ float softmax_scale(float m, float l, float sink) {
+  if (!(l > 0.0f)) return 0.0f;
+  if (sink <= m) return 1.0f / (l + exp2f(sink - m));
+  const float f = exp2f(m - sink);
+  return f / fmaf(l, f, 1.0f);
 }
 
 // Table row and number of visible keys of query row `row`.

@@ -228,7 +228,7 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
                                             int value_dim, int dtype, const int32_t* block_tables, int sequences,
                                             int table_width, const int32_t* context_lengths, const int32_t* cu_seqlens_q,
                                             int rows, int max_new, float scale, float temp_coef, int temp_every,
-                                            int distance_bias, int window, int planned, void* workspace, size_t workspace_bytes,
+                                            int distance_bias, int window, const float* sink, int planned, void* workspace, size_t workspace_bytes,
                                             rlt_stream_t stream) {
   using namespace rlt;
   AttentionArgs a;
@@ -240,7 +240,7 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
   a.value_dim = value_dim; a.v_block_stride = v_block_stride; a.v_token_stride = v_token_stride;
   a.q_stride = q_stride; a.out_stride = out_stride;
   a.terms.scale = scale; a.terms.temp_coef = temp_coef; a.terms.temp_every = temp_every; a.terms.distance_bias = distance_bias;
-  a.terms.window = window;
+  a.terms.window = window; a.terms.sink = sink;
   RLT_REQUIRE(value_dim > 0 && temp_every > 0 && window >= 0, "scored_attention: value_dim and temp_every must be positive, window not negative");
   RLT_REQUIRE(cu_seqlens_q != nullptr || rows == 0, "scored_attention: cu_seqlens_q is required");
   int status = check_args(a);
@@ -254,8 +254,8 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
     status = launch_attention_latent(a, max_new, workspace, workspace_bytes, s);
     if (status != RLT_ERR_UNSUPPORTED) return status;
   }
-  if (window > 0) {
-    // the page kernels walk whole contexts: windowed rows go to the tile or generic kernel
+  if (window > 0 || sink != nullptr) {
+    // the page kernels walk whole contexts and know no sinks: such rows go to the tile or generic kernel
   } else if (max_new > 16) {
     if (prefill_sm100_supported(a)) {
       status = launch_prefill_sm100(a, workspace, workspace_bytes, s);

@@ -1,5 +1,5 @@
 // Shape-generic paged attention: any head_dim <= 640 (keys and values may differ), any block size,
-// any GQA ratio, fp32 / fp16 / bf16, with the score terms of attention.cuh.  One CTA per (query row, query head); four warps stride over the
+// any GQA ratio, fp32 / fp16 / bf16, with the score terms and sinks of attention.cuh.  One CTA per (query row, query head); four warps stride over the
 // row's tokens with an fp32 online softmax each and are merged in warp order, so a row's
 // result depends on nothing but its own query, length and K/V.  This is the path for
 // shapes the tiled sm_100a kernel (attention_sm100.cu) does not cover — the fp32 tiny
@@ -83,8 +83,10 @@ attention_generic_kernel(AttentionArgs a, float scale) {
   float big = -INFINITY;
 #pragma unroll
   for (int w = 0; w < kWarps; ++w) big = fmaxf(big, sm_m[w]);
+  const float sink = a.terms.sink == nullptr ? -INFINITY : a.terms.sink[head];
+  big = fmaxf(big, sink);
   for (int d = threadIdx.x; d < DV; d += kThreads) {
-    float total = 0.0f, acc = 0.0f;
+    float total = sink == -INFINITY ? 0.0f : expf(sink - big), acc = 0.0f;
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) {
       if (sm_m[w] == -INFINITY) continue;

@@ -1,9 +1,10 @@
-// Prompt attention of latent layers on the 5th-generation tensor cores: packed keys and values that were expanded from the
-// latents, a key part shared by all heads, a sliding window, bf16.
+// Prompt attention over packed keys and values on the 5th-generation tensor cores, bf16: expanded from the latents of a latent layer,
+// with a key part shared by all heads, or gathered from the pages of a windowed layer, one key/value head for several query heads.
+// Sliding windows, sinks, and an output gate that is applied on the way out.
 //
-// A head's key is [k (dim, its own) | r (rot_dim, the same for every head)], its value has vdim columns.  Three tensors, none of
-// them copied together: the expanded projection [key rows][heads * dim | heads * vdim], and the gathered cache rows, whose tail
-// is r.  Each is a tensor map of its own whose 64-wide boxes read as zero beyond their head's columns, so the product
+// A head's key is [k (dim, its key/value head's) | r (rot_dim, the same for every head; may be absent)], its value has vdim columns.
+// Three tensors, none of them copied together: keys, values, and for latent layers the gathered cache rows, whose tail is r.  Each is
+// a tensor map of its own whose 64-wide boxes read as zero beyond their head's columns, so the product
 // Q K^T is the sum of two: the unrotated blocks of q with k, the rotated block with r.
 //
 // 256 query tokens of one head per CTA (two tiles of 128 rows that share every stage of 64 keys), 13 warps:
@@ -15,6 +16,7 @@
 // ones, and a stage that only one of them reads is released by the other's hand.
 // TMEM columns: S0 0..63, P0 64..95 | S1 96..159, P1 160..191 | O0 256..383 | O1 384..511.
 #include "latent_attention.cuh"
+#include "layer_math.cuh"
 #include "sm100_primitives.cuh"
 
 namespace rlt {
@@ -27,29 +29,47 @@ constexpr int kBlock = kKeys * 128;        // a stage's 64-wide block of one ope
 constexpr int kQBlock = kRows * 128;
 constexpr uint32_t kColumns = 512, kTileCols = 96, kColP = 64, kColO = 256;
 
-// kK: 64-wide blocks of the unrotated key, kV: of the value.
-template <int kK, int kV>
+// kK: 64-wide blocks of the unrotated key, kR: of the shared part (0 or 1), kV: of the value.
+template <int kK, int kR, int kV>
 struct PromptShared {
-  static constexpr int kStageBytes = (kK + 1 + kV) * kBlock;
-  static constexpr int kFit = (220 * 1024 - 2 * (kK + 1) * kQBlock) / kStageBytes;
+  static constexpr int kStageBytes = (kK + kR + kV) * kBlock;
+  static constexpr int kFit = (220 * 1024 - 2 * (kK + kR) * kQBlock) / kStageBytes;
   static constexpr int kStages = kFit < 6 ? kFit : 6;
   static_assert(kStages > kRows / kKeys, "tile 1 may start kRows keys behind tile 0: its first stage must be in the ring's first round");
-  unsigned char q[2][kK + 1][kQBlock];     // [tile][block][row][64], 128-byte swizzle; the output's staging rows in the end
-  unsigned char k[kStages][kK + 1][kBlock];
+  unsigned char q[2][kK + kR][kQBlock];     // [tile][block][row][64], 128-byte swizzle; the output's staging rows in the end
+  unsigned char k[kStages][kK + kR][kBlock];
   unsigned char v[kStages][kV][kBlock];
   unsigned long long full_q, full_k[kStages], full_v[kStages], free_k[kStages], free_v[kStages];
   unsigned long long s_ready[2], s_free[2], p_ready[2], pv_done[2];
   uint32_t tmem_base;
 };
 
+// Eight output elements times the sigmoid of their gates.
+__device__ __forceinline__ uint4 gated(uint4 piece, const __nv_bfloat16* gate, int column, bool per_head) {
+  const __nv_bfloat16* y = reinterpret_cast<const __nv_bfloat16*>(&piece);
+  float v[8], g[8];
+  if (per_head) {
+    const float one = sigmoid<__nv_bfloat16>(__bfloat162float(*gate));
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = one;
+  } else {
+    load_floats<__nv_bfloat16, 8>(gate + column, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = sigmoid<__nv_bfloat16>(g[e]);
+  }
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] = __bfloat162float(y[e]) * g[e];
+  return make_uint4(pack2<true>(v[0], v[1]), pack2<true>(v[2], v[3]), pack2<true>(v[4], v[5]), pack2<true>(v[6], v[7]));
+}
+
 // Stages [begin, end) of a query tile.
 struct Span { int begin, end; };
 
 // The issue loop of one warp: the scores (kScores) or the output product of query tile `t`.  The whole warp runs it, one elected lane
 // issues.  S(j) waits for Q (first) or for S(j - 1) to be read, and K(j); O(j) for P(j) and V(j).  True when a wait gave up.
-template <bool kScores, int kK, int kV>
-__device__ __forceinline__ bool issue_products(PromptShared<kK, kV>& sm, uint32_t tmem, int t, Span mine, Span other, uint32_t idesc) {
-  constexpr int kStages = PromptShared<kK, kV>::kStages;
+template <bool kScores, int kK, int kR, int kV>
+__device__ __forceinline__ bool issue_products(PromptShared<kK, kR, kV>& sm, uint32_t tmem, int t, Span mine, Span other, uint32_t idesc) {
+  constexpr int kStages = PromptShared<kK, kR, kV>::kStages;
   const uint32_t s_col = tmem + t * kTileCols, o_col = tmem + kColO + t * kRows;
   if (kScores && mine.begin < mine.end && !__all_sync(0xffffffffu, mbar_wait(smem_u32(&sm.full_q), 0))) return true;
   const uint64_t q_desc = umma_desc(smem_u32(&sm.q[t][0][0]), 16, 1024);
@@ -70,7 +90,7 @@ __device__ __forceinline__ bool issue_products(PromptShared<kK, kV>& sm, uint32_
       const uint64_t k_desc = umma_desc(smem_u32(&sm.k[stage][0][0]), 16, 1024);
       if (elect_one()) {
 #pragma unroll
-        for (int ks = 0; ks < 4 * (kK + 1); ++ks)
+        for (int ks = 0; ks < 4 * (kK + kR); ++ks)
           umma_issue(s_col, q_desc + static_cast<uint64_t>(((ks >> 2) * kQBlock + (ks & 3) * 32) >> 4),
                      k_desc + static_cast<uint64_t>(((ks >> 2) * kBlock + (ks & 3) * 32) >> 4), idesc, ks > 0);
         umma_commit(smem_u32(&sm.s_ready[t]));
@@ -93,17 +113,17 @@ __device__ __forceinline__ bool issue_products(PromptShared<kK, kV>& sm, uint32_
   return false;
 }
 
-template <int kK, int kV>
+template <int kK, int kR, int kV>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap qr_map, const __grid_constant__ CUtensorMap k_map,
                      const __grid_constant__ CUtensorMap r_map, const __grid_constant__ CUtensorMap v_map, LatentPromptArgs a, float scale_log2) {
-  using Shared = PromptShared<kK, kV>;
+  using Shared = PromptShared<kK, kR, kV>;
   constexpr int kStages = Shared::kStages;
   extern __shared__ unsigned char smem_raw[];
   Shared& sm = *reinterpret_cast<Shared*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const int lane = threadIdx.x & 31, warp = __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0);
   const PromptTile tile = a.tiles[blockIdx.x];
-  const int head = blockIdx.y;
+  const int head = blockIdx.y, kv_head = head / a.share;
   const int window = a.window > 0 ? a.window : 0x40000000;
   // positions: rows tile.position .., keys tile.key_first .. ; stage j holds keys lo + 64 j ..
   const int lo = max(max(tile.position - window + 1, tile.key_first), 0);
@@ -149,33 +169,33 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
   if (warp == 12) {
     if (lane == 0) {
       const int tiles = count[1] > 0 ? 2 : 1;
-      mbar_expect_tx(smem_u32(&sm.full_q), tiles * (kK + 1) * kQBlock);
+      mbar_expect_tx(smem_u32(&sm.full_q), tiles * (kK + kR) * kQBlock);
       for (int t = 0; t < tiles; ++t) {
 #pragma unroll
         for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.q[t][b][0]), &q_map, b * 64, head, tile.q_row + t * kRows, smem_u32(&sm.full_q));
-        tma_load_3d(smem_u32(&sm.q[t][kK][0]), &qr_map, 0, head, tile.q_row + t * kRows, smem_u32(&sm.full_q));
+        if constexpr (kR > 0) tma_load_3d(smem_u32(&sm.q[t][kK][0]), &qr_map, 0, head, tile.q_row + t * kRows, smem_u32(&sm.full_q));
       }
       for (int j = 0; j < all_stages && !failed; ++j) {
         const int stage = j % kStages, use = j / kStages, row = tile.key_row + lo - tile.key_first + j * kKeys;
         if (use > 0 && !mbar_wait(smem_u32(&sm.free_k[stage]), (use - 1) & 1)) { failed = true; break; }
         uint32_t bar = smem_u32(&sm.full_k[stage]);
-        mbar_expect_tx(bar, (kK + 1) * kBlock);
+        mbar_expect_tx(bar, (kK + kR) * kBlock);
 #pragma unroll
-        for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.k[stage][b][0]), &k_map, b * 64, head, row, bar);
-        tma_load_3d(smem_u32(&sm.k[stage][kK][0]), &r_map, 0, 0, row, bar);
+        for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.k[stage][b][0]), &k_map, b * 64, kv_head, row, bar);
+        if constexpr (kR > 0) tma_load_3d(smem_u32(&sm.k[stage][kK][0]), &r_map, 0, 0, row, bar);
         if (use > 0 && !mbar_wait(smem_u32(&sm.free_v[stage]), (use - 1) & 1)) { failed = true; break; }
         bar = smem_u32(&sm.full_v[stage]);
         mbar_expect_tx(bar, kV * kBlock);
 #pragma unroll
-        for (int b = 0; b < kV; ++b) tma_load_3d(smem_u32(&sm.v[stage][b][0]), &v_map, b * 64, head, row, bar);
+        for (int b = 0; b < kV; ++b) tma_load_3d(smem_u32(&sm.v[stage][b][0]), &v_map, b * 64, kv_head, row, bar);
       }
     }
     __syncwarp();
   } else if (warp >= 8) {
-    if (warp == 8) failed = issue_products<true, kK, kV>(sm, tmem, 0, span0, span1, kIdescQK);
-    else if (warp == 9) failed = issue_products<true, kK, kV>(sm, tmem, 1, span1, span0, kIdescQK);
-    else if (warp == 10) failed = issue_products<false, kK, kV>(sm, tmem, 0, span0, span1, kIdescPV);
-    else failed = issue_products<false, kK, kV>(sm, tmem, 1, span1, span0, kIdescPV);
+    if (warp == 8) failed = issue_products<true, kK, kR, kV>(sm, tmem, 0, span0, span1, kIdescQK);
+    else if (warp == 9) failed = issue_products<true, kK, kR, kV>(sm, tmem, 1, span1, span0, kIdescQK);
+    else if (warp == 10) failed = issue_products<false, kK, kR, kV>(sm, tmem, 0, span0, span1, kIdescPV);
+    else failed = issue_products<false, kK, kR, kV>(sm, tmem, 1, span1, span0, kIdescPV);
   } else {
     // ---- softmax rows ----
     const int t = warp >> 2, warp_row = (warp & 3) * 32, row = warp_row + lane;
@@ -265,9 +285,10 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       // 64 output columns at a time through the warp's share of the tile's query operand, which nothing reads any more
       unsigned char* staging = &sm.q[t][0][0] + (warp & 3) * 4096;
       const int warp_count = min(max(count[t] - warp_row, 0), 32);
-      const float inv = l > 0.f ? 1.0f / l : 0.f;
-      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + (static_cast<int64_t>(tile.q_row) + t * kRows + warp_row) * a.out_stride +
-                           static_cast<int64_t>(head) * a.vdim;
+      const float inv = softmax_scale(m, l, a.sink == nullptr ? -INFINITY : 1.4426950408889634f * a.sink[head]);
+      const int64_t first_out = static_cast<int64_t>(tile.q_row) + t * kRows + warp_row;
+      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + first_out * a.out_stride + static_cast<int64_t>(head) * a.vdim;
+      const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(a.gate) + first_out * a.gate_stride + static_cast<int64_t>(head) * (a.gate_per_head ? 1 : a.vdim);
 #pragma unroll
       for (int b = 0; b < kV; ++b) {
         uint32_t r0[32], r1[32];
@@ -285,9 +306,11 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           const int r = 4 * i + (lane >> 3);
-          if (r < warp_count && b * 64 + (lane & 7) * 8 < a.vdim)
-            reinterpret_cast<uint4*>(dst + r * a.out_stride + b * 64)[lane & 7] =
-                *reinterpret_cast<const uint4*>(staging + r * 128 + (((lane & 7) ^ (r & 7)) << 4));
+          if (r < warp_count && b * 64 + (lane & 7) * 8 < a.vdim) {
+            uint4 piece = *reinterpret_cast<const uint4*>(staging + r * 128 + (((lane & 7) ^ (r & 7)) << 4));
+            if (a.gate != nullptr) piece = gated(piece, gate + r * a.gate_stride, b * 64 + (lane & 7) * 8, a.gate_per_head);
+            reinterpret_cast<uint4*>(dst + r * a.out_stride + b * 64)[lane & 7] = piece;
+          }
         }
         __syncwarp();
       }
@@ -304,10 +327,10 @@ int make_head_rows_map(CUtensorMap* map, const void* base, int width, int heads,
   return make_box_map<3>(map, base, {width, heads, rows}, {1, head_stride, row_stride}, {64, 1, box_rows});
 }
 
-template <int kK, int kV>
+template <int kK, int kR, int kV>
 int launch(const LatentPromptArgs& a, const CUtensorMap (&maps)[5], cudaStream_t stream) {
-  auto kernel = latent_prompt_kernel<kK, kV>;
-  const size_t smem = sizeof(PromptShared<kK, kV>) + 1024;
+  auto kernel = latent_prompt_kernel<kK, kR, kV>;
+  const size_t smem = sizeof(PromptShared<kK, kR, kV>) + 1024;
   RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   const dim3 grid(static_cast<unsigned>(a.tile_count), static_cast<unsigned>(a.heads));
   kernel<<<grid, kThreads, smem, stream>>>(maps[0], maps[1], maps[2], maps[3], maps[4], a, static_cast<float>(1.4426950408889634 * static_cast<double>(a.scale)));
@@ -324,36 +347,49 @@ bool latent_prompt_supported(int dim, int rot_dim, int vdim, int dtype) {
 
 extern "C" RLT_API int rlt_latent_prompt_supported(int dim, int rot_dim, int vdim, int dtype) { return rlt::latent_prompt_supported(dim, rot_dim, vdim, dtype) ? 1 : 0; }
 
-extern "C" RLT_API int rlt_latent_prompt_attention(const void* q, int64_t q_stride, const void* kv, int64_t kv_stride, const void* shared_keys,
-                                                   int64_t shared_stride, void* out, int64_t out_stride, int rows, int key_rows, int heads, int dim,
-                                                   int rot_dim, int vdim, const int32_t* tiles, int tile_count, float scale, int window, int dtype,
-                                                   void* workspace, rlt_stream_t stream) {
+extern "C" RLT_API int rlt_latent_prompt_attention(const void* q, int64_t q_stride, const void* keys, int64_t key_stride, const void* values,
+                                                   int64_t value_stride, const void* shared_keys, int64_t shared_stride, void* out,
+                                                   int64_t out_stride, int rows, int key_rows, int heads, int kv_heads, int dim, int rot_dim, int vdim,
+                                                   const int32_t* tiles, int tile_count, float scale, int window, const float* sink,
+                                                   const void* gate, int64_t gate_stride, int gate_per_head, int dtype, void* workspace,
+                                                   rlt_stream_t stream) {
   using namespace rlt;
-  RLT_REQUIRE(rows >= 0 && key_rows >= 0 && heads > 0 && dim > 0 && rot_dim > 0 && vdim > 0 && tile_count >= 0 && window >= 0, "latent_prompt_attention: invalid shape");
+  RLT_REQUIRE(rows >= 0 && key_rows >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && rot_dim >= 0 && vdim > 0 && tile_count >= 0 && window >= 0,
+              "latent_prompt_attention: invalid shape");
   if (rows == 0 || tile_count == 0) return RLT_OK;
-  RLT_REQUIRE(q && kv && shared_keys && out && tiles && workspace && key_rows > 0, "latent_prompt_attention: null pointer");
-  RLT_REQUIRE(q_stride >= static_cast<int64_t>(heads) * (dim + rot_dim) && kv_stride >= static_cast<int64_t>(heads) * (dim + vdim) && shared_stride >= rot_dim &&
+  RLT_REQUIRE(q && keys && values && (shared_keys || rot_dim == 0) && out && tiles && workspace && key_rows > 0, "latent_prompt_attention: null pointer");
+  RLT_REQUIRE(q_stride >= static_cast<int64_t>(heads) * (dim + rot_dim) && key_stride >= static_cast<int64_t>(kv_heads) * dim &&
+                  value_stride >= static_cast<int64_t>(kv_heads) * vdim && (rot_dim == 0 || shared_stride >= rot_dim) &&
                   out_stride >= static_cast<int64_t>(heads) * vdim && heads <= 65535, "latent_prompt_attention: row strides smaller than a row");
+  RLT_REQUIRE(gate == nullptr || gate_stride >= (gate_per_head != 0 ? heads : static_cast<int64_t>(heads) * vdim), "latent_prompt_attention: gate rows overlap");
   RLT_REQUIRE((reinterpret_cast<uintptr_t>(tiles) & 3u) == 0, "latent_prompt_attention: misaligned tiles");
-  if (!latent_prompt_supported(dim, rot_dim, vdim, dtype) || q_stride % 8 != 0 || kv_stride % 8 != 0 || shared_stride % 8 != 0 || out_stride % 8 != 0 ||
-      !aligned16(q) || !aligned16(kv) || !aligned16(shared_keys) || !aligned16(out)) {
+  if (!latent_prompt_supported(dim, rot_dim, vdim, dtype) || q_stride % 8 != 0 || key_stride % 8 != 0 || value_stride % 8 != 0 ||
+      (rot_dim > 0 && shared_stride % 8 != 0) || out_stride % 8 != 0 || !aligned16(q) || !aligned16(keys) || !aligned16(values) ||
+      !aligned16(shared_keys) || !aligned16(out) || (gate != nullptr && gate_per_head == 0 && (gate_stride % 8 != 0 || !aligned16(gate)))) {
     set_last_error_text("latent_prompt_attention: bf16, sizes in multiples of 8, dim and vdim up to 128, rot_dim up to 64, 16-byte aligned rows");
     return RLT_ERR_UNSUPPORTED;
   }
   LatentPromptArgs a;
-  a.out = out; a.out_stride = out_stride; a.heads = heads; a.vdim = vdim; a.tiles = reinterpret_cast<const PromptTile*>(tiles); a.tile_count = tile_count;
-  a.scale = scale; a.window = window; a.error = static_cast<unsigned*>(workspace);
+  a.out = out; a.out_stride = out_stride; a.heads = heads; a.share = heads / kv_heads; a.vdim = vdim;
+  a.tiles = reinterpret_cast<const PromptTile*>(tiles); a.tile_count = tile_count;
+  a.scale = scale; a.window = window; a.sink = sink; a.gate = gate; a.gate_stride = gate_stride; a.gate_per_head = gate_per_head != 0;
+  a.error = static_cast<unsigned*>(workspace);
   CUtensorMap maps[5];
   const auto at = [](const void* p, int64_t elements) { return static_cast<const void*>(static_cast<const uint16_t*>(p) + elements); };
   if (make_head_rows_map(&maps[0], q, dim, heads, rows, dim + rot_dim, q_stride, kRows) != RLT_OK ||
-      make_head_rows_map(&maps[1], at(q, dim), rot_dim, heads, rows, dim + rot_dim, q_stride, kRows) != RLT_OK ||
-      make_head_rows_map(&maps[2], kv, dim, heads, key_rows, dim, kv_stride, kKeys) != RLT_OK ||
-      make_head_rows_map(&maps[3], shared_keys, rot_dim, 1, key_rows, shared_stride, shared_stride, kKeys) != RLT_OK ||
-      make_head_rows_map(&maps[4], at(kv, static_cast<int64_t>(heads) * dim), vdim, heads, key_rows, vdim, kv_stride, kKeys) != RLT_OK) {
+      make_head_rows_map(&maps[2], keys, dim, kv_heads, key_rows, dim, key_stride, kKeys) != RLT_OK ||
+      make_head_rows_map(&maps[4], values, vdim, kv_heads, key_rows, vdim, value_stride, kKeys) != RLT_OK ||
+      (rot_dim > 0 && (make_head_rows_map(&maps[1], at(q, dim), rot_dim, heads, rows, dim + rot_dim, q_stride, kRows) != RLT_OK ||
+                       make_head_rows_map(&maps[3], shared_keys, rot_dim, 1, key_rows, shared_stride, shared_stride, kKeys) != RLT_OK))) {
     set_last_error_text("latent_prompt_attention: cuTensorMapEncodeTiled rejected the operands");
     return RLT_ERR_UNSUPPORTED;
   }
+  if (rot_dim == 0) { maps[1] = maps[0]; maps[3] = maps[2]; }      // not read
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dim <= 64) return vdim <= 64 ? launch<1, 1>(a, maps, s) : launch<1, 2>(a, maps, s);
-  return vdim <= 64 ? launch<2, 1>(a, maps, s) : launch<2, 2>(a, maps, s);
+  if (rot_dim == 0) {
+    if (dim <= 64) return vdim <= 64 ? launch<1, 0, 1>(a, maps, s) : launch<1, 0, 2>(a, maps, s);
+    return vdim <= 64 ? launch<2, 0, 1>(a, maps, s) : launch<2, 0, 2>(a, maps, s);
+  }
+  if (dim <= 64) return vdim <= 64 ? launch<1, 1, 1>(a, maps, s) : launch<1, 1, 2>(a, maps, s);
+  return vdim <= 64 ? launch<2, 1, 1>(a, maps, s) : launch<2, 1, 2>(a, maps, s);
 }

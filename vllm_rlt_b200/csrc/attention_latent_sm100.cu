@@ -323,7 +323,10 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
         if (g == 0) sm.folded[warp][(i >> 1) * 8 + 2 * t + (i & 1)] = sum[i];
       }
       rows_any(false);
-      for (int i = threadIdx.x; i < kN; i += kRowThreads) sm.alpha[i] = (sm.folded[0][i] + sm.folded[1][i]) + (sm.folded[2][i] + sm.folded[3][i]);
+      for (int i = threadIdx.x; i < kN; i += kRowThreads) {
+        const float total = (sm.folded[0][i] + sm.folded[1][i]) + (sm.folded[2][i] + sm.folded[3][i]);
+        sm.alpha[i] = splits > 1 ? total : softmax_scale(sm.m[i], total, sink_log2(a.terms, (r_base + i) % heads));   // of several splits the merge adds the sink
+      }
       rows_any(false);
       const int count = min(kN, all_rows - r_base);
       const int64_t first_pair = static_cast<int64_t>(first_row) * heads + r_base;      // (token, head) pairs are consecutive rows
@@ -348,8 +351,7 @@ attention_latent_kernel(const __grid_constant__ CUtensorMap map, const __grid_co
 #pragma unroll
             for (int i = 0; i < kPart; ++i) {
               const int n = part * kPart + i;
-              const float total = sm.alpha[n];
-              if (live && n < count) to[i * a.value_dim] = __float2bfloat16_rn(total > 0.f ? __fdividef(__uint_as_float(r[i]), total) : 0.f);
+              if (live && n < count) to[i * a.value_dim] = __float2bfloat16_rn(__uint_as_float(r[i]) * sm.alpha[n]);
             }
           } else {
             const int64_t step = static_cast<int64_t>(splits) * (a.value_dim + 2);

@@ -1,5 +1,5 @@
 // Tensor-core paged attention for head sizes the sm_100a page kernels do not cover: bf16, key and value sizes of
-// their own (multiples of 8, up to 256), any page size and GQA ratio, with the score terms of attention.cuh (windows included).
+// their own (multiples of 8, up to 256), any page size and GQA ratio, with the score terms of attention.cuh (windows and sinks included).
 //
 // The query rows of one KV head are the (token, query head of the group) pairs of a sequence's portion, token
 // major, so a K / V stage serves every head of the group.  Keys come in stages of 64, gathered row by row with
@@ -234,9 +234,12 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
     }
     __syncthreads();
     for (int r = warp; r < 16 && r_base + r < all_rows; r += kWarps) {
-      float big = -INFINITY, total = 0.f, f[kWarps];
+      const int head = kv_head * gqa + (r_base + r) % gqa;
+      const float sink = splits == 1 ? sink_log2(a.terms, head) : -INFINITY;      // of several splits the merge adds it
+      float big = sink, f[kWarps];
 #pragma unroll
       for (int w = 0; w < kWarps; ++w) big = fmaxf(big, fold[(w * 16 + r) * kStride + kD]);
+      float total = sink == -INFINITY ? 0.f : fast_exp2(sink - big);
 #pragma unroll
       for (int w = 0; w < kWarps; ++w) {
         const float m = fold[(w * 16 + r) * kStride + kD];
@@ -244,7 +247,6 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
         total = fmaf(fold[(w * 16 + r) * kStride + kD + 1], f[w], total);
       }
       const int64_t row = first_row + (r_base + r) / gqa;
-      const int head = kv_head * gqa + (r_base + r) % gqa;
       float* part = partials + ((row * a.q_heads + head) * splits + split) * (a.value_dim + 2);
       T* out = static_cast<T*>(a.out) + row * a.out_stride + static_cast<int64_t>(head) * a.value_dim;
       const float inv = total > 0.f ? 1.f / total : 0.f;
@@ -258,7 +260,7 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
       if (splits > 1 && lane == 0) { part[a.value_dim] = big; part[a.value_dim + 1] = total; }
     }
   } else {
-    const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+    const float inv0 = softmax_scale(m0, l0, sink_log2(a.terms, head0)), inv1 = softmax_scale(m1, l1, sink_log2(a.terms, head1));
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int r = r_base + (half == 0 ? row0 : row1);
@@ -291,13 +293,15 @@ merge_splits_kernel(AttentionArgs a, int splits, const float* partials) {
   float2 first[4];
 #pragma unroll
   for (int s = 0; s < 4; ++s) first[s] = live && s < splits ? *reinterpret_cast<const float2*>(part + s * stride + d) : make_float2(0.f, 0.f);
-  float big = m;
+  const float sink = sink_log2(a.terms, static_cast<int>(pair - row * a.q_heads));
+  float big = fmaxf(m, sink);
 #pragma unroll
   for (int x = 16; x > 0; x >>= 1) big = fmaxf(big, __shfl_xor_sync(0xffffffffu, big, x));
   const float f = m == -INFINITY ? 0.f : fast_exp2(m - big);
   float total = sum * f;
 #pragma unroll
   for (int x = 16; x > 0; x >>= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
+  if (sink != -INFINITY) total += fast_exp2(sink - big);
   const float inv = total > 0.f ? 1.f / total : 0.f;
   float2 acc = make_float2(0.f, 0.f);
 #pragma unroll

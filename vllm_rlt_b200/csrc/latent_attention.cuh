@@ -1,4 +1,4 @@
-// Arguments of the prompt kernel of latent attention (attention_latent_prompt_sm100.cu explains the operands).
+// Arguments of the prompt kernel over packed keys and values (attention_latent_prompt_sm100.cu explains the operands).
 #pragma once
 
 #include "attention.cuh"
@@ -17,9 +17,11 @@ struct PromptTile {
 
 struct LatentPromptArgs {
   void* out; int64_t out_stride;
-  int heads, vdim;
+  int heads, share, vdim;   // query heads, query heads per key/value head
   const PromptTile* tiles; int tile_count;
   float scale; int window;
+  const float* sink;                                               // [heads], or null
+  const void* gate; int64_t gate_stride; bool gate_per_head;       // null: no gate
   unsigned* error;   // set when a bounded wait gave up
 };
 

@@ -7,8 +7,9 @@
 //   latent_gather_kernel  the cache rows of a range of positions of every sequence, side by side: what a prompt expands
 //                         into keys and values
 //
-// Rotation: dimensions 2i and 2i + 1 are a pair, turned by position * frequency_i.  The product is formed and reduced to one
-// turn in double, so that angles far into a sequence keep 32-bit precision.
+// Rotation: dimensions 2i and 2i + 1 — in the `halves` layout i and i + rot_dims / 2 — are a pair, turned by position * frequency_i
+// and multiplied by an amplitude.  The product is formed and reduced to one turn in double, so that angles far into a sequence keep
+// 32-bit precision.
 #include <math.h>
 
 #include "layer_math.cuh"
@@ -18,18 +19,20 @@ namespace {
 
 constexpr int kThreads = 256;
 
-__device__ __forceinline__ void rotation(int position, double frequency, float* cosine, float* sine) {
+__device__ __forceinline__ void rotation(int position, double frequency, float amplitude, float* cosine, float* sine) {
   constexpr double kTurn = 6.283185307179586476925286766559;
   double angle = static_cast<double>(position) * frequency;
   angle -= rint(angle * (1.0 / kTurn)) * kTurn;
   sincosf(static_cast<float>(angle), sine, cosine);
+  *cosine *= amplitude;
+  *sine *= amplitude;
 }
 
 struct LatentArgs {
   const void* proj; int64_t proj_stride;
   int q_col, q_rank, kv_col, kv_rank, rot_dim, rot_dims;   // rot_dims of the rot_dim are turned
   const float* q_weight; const float* kv_weight; float eps;
-  const double* frequencies;
+  const double* frequencies; int halves; float amplitude;
   void* q_out; int64_t q_out_stride;
   void* cache; int64_t block_stride, token_stride, num_blocks; int block_size;
   const int32_t* tables; int table_width; const int32_t* row_seq; const int32_t* positions;
@@ -55,13 +58,16 @@ latent_write_kernel(LatentArgs a, int rows, int parts) {
   T* dst = static_cast<T*>(a.q_out) + row * a.q_out_stride;
   int position = 0;
   float turned[2] = {0.0f, 0.0f};             // the lane's first pair of the rotated part
+  const int half = a.rot_dims / 2;            // pairs that are turned; the elements behind them go two by two
+  auto first_of = [&](int i) { return a.halves != 0 && i < half ? i : 2 * i; };
+  auto second_of = [&](int i) { return a.halves != 0 && i < half ? i + half : 2 * i + 1; };
   if (!query) {
     const int seq = a.row_seq[row];
     if (seq < 0) return;                      // a padding row of a captured step
     position = a.positions[row];
     if (2 * lane < a.rot_dim) {
-      turned[0] = Elem<T>::to_float(proj[a.kv_rank + 2 * lane]);
-      if (2 * lane + 1 < a.rot_dim) turned[1] = Elem<T>::to_float(proj[a.kv_rank + 2 * lane + 1]);
+      turned[0] = Elem<T>::to_float(proj[a.kv_rank + first_of(lane)]);
+      if (2 * lane + 1 < a.rot_dim) turned[1] = Elem<T>::to_float(proj[a.kv_rank + second_of(lane)]);
     }
     const int page_index = position / a.block_size;
     if (position < 0 || page_index >= a.table_width) return;
@@ -106,59 +112,80 @@ latent_write_kernel(LatentArgs a, int rows, int parts) {
   for (int i = (kKeep * 32 + lane) * kVec; i < width; i += 32 * kVec) write(i, *reinterpret_cast<const Vec*>(proj + i));
   if (query) return;
   for (int i = lane; 2 * i < a.rot_dim; i += 32) {
-    const int d = 2 * i;
+    const bool whole = 2 * i + 1 < a.rot_dim;   // the last element of an odd part has no partner
     if (i != lane) {
-      turned[0] = Elem<T>::to_float(proj[a.kv_rank + d]);
-      turned[1] = d + 1 < a.rot_dim ? Elem<T>::to_float(proj[a.kv_rank + d + 1]) : 0.0f;
+      turned[0] = Elem<T>::to_float(proj[a.kv_rank + first_of(i)]);
+      turned[1] = whole ? Elem<T>::to_float(proj[a.kv_rank + second_of(i)]) : 0.0f;
     }
     float u = turned[0], v = turned[1];
-    if (d < a.rot_dims) {
+    if (i < half) {
       float c, s;
-      rotation(position, a.frequencies[i], &c, &s);
+      rotation(position, a.frequencies[i], a.amplitude, &c, &s);
       u = turned[0] * c - turned[1] * s;
       v = turned[1] * c + turned[0] * s;
     }
-    dst[a.kv_rank + d] = Elem<T>::from_float(u);
-    if (d + 1 < a.rot_dim) dst[a.kv_rank + d + 1] = Elem<T>::from_float(v);
+    dst[a.kv_rank + first_of(i)] = Elem<T>::from_float(u);
+    if (whole) dst[a.kv_rank + second_of(i)] = Elem<T>::from_float(v);
   }
 }
 
-// `per_cta` rows: their angles once, then every head's elements, kVec (an even number, or one pair whose second half may lie outside).
-template <typename T, int kVec>
+// `per_cta` rows: their angles once, then every head's elements, kVec neighbouring ones per access (an even number, or one: then a thread
+// takes one pair, whose second element may lie outside).  kHalves: a thread of the turned part holds an access of either half.
+template <typename T, int kVec, bool kHalves>
 __global__ void __launch_bounds__(kThreads)
 rotate_heads_kernel(const T* src, int64_t src_row, int64_t src_head, T* dst, int64_t dst_row, int64_t dst_head, int heads, int dim,
-                    int rot_dims, const double* __restrict__ frequencies, const int32_t* __restrict__ positions, int rows, int per_cta) {
+                    int rot_dims, const double* __restrict__ frequencies, float amplitude, const int32_t* __restrict__ positions, int rows, int per_cta) {
   extern __shared__ float2 turns[];
   const int pairs = rot_dims / 2, first = blockIdx.x * per_cta, count = min(per_cta, rows - first);
-  for (int i = threadIdx.x; i < count * pairs; i += kThreads) rotation(positions[first + i / pairs], frequencies[i % pairs], &turns[i].x, &turns[i].y);
+  for (int i = threadIdx.x; i < count * pairs; i += kThreads)
+    rotation(positions[first + i / pairs], frequencies[i % pairs], amplitude, &turns[i].x, &turns[i].y);
   __syncthreads();
   constexpr int kStep = kVec < 2 ? 2 : kVec;
-  const int pieces = (dim + kStep - 1) / kStep, per_row = heads * pieces;
+  const int joint = kHalves ? pairs / (kVec < 2 ? 1 : kVec) : 0;                     // pieces that hold both halves of their pairs
+  const int pieces = joint + (kHalves ? dim - rot_dims + kStep - 1 : dim + kStep - 1) / kStep, per_row = heads * pieces;
   for (int i = threadIdx.x; i < count * per_row; i += kThreads) {
-    const int r = i / per_row, rest = i - r * per_row, head = rest / pieces, d = (rest - head * pieces) * kStep;
-    const T* from = src + (first + r) * src_row + head * src_head + d;
-    T* to = dst + (first + r) * dst_row + head * dst_head + d;
-    const float2* turn = turns + r * pairs + d / 2;
+    const int r = i / per_row, rest = i - r * per_row, head = rest / pieces, piece = rest - head * pieces;
+    const T* from = src + (first + r) * src_row + head * src_head;
+    T* to = dst + (first + r) * dst_row + head * dst_head;
+    if (kHalves && piece < joint) {
+      const int d = piece * kVec;
+      float u[kVec], v[kVec];
+      load_floats<T, kVec>(from + d, u);
+      load_floats<T, kVec>(from + pairs + d, v);
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) {
+        const float2 t = turns[r * pairs + d + e];
+        const float x = u[e];
+        u[e] = x * t.x - v[e] * t.y;
+        v[e] = v[e] * t.x + x * t.y;
+      }
+      store_floats<T, kVec>(to + d, u);
+      store_floats<T, kVec>(to + pairs + d, v);
+      continue;
+    }
+    const int d = kHalves ? rot_dims + (piece - joint) * kStep : piece * kStep;
     float v[kStep];
     if constexpr (kVec > 1) {
-      load_floats<T, kVec>(from, v);
+      load_floats<T, kVec>(from + d, v);
     } else {
-      v[0] = Elem<T>::to_float(from[0]);
-      v[1] = d + 1 < dim ? Elem<T>::to_float(from[1]) : 0.0f;
+      v[0] = Elem<T>::to_float(from[d]);
+      v[1] = d + 1 < dim ? Elem<T>::to_float(from[d + 1]) : 0.0f;
     }
+    if (!kHalves) {
 #pragma unroll
-    for (int e = 0; e < kStep; e += 2)
-      if (d + e < rot_dims) {
-        const float2 t = turn[e / 2];
-        const float u = v[e];
-        v[e] = u * t.x - v[e + 1] * t.y;
-        v[e + 1] = v[e + 1] * t.x + u * t.y;
-      }
+      for (int e = 0; e < kStep; e += 2)
+        if (d + e < rot_dims) {
+          const float2 t = turns[r * pairs + (d + e) / 2];
+          const float u = v[e];
+          v[e] = u * t.x - v[e + 1] * t.y;
+          v[e + 1] = v[e + 1] * t.x + u * t.y;
+        }
+    }
     if constexpr (kVec > 1) {
-      store_floats<T, kVec>(to, v);
+      store_floats<T, kVec>(to + d, v);
     } else {
-      to[0] = Elem<T>::from_float(v[0]);
-      if (d + 1 < dim) to[1] = Elem<T>::from_float(v[1]);
+      to[d] = Elem<T>::from_float(v[0]);
+      if (d + 1 < dim) to[d + 1] = Elem<T>::from_float(v[1]);
     }
   }
 }
@@ -192,8 +219,8 @@ latent_gather_kernel(const unsigned char* __restrict__ cache, int64_t block_byte
 
 extern "C" RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, int q_col, int q_rank, int kv_col, int kv_rank,
                                         int rot_dim, int rot_dims, const float* q_weight, const float* kv_weight, float eps,
-                                        const double* frequencies, void* q_out, int64_t q_out_stride, void* cache, int64_t block_stride,
-                                        int64_t token_stride, int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
+                                        const double* frequencies, int halves, float amplitude, void* q_out, int64_t q_out_stride, void* cache,
+                                        int64_t block_stride, int64_t token_stride, int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
                                         const int32_t* row_seq, const int32_t* positions, int rows, int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "latent_write: dtype must be float32, float16 or bfloat16");
@@ -207,7 +234,7 @@ extern "C" RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, i
   RLT_REQUIRE(token_stride >= kv_rank + rot_dim && block_stride >= token_stride * block_size, "latent_write: cache rows overlap");
   LatentArgs a;
   a.proj = proj; a.proj_stride = proj_stride; a.q_col = q_col; a.q_rank = q_rank; a.kv_col = kv_col; a.kv_rank = kv_rank;
-  a.rot_dim = rot_dim; a.rot_dims = rot_dims; a.q_weight = q_weight; a.kv_weight = kv_weight; a.eps = eps; a.frequencies = frequencies;
+  a.rot_dim = rot_dim; a.rot_dims = rot_dims; a.q_weight = q_weight; a.kv_weight = kv_weight; a.eps = eps; a.frequencies = frequencies; a.halves = halves; a.amplitude = amplitude;
   a.q_out = q_out; a.q_out_stride = q_out_stride; a.cache = cache; a.block_stride = block_stride; a.token_stride = token_stride;
   a.num_blocks = num_blocks; a.block_size = block_size; a.tables = tables; a.table_width = table_width; a.row_seq = row_seq; a.positions = positions;
   const int parts = q_rank > 0 ? 2 : 1;
@@ -225,8 +252,8 @@ extern "C" RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, i
 }
 
 extern "C" RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head, void* dst, int64_t dst_row, int64_t dst_head,
-                                        int heads, int dim, int rot_dims, const double* frequencies, const int32_t* positions, int rows,
-                                        int dtype, rlt_stream_t stream) {
+                                        int heads, int dim, int rot_dims, const double* frequencies, int halves, float amplitude, const int32_t* positions,
+                                        int rows, int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "rotate_heads: dtype must be float32, float16 or bfloat16");
   RLT_REQUIRE(rows >= 0 && heads > 0 && dim >= 0 && rot_dims >= 0 && rot_dims <= dim && rot_dims % 2 == 0 && rot_dims <= 4096, "rotate_heads: invalid shape");
@@ -235,14 +262,18 @@ extern "C" RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int vec = static_cast<int>(16 / dtype_size(dtype));
   auto whole = [&](int64_t n) { return n % vec == 0; };
-  const bool wide = whole(dim) && whole(rot_dims) && whole(src_row) && whole(src_head) && whole(dst_row) && whole(dst_head) && aligned16(src) && aligned16(dst);
+  const bool wide = whole(dim) && whole(halves != 0 ? rot_dims / 2 : rot_dims) && whole(src_row) && whole(src_head) && whole(dst_row) && whole(dst_head) && aligned16(src) && aligned16(dst);
   int per_cta = rows >= 4096 ? 4 : 1;                       // enough CTAs for every SM first
   if (static_cast<size_t>(per_cta) * (rot_dims / 2) * sizeof(float2) > 40u * 1024u) per_cta = 1;
   const size_t smem = static_cast<size_t>(per_cta) * (rot_dims / 2) * sizeof(float2);
   const unsigned grid = static_cast<unsigned>((rows + per_cta - 1) / per_cta);
-#define RLT_LAUNCH(T, V) rotate_heads_kernel<T, V><<<grid, kThreads, smem, s>>>(static_cast<const T*>(src), src_row, src_head, static_cast<T*>(dst), dst_row, \
-                                                                               dst_head, heads, dim, rot_dims, frequencies, positions, rows, per_cta)
-  RLT_DISPATCH_DTYPE(dtype, T, { if (wide) RLT_LAUNCH(T, static_cast<int>(16 / sizeof(T))); else RLT_LAUNCH(T, 1); });
+#define RLT_LAUNCH(T, V, H) rotate_heads_kernel<T, V, H><<<grid, kThreads, smem, s>>>(static_cast<const T*>(src), src_row, src_head, static_cast<T*>(dst), dst_row, \
+                                                                                     dst_head, heads, dim, rot_dims, frequencies, amplitude, positions, rows, per_cta)
+  RLT_DISPATCH_DTYPE(dtype, T, {
+    constexpr int kWide = static_cast<int>(16 / sizeof(T));
+    if (halves != 0) { if (wide) RLT_LAUNCH(T, kWide, true); else RLT_LAUNCH(T, 1, true); }
+    else { if (wide) RLT_LAUNCH(T, kWide, false); else RLT_LAUNCH(T, 1, false); }
+  });
 #undef RLT_LAUNCH
   return launch_status("rotate_heads_kernel");
 }

@@ -34,7 +34,9 @@ __device__ __forceinline__ float activate(float x, int act) {
   }
   if (act == kActSilu) return x * sigmoid<T>(x);
   if (act == kActSquaredRelu) { const float r = fmaxf(x, 0.0f); return r * r; }
-  return 0.5f * x * (1.0f + tanhf(0.79788456080286536f * (x + 0.044715f * x * x * x)));
+  const float u = 0.79788456080286536f * (x + 0.044715f * x * x * x);
+  if (sizeof(T) < 4) return x * sigmoid<T>(2.0f * u);      // (1 + tanh u) / 2 is the sigmoid of 2 u
+  return 0.5f * x * (1.0f + tanhf(u));
 }
 
 // kVec consecutive elements as fp32, in one access of kVec * sizeof(T) bytes (the caller guarantees the alignment).

@@ -3,7 +3,8 @@
 // stacked output projections — and between them
 //
 //   residual_norm_kernel   residual += delta (or residual = embed[token]), h = rmsnorm(residual) * (offset + w):
-//                          the tail of one layer and the head of the next in one pass over the row
+//                          the tail of one layer and the head of the next in one pass over the row; for models with a norm
+//                          on both sides of a sublayer residual += scale * norm(delta) * w', and layer norms for RMS norms
 //   block_epilogue_kernel  columns of the stacked input projection: keys and values to their pages,
 //                          the feed-forward columns through their activation into the stacked output operand
 //   gated_norm_kernel      y * silu(z), RMS-normed in equal parts, into the stacked output operand; or y RMS-normed first
@@ -20,48 +21,97 @@ namespace {
 
 constexpr int kThreads = 256;
 
-template <typename T, int kVec>
+struct NormArgs {
+  float* residual; const void* delta;
+  const int64_t* tokens; const void* embed; int64_t vocab;
+  const int64_t* row_index; int store_residual;
+  const float* weight; float weight_offset;
+  const float* delta_weight; float delta_scale;   // null: delta is added as it is
+  int centred;
+  void* out; int width; float eps;
+};
+
+// One row per CTA, kPer accesses of kVec elements per thread, in registers from the first load to the last store.
+template <typename T, int kVec, int kPer>
 __global__ void __launch_bounds__(kThreads)
-residual_norm_kernel(float* residual, const T* __restrict__ delta, const int64_t* __restrict__ tokens,
-                     const T* __restrict__ embed, int64_t vocab, const int64_t* __restrict__ row_index, int store_residual,
-                     const float* __restrict__ weight, float weight_offset, T* __restrict__ out, int width, float eps) {
-  extern __shared__ __align__(16) float row_values[];
+residual_norm_kernel(NormArgs a) {
   __shared__ float scratch[kThreads / 32];
-  const int64_t source = row_index != nullptr ? row_index[blockIdx.x] : static_cast<int64_t>(blockIdx.x);
-  float* res = residual + source * width;
-  const T* del = delta == nullptr ? nullptr : delta + source * width;
+  const int width = a.width;
+  const int64_t source = a.row_index != nullptr ? a.row_index[blockIdx.x] : static_cast<int64_t>(blockIdx.x);
+  float* res = a.residual + source * width;
   const T* emb = nullptr;
-  if (tokens != nullptr) {
-    int64_t token = tokens[source];
-    token = token < 0 ? 0 : (token >= vocab ? vocab - 1 : token);   // the host refuses such tokens; a device id never leaves the table
-    emb = embed + token * width;
+  if (a.tokens != nullptr) {
+    int64_t token = a.tokens[source];
+    token = token < 0 ? 0 : (token >= a.vocab ? a.vocab - 1 : token);   // the host refuses such tokens; a device id never leaves the table
+    emb = static_cast<const T*>(a.embed) + token * width;
   }
-  float ss = 0.0f;
-  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
-    float v[kVec];
-    if (emb != nullptr) load_floats<T, kVec>(emb + i, v);
-    else load_floats<float, kVec>(res + i, v);
-    if (del != nullptr) {
-      float d[kVec];
-      load_floats<T, kVec>(del + i, d);
+  float v[kPer][kVec], d[kPer][kVec];
+  auto at = [&](int k) { return (k * kThreads + static_cast<int>(threadIdx.x)) * kVec; };
 #pragma unroll
-      for (int e = 0; e < kVec; ++e) v[e] += d[e];
+  for (int k = 0; k < kPer; ++k)
+    if (at(k) < width) {
+      if (emb != nullptr) load_floats<T, kVec>(emb + at(k), v[k]);
+      else load_floats<float, kVec>(res + at(k), v[k]);
+      if (a.delta != nullptr) load_floats<T, kVec>(static_cast<const T*>(a.delta) + source * width + at(k), d[k]);
     }
-    if (store_residual) store_floats<float, kVec>(res + i, v);
+  // the row minus its mean (`centred`), and 1 / sqrt(mean of squares + eps) of it; deviations from the mean, not differences of sums
+  auto normalise = [&](float (&x)[kPer][kVec]) {
+    float sum = 0.0f;
+    if (a.centred != 0) {
 #pragma unroll
-    for (int e = 0; e < kVec; ++e) {
-      row_values[i + e] = v[e];
-      ss = fmaf(v[e], v[e], ss);
+      for (int k = 0; k < kPer; ++k)
+        if (at(k) < width) {
+#pragma unroll
+          for (int e = 0; e < kVec; ++e) sum += x[k][e];
+        }
+      const float mean = block_sum<kThreads>(sum, scratch) / static_cast<float>(width);
+#pragma unroll
+      for (int k = 0; k < kPer; ++k)
+#pragma unroll
+        for (int e = 0; e < kVec; ++e) x[k][e] -= mean;
+      sum = 0.0f;
     }
-  }
-  const float r = 1.0f / sqrtf(block_sum<kThreads>(ss, scratch) / static_cast<float>(width) + eps);
-  for (int i = threadIdx.x * kVec; i < width; i += kThreads * kVec) {
-    float v[kVec], w[kVec];
-    load_floats<float, kVec>(weight + i, w);
 #pragma unroll
-    for (int e = 0; e < kVec; ++e) v[e] = row_values[i + e] * r * (weight_offset + w[e]);
-    store_floats<T, kVec>(out + static_cast<int64_t>(blockIdx.x) * width + i, v);
+    for (int k = 0; k < kPer; ++k)
+      if (at(k) < width) {
+#pragma unroll
+        for (int e = 0; e < kVec; ++e) sum = fmaf(x[k][e], x[k][e], sum);
+      }
+    return 1.0f / sqrtf(block_sum<kThreads>(sum, scratch) / static_cast<float>(width) + a.eps);
+  };
+  if (a.delta != nullptr) {
+    if (a.delta_weight != nullptr) {
+      const float r = normalise(d) * a.delta_scale;
+#pragma unroll
+      for (int k = 0; k < kPer; ++k)
+        if (at(k) < width) {
+          float w[kVec];
+          load_floats<float, kVec>(a.delta_weight + at(k), w);
+#pragma unroll
+          for (int e = 0; e < kVec; ++e) d[k][e] *= r * w[e];
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < kPer; ++k)
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) v[k][e] += d[k][e];
   }
+  if (a.store_residual) {
+#pragma unroll
+    for (int k = 0; k < kPer; ++k)
+      if (at(k) < width) store_floats<float, kVec>(res + at(k), v[k]);
+  }
+  const float r = normalise(v);
+  T* out = static_cast<T*>(a.out) + static_cast<int64_t>(blockIdx.x) * width;
+#pragma unroll
+  for (int k = 0; k < kPer; ++k)
+    if (at(k) < width) {
+      float w[kVec];
+      load_floats<float, kVec>(a.weight + at(k), w);
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) w[e] = v[k][e] * r * (a.weight_offset + w[e]);
+      store_floats<T, kVec>(out + at(k), w);
+    }
 }
 
 struct EpilogueArgs {
@@ -149,6 +199,7 @@ gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict
   }
 }
 
+constexpr int kMaxPer = 12;   // accesses of 4 elements per thread of a residual row
 constexpr size_t kMaxRowBytes = 48u * 1024u;   // a staged row of fp32 values
 
 }  // namespace
@@ -156,26 +207,34 @@ constexpr size_t kMaxRowBytes = 48u * 1024u;   // a staged row of fp32 values
 
 extern "C" RLT_API int rlt_residual_norm(float* residual, const void* delta, const int64_t* tokens, const void* embed,
                                          int64_t vocab, const int64_t* row_index, int store_residual, const float* weight,
-                                         float weight_offset, void* out, int rows, int width, float eps, int dtype,
-                                         rlt_stream_t stream) {
+                                         float weight_offset, const float* delta_weight, float delta_scale, int centred, void* out,
+                                         int rows, int width, float eps, int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "residual_norm: dtype must be float32, float16 or bfloat16");
   RLT_REQUIRE(rows >= 0 && width > 0 && eps >= 0.0f, "residual_norm: invalid shape or eps");
   if (rows == 0) return RLT_OK;
   RLT_REQUIRE(residual && weight && out, "residual_norm: null pointer");
   RLT_REQUIRE((tokens == nullptr) == (embed == nullptr) && (tokens == nullptr || vocab > 0), "residual_norm: tokens and embed go together");
-  const size_t smem = static_cast<size_t>(width) * sizeof(float);
-  if (smem > kMaxRowBytes - 1024) {
-    set_last_error_text("residual_norm: widths above 12032 are not supported");
+  if (width > kMaxPer * kThreads * 4) {
+    set_last_error_text("residual_norm: widths above 12288 are not supported");
     return RLT_ERR_UNSUPPORTED;
   }
+  NormArgs a;
+  a.residual = residual; a.delta = delta; a.tokens = tokens; a.embed = embed; a.vocab = vocab; a.row_index = row_index;
+  a.store_residual = store_residual; a.weight = weight; a.weight_offset = weight_offset; a.delta_weight = delta_weight;
+  a.delta_scale = delta_scale; a.centred = centred; a.out = out; a.width = width; a.eps = eps;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool wide = width % 4 == 0 && aligned16(residual) && aligned16(weight) && aligned16(delta) && aligned16(embed) && aligned16(out);
-#define RLT_LAUNCH(T, V)                                                                                              \
-  residual_norm_kernel<T, V><<<rows, kThreads, smem, s>>>(residual, static_cast<const T*>(delta), tokens,             \
-      static_cast<const T*>(embed), vocab, row_index, store_residual, weight, weight_offset, static_cast<T*>(out), width, eps)
-  RLT_DISPATCH_DTYPE(dtype, T, { if (wide) RLT_LAUNCH(T, 4); else RLT_LAUNCH(T, 1); });
-#undef RLT_LAUNCH
+  const bool wide = width % 4 == 0 && aligned16(residual) && aligned16(weight) && aligned16(delta) && aligned16(embed) && aligned16(out) &&
+                    aligned16(delta_weight);
+  const int per = (width + kThreads * 4 - 1) / (kThreads * 4);
+  RLT_DISPATCH_DTYPE(dtype, T, {
+    if (!wide && per == 1) residual_norm_kernel<T, 1, 4><<<rows, kThreads, 0, s>>>(a);
+    else if (!wide) residual_norm_kernel<T, 1, 4 * kMaxPer><<<rows, kThreads, 0, s>>>(a);
+    else if (per == 1) residual_norm_kernel<T, 4, 1><<<rows, kThreads, 0, s>>>(a);
+    else if (per == 2) residual_norm_kernel<T, 4, 2><<<rows, kThreads, 0, s>>>(a);
+    else if (per <= 4) residual_norm_kernel<T, 4, 4><<<rows, kThreads, 0, s>>>(a);
+    else residual_norm_kernel<T, 4, kMaxPer><<<rows, kThreads, 0, s>>>(a);
+  });
   return launch_status("residual_norm_kernel");
 }
 

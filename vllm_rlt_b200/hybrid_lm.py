@@ -25,7 +25,7 @@ import torch.nn.functional as F
 
 from .attention import B200PagedAttention, ScoreTerms
 from .layers import block_epilogue, residual_norm
-from .model_parts import check_positive, check_shapes, full_accumulation, stack_blocks, take_keys
+from .model_parts import check_positive, check_shapes, full_accumulation, product32, stack_blocks, take_keys
 from .recurrent import causal_conv, gated_norm, ssd_scan
 from .sequence_cache import CacheSpec, KVSpec, StateSpec
 
@@ -279,6 +279,4 @@ class HybridLM:
         with full_accumulation():
             h = residual_norm(residual, self.final_norm, self.config.eps, self.dtype, delta=delta, row_index=rows,
                               weight_offset=self.norm_offset, store=False)
-            if self.dtype == torch.float32:
-                return F.linear(h, self.head)
-            return torch.mm(h, self.head.t(), out_dtype=torch.float32)
+            return product32(h, self.head)

@@ -105,21 +105,26 @@ ACTIVATIONS = {"gelu": 1, "gelu_tanh": 2, "silu": 3, "squared_relu": 4}      # g
 
 
 def residual_norm(residual, weight, eps: float, dtype, *, delta=None, tokens=None, embed=None, row_index=None,
-                  weight_offset: float = 0.0, store: bool = True):
-    """The 32-bit residual stream of a parallel-block model and the norm that opens a layer, in one pass:
+                  weight_offset: float = 0.0, store: bool = True, behind=None, centred: bool = False):
+    """The 32-bit residual stream and the norm that opens a layer or sublayer, in one pass:
 
         r = embed[tokens] or residual;  r += delta;  residual <- r (with `store`)
-        returns r / sqrt(mean(r^2) + eps) * (weight_offset + weight), in `dtype`
+        returns norm(r) * (weight_offset + weight), in `dtype`
 
-    residual: float32 [rows, width], updated in place.  `row_index` (int64) selects rows: the result has one
-    row per entry, and the residual is not stored.  `weight`: float32 [width] (`weight_offset` 1 for weights
-    stored around zero)."""
-    _capi.require_cuda(residual, weight, delta, tokens, embed, row_index)
+    norm(r) = r / sqrt(mean(r^2) + eps), with `centred` (a layer norm) of r minus its mean.  behind = (weight, scale): the sublayer has a
+    norm behind it too, r += scale * norm(delta) * weight.  residual: float32 [rows, width], updated in place.  `row_index` (int64)
+    selects rows: the result has one row per entry, and the residual is not stored.  `weight`: float32 [width]
+    (`weight_offset` 1 for weights stored around zero)."""
+    delta_weight, delta_scale = behind if behind is not None else (None, 1.0)
+    _capi.require_cuda(residual, weight, delta, tokens, embed, row_index, delta_weight)
     if residual.dim() != 2 or residual.dtype != torch.float32 or not residual.is_contiguous():
         raise ValueError("residual must be contiguous float32 [rows, width]")
     rows, width = residual.shape
     if weight.dtype != torch.float32 or weight.shape != (width,) or not weight.is_contiguous():
         raise ValueError("weight must be contiguous float32 [width]")
+    if delta_weight is not None and (delta is None or delta_weight.dtype != torch.float32 or delta_weight.shape != (width,)
+                                     or not delta_weight.is_contiguous()):
+        raise ValueError("the norm behind a sublayer needs a delta and a contiguous float32 [width] weight")
     if dtype not in _capi.DTYPE_CODES:
         raise ValueError("dtype must be float32 / float16 / bfloat16")
     if delta is not None and (delta.shape != residual.shape or delta.dtype != dtype or not delta.is_contiguous()):
@@ -143,8 +148,8 @@ def residual_norm(residual, weight, eps: float, dtype, *, delta=None, tokens=Non
     with torch.cuda.device(residual.device):
         code = _capi.load().rlt_residual_norm(
             _capi.ptr(residual), _capi.ptr(delta), _capi.ptr(tokens), _capi.ptr(embed), 0 if embed is None else embed.shape[0],
-            _capi.ptr(row_index), int(store), _capi.ptr(weight), float(weight_offset), _capi.ptr(out), count, width, float(eps),
-            _capi.DTYPE_CODES[dtype], _capi.stream_of(residual))
+            _capi.ptr(row_index), int(store), _capi.ptr(weight), float(weight_offset), _capi.ptr(delta_weight), float(delta_scale),
+            int(centred), _capi.ptr(out), count, width, float(eps), _capi.DTYPE_CODES[dtype], _capi.stream_of(residual))
     _capi.check(code, "residual_norm")
     return out
 
@@ -271,3 +276,55 @@ def clamped_glu(gate_up, up_col: int, cols: int, limit: float, slope: float):
                                             cols, float(limit), float(slope), _capi.DTYPE_CODES[gate_up.dtype], _capi.stream_of(gate_up))
     _capi.check(code, "clamped_glu")
     return out
+
+
+def gated_unit(gate_up, up_col: int, cols: int, act: str):
+    """`act(gate) * up` over columns 0 .. and `up_col` .. of one projection output; returns contiguous `[rows, cols]`."""
+    _capi.require_cuda(gate_up)
+    if gate_up.dim() != 2 or gate_up.stride(1) != 1 or gate_up.dtype not in _capi.DTYPE_CODES or up_col + cols > gate_up.shape[1]:
+        raise ValueError("gate_up must be [rows, columns] with unit inner stride that holds both halves")
+    out = torch.empty(gate_up.shape[0], cols, dtype=gate_up.dtype, device=gate_up.device)
+    with torch.cuda.device(gate_up.device):
+        code = _capi.load().rlt_gated_unit(_capi.ptr(gate_up), gate_up.stride(0), up_col, _capi.ptr(out), out.stride(0), out.shape[0],
+                                           cols, ACTIVATIONS[act], _capi.DTYPE_CODES[gate_up.dtype], _capi.stream_of(gate_up))
+    _capi.check(code, "gated_unit")
+    return out
+
+
+def check_gate(gate, rows: int, heads: int, dim: int) -> None:
+    if gate is not None and gate.shape not in ((rows, heads * dim), (rows, heads)):
+        raise ValueError("gate must be [rows, heads * dim] or [rows, heads]")
+
+
+def per_head(gate, heads: int, dim: int) -> bool:
+    """Whether a gate has one value per head and not one per element (with heads of one element both are the same)."""
+    return gate.shape[1] == heads and dim != 1
+
+
+def head_gate(y, gate, out=None):
+    """`y * sigmoid(gate)`: y `[rows, heads, dim]` with heads side by side, gate `[rows, heads * dim]` or `[rows, heads]`; out None: in place."""
+    out = y if out is None else out
+    _capi.require_cuda(y, gate, out)
+    rows, heads, dim = y.shape
+    check_gate(gate, rows, heads, dim)
+    if out.shape != y.shape or any(t.stride(2) != 1 or t.stride(1) != dim for t in (y, out)) or gate.stride(1) != 1 \
+            or y.dtype not in _capi.DTYPE_CODES or gate.dtype != y.dtype or out.dtype != y.dtype:
+        raise ValueError("y and out must be [rows, heads, dim] with heads side by side, gate of the same dtype with unit inner stride")
+    if rows == 0:
+        return out
+    with torch.cuda.device(y.device):
+        code = _capi.load().rlt_head_gate(_capi.ptr(y), y.stride(0), _capi.ptr(gate), gate.stride(0), _capi.ptr(out), out.stride(0), rows, heads,
+                                          dim, int(per_head(gate, heads, dim)), _capi.DTYPE_CODES[y.dtype], _capi.stream_of(y))
+    _capi.check(code, "head_gate")
+    return out
+
+
+def soft_cap(x, cap: float):
+    """`cap * tanh(x / cap)` of a contiguous float32 tensor, in place."""
+    _capi.require_cuda(x)
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise ValueError("x must be contiguous float32")
+    with torch.cuda.device(x.device):
+        code = _capi.load().rlt_soft_cap(_capi.ptr(x), x.numel(), float(cap), _capi.stream_of(x))
+    _capi.check(code, "soft_cap")
+    return x

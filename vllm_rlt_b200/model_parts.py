@@ -61,3 +61,8 @@ def full_accumulation():
         yield
     finally:
         m.allow_tf32, m.allow_bf16_reduced_precision_reduction = saved
+
+
+def product32(x, weight):
+    """x W^T with an fp32 result."""
+    return F.linear(x, weight) if x.dtype == torch.float32 else torch.mm(x, weight.t(), out_dtype=torch.float32)

@@ -1,5 +1,5 @@
-"""Recurrent layers over packed sequences with per-sequence state slots: short causal convolution, the Mamba-2
-state-space recurrence, linear attention with constant decays, and the gated norm behind them.
+"""Recurrent layers over packed sequences with per-sequence state slots: short causal convolution (also as part of what prepares
+an attention layer's heads), the Mamba-2 state-space recurrence, linear attention with constant decays, and the gated norm behind them.
 
 `group` arguments are a step's sequence group (`StepGroup`): `cu` (int32 [n + 1], row offsets into the step's
 rows), `starts` (position of each portion's first token), `slots`, and the host-side bound `max_new`.
@@ -45,6 +45,43 @@ def causal_conv(x, weight, bias, state, out, group, act=None):
             _capi.DTYPE_CODES[x.dtype], _capi.stream_of(x))
     _capi.check(code, "causal_conv")
     return out
+
+
+def conv_heads(proj, columns, weight, eps: float, state, q_out, key_cache, value_cache, group, *, unit_norm: bool = True):
+    """What stands between an attention layer's projections and its scores: `out[i, c] = sum_j weight[c, j] * x[i - taps + 1 + j, c]`
+    over the channels of q, k and v, with `unit_norm` q and k of every head divided by their root mean square, k and v into the pages of
+    their positions, q into q_out.
+
+    proj `[rows, columns]` holds q, k and v from the three `columns` on; weight float32 `[channels, taps]` (channels in the order q, k, v);
+    state `[slots, taps - 1, channels]` of proj's dtype, updated in place; q_out `[rows, heads, dim]`; the caches
+    `[pages, block, kv_heads, dim]` views."""
+    device = _capi.require_cuda(proj, weight, state, q_out, key_cache, value_cache, group.cu, group.starts, group.slots, group.lengths, group.tables)
+    rows, heads, key_dim = q_out.shape
+    kv_heads, value_dim = value_cache.shape[2], value_cache.shape[3]
+    channels, taps = weight.shape
+    if proj.dim() != 2 or proj.shape[0] != rows or proj.stride(1) != 1 or proj.dtype not in _capi.DTYPE_CODES \
+            or any(t.dtype != proj.dtype for t in (state, q_out, key_cache, value_cache)):
+        raise ValueError("proj must be [rows, columns] with unit inner stride; state, q_out and caches of its dtype")
+    if key_cache.shape != (*value_cache.shape[:3], key_dim) or any(c.stride(3) != 1 or c.stride(2) != c.shape[3] for c in (key_cache, value_cache)):
+        raise ValueError("caches must be [pages, block, kv_heads, dim] with a contiguous tail, keys as wide as queries")
+    widths = heads * key_dim, kv_heads * key_dim, kv_heads * value_dim
+    if channels != sum(widths) or any(at + n > proj.shape[1] for at, n in zip(columns, widths)):
+        raise ValueError("weight needs a row per channel of q, k and v; their columns must lie in the projection")
+    if weight.dtype != torch.float32 or not weight.is_contiguous() or state.shape[1:] != (taps - 1, channels) or not state.is_contiguous():
+        raise ValueError("weight must be contiguous float32 [channels, taps], state contiguous [slots, taps - 1, channels]")
+    if q_out.stride(2) != 1 or q_out.stride(1) != key_dim:
+        raise ValueError("q_out must be [rows, heads, dim] with heads side by side")
+    if group.sequences == 0:
+        return q_out
+    with torch.cuda.device(device):
+        code = _capi.load().rlt_conv_heads(
+            _capi.ptr(proj), proj.stride(0), *columns, heads, kv_heads, key_dim, value_dim, _capi.ptr(weight), taps, int(unit_norm), float(eps),
+            _capi.ptr(state), state.shape[0], _capi.ptr(q_out), q_out.stride(0), _capi.ptr(key_cache), key_cache.stride(0), key_cache.stride(1),
+            _capi.ptr(value_cache), value_cache.stride(0), value_cache.stride(1), key_cache.shape[0], key_cache.shape[1], _capi.ptr(group.tables),
+            group.tables.shape[1], _capi.ptr(group.cu), _capi.ptr(group.starts), _capi.ptr(group.lengths), _capi.ptr(group.slots), group.sequences,
+            group.max_new, _capi.DTYPE_CODES[proj.dtype], _capi.stream_of(proj))
+    _capi.check(code, "conv_heads")
+    return q_out
 
 
 def ssd_scan(x, b, c, dt, dt_bias, a_log, d, state, out, group):

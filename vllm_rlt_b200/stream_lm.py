@@ -5,10 +5,7 @@ The residual is S 32-bit streams.  Every sublayer (mixer, feed-forward) reads a 
 writes to all of them through a small mixing matrix; `stream_mix` does the writing of one sublayer and the reading of the
 next in one pass, so a layer is
 
-    latent attention   GEMM (both down projections), latent_write (query latent normed, cache row written), GEMM (queries), then
-                       long portions:  rotate_heads, latent_gather, GEMM (keys and values), attention, and
-                       short ones:     per-head GEMM (queries into the latent's space), rotate_heads, attention over the
-                                       cache rows themselves, per-head GEMM (values out of it);  GEMM
+    latent attention   as in `latent_mixer`, with a window
     lightning          GEMM (q, k, v, gate), block_epilogue (silu), decay_scan, gated_norm, GEMM
     dense              GEMM (gate, up), clamped_glu, GEMM
     experts            GEMM (router), expert_route, expert_gather, expert_gemm (up, squared relu), expert_gemm (down); their
@@ -22,59 +19,21 @@ softmax, router and recurrent state are fp32; in float32 everything is.
 from __future__ import annotations
 
 from dataclasses import dataclass
+from functools import partial
 
 import torch
 import torch.nn.functional as F
 
-from .attention import B200PagedAttention, ScoreTerms
+from .attention import B200PagedAttention
 from .experts import expert_gather, expert_gemm, expert_route
-from .latent import latent_gather, latent_prompt_attention, latent_prompt_supported, latent_write, rotate_heads, rotation_frequencies
+from .latent_mixer import LatentAttention, LatentAttentionConfig
 from .layers import block_epilogue, clamped_glu, stream_mix
-from .model_parts import check_positive, check_shapes, full_accumulation, stack_blocks, take_keys
+from .model_parts import check_positive, check_shapes, full_accumulation, product32, stack_blocks, take_keys
 from .recurrent import decay_scan, decay_table, gated_norm
-from .sequence_cache import CacheSpec, KVSpec, StateSpec
-
-SHORT_PORTION = 16      # groups of portions up to this long attend over the cache rows, longer ones over expanded keys and values
+from .sequence_cache import CacheSpec, StateSpec
 
 
 # ---- configuration -----------------------------------------------------------------------------
-@dataclass(frozen=True)
-class LatentAttentionConfig:
-    heads: int
-    dim: int              # unrotated query / key dimensions of a head
-    rot_dim: int          # rotated ones
-    vdim: int
-    q_rank: int
-    kv_rank: int
-    scale: float
-    window: int           # 0: every earlier key
-    rot_base: float
-    rot_dims: int         # how many of rot_dim are turned
-
-    @classmethod
-    def from_json(cls, entry: dict, what: str) -> "LatentAttentionConfig":
-        m = take_keys(entry, what, ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale", "rot"), ("mask",))
-        check_positive(what, **{k: m[k] for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank")})
-        rot = take_keys(m["rot"], what + " rot", ("base", "dims"))
-        check_positive(what + " rot", dims=rot["dims"])
-        if rot["dims"] % 2 or rot["dims"] > m["rot_dim"]:
-            raise ValueError(f"{what}: rot.dims must be even and at most rot_dim")
-        window = 0
-        if m["mask"]:
-            window = take_keys(m["mask"], what + " mask", ("size",))["size"]
-            check_positive(what + " mask", size=window)
-        return cls(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["q_rank"], m["kv_rank"], float(m["scale"]), window,
-                   float(rot["base"]), rot["dims"])
-
-    @property
-    def terms(self) -> ScoreTerms:
-        return ScoreTerms(self.scale, window=self.window)
-
-    @property
-    def row(self) -> int:             # elements of a cache row
-        return self.kv_rank + self.rot_dim
-
-
 @dataclass(frozen=True)
 class LightningConfig:
     heads: int
@@ -92,7 +51,7 @@ class LightningConfig:
         return cls(m["heads"], m["dim"], m["vdim"], decay)
 
 
-MIXERS = {"latent_attention": LatentAttentionConfig, "lightning": LightningConfig}
+MIXERS = {"latent_attention": partial(LatentAttentionConfig.from_json, windowed=True), "lightning": LightningConfig.from_json}
 
 
 @dataclass(frozen=True)
@@ -158,7 +117,7 @@ class StreamLMConfig:
             entry = take_keys(entry, what, ("type", "mixer"), ("mlp",))
             if entry["type"] not in MIXERS:
                 raise ValueError(f"{what}: unknown mixer type {entry['type']!r}; known: {', '.join(MIXERS)}")
-            mixer, ff = MIXERS[entry["type"]].from_json(entry["mixer"], what), None
+            mixer, ff = MIXERS[entry["type"]](entry["mixer"], what), None
             if entry["mlp"]:
                 kind = entry["mlp"].get("kind")
                 if kind not in FEED_FORWARDS:
@@ -200,9 +159,7 @@ def parameter_shapes(config: StreamLMConfig) -> dict[str, tuple]:
         for q in (1, 2) if f else (1,):
             shapes.update({f"{p}norm{q}": (w,), f"{p}hc{q}.in": (s,), f"{p}hc{q}.out": (s,), f"{p}hc{q}.mix": (s, s)})
         if isinstance(m, LatentAttentionConfig):
-            shapes.update({p + "mix.dq": (m.q_rank, w), p + "mix.dq.norm": (m.q_rank,), p + "mix.uq": (m.heads * (m.dim + m.rot_dim), m.q_rank),
-                           p + "mix.dkv": (m.row, w), p + "mix.dkv.norm": (m.kv_rank,), p + "mix.uk": (m.heads * m.dim, m.kv_rank),
-                           p + "mix.uv": (m.heads * m.vdim, m.kv_rank), p + "mix.o": (w, m.heads * m.vdim)})
+            shapes.update(m.parameter_shapes(p + "mix.", w))
         else:
             inner = m.heads * m.vdim
             shapes.update({p + "mix.q": (m.heads * m.dim, w), p + "mix.k": (m.heads * m.dim, w), p + "mix.v": (inner, w),
@@ -246,18 +203,12 @@ class _Layer:
         self.sublayers = [_Sublayer(fp32(f"norm{q}"), fp32(f"hc{q}.in"), (fp32(f"hc{q}.out"), fp32(f"hc{q}.mix")))
                           for q in ((1, 2) if f else (1,))]
         if isinstance(m, LatentAttentionConfig):
-            self.w_down, (self.q_col, self.kv_col), _ = stack_blocks([take(p + "mix.dq"), take(p + "mix.dkv")], 0)
-            self.q_norm, self.kv_norm = fp32("mix.dq.norm"), fp32("mix.dkv.norm")
-            self.w_q = take(p + "mix.uq")
-            keys = m.heads * m.dim
-            self.w_kv = torch.cat([take(p + "mix.uk"), take(p + "mix.uv")])       # all heads' keys, then all values
-            self.w_uk, self.w_uv = self.w_kv[:keys].view(m.heads, m.dim, m.kv_rank), self.w_kv[keys:].view(m.heads, m.vdim, m.kv_rank)
-            self.frequencies = rotation_frequencies(m.rot_base, m.rot_dims, model.device)
+            self.latent = LatentAttention(m, p + "mix.", take, model.attention, model.config.eps, model.device)
         else:
+            self.w_o = take(p + "mix.o")
             self.w_in, (self.q_at, self.k_at, self.v_at, self.g_at), _ = stack_blocks([take(p + "mix." + n) for n in "qkvg"], 0)
             self.out_norm = fp32("mix.norm")
             self.decay = decay_table(m.decay, model.device)
-        self.w_o = take(p + "mix.o")
         if isinstance(f, DenseConfig):
             self.w_gate_up, (_, self.up_col), _ = stack_blocks([take(p + "mlp.gate"), take(p + "mlp.up")], 0)
             self.w_ff_down = take(p + "mlp.down")
@@ -298,7 +249,7 @@ class StreamLM:
         for run, i in enumerate(self.config.runs):
             m = self.config.layers[i].mixer
             if isinstance(m, LatentAttentionConfig):
-                layers[run] = KVSpec(1, m.row, 0)
+                layers[run] = m.cache
             else:
                 states[f"r{run}.state"] = StateSpec((m.heads, m.dim, m.vdim), torch.float32)
         return CacheSpec(layers=layers, states=states, block=64)      # a page is a stage of the attention over cache rows
@@ -327,8 +278,8 @@ class StreamLM:
                     h = self._mix(streams, pending, sub.norm, sub.reads, **start)
                     parts = None
                     if q == 0:
-                        mix = self._latent_attention if isinstance(layer.mixer, LatentAttentionConfig) else self._lightning
-                        delta = mix(run, layer, h, batch, cache)
+                        latent = isinstance(layer.mixer, LatentAttentionConfig)
+                        delta = layer.latent(h, cache.key[run], batch) if latent else self._lightning(run, layer, h, batch, cache)
                     elif isinstance(layer.ff, DenseConfig):
                         act = clamped_glu(F.linear(h, layer.w_gate_up), layer.up_col, layer.ff.ff, layer.ff.limit, self.glu_slope)
                         delta = F.linear(act, layer.w_ff_down)
@@ -340,40 +291,6 @@ class StreamLM:
                     self._mix(total, pending, self.final_norm, None)
                     after_layer(run, total.sum(1))
         return streams, pending
-
-    def _latent_attention(self, run, layer, h, batch, cache):
-        m, rows = layer.mixer, h.shape[0]
-        pages = cache.key[run]
-        latent = latent_write(F.linear(h, layer.w_down), layer.q_col, layer.kv_col, layer.q_norm, layer.kv_norm, self.config.eps,
-                              layer.frequencies, pages, batch)
-        q = F.linear(latent, layer.w_q).view(rows, m.heads, m.dim + m.rot_dim)
-        out = torch.empty(rows, m.heads, m.vdim, dtype=self.dtype, device=self.device)
-        for group in batch.groups:
-            expand = group.max_new > SHORT_PORTION and group.portions is not None and m.kv_rank % 8 == 0 and \
-                latent_prompt_supported(m.dim, m.rot_dim, m.vdim, self.dtype)
-            attend = self._attend_expanded if expand else self._attend_latents
-            attend(layer, q[group.rows], out[group.rows], pages, batch.positions[group.rows], group)
-        return F.linear(out.view(rows, -1), layer.w_o)
-
-    def _attend_expanded(self, layer, q, out, pages, positions, group):
-        """Over keys and values expanded from the latents of every position the portions see."""
-        m = layer.mixer
-        ranges = group.key_ranges(m.window)
-        rows = latent_gather(pages, group.tables, ranges)
-        rotate_heads(q[:, :, m.dim:], q[:, :, m.dim:], layer.frequencies, positions)
-        latent_prompt_attention(q, F.linear(rows[:, :m.kv_rank], layer.w_kv), rows[:, m.kv_rank:], out, m.dim, ranges, m.scale, m.window)
-
-    def _attend_latents(self, layer, q, out, pages, positions, group):
-        """Over the cache rows themselves: a head's query is taken into the latent's space (q . W_uk c = W_uk^T q . c), so all
-        heads score the one row of a key, and the weighted sum of latents is taken out of it by W_uv."""
-        m, rows = layer.mixer, q.shape[0]
-        operand = torch.empty(rows, m.heads, m.row, dtype=self.dtype, device=self.device)
-        torch.bmm(q[:, :, :m.dim].transpose(0, 1), layer.w_uk, out=operand[:, :, :m.kv_rank].transpose(0, 1))
-        rotate_heads(q[:, :, m.dim:], operand[:, :, m.kv_rank:], layer.frequencies, positions)
-        latents = torch.empty(rows, m.heads, m.kv_rank, dtype=self.dtype, device=self.device)
-        self.attention.scored(operand, latents, pages, pages[..., :m.kv_rank], group.tables, group.lengths, group.local_cu, group.max_new,
-                              m.terms)
-        torch.bmm(latents.transpose(0, 1), layer.w_uv.transpose(1, 2), out=out.transpose(0, 1))
 
     def _lightning(self, run, layer, h, batch, cache):
         m, rows = layer.mixer, h.shape[0]
@@ -390,17 +307,13 @@ class StreamLM:
         return F.linear(gated, layer.w_o)
 
     def _experts(self, layer, h, queue):
-        routing = expert_route(self._product32(h, layer.router), layer.correction, layer.ff.top, counts=queue)
+        routing = expert_route(product32(h, layer.router), layer.correction, layer.ff.top, counts=queue)
         x = expert_gather(h, routing)
         y = expert_gemm(expert_gemm(x, layer.e_up, routing.counts, "squared_relu"), layer.e_down, routing.counts)
         return y, (routing.places, routing.weights)
-
-    def _product32(self, x, weight):
-        """x W^T with an fp32 result."""
-        return F.linear(x, weight) if self.dtype == torch.float32 else torch.mm(x, weight.t(), out_dtype=torch.float32)
 
     def step_logits(self, hidden, rows=None):
         """fp32 logits of the given rows (int64 indices; None: all)."""
         streams, pending = hidden
         with full_accumulation():
-            return self._product32(self._mix(streams, pending, self.final_norm, None, row_index=rows, store=False), self.head)
+            return product32(self._mix(streams, pending, self.final_norm, None, row_index=rows, store=False), self.head)
