@@ -46,6 +46,9 @@ Other entry points (each prints its own JSON line; none is the contract line abo
     --workload stream [--steps K --warmup W]
                       the same for Sugosun-shaped models (hyper-connected streams, latent / lightning attention, dense and
                       mixture-of-experts feed-forwards)
+    --workload sandwich [--steps K --warmup W]
+                      the same for Kezuvik-shaped models (norms on both sides of a sublayer, latent attention with sinks and gates,
+                      windowed attention behind a convolution), beside Sugosun and the looped model
     --only attention  [--requests --layers --tokens --depths --kv-heads --context-min --context-max --shared-plan]
     --only prefill    [--requests --tokens --kv-heads --eager]   packed causal prefill, TFLOP/s
     --only accept | --only silu                                  the small kernels at the step's shapes
@@ -990,6 +993,25 @@ def ring_us(calls, replays: int) -> float:
     return ms / len(calls) * 1e3
 
 
+class KernelRows:
+    """Rows of a kernel table: time of a call in a ring of calls, and its fraction of the measured roofline (the later of the two bounds)."""
+
+    def __init__(self, steps):
+        self.steps, self.rows = steps, []
+        self.peak_gbs, _ = measured_peaks()
+        peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
+        self.peak_tflops = float(peaks.get("bf16_tflops", 1590.0))
+
+    def __call__(self, kernel, phase, like, make, nbytes=0.0, flops=0.0, copies=None):
+        """make(i) -> a call on the i-th set of tensors."""
+        copies = copies or max(2, min(48, int(400e6 // max(nbytes, 1)) + 1))
+        us = ring_us([make(i) for i in range(copies)], self.steps)
+        tensor = flops / self.peak_tflops / 1e6 > nbytes / self.peak_gbs / 1e3
+        frac = flops / us / 1e6 / self.peak_tflops if tensor else nbytes / us / 1e3 / self.peak_gbs
+        self.rows.append({"kernel": kernel, "phase": phase, "like": like, "us": us, "bound": "tensor" if tensor else "hbm", "roofline_frac": frac})
+        torch.cuda.empty_cache()
+
+
 @torch.no_grad()
 def hybrid_kernel_rows(size, steps):
     """Every kernel of a hybrid layer at prefill (16384 rows: 8 x 2048) and decode (64 rows, context 2048), with its
@@ -1195,25 +1217,12 @@ def stream_kernel_rows(size, steps):
     from vllm_rlt_b200.engine import KeyRanges
 
     device = torch.device("cuda", 0)
-    peak_gbs, _ = measured_peaks()
-    peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
-    peak_tflops = float(peaks.get("bf16_tflops", 1590.0))
     width, heads, rank, rot, q_rank = size["width"], size["heads"], size["kv_rank"], size["rot_dim"], size["q_rank"]
     ff, experts, top, expert_ff, s_count = size["ff"], size["experts"], size["top"], size["expert_ff"], size["streams"]
     row_dim, inner, key_dim = rank + rot, heads * HEAD_DIM, HEAD_DIM + rot
     bf16 = lambda *shape: torch.randn(*shape, device=device).to(torch.bfloat16)
     f32 = lambda *shape: torch.randn(*shape, device=device)
-    rows_out = []
-
-    def add(kernel, phase, like, make, nbytes=0.0, flops=0.0, copies=None):
-        """make(i) -> a call on the i-th set of tensors.  The roofline is the later of the two bounds."""
-        copies = copies or max(2, min(48, int(400e6 // max(nbytes, 1)) + 1))
-        us = ring_us([make(i) for i in range(copies)], steps)
-        tensor = flops / peak_tflops / 1e6 > nbytes / peak_gbs / 1e3
-        frac = flops / us / 1e6 / peak_tflops if tensor else nbytes / us / 1e3 / peak_gbs
-        rows_out.append({"kernel": kernel, "phase": phase, "like": like, "us": us, "bound": "tensor" if tensor else "hbm", "roofline_frac": frac})
-        torch.cuda.empty_cache()
-
+    add = KernelRows(steps)
     for phase, seqs, new, context in (("prefill", 8, 2048, 2048), ("decode", 64, 1, 2048)):
         rows, page = seqs * new, 64
         pages = context // page
@@ -1339,7 +1348,7 @@ def stream_kernel_rows(size, steps):
         add("cuBLAS GEMM (gate and up)", phase, None, lambda i: (lambda: torch.nn.functional.linear(inputs, dense[i])),
             (2 * ff * width + rows * (width + 2 * ff)) * 2.0, 2.0 * rows * width * 2 * ff, copies=8)
         del dense, inputs
-    return rows_out
+    return add.rows
 
 
 def run_stream_workload(args):
@@ -1369,6 +1378,213 @@ def run_stream_workload(args):
             del model
             torch.cuda.empty_cache()
             report["sizes"][name] = {"shape": dict(size), "throughput": rows, "kernels": stream_kernel_rows(size, args.steps)}
+            torch.cuda.empty_cache()
+    report["clocks"] = clocks.summary()
+    print(json.dumps(report))
+
+
+# Layer shapes of the sandwich workload: those of the stream workload's latent and dense layers, with windowed attention of grouped heads.
+SANDWICH_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, q_rank=1536, kv_rank=512, rot_dim=64, window=1024, taps=4, ff=5632, layers=8, vocab=49152),
+    "4096": dict(width=4096, heads=32, kv_heads=8, q_rank=1536, kv_rank=512, rot_dim=64, window=1024, taps=4, ff=9600, layers=6, vocab=49152),
+}
+
+
+def sandwich_config(size, pattern):
+    """config.json of a Kezuvik model whose layers repeat `pattern` ('e' latent attention with a gate per element, 's' latent attention with
+    sinks, scaled rotation and a gate per head, 'w' windowed attention)."""
+    latent = {"heads": size["heads"], "dim": HEAD_DIM, "rot_dim": size["rot_dim"], "vdim": HEAD_DIM, "q_rank": size["q_rank"], "kv_rank": size["kv_rank"],
+              "scale": (HEAD_DIM + size["rot_dim"]) ** -0.5}
+    rot = {"base": 10000.0, "dims": size["rot_dim"]}
+    kinds = {"e": ("latent_attention", dict(latent, rot=rot)),
+             "s": ("latent_attention_2", dict(latent, rot=dict(rot, scaling={"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}))),
+             "w": ("attention", {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": HEAD_DIM, "vdim": HEAD_DIM, "conv": size["taps"],
+                                 "mask": {"size": size["window"]}, "scale": HEAD_DIM ** 0.5})}
+    layers = []
+    for i in range(size["layers"]):
+        kind, mixer = kinds[pattern[i % len(pattern)]]
+        layers.append({"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": size["ff"]}})
+    return {"architecture": "Kezuvik", "vocab": size["vocab"], "width": size["width"], "residual_mult": 0.5, "logit_softcap": 30.0,
+            "norm": {"eps": 1e-6}, "layers": layers}
+
+
+@torch.no_grad()
+def sandwich_kernel_rows(size, steps):
+    """Every kernel of a Kezuvik layer at prefill (16384 rows: 8 x 2048) and decode (64 rows, context 2048), with its algorithmic bytes
+    or flops against the measured peak, beside the like kernel of the nearest model (Sugosun, Sobipel, looped)."""
+    from types import SimpleNamespace
+
+    import vllm_rlt_b200 as rlt
+    from vllm_rlt_b200.engine import KeyRanges
+
+    device = torch.device("cuda", 0)
+    width, heads, kv_heads, rank, rot, q_rank = (size[k] for k in ("width", "heads", "kv_heads", "kv_rank", "rot_dim", "q_rank"))
+    ff, window, taps = size["ff"], size["window"], size["taps"]
+    row_dim, inner, key_dim, kv_inner = rank + rot, heads * HEAD_DIM, HEAD_DIM + rot, kv_heads * HEAD_DIM
+    bf16 = lambda *shape: torch.randn(*shape, device=device).to(torch.bfloat16)
+    f32 = lambda *shape: torch.randn(*shape, device=device)
+    add = KernelRows(steps)
+    sink = f32(heads)
+    for phase, seqs, new, context in (("prefill", 8, 2048, 2048), ("decode", 64, 1, 2048)):
+        rows, page = seqs * new, 64
+        pages = context // page
+        tables = torch.randperm(seqs * pages, device=device).int().view(seqs, pages)
+        lengths = torch.full((seqs,), context, dtype=torch.int32, device=device)
+        cu = (torch.arange(seqs + 1, device=device) * new).int()
+        positions = (torch.arange(rows, device=device) % new).int() + (context - new)
+        row_seq = torch.arange(seqs, device=device, dtype=torch.int32).repeat_interleave(new)
+        batch = SimpleNamespace(tables=tables[None], row_seq=row_seq, positions=positions)
+        group = SimpleNamespace(sequences=seqs, max_new=new, cu=cu, starts=lengths - new, slots=torch.arange(seqs, device=device, dtype=torch.int32),
+                                lengths=lengths, tables=tables)
+        kernels = rlt.B200PagedAttention()
+        small = lambda nbytes: max(2, min(48, int(400e6 // nbytes) + 1))
+
+        # latent attention: sinks and gates against none
+        pairs = sum(range(context - new + 1, context + 1)) * seqs
+        if new > 1:
+            ranges = KeyRanges.of([(0, new)] * seqs, 0, device)
+            q, kv, latent, out = [bf16(rows, heads, key_dim) for _ in range(2)], [bf16(rows, 2 * inner) for _ in range(2)], bf16(rows, row_dim), bf16(rows, heads, HEAD_DIM)
+            gates = {"head": bf16(rows, heads), "element": bf16(rows, inner)}
+            for name, like, extra in (("latent attention, sink, gate per head", "latent attention (Sugosun)", dict(sink=sink, gate=gates["head"])),
+                                      ("latent attention, gate per element", "latent attention (Sugosun)", dict(gate=gates["element"])),
+                                      ("latent attention (Sugosun)", None, {})):
+                nbytes = rows * (heads * key_dim + 3 * inner + row_dim) * 2.0 + (extra["gate"].numel() * 2.0 if extra else 0.0)
+                add(name, phase, like, lambda i: (lambda: rlt.latent_prompt_attention(q[i % 2], kv[i % 2], latent[:, rank:], out, HEAD_DIM, ranges, key_dim ** -0.5, 0, **extra)),
+                    nbytes, 2.0 * pairs * heads * (key_dim + HEAD_DIM), copies=4)
+            del q, kv, latent, out, gates
+        else:
+            copies = small(seqs * context * row_dim * 2)
+            pools = [bf16(seqs * pages, page, 1, row_dim) for _ in range(copies)]
+            q, out = bf16(rows, heads, row_dim), bf16(rows, heads, rank)
+            for name, like, terms in (("latent attention, sink", "latent attention (Sugosun)", rlt.ScoreTerms(key_dim ** -0.5, sink=sink)),
+                                      ("latent attention (Sugosun)", None, rlt.ScoreTerms(key_dim ** -0.5))):
+                add(name, phase, like, lambda i: (lambda: kernels.scored(q, out, pools[i], pools[i][..., :rank], tables, lengths, cu, 1, terms)),
+                    seqs * context * row_dim * 2.0 + rows * heads * (row_dim + rank) * 2.0, 2.0 * seqs * context * heads * (row_dim + rank), copies=copies)
+            del pools, q, out
+
+        # windowed attention of grouped heads, and the page kernels' over whole contexts with the same heads
+        seen = sum(min(p + 1, window) for p in range(context - new, context)) * seqs
+        stored = seqs * min(context, new + window - 1)
+        q, out = [bf16(rows, heads, HEAD_DIM) for _ in range(2)], bf16(rows, heads, HEAD_DIM)
+        terms = rlt.ScoreTerms(HEAD_DIM ** -0.5, window=window)
+        kv_bytes, qo_bytes = stored * kv_inner * 4.0, rows * inner * 4.0
+        if new > 1:
+            ranges = KeyRanges.of([(0, new)] * seqs, window, device)
+            k, v, gate = bf16(ranges.rows, kv_heads, HEAD_DIM), bf16(ranges.rows, kv_heads, HEAD_DIM), bf16(rows, inner)
+            add("windowed attention, gate per element", phase, "attention of grouped heads (Sobipel)",
+                lambda i: (lambda: rlt.packed_attention(q[i % 2], k, v, out, ranges, HEAD_DIM ** -0.5, window, gate=gate)), kv_bytes + 1.5 * qo_bytes, 4.0 * seen * inner, copies=4)
+            del k, v, gate
+            caches = [bf16(seqs * pages, page, 1, kv_inner) for _ in range(12)]
+            add("latent_gather (keys of a window)", phase, "latent_gather (Sugosun)", lambda i: (lambda: rlt.latent_gather(caches[i], tables, ranges)),
+                ranges.rows * kv_inner * 4.0, copies=12)
+            caches = [bf16(seqs * pages, page, 1, row_dim) for _ in range(12)]
+            add("latent_gather (Sugosun)", phase, None, lambda i: (lambda: rlt.latent_gather(caches[i], tables, ranges)), ranges.rows * row_dim * 4.0, copies=12)
+            del caches
+        else:
+            copies = small(kv_bytes)
+            pools = [bf16(2, seqs * pages, page, kv_heads, HEAD_DIM) for _ in range(copies)]
+            add("windowed attention", phase, "attention of grouped heads (Sobipel)",
+                lambda i: (lambda: kernels.scored(q[i % 2], out, pools[i][0], pools[i][1], tables, lengths, cu, 1, terms)), kv_bytes + qo_bytes, copies=copies)
+            del pools
+        small_pages = context // BLOCK
+        small_tables = torch.randperm(seqs * small_pages, device=device).int().view(seqs, small_pages)
+        copies = max(2, min(12, small(seqs * context * kv_inner * 4)))
+        pools = [bf16(2, seqs * small_pages, BLOCK, kv_heads, HEAD_DIM) for _ in range(copies)]
+        plain = rlt.ScoreTerms(HEAD_DIM ** -0.5, 0.1, 2048, True)
+        add("attention of grouped heads (Sobipel)", phase, None,
+            lambda i: (lambda: kernels.scored(q[i % 2], out, pools[i][0], pools[i][1], small_tables, lengths, cu, new, plain)),
+            seqs * context * kv_inner * 4.0 + qo_bytes, 4.0 * pairs * inner, copies=copies)
+        del pools, q, out
+
+        # between projections and scores
+        channels = inner + 2 * kv_inner
+        nbytes = rows * channels * 4.0 + (seqs * (taps - 1) * channels * 4.0 if new == 1 else 0.0)
+        copies = small(rows * (channels + inner) * 2)
+        proj = [bf16(rows, channels + inner) for _ in range(copies)]
+        weight, state = f32(channels, taps), torch.zeros(seqs, taps - 1, channels, dtype=torch.bfloat16, device=device)
+        q_out, cache = bf16(rows, heads, HEAD_DIM), bf16(2, seqs * pages, page, kv_heads, HEAD_DIM)
+        add("conv_heads", phase, "causal_conv (Sobipel)",
+            lambda i: (lambda: rlt.conv_heads(proj[i], (0, inner, inner + kv_inner), weight, 1e-6, state, q_out, cache[0], cache[1], group)), nbytes, copies=copies)
+        bias, mixed = f32(channels), bf16(rows, channels)
+        add("causal_conv (Sobipel)", phase, None, lambda i: (lambda: rlt.causal_conv(proj[i][:, :channels], weight, bias, state, mixed, group)), nbytes, copies=copies)
+        del proj, q_out, cache, mixed
+        nbytes = rows * heads * rot * 4.0
+        copies = small(rows * heads * key_dim * 2)
+        q = [bf16(rows, heads, key_dim) for _ in range(copies)]
+        frequencies = rlt.rotation_frequencies(10000.0, rot, device)
+        for name, like, turn in (("rotate_heads (halves)", "rotate_heads (Sugosun)", dict(halves=True, amplitude=1.2)), ("rotate_heads (Sugosun)", None, {})):
+            add(name, phase, like, lambda i: (lambda: rlt.rotate_heads(q[i][:, :, HEAD_DIM:], q[i][:, :, HEAD_DIM:], frequencies, positions, **turn)), nbytes, copies=copies)
+        del q
+        down = q_rank + row_dim
+        copies = small(rows * down * 4)
+        proj, cache = [bf16(rows, down) for _ in range(copies)], bf16(seqs * pages, page, 1, row_dim)
+        q_norm, kv_norm = f32(q_rank), f32(rank)
+        for name, like, turn in (("latent_write (halves)", "latent_write (Sugosun)", dict(halves=True, amplitude=1.2)), ("latent_write (Sugosun)", None, {})):
+            add(name, phase, like, lambda i: (lambda: rlt.latent_write(proj[i], 0, q_rank, q_norm, kv_norm, 1e-6, frequencies, cache, batch, **turn)), rows * down * 4.0, copies=copies)
+        del proj, cache
+
+        # between the sublayers
+        nbytes = rows * width * 12.0
+        copies = small(nbytes)
+        residual, delta = [f32(rows, width) for _ in range(copies)], [bf16(rows, width) for _ in range(copies)]
+        before, behind = f32(width), f32(width)
+        add("residual_norm, layer norms on both sides", phase, "sandwich_norm (looped)",
+            lambda i: (lambda: rlt.residual_norm(residual[i], before, 1e-6, torch.bfloat16, delta=delta[i], behind=(behind, 0.5), centred=True)), nbytes, copies=copies)
+        add("residual_norm (Sobipel)", phase, None, lambda i: (lambda: rlt.residual_norm(residual[i], before, 1e-6, torch.bfloat16, delta=delta[i])), nbytes, copies=copies)
+        w16, res16 = bf16(width), [bf16(rows, width) for _ in range(copies)]
+        add("sandwich_norm (looped)", phase, None, lambda i: (lambda: rlt.sandwich_norm(delta[i], w16, 1e-6, res16[i], w16, in_place=True)), rows * width * 8.0, copies=copies)
+        del residual, delta, res16
+
+        # gates and units
+        copies = small(rows * inner * 4)
+        y, gate = [bf16(rows, heads, HEAD_DIM) for _ in range(copies)], [bf16(rows, inner) for _ in range(copies)]
+        add("head_gate, per element", phase, "gated_norm (Sugosun)", lambda i: (lambda: rlt.head_gate(y[i], gate[i])), rows * inner * 6.0, copies=copies)
+        add("head_gate, per head", phase, "gated_norm (Sugosun)", lambda i: (lambda: rlt.head_gate(y[i], gate[i][:, :heads])), rows * inner * 4.0, copies=copies)
+        norm_w, gated = f32(inner), bf16(rows, inner)
+        add("gated_norm (Sugosun)", phase, None, lambda i: (lambda: rlt.gated_norm(y[i].view(rows, -1), gate[i], norm_w, gated, 1, 1e-6, gate_behind=True)), rows * inner * 6.0, copies=copies)
+        del y, gate, gated
+        copies = small(rows * ff * 6)
+        gate_up = [bf16(rows, 2 * ff) for _ in range(copies)]
+        add("gated_unit (tanh gelu)", phase, "clamped_glu (Sugosun)", lambda i: (lambda: rlt.gated_unit(gate_up[i], ff, ff, "gelu_tanh")), rows * ff * 6.0, copies=copies)
+        add("clamped_glu (Sugosun)", phase, None, lambda i: (lambda: rlt.clamped_glu(gate_up[i], ff, ff, 7.0, 1.702)), rows * ff * 6.0, copies=copies)
+        del gate_up
+        if new == 1:
+            copies = small(rows * size["vocab"] * 4)
+            logits = [f32(rows, size["vocab"]) for _ in range(copies)]
+            add("soft_cap", phase, "gated_norm (Sugosun)", lambda i: (lambda: rlt.soft_cap(logits[i], 30.0)), rows * size["vocab"] * 8.0, copies=copies)
+            del logits
+    return add.rows
+
+
+def run_sandwich_workload(args):
+    """`--workload sandwich`: one JSON line with throughput rows, kernel rows and the clocks under them."""
+    import vllm_rlt_b200 as rlt
+    from vllm_rlt_b200.looped_lm import parameter_shapes as looped_shapes
+    from vllm_rlt_b200.sandwich_lm import parameter_shapes as sandwich_shapes
+    from vllm_rlt_b200.stream_lm import parameter_shapes as stream_shapes
+
+    torch.cuda.set_device(0)
+    device = torch.device("cuda", 0)
+    report = {"workload": "sandwich", "data": "synthetic, random weights", "dtype": "bf16", "steps": args.steps, "sizes": {}}
+    with ClockSampler(0) as clocks:
+        for name, size in SANDWICH_SIZES.items():
+            rows = []
+            builds = [(f"Kezuvik, {label}", lambda pattern=pattern: rlt.SandwichLM(config := rlt.SandwichLMConfig.from_json(sandwich_config(size, pattern)),
+                                                                                   device_weights(sandwich_shapes(config), device), device))
+                      for label, pattern in (("latent attention, gate per element", "e"), ("latent attention, sinks", "s"), ("windowed attention", "w"),
+                                             ("all three", "sew"))]
+            builds.append(("Sugosun, latent attention and dense", lambda: rlt.StreamLM(
+                config := rlt.StreamLMConfig.from_json(stream_config(STREAM_SIZES[name], ["ad"])), device_weights(stream_shapes(config), device), device)))
+            looped = rlt.LoopedLMConfig(vocab_size=size["vocab"], hidden_size=size["width"], intermediate_size=size["ff"],
+                                        num_hidden_layers=size["layers"], num_attention_heads=size["heads"],
+                                        num_key_value_heads=size["heads"], head_dim=HEAD_DIM, total_ut_steps=1)
+            builds.append(("looped model, one loop", lambda: rlt.LoopedLM(looped, device_weights(looped_shapes(looped), device), device, torch.bfloat16)))
+            for label, build in builds:
+                model = build()
+                rows += hybrid_model_rows(label, model, args.steps, args.warmup)
+                del model
+                torch.cuda.empty_cache()
+            report["sizes"][name] = {"shape": dict(size), "throughput": rows, "kernels": sandwich_kernel_rows(size, args.steps)}
             torch.cuda.empty_cache()
     report["clocks"] = clocks.summary()
     print(json.dumps(report))
@@ -1666,7 +1882,7 @@ def main():
     parser.add_argument("--no-cpu-baseline", action="store_true")
     parser.add_argument("--only", default=None, choices=["attention", "accept", "silu", "prefill"],
                         help="profiling aid: run only this kernel family (not a bench line)")
-    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded", "hybrid", "stream"],
+    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded", "hybrid", "stream", "sandwich"],
                         help="rounds: timed speculative rounds (the bench line); decode: one complete generation; "
                              "sharded: a fixed request set shared out over the ranks, decoded to completion")
     parser.add_argument("--engine", default="b200", choices=["b200", "reference"],
@@ -1714,6 +1930,9 @@ def main():
             setattr(args, name, sharded_default if sharded else decode_default)
     if sharded:
         run_sharded_workload(args)
+        return
+    if args.workload == "sandwich":
+        run_sandwich_workload(args)
         return
     if args.workload == "stream":
         run_stream_workload(args)

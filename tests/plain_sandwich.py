@@ -62,16 +62,20 @@ def attention(q, k, v, scale, window=0, sink=None, first=0):
     """q [n, H, d] at positions first .. over k [T, G, d], v [T, G, e]: query head h reads key/value head h // (H / G); a row sees
     itself and the window - 1 keys before it (window 0: all of them); sink [H]: one more term of a head's denominator."""
     n, heads, share = q.shape[0], q.shape[1], q.shape[1] // k.shape[1]
+    group = torch.arange(heads) // share
     out = torch.zeros(n, heads, v.shape[2], dtype=torch.float64)
     for i in range(n):
         p = first + i
         lo = max(p - window + 1, 0) if window else 0
-        for h in range(heads):
-            scores = k[lo:p + 1, h // share] @ q[i, h] * scale
-            top = scores.max() if sink is None else torch.maximum(scores.max(), sink[h])
-            weights = torch.exp(scores - top)
-            total = weights.sum() if sink is None else weights.sum() + torch.exp(sink[h] - top)
-            out[i, h] = weights @ v[lo:p + 1, h // share] / total
+        scores = torch.einsum("hd,thd->ht", q[i], k[lo:p + 1, group]) * scale
+        top = scores.amax(1)
+        if sink is not None:
+            top = torch.maximum(top, sink)
+        weights = torch.exp(scores - top[:, None])
+        total = weights.sum(1)
+        if sink is not None:
+            total = total + torch.exp(sink - top)
+        out[i] = torch.einsum("ht,the->he", weights, v[lo:p + 1, group]) / total[:, None]
     return out
 
 
@@ -106,7 +110,7 @@ class PlainSandwich:
     def latent(self, p, m, h, second):
         """`second`: the kind with a sink, scaled frequencies and one gate per head; else one gate per element."""
         w, r, n, heads, d = self.w, self.r, h.shape[0], m["heads"], m["dim"]
-        turns, amplitude = frequencies(m["rot"]["base"], m["rot"]["dims"], m["rot"]["scaling"] if second else None)
+        turns, amplitude = frequencies(m["rot"]["base"], m["rot"]["dims"], m["rot"].get("scaling") if second else None)
         turn = lambda x: r(rotate(x, torch.arange(n), turns, amplitude))
         c_q = r(rms_norm(r(h @ w[p + "dq"].T), w[p + "dq.norm"], self.eps))
         q = r(c_q @ w[p + "uq"].T).reshape(n, heads, -1)
