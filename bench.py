@@ -1501,12 +1501,12 @@ def sandwich_kernel_rows(size, steps):
         nbytes = rows * channels * 4.0 + (seqs * (taps - 1) * channels * 4.0 if new == 1 else 0.0)
         copies = small(rows * (channels + inner) * 2)
         proj = [bf16(rows, channels + inner) for _ in range(copies)]
-        weight, state = f32(channels, taps), torch.zeros(seqs, taps - 1, channels, dtype=torch.bfloat16, device=device)
+        weight, state = f32(taps, channels), torch.zeros(seqs, taps - 1, channels, dtype=torch.bfloat16, device=device)
         q_out, cache = bf16(rows, heads, HEAD_DIM), bf16(2, seqs * pages, page, kv_heads, HEAD_DIM)
         add("conv_heads", phase, "causal_conv (Sobipel)",
             lambda i: (lambda: rlt.conv_heads(proj[i], (0, inner, inner + kv_inner), weight, 1e-6, state, q_out, cache[0], cache[1], group)), nbytes, copies=copies)
-        bias, mixed = f32(channels), bf16(rows, channels)
-        add("causal_conv (Sobipel)", phase, None, lambda i: (lambda: rlt.causal_conv(proj[i][:, :channels], weight, bias, state, mixed, group)), nbytes, copies=copies)
+        channel_weight, bias, mixed = f32(channels, taps), f32(channels), bf16(rows, channels)
+        add("causal_conv (Sobipel)", phase, None, lambda i: (lambda: rlt.causal_conv(proj[i][:, :channels], channel_weight, bias, state, mixed, group)), nbytes, copies=copies)
         del proj, q_out, cache, mixed
         nbytes = rows * heads * rot * 4.0
         copies = small(rows * heads * key_dim * 2)

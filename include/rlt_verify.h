@@ -679,7 +679,7 @@ RLT_API int rlt_soft_cap(float* x, int64_t count, float cap, rlt_stream_t stream
 
 /* What stands between the projections of an attention layer and its scores: a causal convolution over time per channel of q, k and v
  * (no bias, no activation), then with unit_norm != 0 q and k of every head divided by their root mean square, then k and v into the
- * pages of the row's position and q into q_out [rows][q_heads * key_dim].  Channels are ordered q, k, v in weight (fp32 [channels][taps])
+ * pages of the row's position and q into q_out [rows][q_heads * key_dim].  Channels are ordered q, k, v in weight (fp32 [taps][channels])
  * and in state ([slots][taps - 1][channels] of `dtype`, the last inputs, updated in place); q_col, k_col, v_col: their columns in proj.
  * Sequences and slots as in rlt_causal_conv; lengths[s]: tokens of sequence s after the portion (0: padding, nothing is written to pages). */
 RLT_API int rlt_conv_heads(const void* proj, int64_t proj_stride, int q_col, int k_col, int v_col, int q_heads, int kv_heads,

@@ -110,7 +110,8 @@ def test_latent_rows_with_turned_halves(dtype, q_rank, kv_rank, rot_dim, dims):
 # ---- convolution and unit norm in front of the scores --------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,taps", [(4, 2, 24, 40, 4), (3, 1, 10, 7, 1), (1, 1, 5, 3, 6), (8, 2, 128, 128, 3), (2, 2, 72, 136, 2),
-                                                          (5, 5, 256, 64, 4), (2, 1, 16, 12, 33), (1, 1, 300, 20, 3)])
+                                                          (5, 5, 256, 64, 4), (2, 1, 16, 12, 33), (1, 1, 300, 20, 3), (6, 3, 128, 64, 4),
+                                                          (2, 1, 32, 64, 1), (3, 3, 8, 8, 4)])
 @pytest.mark.parametrize("unit_norm", [True, False])
 def test_heads_behind_a_convolution(dtype, heads, kv_heads, dim, vdim, taps, unit_norm):
     """Two sequences in portions of unequal size, one of which starts late; pages, queries and the state that is carried on."""
@@ -134,7 +135,7 @@ def test_heads_behind_a_convolution(dtype, heads, kv_heads, dim, vdim, taps, uni
                                 starts=as_int([at[s] for s, _ in parts]), lengths=as_int([at[s] + n for s, n in parts]), slots=as_int([slots[s] for s, _ in parts]),
                                 tables=tables[[s for s, _ in parts]].contiguous().cuda())
         q = torch.empty(rows, heads, dim, dtype=dtype, device="cuda")
-        rlt.conv_heads(torch.cat([texts[s][at[s]:at[s] + n] for s, n in parts]).cuda(), columns, weight.cuda(), 1e-2, state, q, key, value, group, unit_norm=unit_norm)
+        rlt.conv_heads(torch.cat([texts[s][at[s]:at[s] + n] for s, n in parts]).cuda(), columns, weight.t().contiguous().cuda(), 1e-2, state, q, key, value, group, unit_norm=unit_norm)
         first = 0
         for s, n in parts:
             got[s].append(q[first:first + n])
@@ -162,7 +163,7 @@ def test_padding_rows_of_a_captured_step_write_no_page(dtype):
                             slots=zero + 1, tables=torch.zeros(1, 2, dtype=torch.int32, device="cuda"))
     state = torch.full((2, 2, 48), 5.0, dtype=dtype, device="cuda")
     q = torch.empty(1, 1, 16, dtype=dtype, device="cuda")
-    rlt.conv_heads(torch.ones(1, 48, dtype=dtype, device="cuda"), (0, 16, 32), torch.ones(48, 3, device="cuda"), 1e-5, state, q, key, value, group)
+    rlt.conv_heads(torch.ones(1, 48, dtype=dtype, device="cuda"), (0, 16, 32), torch.ones(3, 48, device="cuda"), 1e-5, state, q, key, value, group)
     assert bool((key == 9.0).all()) and bool((value == 9.0).all()) and bool((state[0] == 5.0).all()) and bool(torch.isfinite(q).all())
 
 

@@ -33,7 +33,7 @@ def test_configurations_parse_and_name_every_tensor(name):
             for at, n in zip(mixer.columns, "qkv"):
                 assert torch.equal(mixer.w_in[at:at + w(n).shape[0]], w(n)) and torch.equal(mixer.bias[at:at + w(n).shape[0]], w(n + ".b"))
             assert torch.equal(mixer.w_in[mixer.g_col:mixer.g_col + m.heads * m.vdim], w("g"))
-            assert not mixer.bias[mixer.g_col:].any() and mixer.conv.shape == (sum(m.projections.values()), entry["mixer"]["conv"])
+            assert not mixer.bias[mixer.g_col:].any() and mixer.conv.shape == (entry["mixer"]["conv"], sum(m.projections.values()))
         else:
             second = entry["type"] == "latent_attention_2"
             assert (mixer.sink is not None) == (f"{p}mix.sink" in shapes) == second

@@ -45,20 +45,11 @@ struct PromptShared {
 };
 
 // Eight output elements times the sigmoid of their gates.
-__device__ __forceinline__ uint4 gated(uint4 piece, const __nv_bfloat16* gate, int column, bool per_head) {
-  const __nv_bfloat16* y = reinterpret_cast<const __nv_bfloat16*>(&piece);
-  float v[8], g[8];
-  if (per_head) {
-    const float one = sigmoid<__nv_bfloat16>(__bfloat162float(*gate));
+__device__ __forceinline__ uint4 gated(const uint4& piece, const uint4& gate) {
+  const __nv_bfloat16 *y = reinterpret_cast<const __nv_bfloat16*>(&piece), *g = reinterpret_cast<const __nv_bfloat16*>(&gate);
+  float v[8];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) g[e] = one;
-  } else {
-    load_floats<__nv_bfloat16, 8>(gate + column, g);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) g[e] = sigmoid<__nv_bfloat16>(g[e]);
-  }
-#pragma unroll
-  for (int e = 0; e < 8; ++e) v[e] = __bfloat162float(y[e]) * g[e];
+  for (int e = 0; e < 8; ++e) v[e] = __bfloat162float(y[e]) * sigmoid<__nv_bfloat16>(__bfloat162float(g[e]));
   return make_uint4(pack2<true>(v[0], v[1]), pack2<true>(v[2], v[3]), pack2<true>(v[4], v[5]), pack2<true>(v[6], v[7]));
 }
 
@@ -278,17 +269,28 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&sm.p_ready[t]));
     }
+    const int64_t first_out = static_cast<int64_t>(tile.q_row) + t * kRows + warp_row;
+    const int warp_count = min(max(count[t] - warp_row, 0), 32);
+    const bool gate_elements = a.gate != nullptr && !a.gate_per_head;
+    const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(a.gate) + first_out * a.gate_stride + static_cast<int64_t>(head) * (gate_elements ? a.vdim : 1);
+    uint4 gates[8];                 // of a block of 64 output columns, loaded ahead of the output
+    auto load_gates = [&](int b) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int r = 4 * i + (lane >> 3), column = b * 64 + (lane & 7) * 8;
+        if (r < warp_count && column < a.vdim) gates[i] = *reinterpret_cast<const uint4*>(gate + r * a.gate_stride + column);
+      }
+    };
+    if (gate_elements) load_gates(0);
+    const float head_gate = a.gate != nullptr && a.gate_per_head && live ? sigmoid<__nv_bfloat16>(__bfloat162float(gate[lane * a.gate_stride])) : 1.0f;
     if (!failed && stages > 0 && !mbar_wait(smem_u32(&sm.pv_done[t]), (stages - 1) & 1)) failed = true;
     tcgen05_after_sync();
     failed = __any_sync(0xffffffffu, failed);
     if (!failed && stages > 0) {
       // 64 output columns at a time through the warp's share of the tile's query operand, which nothing reads any more
       unsigned char* staging = &sm.q[t][0][0] + (warp & 3) * 4096;
-      const int warp_count = min(max(count[t] - warp_row, 0), 32);
-      const float inv = softmax_scale(m, l, a.sink == nullptr ? -INFINITY : 1.4426950408889634f * a.sink[head]);
-      const int64_t first_out = static_cast<int64_t>(tile.q_row) + t * kRows + warp_row;
+      const float inv = head_gate * softmax_scale(m, l, a.sink == nullptr ? -INFINITY : 1.4426950408889634f * a.sink[head]);
       __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + first_out * a.out_stride + static_cast<int64_t>(head) * a.vdim;
-      const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(a.gate) + first_out * a.gate_stride + static_cast<int64_t>(head) * (a.gate_per_head ? 1 : a.vdim);
 #pragma unroll
       for (int b = 0; b < kV; ++b) {
         uint32_t r0[32], r1[32];
@@ -308,10 +310,11 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_con
           const int r = 4 * i + (lane >> 3);
           if (r < warp_count && b * 64 + (lane & 7) * 8 < a.vdim) {
             uint4 piece = *reinterpret_cast<const uint4*>(staging + r * 128 + (((lane & 7) ^ (r & 7)) << 4));
-            if (a.gate != nullptr) piece = gated(piece, gate + r * a.gate_stride, b * 64 + (lane & 7) * 8, a.gate_per_head);
+            if (gate_elements) piece = gated(piece, gates[i]);
             reinterpret_cast<uint4*>(dst + r * a.out_stride + b * 64)[lane & 7] = piece;
           }
         }
+        if (gate_elements && b + 1 < kV) load_gates(b + 1);
         __syncwarp();
       }
     }

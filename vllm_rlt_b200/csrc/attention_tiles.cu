@@ -72,19 +72,31 @@ attention_tiles_kernel(AttentionArgs a, float scale_log2, int splits, float* par
   const T* key_head = static_cast<const T*>(a.key_cache) + static_cast<int64_t>(kv_head) * a.head_dim;
   const T* value_head = static_cast<const T*>(a.value_cache) + static_cast<int64_t>(kv_head) * a.value_dim;
 
+  // keys that certainly share a page, counted from a stage's first (a multiple of kKeys): one table lookup for all of them
+  const int together = a.block_size % kKeys == 0 ? kKeys : (a.block_size % 16 == 0 ? 16 : 1);
   auto load_stage = [&](int j) {
-    constexpr int kPieces = kD / 8;
-    for (int i = threadIdx.x; i < kKeys * kPieces; i += kThreads) {
-      const int r = i / kPieces, c = (i % kPieces) * 8;
-      const int pos = key_begin + j * kKeys + r;
-      int64_t page = -1;
-      if (pos < key_end) page = table[pos / a.block_size];
-      const bool live = page >= 0 && page < a.num_blocks;   // a corrupt table entry is never dereferenced
-      const int offset = pos % a.block_size;
-      const T* ks = live && c < a.head_dim ? key_head + page * a.block_stride + offset * a.token_stride + c : key_head;
-      const T* vs = live && c < a.value_dim ? value_head + page * a.v_block_stride + offset * a.v_token_stride + c : value_head;
-      copy16(smem_u32(&sm.k[j & 1][r][c]), ks, live && c < a.head_dim);
-      copy16(smem_u32(&sm.v[j & 1][r][c]), vs, live && c < a.value_dim);
+    constexpr int kPieces = kD / 8, kStep = kThreads / kPieces;        // a thread copies the same columns of every kStep-th key
+    const int r0 = threadIdx.x / kPieces, c = (threadIdx.x % kPieces) * 8, first = key_begin + j * kKeys + r0;
+    const bool has_k = c < a.head_dim, has_v = c < a.value_dim;
+    const T *ks = key_head, *vs = value_head;
+    bool live = false;
+#pragma unroll
+    for (int i = 0; i < kKeys / kStep; ++i) {
+      const int r = r0 + i * kStep, pos = first + i * kStep;
+      if (i == 0 || together == 1 || (together == 16 && (i * kStep) % 16 == 0)) {
+        int64_t page = -1;
+        const int page_index = pos / a.block_size, offset = pos - page_index * a.block_size;
+        if (pos < key_end) page = table[page_index];
+        live = page >= 0 && page < a.num_blocks;   // a corrupt table entry is never dereferenced
+        ks = live ? key_head + page * a.block_stride + offset * a.token_stride + c : key_head;
+        vs = live ? value_head + page * a.v_block_stride + offset * a.v_token_stride + c : value_head;
+      } else {
+        ks += kStep * a.token_stride;
+        vs += kStep * a.v_token_stride;
+      }
+      const bool valid = live && pos < key_end;
+      copy16(smem_u32(&sm.k[j & 1][r][c]), valid && has_k ? ks : key_head, valid && has_k);
+      copy16(smem_u32(&sm.v[j & 1][r][c]), valid && has_v ? vs : value_head, valid && has_v);
     }
     copy_commit();
   };

@@ -4,8 +4,8 @@
 //
 //   y_t = sum_j w[:, j] u_(t - taps + 1 + j),   q, k: y / sqrt(mean over the head of y^2 + eps)
 //
-// One warp per (head, up to 32 tokens of a portion); a lane keeps its channels' last inputs in registers.  Inputs before a portion's
-// first token come from the sequence's state slot (zeros where the portion starts the sequence).  Only the first tile of a portion
+// A group of lanes takes one head and up to 32 tokens of a portion, and keeps its channels' last inputs in registers.  Inputs before a
+// portion's first token come from the sequence's state slot (zeros where the portion starts the sequence).  Only the first tile of a portion
 // reads the slot, and the same threads write the new one, each for its own channels, after they have read it.
 #include <math.h>
 
@@ -21,7 +21,7 @@ constexpr int kMaxTaps = kTile + 1;
 struct ConvHeadsArgs {
   const void* proj; int64_t proj_stride;
   int q_col, k_col, v_col, q_heads, kv_heads, key_dim, value_dim;
-  const float* weight; int taps;                 // [channels][taps], channels of q, k, v in this order
+  const float* weight; int taps;                 // [taps][channels], channels of q, k, v in this order
   int unit_norm; float eps;
   void* state; int64_t slots;                    // [slots][taps - 1][channels]
   void* q_out; int64_t q_out_stride;
@@ -32,143 +32,204 @@ struct ConvHeadsArgs {
   const int32_t* cu; const int32_t* starts; const int32_t* lengths; const int32_t* slot_of;
 };
 
-// A lane owns kChunks groups of kVec neighbouring channels of a head.  kTaps 4: up to four taps, inputs in registers; 0: any number of
-// taps, inputs re-read (from L1) for every output.
-template <typename T, int kTaps, int kVec, int kChunks>
-__global__ void __launch_bounds__(kThreads)
+// Where a head of q, k or v lies.
+struct HeadPlace {
+  bool is_q, is_v;
+  int index, dim, column, channel;               // among its kind; first column of the projection, first channel of weight and state
+};
+
+__device__ __forceinline__ HeadPlace place_of(const ConvHeadsArgs& a, int head) {
+  HeadPlace p;
+  p.is_q = head < a.q_heads;
+  p.is_v = head >= a.q_heads + a.kv_heads;
+  p.index = p.is_q ? head : (p.is_v ? head - a.q_heads - a.kv_heads : head - a.q_heads);
+  p.dim = p.is_v ? a.value_dim : a.key_dim;
+  p.column = (p.is_q ? a.q_col : (p.is_v ? a.v_col : a.k_col)) + p.index * p.dim;
+  p.channel = p.index * p.dim + (p.is_q ? 0 : (p.is_v ? (a.q_heads + a.kv_heads) * a.key_dim : a.q_heads * a.key_dim));
+  return p;
+}
+
+__device__ __forceinline__ int channels_of(const ConvHeadsArgs& a) { return (a.q_heads + a.kv_heads) * a.key_dim + a.kv_heads * a.value_dim; }
+
+// Where the heads of consecutive tokens go: rows of q_out, or slots of the sequence's pages, looked up once per page.
+template <typename T>
+struct Destination {
+  const ConvHeadsArgs& a;
+  const HeadPlace& p;
+  int seq, row, position, offset;
+  T* base;                                       // q: the first row; k, v: the current page, or null where nothing is to be written
+  bool padding;
+
+  __device__ __forceinline__ Destination(const ConvHeadsArgs& args, const HeadPlace& place, int sequence, int first_row, int first_position)
+      : a(args), p(place), seq(sequence), row(first_row), position(first_position), offset(0), base(nullptr), padding(args.lengths[sequence] <= 0) {
+    if (p.is_q) base = static_cast<T*>(a.q_out) + row * a.q_out_stride + static_cast<int64_t>(p.index) * p.dim;
+    else look_up();
+  }
+  __device__ __forceinline__ void look_up() {
+    const int page_index = position / a.block_size;
+    offset = position - page_index * a.block_size;
+    base = nullptr;
+    if (padding || position < 0 || page_index >= a.table_width) return;
+    const int64_t page = a.tables[static_cast<int64_t>(seq) * a.table_width + page_index];
+    if (page < 0 || page >= a.num_blocks) return;
+    base = (p.is_v ? static_cast<T*>(a.value_cache) + page * a.v_block_stride : static_cast<T*>(a.key_cache) + page * a.k_block_stride) +
+           static_cast<int64_t>(p.index) * p.dim;
+  }
+  __device__ __forceinline__ T* next() {         // of the next token
+    if (p.is_q) {
+      T* dst = base;
+      base += a.q_out_stride;
+      return dst;
+    }
+    if (offset == a.block_size) look_up();
+    T* dst = base == nullptr ? nullptr : base + offset * (p.is_v ? a.v_token_stride : a.k_token_stride);
+    ++offset;
+    ++position;
+    return dst;
+  }
+};
+
+// Up to four taps (fewer: the missing ones are leading zeros).  kLanes lanes take a head, 16 bytes each.
+template <typename T, int kLanes>
+__global__ void __launch_bounds__(kThreads, 4)
 conv_heads_kernel(ConvHeadsArgs a) {
-  struct alignas(sizeof(T) * kVec) Vec { T e[kVec]; };
+  constexpr int kTaps = 4, kVec = static_cast<int>(16 / sizeof(T)), kAhead = 4;
+  struct alignas(16) Vec { T e[kVec]; };
+  const int lane = threadIdx.x % kLanes, head = blockIdx.x * (kThreads / kLanes) + threadIdx.x / kLanes;
+  const int seq = blockIdx.z, first = blockIdx.y * kTile;
+  const int row0 = a.cu[seq], n = a.cu[seq + 1] - row0, start = a.starts[seq];
+  const int64_t slot = a.slot_of[seq];
+  if (first >= n) return;
+  const int at = lane * kVec;                                // first channel of the lane within its head
+  const bool alive = head < a.q_heads + 2 * a.kv_heads;      // the others stay for the shuffles
+  const HeadPlace p = place_of(a, alive ? head : 0);
+  const int dim = alive ? p.dim : 0, channels = channels_of(a), taps = a.taps, count = min(kTile, n - first);
+  const bool slot_ok = slot >= 0 && slot < a.slots, resumed = start > 0 && slot_ok, carries = first == 0 && slot_ok;
+  const T* in = static_cast<const T*>(a.proj) + static_cast<int64_t>(row0) * a.proj_stride + p.column;   // in[i * stride]: token i of the portion
+  T* state = static_cast<T*>(a.state) + slot * (taps - 1) * static_cast<int64_t>(channels) + p.channel;
+  auto zero = [] {
+    Vec z;
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) z.e[e] = Elem<T>::from_float(0.0f);
+    return z;
+  };
+  auto input = [&](int i, int d) {   // channels d .. of token i of the portion; negative: one of the taps - 1 inputs before it
+    if (i >= 0) return *reinterpret_cast<const Vec*>(in + i * a.proj_stride + d);
+    if (resumed && i + taps - 1 >= 0) return *reinterpret_cast<const Vec*>(state + static_cast<int64_t>(i + taps - 1) * channels + d);
+    return zero();
+  };
+  // all loads of the beginning together: the inputs before the tile, the weights, and what the state becomes; lanes behind the head hold zeros
+  Vec kept[kTaps - 1];
+  float w[kTaps][kVec], window[kTaps][kVec];
+  const int skip = kTaps - taps;
+#pragma unroll
+  for (int j = 0; j < kTaps; ++j)
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) w[j][e] = window[j][e] = 0.0f;
+  if (at < dim) {
+    Vec before[kTaps - 1];
+#pragma unroll
+    for (int j = 0; j + 1 < kTaps; ++j) before[j] = input(first - kTaps + 1 + j, at);
+#pragma unroll
+    for (int k = 0; k + 1 < kTaps; ++k)
+      if (carries && k < taps - 1) kept[k] = input(n + k - taps + 1, at);
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j)
+      if (j >= skip) {
+#pragma unroll
+        for (int e = 0; e < kVec; e += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(a.weight + static_cast<int64_t>(j - skip) * channels + p.channel + at + e);
+          w[j][e] = x.x; w[j][e + 1] = x.y; w[j][e + 2] = x.z; w[j][e + 3] = x.w;
+        }
+      }
+#pragma unroll
+    for (int j = 0; j + 1 < kTaps; ++j)
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) window[j + 1][e] = Elem<T>::to_float(before[j].e[e]);
+  }
+  Destination<T> to(a, p, seq, row0 + first, start + first);
+  const bool normed = !p.is_v && a.unit_norm != 0;
+  const float share = 1.0f / static_cast<float>(p.dim);
+  in += first * a.proj_stride + at;
+  for (int base = 0; base < count; base += kAhead) {
+    Vec now[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      if (base + i < count && at < dim) now[i] = *reinterpret_cast<const Vec*>(in + i * a.proj_stride);
+      else now[i] = zero();
+    }
+    in += kAhead * a.proj_stride;
+    const int steps = min(kAhead, count - base);
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      if (i >= steps) break;
+      float y[kVec], ss = 0.0f;
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) {
+#pragma unroll
+        for (int j = 0; j + 1 < kTaps; ++j) window[j][e] = window[j + 1][e];
+        window[kTaps - 1][e] = Elem<T>::to_float(now[i].e[e]);
+        y[e] = 0.0f;
+#pragma unroll
+        for (int j = 0; j < kTaps; ++j) y[e] = fmaf(w[j][e], window[j][e], y[e]);
+        ss = fmaf(y[e], y[e], ss);
+      }
+      T* dst = to.next();
+#pragma unroll
+      for (int x = kLanes / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);   // a warp may hold heads of several kinds: all take part
+      const float r = normed ? rsqrtf(fmaf(ss, share, a.eps)) : 1.0f;
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) y[e] *= r;
+      if (at < dim && dst != nullptr) store_floats<T, kVec>(dst + at, y);
+    }
+  }
+  if (!carries) return;
+#pragma unroll
+  for (int k = 0; k + 1 < kTaps; ++k)
+    if (k < taps - 1 && at < dim) *reinterpret_cast<Vec*>(state + static_cast<int64_t>(k) * channels + at) = kept[k];
+}
+
+// Any number of taps and any head size: a warp per head, inputs re-read (from L1) for every output.
+template <typename T, int kPer>
+__global__ void __launch_bounds__(kThreads)
+conv_heads_any_kernel(ConvHeadsArgs a) {
   const int lane = threadIdx.x & 31, head = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
   const int seq = blockIdx.z, first = blockIdx.y * kTile;
   if (head >= a.q_heads + 2 * a.kv_heads) return;
   const int row0 = a.cu[seq], n = a.cu[seq + 1] - row0, start = a.starts[seq];
   if (first >= n) return;
+  const HeadPlace p = place_of(a, head);
   const int64_t slot = a.slot_of[seq];
-  const bool slot_ok = slot >= 0 && slot < a.slots, resumed = start > 0 && slot_ok, padding = a.lengths[seq] <= 0;
-  const int count = min(kTile, n - first);
-  const bool is_q = head < a.q_heads, is_v = head >= a.q_heads + a.kv_heads;
-  const int of_kind = is_q ? head : (is_v ? head - a.q_heads - a.kv_heads : head - a.q_heads);
-  const int dim = is_v ? a.value_dim : a.key_dim;
-  const int column = (is_q ? a.q_col : (is_v ? a.v_col : a.k_col)) + of_kind * dim;
-  const int channels = (a.q_heads + a.kv_heads) * a.key_dim + a.kv_heads * a.value_dim;
-  const int channel = of_kind * dim + (is_q ? 0 : (is_v ? (a.q_heads + a.kv_heads) * a.key_dim : a.q_heads * a.key_dim));
-  const int taps = a.taps;
-  const T* in = static_cast<const T*>(a.proj) + static_cast<int64_t>(row0) * a.proj_stride + column;   // in[i * stride]: token i of the portion
-  T* state = static_cast<T*>(a.state) + slot * (taps - 1) * static_cast<int64_t>(channels) + channel;
-  const float* weight = a.weight + static_cast<int64_t>(channel) * taps;
-  auto at = [&](int c) { return (c * 32 + lane) * kVec; };                       // first channel of the lane's chunk c, within the head
-  auto input = [&](int i, int d) {   // channels d .. of token i of the portion; negative: one of the taps - 1 inputs before it
-    if (i >= 0) return *reinterpret_cast<const Vec*>(in + i * a.proj_stride + d);
-    if (resumed && i + taps - 1 >= 0) return *reinterpret_cast<const Vec*>(state + static_cast<int64_t>(i + taps - 1) * channels + d);
-    Vec zero;
-#pragma unroll
-    for (int e = 0; e < kVec; ++e) zero.e[e] = Elem<T>::from_float(0.0f);
-    return zero;
+  const bool slot_ok = slot >= 0 && slot < a.slots, resumed = start > 0 && slot_ok;
+  const int channels = channels_of(a), taps = a.taps, last = min(first + kTile, n);
+  const T* in = static_cast<const T*>(a.proj) + static_cast<int64_t>(row0) * a.proj_stride + p.column;
+  T* state = static_cast<T*>(a.state) + slot * (taps - 1) * static_cast<int64_t>(channels) + p.channel;
+  auto input = [&](int i, int d) {
+    if (i >= 0) return in[i * a.proj_stride + d];
+    return resumed ? state[static_cast<int64_t>(i + taps - 1) * channels + d] : Elem<T>::from_float(0.0f);
   };
-  const int32_t* table = a.tables + static_cast<int64_t>(seq) * a.table_width;
-  // the token's head: normed and stored where it belongs
-  auto finish = [&](int i, float (&y)[kChunks][kVec]) {
-    if (!is_v && a.unit_norm != 0) {
-      float ss = 0.0f;
+  Destination<T> to(a, p, seq, row0 + first, start + first);
+  for (int i = first; i < last; ++i) {
+    float y[kPer], ss = 0.0f;
 #pragma unroll
-      for (int c = 0; c < kChunks; ++c)
-        if (at(c) < dim) {
-#pragma unroll
-          for (int e = 0; e < kVec; ++e) ss = fmaf(y[c][e], y[c][e], ss);
-        }
-#pragma unroll
-      for (int x = 16; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
-      const float r = 1.0f / sqrtf(ss / static_cast<float>(dim) + a.eps);
-#pragma unroll
-      for (int c = 0; c < kChunks; ++c)
-#pragma unroll
-        for (int e = 0; e < kVec; ++e) y[c][e] *= r;
+    for (int c = 0; c < kPer; ++c) {
+      const int d = c * 32 + lane;
+      y[c] = 0.0f;
+      if (d < p.dim)
+        for (int j = 0; j < taps; ++j) y[c] = fmaf(a.weight[static_cast<int64_t>(j) * channels + p.channel + d], Elem<T>::to_float(input(i - taps + 1 + j, d)), y[c]);
+      ss = fmaf(y[c], y[c], ss);
     }
-    T* dst = nullptr;
-    if (is_q) {
-      dst = static_cast<T*>(a.q_out) + static_cast<int64_t>(row0 + i) * a.q_out_stride + static_cast<int64_t>(head) * dim;
-    } else if (!padding) {
-      const int position = start + i, page_index = position / a.block_size;
-      const int64_t page = position >= 0 && page_index < a.table_width ? table[page_index] : -1;
-      if (page >= 0 && page < a.num_blocks) {
-        const int offset = position - page_index * a.block_size;
-        dst = (is_v ? static_cast<T*>(a.value_cache) + page * a.v_block_stride + offset * a.v_token_stride
-                    : static_cast<T*>(a.key_cache) + page * a.k_block_stride + offset * a.k_token_stride) + static_cast<int64_t>(of_kind) * dim;
-      }
-    }
-    if (dst == nullptr) return;
 #pragma unroll
-    for (int c = 0; c < kChunks; ++c)
-      if (at(c) < dim) store_floats<T, kVec>(dst + at(c), y[c]);
-  };
-  if constexpr (kTaps > 0) {
-    const int skip = kTaps - taps;               // missing taps are leading zeros
-    float w[kChunks][kVec][kTaps], window[kTaps][kChunks][kVec];
+    for (int x = 16; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    const float r = !p.is_v && a.unit_norm != 0 ? 1.0f / sqrtf(ss / static_cast<float>(p.dim) + a.eps) : 1.0f;
+    T* dst = to.next();
 #pragma unroll
-    for (int c = 0; c < kChunks; ++c)
-      if (at(c) < dim) {
-#pragma unroll
-        for (int e = 0; e < kVec; ++e)
-#pragma unroll
-          for (int j = 0; j < kTaps; ++j) w[c][e][j] = j >= skip ? weight[(at(c) + e) * taps + j - skip] : 0.0f;
-#pragma unroll
-        for (int j = 1; j < kTaps; ++j) {
-          Vec x = input(first - kTaps + j, at(c));
-#pragma unroll
-          for (int e = 0; e < kVec; ++e) window[j][c][e] = Elem<T>::to_float(x.e[e]);
-        }
-      }
-    constexpr int kAhead = kChunks == 1 ? 4 : 2;
-    Vec next[kAhead][kChunks];
-    for (int base = 0; base < count; base += kAhead) {
-#pragma unroll
-      for (int i = 0; i < kAhead; ++i)
-        if (base + i < count) {
-#pragma unroll
-          for (int c = 0; c < kChunks; ++c)
-            if (at(c) < dim) next[i][c] = *reinterpret_cast<const Vec*>(in + (first + base + i) * a.proj_stride + at(c));
-        }
-#pragma unroll
-      for (int i = 0; i < kAhead; ++i) {
-        if (base + i < count) {
-          float y[kChunks][kVec];
-#pragma unroll
-          for (int c = 0; c < kChunks; ++c)
-#pragma unroll
-            for (int e = 0; e < kVec; ++e) {
-#pragma unroll
-              for (int j = 0; j + 1 < kTaps; ++j) window[j][c][e] = window[j + 1][c][e];
-              window[kTaps - 1][c][e] = Elem<T>::to_float(next[i][c].e[e]);
-              y[c][e] = 0.0f;
-#pragma unroll
-              for (int j = 0; j < kTaps; ++j) y[c][e] = fmaf(w[c][e][j], window[j][c][e], y[c][e]);
-            }
-          finish(first + base + i, y);
-        }
-      }
-    }
-  } else {
-    for (int i = first; i < first + count; ++i) {
-      float y[kChunks][kVec];
-#pragma unroll
-      for (int c = 0; c < kChunks; ++c) {
-#pragma unroll
-        for (int e = 0; e < kVec; ++e) y[c][e] = 0.0f;
-        if (at(c) < dim)
-          for (int j = 0; j < taps; ++j) {
-            const Vec x = input(i - taps + 1 + j, at(c));
-#pragma unroll
-            for (int e = 0; e < kVec; ++e) y[c][e] = fmaf(weight[(at(c) + e) * taps + j], Elem<T>::to_float(x.e[e]), y[c][e]);
-          }
-      }
-      finish(i, y);
-    }
+    for (int c = 0; c < kPer; ++c)
+      if (c * 32 + lane < p.dim && dst != nullptr) dst[c * 32 + lane] = Elem<T>::from_float(y[c] * r);
   }
   if (first == 0 && slot_ok)   // ascending: entry k is written after every entry it is shifted from has been read
     for (int k = 0; k + 1 < taps; ++k)
-#pragma unroll
-      for (int c = 0; c < kChunks; ++c)
-        if (at(c) < dim) *reinterpret_cast<Vec*>(state + static_cast<int64_t>(k) * channels + at(c)) = input(n + k - taps + 1, at(c));
+      for (int d = lane; d < p.dim; d += 32) state[static_cast<int64_t>(k) * channels + d] = input(n + k - taps + 1, d);
 }
 
 }  // namespace
@@ -204,21 +265,23 @@ extern "C" RLT_API int rlt_conv_heads(const void* proj, int64_t proj_stride, int
   a.k_token_stride = k_token_stride; a.value_cache = value_cache; a.v_block_stride = v_block_stride; a.v_token_stride = v_token_stride;
   a.num_blocks = num_blocks; a.block_size = block_size; a.tables = tables; a.table_width = table_width; a.cu = cu_seqlens; a.starts = starts;
   a.lengths = lengths; a.slot_of = slot_of;
-  bool wide = taps <= 4 && widest <= 256;
+  const int vec = static_cast<int>(16 / dtype_size(dtype));
+  bool wide = taps <= 4 && widest <= 32 * vec && aligned16(weight);
   for (const int64_t x : {proj_stride, static_cast<int64_t>(q_col), static_cast<int64_t>(k_col), static_cast<int64_t>(v_col), static_cast<int64_t>(key_dim),
                           static_cast<int64_t>(value_dim), q_out_stride, k_block_stride, k_token_stride, v_block_stride, v_token_stride})
-    wide = wide && x % 4 == 0;
+    wide = wide && x % vec == 0;
   for (const void* p : {proj, static_cast<const void*>(state), static_cast<const void*>(q_out), static_cast<const void*>(key_cache), static_cast<const void*>(value_cache)})
     wide = wide && aligned16(p);
-  const int heads = q_heads + 2 * kv_heads;
-  const dim3 grid(static_cast<unsigned>((heads + kThreads / 32 - 1) / (kThreads / 32)), static_cast<unsigned>((max_tokens + kTile - 1) / kTile),
+  const int lanes = !wide || widest > 16 * vec ? 32 : (widest > 8 * vec ? 16 : 8), heads = q_heads + 2 * kv_heads, per_cta = kThreads / lanes;
+  const dim3 grid(static_cast<unsigned>((heads + per_cta - 1) / per_cta), static_cast<unsigned>((max_tokens + kTile - 1) / kTile),
                   static_cast<unsigned>(sequences));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   RLT_DISPATCH_DTYPE(dtype, T, {
-    if (wide && widest <= 128) conv_heads_kernel<T, 4, 4, 1><<<grid, kThreads, 0, s>>>(a);
-    else if (wide) conv_heads_kernel<T, 4, 4, 2><<<grid, kThreads, 0, s>>>(a);
-    else if (widest <= 256) conv_heads_kernel<T, 0, 1, 8><<<grid, kThreads, 0, s>>>(a);
-    else conv_heads_kernel<T, 0, 1, 20><<<grid, kThreads, 0, s>>>(a);
+    if (wide && lanes == 8) conv_heads_kernel<T, 8><<<grid, kThreads, 0, s>>>(a);
+    else if (wide && lanes == 16) conv_heads_kernel<T, 16><<<grid, kThreads, 0, s>>>(a);
+    else if (wide) conv_heads_kernel<T, 32><<<grid, kThreads, 0, s>>>(a);
+    else if (widest <= 256) conv_heads_any_kernel<T, 8><<<grid, kThreads, 0, s>>>(a);
+    else conv_heads_any_kernel<T, 20><<<grid, kThreads, 0, s>>>(a);
   });
   return launch_status("conv_heads_kernel");
 }

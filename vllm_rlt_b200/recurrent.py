@@ -48,17 +48,17 @@ def causal_conv(x, weight, bias, state, out, group, act=None):
 
 
 def conv_heads(proj, columns, weight, eps: float, state, q_out, key_cache, value_cache, group, *, unit_norm: bool = True):
-    """What stands between an attention layer's projections and its scores: `out[i, c] = sum_j weight[c, j] * x[i - taps + 1 + j, c]`
+    """What stands between an attention layer's projections and its scores: `out[i, c] = sum_j weight[j, c] * x[i - taps + 1 + j, c]`
     over the channels of q, k and v, with `unit_norm` q and k of every head divided by their root mean square, k and v into the pages of
     their positions, q into q_out.
 
-    proj `[rows, columns]` holds q, k and v from the three `columns` on; weight float32 `[channels, taps]` (channels in the order q, k, v);
+    proj `[rows, columns]` holds q, k and v from the three `columns` on; weight float32 `[taps, channels]` (channels in the order q, k, v);
     state `[slots, taps - 1, channels]` of proj's dtype, updated in place; q_out `[rows, heads, dim]`; the caches
     `[pages, block, kv_heads, dim]` views."""
     device = _capi.require_cuda(proj, weight, state, q_out, key_cache, value_cache, group.cu, group.starts, group.slots, group.lengths, group.tables)
     rows, heads, key_dim = q_out.shape
     kv_heads, value_dim = value_cache.shape[2], value_cache.shape[3]
-    channels, taps = weight.shape
+    taps, channels = weight.shape
     if proj.dim() != 2 or proj.shape[0] != rows or proj.stride(1) != 1 or proj.dtype not in _capi.DTYPE_CODES \
             or any(t.dtype != proj.dtype for t in (state, q_out, key_cache, value_cache)):
         raise ValueError("proj must be [rows, columns] with unit inner stride; state, q_out and caches of its dtype")
@@ -66,9 +66,9 @@ def conv_heads(proj, columns, weight, eps: float, state, q_out, key_cache, value
         raise ValueError("caches must be [pages, block, kv_heads, dim] with a contiguous tail, keys as wide as queries")
     widths = heads * key_dim, kv_heads * key_dim, kv_heads * value_dim
     if channels != sum(widths) or any(at + n > proj.shape[1] for at, n in zip(columns, widths)):
-        raise ValueError("weight needs a row per channel of q, k and v; their columns must lie in the projection")
+        raise ValueError("weight needs a column per channel of q, k and v; their columns must lie in the projection")
     if weight.dtype != torch.float32 or not weight.is_contiguous() or state.shape[1:] != (taps - 1, channels) or not state.is_contiguous():
-        raise ValueError("weight must be contiguous float32 [channels, taps], state contiguous [slots, taps - 1, channels]")
+        raise ValueError("weight must be contiguous float32 [taps, channels], state contiguous [slots, taps - 1, channels]")
     if q_out.stride(2) != 1 or q_out.stride(1) != key_dim:
         raise ValueError("q_out must be [rows, heads, dim] with heads side by side")
     if group.sequences == 0:

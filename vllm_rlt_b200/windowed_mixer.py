@@ -78,7 +78,7 @@ class WindowedAttention:
         self.bias = torch.zeros(total, dtype=self.w_in.dtype, device=self.w_in.device)
         for name, at in zip(names, self.columns):
             self.bias[at:at + m.projections[name]] = take(f"{prefix}{name}.b")
-        self.conv = torch.cat([take(f"{prefix}{name}.conv", torch.float32) for name in names])
+        self.conv = torch.cat([take(f"{prefix}{name}.conv", torch.float32) for name in names]).t().contiguous()
         self.w_o = take(prefix + "o")
         self.terms = ScoreTerms(m.scale, window=m.window)
 
