@@ -212,7 +212,7 @@ def test_attention_over_cache_rows_with_sinks(dtype, heads, rank, rot, window, p
                 assert float(got[:, h].abs().max()) < 1e-20
 
 
-def test_a_sink_counts_once_and_is_not_scaled():
+def test_the_scale_leaves_a_sink_alone():
     """One key of score zero: the sink's share is exp(sink) / (1 + exp(sink)), whatever the scale."""
     for scale in (1e-3, 1.0, 30.0):
         for context in (1, 16):                  # equal keys: their weights add

@@ -48,8 +48,8 @@ class ScoreTerms:
         score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
                 - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
 
-    over the keys j <= p, with `window` > 0 only those with p - j < window.  `sink` (float32 [H]): the softmax's denominator
-    has one more term, exp(sink[h]), which is not scaled and has neither key nor value.
+    over the keys j <= p, with `window` > 0 only those with p - j < window.  `sink` (float32 [H]): exp(sink[h]) joins the
+    softmax's denominator (`scale` leaves it alone), and nothing joins its numerator.
     """
 
     scale: float

@@ -11,7 +11,7 @@ namespace rlt {
 // the row's length minus one), query head h of H, key at position j:
 //   score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
 //           - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
-// With a sink the softmax's denominator has one more term, exp(sink[h]), which has no key and no value.
+// With a sink, exp(sink[h]) joins the softmax's denominator, and nothing joins its numerator.
 // The default is the plain 1 / sqrt(head_dim) of the looped models.
 struct ScoreTerms {
   float scale = 0.0f;        // 0: 1 / sqrt(head_dim)
