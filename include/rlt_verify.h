@@ -530,7 +530,9 @@ RLT_API int rlt_sandwich_norm(const void* x, const void* weight, const void* res
  *             - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
  * softmax over the visible keys, weighted sum of the values.  Keys and values may have different head
  * sizes and cache strides; query and output rows may be column slices (strides in elements).
- * window > 0: only keys with p - j < window.  sink (fp32 [q_heads], or null): one more term exp(sink_h) of the denominator.  value_cache may be key_cache with one KV head: a value is then the first value_dim
+ * then multiplied by head_scale[h] (fp32 [q_heads], or null), and with softcap > 0 bounded: softcap * tanh(score / softcap).
+ * all_values != 0: head h is applied to the values of every key/value head, out [rows][q_heads][kv_heads * value_dim].
+ * window > 0: only keys with p - j < window, or j < keep_first.  sink (fp32 [q_heads], or null): one more term exp(sink_h) of the denominator.  value_cache may be key_cache with one KV head: a value is then the first value_dim
  * elements of its key row.
  * context_lengths[s]: tokens of sequence s after this portion.  planned != 0: the workspace holds the
  * plan of rlt_verify_attention_plan for the same tables, lengths and packing (max_new <= 16 only). */
@@ -543,17 +545,20 @@ RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, void* out, int
                          int value_dim, int dtype, const int32_t* block_tables, int sequences, int table_width,
                          const int32_t* context_lengths, const int32_t* cu_seqlens_q, int rows, int max_new,
                          float scale, float temp_coef, int temp_every, int distance_bias, int window,
-                         const float* sink, int planned, void* workspace, size_t workspace_bytes, rlt_stream_t stream);
+                         const float* sink, int keep_first, float softcap, const float* head_scale, int all_values, int planned, void* workspace, size_t workspace_bytes, rlt_stream_t stream);
 
 /* The fp32 residual stream and the norm that opens a layer:
  *   r = tokens ? embed[tokens[i]] : residual[i];  r += delta[i];  residual[i] = r (store_residual != 0)
  *   out[row] = r / sqrt(mean(r^2) + eps) * (weight_offset + weight)
  * i = row_index ? row_index[row] : row.  delta, embed, out: `dtype`; residual, weight, delta_weight: fp32.
  * delta_weight (may be null): r += delta_scale * norm(delta[i]) * delta_weight instead, a norm of its own behind the sublayer.
+ * parts > 0: the delta is the sum over p of part_weights[i][p] * part_values[part_rows[i][p]], plus delta (which may be null).
+ * weight null: out[row] = r, as it is.
  * centred != 0: both norms subtract the mean first (layer norm), mean(.^2) is then the variance. */
 RLT_API int rlt_residual_norm(float* residual, const void* delta, const int64_t* tokens, const void* embed, int64_t vocab,
                       const int64_t* row_index, int store_residual, const float* weight, float weight_offset,
-                      const float* delta_weight, float delta_scale, int centred, void* out, int rows, int width, float eps,
+                      const float* delta_weight, float delta_scale, int centred, const void* part_values,
+                      const int32_t* part_rows, const float* part_weights, int parts, void* out, int rows, int width, float eps,
                       int dtype, rlt_stream_t stream);
 
 /* Columns of a stacked projection to where they are needed: k_width columns from k_col and v_width from v_col into
@@ -584,9 +589,9 @@ RLT_API int rlt_ssd_scan(const void* x, const void* b, const void* c, int64_t xb
                  int head_dim, int dtype, void* workspace, size_t workspace_bytes, rlt_stream_t stream);
 
 /* out = rmsnorm_parts(y * silu(z)) * weight: the row is normed in `parts` equal parts, each by its own root mean square.
- * gate_behind != 0: out = rmsnorm_parts(y) * weight * sigmoid(z). */
+ * gate 1: out = rmsnorm_parts(y) * weight * sigmoid(z), 2: with silu(z).  weight may be null (ones). */
 RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight,
-                   void* out, int64_t out_stride, int rows, int width, int parts, float eps, int gate_behind,
+                   void* out, int64_t out_stride, int rows, int width, int parts, float eps, int gate,
                    int dtype, rlt_stream_t stream);
 
 /* Linear attention with a constant decay per head: S_t = decay_h S_(t-1) + k_t v_t^T, out_t = S_t^T q_t.  q, k
@@ -623,10 +628,11 @@ RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, int q_col, i
                      void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks, int block_size, const int32_t* tables, int table_width,
                      const int32_t* row_seq, const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
 
-/* The same rotation of `dim` elements of every head, from src to dst (which may be one); strides in elements. */
+/* The same rotation of `dim` elements of every head, from src to dst (which may be one); strides in elements.  Heads from scaled_from on
+ * are multiplied by scale, all of their elements. */
 RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head, void* dst, int64_t dst_row,
                      int64_t dst_head, int heads, int dim, int rot_dims, const double* frequencies, int halves,
-                     float amplitude, const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
+                     float amplitude, float scale, int scaled_from, const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
 
 /* Cache rows of positions first[s] .. of every sequence s, packed: row cu[s] + i holds position first[s] + i. */
 RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks,
@@ -650,17 +656,18 @@ RLT_API int rlt_latent_prompt_attention(const void* q, int64_t q_stride, const v
                                 const float* sink, const void* gate, int64_t gate_stride, int gate_per_head, int dtype,
                                 void* workspace, rlt_stream_t stream);
 
-/* Mixture of experts.  route: s = softmax(logits) in fp32, the `top` largest of s + correction (null: none), weights =
+/* Mixture of experts.  route: s = softmax(logits + bias) in fp32 (bias null: none), the `top` largest of s + correction (null: of logits + bias), weights =
  * chosen s / (their sum + floor_sum); counts [experts] must be zero before.  gather: rows sorted by expert, and every
- * choice's place among them.  gemm: y = act(x W_e^T) over sorted rows (act 0: none); workspace: 256 bytes for an error word. */
-RLT_API int rlt_expert_route(const float* logits, int64_t logit_stride, const float* correction, int rows, int experts,
+ * choice's place among them.  gemm: y = act(x W_e^T) over sorted rows (act 0: none); paired != 0: rows 2i and 2i + 1 of W_e are a
+ * gate and what it multiplies, y [rows][out / 2] = act(gate) * up; workspace: 256 bytes for an error word. */
+RLT_API int rlt_expert_route(const float* logits, int64_t logit_stride, const float* bias, const float* correction, int rows, int experts,
                      int top, float floor_sum, int32_t* counts, int32_t* chosen, int32_t* rank, float* weights,
                      rlt_stream_t stream);
 RLT_API int rlt_expert_gather(const void* x, int64_t x_stride, const int32_t* counts, const int32_t* chosen,
                       const int32_t* rank, int rows, int top, int width, void* sorted, int32_t* places, int dtype,
                       rlt_stream_t stream);
 RLT_API int rlt_expert_gemm(const void* x, int64_t x_stride, const void* w, void* y, int64_t y_stride, const int32_t* counts,
-                    int rows, int experts, int in, int out, int act, int dtype, void* workspace, rlt_stream_t stream);
+                    int rows, int experts, int in, int out, int act, int paired, int dtype, void* workspace, rlt_stream_t stream);
 
 /* g = min(gate, limit), u = clamp(up, -limit, limit): out = g * sigmoid(slope * g) * (u + 1); gate at column 0, up at up_col. */
 RLT_API int rlt_clamped_glu(const void* gate_up, int64_t row_stride, int up_col, void* out, int64_t out_stride, int64_t rows,
@@ -689,6 +696,33 @@ RLT_API int rlt_conv_heads(const void* proj, int64_t proj_stride, int q_col, int
                    int64_t num_blocks, int block_size, const int32_t* tables, int table_width, const int32_t* cu_seqlens,
                    const int32_t* starts, const int32_t* lengths, const int32_t* slot_of, int sequences, int max_tokens,
                    int dtype, rlt_stream_t stream);
+
+/* The same without convolution: with weights (fp32 [key_dim], or null) q and k of every head divided by their root mean square times the weight,
+ * then their first rot_dims dimensions turned as in rlt_rotate_heads; k and v into the pages of (row_seq[row], positions[row]) — row_seq -1: a
+ * padding row, nothing is written to pages — and q into q_out. */
+RLT_API int rlt_norm_rotate(const void* proj, int64_t proj_stride, int q_col, int k_col, int v_col, int q_heads, int kv_heads, int key_dim,
+                    int value_dim, const float* q_weight, const float* k_weight, float eps, const double* frequencies, int rot_dims,
+                    int halves, const int32_t* row_seq, const int32_t* positions, void* q_out, int64_t q_out_stride, void* key_cache,
+                    int64_t k_block_stride, int64_t k_token_stride, void* value_cache, int64_t v_block_stride, int64_t v_token_stride,
+                    int64_t num_blocks, int block_size, const int32_t* tables, int table_width, int rows, int dtype, rlt_stream_t stream);
+
+/* out[h] = sum_g talk[h][g] y[g][h / (heads / kv_heads)]: y [rows][heads][kv_heads * dim] as all_values attention leaves it, talk fp32
+ * [heads][heads], out [rows][heads * dim]. */
+RLT_API int rlt_head_mix(const void* y, int64_t y_stride, const float* talk, void* out, int64_t out_stride, int rows, int heads, int kv_heads,
+                 int dim, int dtype, rlt_stream_t stream);
+
+/* The gated delta rule with a decay per head and key channel, state fp32 [slots][heads][dim][vdim], updated in place.  Per head, with k and q
+ * divided by sqrt(sum of squares + 1e-6), q also by sqrt(dim), g = exp(-exp(a_log) softplus(decay + dt_bias)) and beta sigmoid of its raw value:
+ *   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  out = S^T q
+ * q, k [rows][kv_heads * dim] and v [rows][heads * vdim] are column slices of rows of one stride; head h reads q and k of head
+ * h / (heads / kv_heads).  decay [rows][heads * dim], beta [rows][heads], dt_bias fp32 [heads * dim], a_log fp32 [heads].  Sequences and slots
+ * as in rlt_ssd_scan; rows: rows of all sequences together. */
+RLT_API size_t rlt_delta_scan_workspace_bytes(int sequences, int max_tokens, int rows, int heads, int dim, int vdim, int dtype);
+RLT_API int rlt_delta_scan(const void* q, const void* k, const void* v, int64_t qkv_stride, const void* decay, int64_t decay_stride,
+                   const void* beta, int64_t beta_stride, const float* dt_bias, const float* a_log, void* out, int64_t out_stride,
+                   float* state, int64_t slots, const int32_t* cu_seqlens, const int32_t* starts, const int32_t* slot_of, int sequences,
+                   int max_tokens, int rows, int heads, int kv_heads, int dim, int vdim, int dtype, void* workspace, size_t workspace_bytes,
+                   rlt_stream_t stream);
 
 #ifdef __cplusplus
 }

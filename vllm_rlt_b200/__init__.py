@@ -17,12 +17,14 @@ from .prefix_cache import PrefixIndex
 from .engine import Engine, StepEntry
 from .hybrid_lm import HybridLM, HybridLMConfig
 from .kv_cache import RollbackResult, finalize_tokens, kv_write, rollback
-from .experts import expert_gather, expert_gemm, expert_route
+from .experts import expert_gather, expert_gemm, expert_route, paired_rows
 from .latent import (YarnScaling, latent_gather, latent_prompt_attention, latent_prompt_supported, latent_write, packed_attention,
                      rotate_heads, rotation_frequencies)
-from .layers import block_epilogue, clamped_glu, gated_unit, head_gate, residual_norm, rope_kv_write, sandwich_norm, soft_cap, stream_mix
+from .layers import (block_epilogue, clamped_glu, gated_unit, head_gate, head_mix, norm_rotate, residual_norm, rope_kv_write, sandwich_norm,
+                     soft_cap, stream_mix)
 from .looped_lm import LoopedLM, LoopedLMConfig, seeded_state_dict
-from .recurrent import causal_conv, conv_heads, decay_scan, decay_table, gated_norm, ssd_scan
+from .postnorm_lm import PostNormLM, PostNormLMConfig
+from .recurrent import causal_conv, conv_heads, decay_scan, decay_table, delta_scan, gated_norm, ssd_scan
 from .registry import load_model, register_model, registered_architectures
 from .runner import (B200SpeculativeRunner, KVCacheManagerView, ModelRunnerOutput, Request, SamplingParams, ScheduledRequest,
                      SchedulerOutput, SpeculativeConfig, SpeculativeRoundTicket, SpeculativeStats)
@@ -47,4 +49,5 @@ __all__ = [
     "StreamLM", "StreamLMConfig", "clamped_glu", "decay_scan", "decay_table", "expert_gather", "expert_gemm", "expert_route",
     "latent_gather", "latent_prompt_attention", "latent_prompt_supported", "latent_write", "rotate_heads", "rotation_frequencies", "stream_mix",
     "SandwichLM", "SandwichLMConfig", "YarnScaling", "conv_heads", "gated_unit", "head_gate", "packed_attention", "soft_cap",
+    "PostNormLM", "PostNormLMConfig", "delta_scan", "head_mix", "norm_rotate", "paired_rows",
 ]

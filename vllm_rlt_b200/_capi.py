@@ -54,8 +54,8 @@ SIGNATURES = {
     "rlt_sandwich_norm": (_I, [_P, _P, _P, _P, _P, _P, _I, _I, _F, _I, _P]),
     "rlt_scored_attention_workspace_bytes": (_Z, [_I, _I, _I, _I, _I, _I, _I, _I, _I, _I]),
     "rlt_scored_attention": (_I, [_P, _L, _P, _L, _P, _L, _L, _P, _L, _L, _L, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _I, _I,
-                                  _F, _F, _I, _I, _I, _P, _I, _P, _Z, _P]),
-    "rlt_residual_norm": (_I, [_P, _P, _P, _P, _L, _P, _I, _P, _F, _P, _F, _I, _P, _I, _I, _F, _I, _P]),
+                                  _F, _F, _I, _I, _I, _P, _I, _F, _P, _I, _I, _P, _Z, _P]),
+    "rlt_residual_norm": (_I, [_P, _P, _P, _P, _L, _P, _I, _P, _F, _P, _F, _I, _P, _P, _P, _I, _P, _I, _I, _F, _I, _P]),
     "rlt_block_epilogue": (_I, [_P, _L, _I, _I, _I, _I, _P, _L, _L, _P, _L, _L, _L, _I, _P, _I, _P, _P, _I, _I, _I, _P, _L, _I,
                                 _I, _I, _P]),
     "rlt_causal_conv": (_I, [_P, _L, _P, _P, _P, _L, _P, _L, _I, _I, _P, _P, _P, _I, _I, _P, _P, _L, _I, _I, _I, _P]),
@@ -67,20 +67,25 @@ SIGNATURES = {
                             _I, _P]),
     "rlt_latent_write": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _I, _F, _P, _L, _P, _L, _L, _L, _I, _P, _I, _P, _P, _I, _I,
                               _P]),
-    "rlt_rotate_heads": (_I, [_P, _L, _L, _P, _L, _L, _I, _I, _I, _P, _I, _F, _P, _I, _I, _P]),
+    "rlt_rotate_heads": (_I, [_P, _L, _L, _P, _L, _L, _I, _I, _I, _P, _I, _F, _F, _I, _P, _I, _I, _P]),
     "rlt_latent_gather": (_I, [_P, _L, _L, _L, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _P]),
     "rlt_latent_prompt_supported": (_I, [_I, _I, _I, _I]),
     "rlt_latent_prompt_attention": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _I, _F, _I, _P, _P, _L, _I,
                                          _I, _P, _P]),
-    "rlt_expert_route": (_I, [_P, _L, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P]),
+    "rlt_expert_route": (_I, [_P, _L, _P, _P, _I, _I, _I, _F, _P, _P, _P, _P, _P]),
     "rlt_expert_gather": (_I, [_P, _L, _P, _P, _P, _I, _I, _I, _P, _P, _I, _P]),
-    "rlt_expert_gemm": (_I, [_P, _L, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _P, _P]),
+    "rlt_expert_gemm": (_I, [_P, _L, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P]),
     "rlt_clamped_glu": (_I, [_P, _L, _I, _P, _L, _L, _I, _F, _F, _I, _P]),
     "rlt_gated_unit": (_I, [_P, _L, _I, _P, _L, _L, _I, _I, _I, _P]),
     "rlt_head_gate": (_I, [_P, _L, _P, _L, _P, _L, _L, _I, _I, _I, _I, _P]),
     "rlt_soft_cap": (_I, [_P, _L, _F, _P]),
     "rlt_conv_heads": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P, _L, _P, _L, _P, _L, _L, _P, _L, _L, _L, _I, _P, _I, _P, _P,
                             _P, _P, _I, _I, _I, _P]),
+    "rlt_norm_rotate": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _P, _L, _P, _L, _L, _P, _L, _L, _L, _I, _P, _I,
+                             _I, _I, _P]),
+    "rlt_head_mix": (_I, [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P]),
+    "rlt_delta_scan_workspace_bytes": (_Z, [_I, _I, _I, _I, _I, _I, _I]),
+    "rlt_delta_scan": (_I, [_P, _P, _P, _L, _P, _L, _P, _L, _P, _P, _P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _Z, _P]),
     "rlt_rollback": (_I, [_P, _P, _I, _P, _I, _I, _I, _P, _P, _L, _P, _I, _P, _P, _P, _P, _P, _P]),
 }
 

@@ -48,7 +48,8 @@ class ScoreTerms:
         score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
                 - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
 
-    over the keys j <= p, with `window` > 0 only those with p - j < window.  `sink` (float32 [H]): exp(sink[h]) joins the
+    over the keys j <= p, with `window` > 0 only those with p - j < window or j < keep_first.  `head_scale` (float32 [H]) multiplies a
+    head's scores, and `softcap` > 0 then bounds them: softcap * tanh(score / softcap).  `sink` (float32 [H]): exp(sink[h]) joins the
     softmax's denominator (`scale` leaves it alone), and nothing joins its numerator.
     """
 
@@ -58,11 +59,14 @@ class ScoreTerms:
     distance_bias: bool = False
     window: int = 0
     sink: torch.Tensor | None = field(default=None, compare=False)
+    keep_first: int = 0
+    softcap: float = 0.0
+    head_scale: torch.Tensor | None = field(default=None, compare=False)
 
 
-def check_sink(sink, heads: int) -> None:
+def check_sink(sink, heads: int, name: str = "sink") -> None:
     if sink is not None and (sink.dtype != torch.float32 or sink.shape != (heads,) or not sink.is_contiguous()):
-        raise ValueError("sink must be contiguous float32 [heads]")
+        raise ValueError(f"{name} must be contiguous float32 [heads]")
 
 
 @dataclass
@@ -328,8 +332,9 @@ class B200PagedAttention:
         return out
 
     def scored(self, q, out, key_cache, value_cache, block_tables, context_lengths, cu_seqlens_q, max_new: int,
-               terms: ScoreTerms):
-        """Packed causal attention with score terms, into `out` (`rlt_scored_attention`).
+               terms: ScoreTerms, *, all_values: bool = False):
+        """Packed causal attention with score terms, into `out` (`rlt_scored_attention`).  `all_values`: every head is applied to the
+        values of every key/value head, and out is `[rows, heads, kv_heads * value_dim]` (what `head_mix` takes).
 
         q `[rows, heads, key_dim]` and out `[rows, heads, value_dim]` may be column slices of wider rows; the
         caches are `[pages, block, kv_heads, dim]` views with sizes and strides of their own.  One table row and
@@ -337,12 +342,12 @@ class B200PagedAttention:
         heads over 16-token pages in 16 bits run on the tiled kernels (portions of at most 16 tokens on the verify
         kernel, whose plan a `shared_plan` block reuses; longer ones on the prompt kernel), everything else on
         the shape-generic ones."""
-        device = _capi.require_cuda(q, out, key_cache, value_cache, block_tables, context_lengths, cu_seqlens_q, terms.sink)
+        device = _capi.require_cuda(q, out, key_cache, value_cache, block_tables, context_lengths, cu_seqlens_q, terms.sink, terms.head_scale)
         rows, heads, key_dim = q.shape
         if q.dtype not in _capi.DTYPE_CODES or any(t.dtype != q.dtype for t in (out, key_cache, value_cache)):
             raise ValueError("q, out and the caches must share a float32/float16/bfloat16 dtype")
         if key_cache.dim() != 4 or value_cache.dim() != 4 or key_cache.shape[:3] != value_cache.shape[:3] \
-                or key_cache.shape[3] != key_dim or out.shape != (rows, heads, value_cache.shape[3]):
+                or key_cache.shape[3] != key_dim or out.shape != (rows, heads, value_cache.shape[3] * (value_cache.shape[2] if all_values else 1)):
             raise ValueError("caches must be [pages, block, kv_heads, dim]; q and out [rows, heads, key_dim / value_dim]")
         for name, t in (("q", q), ("out", out)):
             if t.stride(2) != 1 or t.stride(1) != t.shape[2]:
@@ -357,6 +362,7 @@ class B200PagedAttention:
         if heads % key_cache.shape[2]:
             raise ValueError("query heads must be a positive multiple of KV heads")
         check_sink(terms.sink, heads)
+        check_sink(terms.head_scale, heads, "head_scale")
         if rows == 0:
             return out
         blocks, block, kv_heads, value_dim = value_cache.shape
@@ -369,7 +375,8 @@ class B200PagedAttention:
             # prompt calls have scratch of their own: a mixed step's plan for its short portions survives them
             workspace = self._workspace(device, stream.value or 0 if max_new <= 16 else ("prompt", stream.value or 0), nbytes)
             planned = False
-            tiled = max_new <= 16 and not terms.window and terms.sink is None and q.dtype != torch.float32 and key_dim == value_dim == 128 and block == 16
+            bounded = bool(all_values or terms.softcap or terms.keep_first or terms.head_scale is not None)
+            tiled = max_new <= 16 and not terms.window and terms.sink is None and not bounded and q.dtype != torch.float32 and key_dim == value_dim == 128 and block == 16
             versions = self._versions(block_tables, context_lengths, cu_seqlens_q) if self._sharing and tiled else None
             if versions is not None:
                 plan_key = (block_tables.data_ptr(), sequences, width, context_lengths.data_ptr(), cu_seqlens_q.data_ptr(), rows,
@@ -389,7 +396,8 @@ class B200PagedAttention:
                 key_cache.stride(1), _capi.ptr(value_cache), value_cache.stride(0), value_cache.stride(1), blocks, block, heads,
                 kv_heads, key_dim, value_dim, dtype, _capi.ptr(block_tables), sequences, width, _capi.ptr(context_lengths),
                 _capi.ptr(cu_seqlens_q), rows, int(max_new), float(terms.scale), float(terms.temp_coef), int(terms.temp_every),
-                int(terms.distance_bias), int(terms.window), _capi.ptr(terms.sink), int(planned), _capi.ptr(workspace), workspace.numel(), stream)
+                int(terms.distance_bias), int(terms.window), _capi.ptr(terms.sink), int(terms.keep_first), float(terms.softcap),
+                _capi.ptr(terms.head_scale), int(all_values), int(planned), _capi.ptr(workspace), workspace.numel(), stream)
         _capi.check(status, "scored_attention")
         return out
 

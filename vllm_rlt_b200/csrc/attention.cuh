@@ -11,6 +11,8 @@ namespace rlt {
 // the row's length minus one), query head h of H, key at position j:
 //   score = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
 //           - distance_bias * 2^(-8 (h + 1) / H) * (p - j)
+// With a soft cap the score then becomes softcap * tanh(score / softcap).  head_scale multiplies the score of head h in front of it.
+// A window's row sees the first keep_first keys too.
 // With a sink, exp(sink[h]) joins the softmax's denominator, and nothing joins its numerator.
 // The default is the plain 1 / sqrt(head_dim) of the looped models.
 struct ScoreTerms {
@@ -20,8 +22,13 @@ struct ScoreTerms {
   int distance_bias = 0;
   int window = 0;            // 0: all keys before the row, else the last `window` of them (the row's own included)
   const float* sink = nullptr;   // [q_heads], or none
+  int keep_first = 0;
+  float softcap = 0.0f;          // 0: no cap
+  const float* head_scale = nullptr;   // [q_heads], or none
+  int all_values = 0;            // a head is applied to the values of every key/value head: out [rows][q_heads][kv_heads * value_dim]
 
-  __host__ __device__ bool plain() const { return temp_coef == 0.0f && distance_bias == 0 && window == 0 && sink == nullptr; }
+  __host__ __device__ bool bounded() const { return keep_first > 0 || softcap > 0.0f || head_scale != nullptr || all_values != 0; }
+  __host__ __device__ bool plain() const { return temp_coef == 0.0f && distance_bias == 0 && window == 0 && sink == nullptr && !bounded(); }
 };
 
 struct AttentionArgs {

@@ -228,7 +228,8 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
                                             int value_dim, int dtype, const int32_t* block_tables, int sequences,
                                             int table_width, const int32_t* context_lengths, const int32_t* cu_seqlens_q,
                                             int rows, int max_new, float scale, float temp_coef, int temp_every,
-                                            int distance_bias, int window, const float* sink, int planned, void* workspace, size_t workspace_bytes,
+                                            int distance_bias, int window, const float* sink, int keep_first, float softcap,
+                                            const float* head_scale, int all_values, int planned, void* workspace, size_t workspace_bytes,
                                             rlt_stream_t stream) {
   using namespace rlt;
   AttentionArgs a;
@@ -240,16 +241,20 @@ extern "C" RLT_API int rlt_scored_attention(const void* q, int64_t q_stride, voi
   a.value_dim = value_dim; a.v_block_stride = v_block_stride; a.v_token_stride = v_token_stride;
   a.q_stride = q_stride; a.out_stride = out_stride;
   a.terms.scale = scale; a.terms.temp_coef = temp_coef; a.terms.temp_every = temp_every; a.terms.distance_bias = distance_bias;
-  a.terms.window = window; a.terms.sink = sink;
+  a.terms.window = window; a.terms.sink = sink; a.terms.keep_first = keep_first; a.terms.softcap = softcap; a.terms.head_scale = head_scale;
+  a.terms.all_values = all_values != 0;
+  RLT_REQUIRE(keep_first >= 0 && softcap >= 0.0f && kv_heads > 0, "scored_attention: keep_first and softcap must not be negative");
+  const int64_t out_width = static_cast<int64_t>(q_heads) * value_dim * (all_values != 0 ? kv_heads : 1);
   RLT_REQUIRE(value_dim > 0 && temp_every > 0 && window >= 0, "scored_attention: value_dim and temp_every must be positive, window not negative");
   RLT_REQUIRE(cu_seqlens_q != nullptr || rows == 0, "scored_attention: cu_seqlens_q is required");
   int status = check_args(a);
   if (status != RLT_OK || rows == 0) return status;
   RLT_REQUIRE(v_token_stride >= static_cast<int64_t>(kv_heads) * value_dim && v_block_stride >= v_token_stride * block_size,
               "scored_attention: the [kv_heads, value_dim] tail of the value cache must be contiguous");
-  RLT_REQUIRE(q_stride >= static_cast<int64_t>(q_heads) * key_dim && out_stride >= static_cast<int64_t>(q_heads) * value_dim,
+  RLT_REQUIRE(q_stride >= static_cast<int64_t>(q_heads) * key_dim && out_stride >= out_width,
               "scored_attention: row strides smaller than a row");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (a.terms.bounded()) return launch_attention_generic(a, s);
   if (attention_latent_supported(a, max_new)) {
     status = launch_attention_latent(a, max_new, workspace, workspace_bytes, s);
     if (status != RLT_ERR_UNSUPPORTED) return status;

@@ -4,7 +4,8 @@
 // result depends on nothing but its own query, length and K/V.  This is the path for
 // shapes the tiled sm_100a kernel (attention_sm100.cu) does not cover — the fp32 tiny
 // model and the odd head sizes the reference's tests use; it reads K/V once per row.
-// With terms.window > 0 a row attends only its last `window` keys (sliding-window layers).
+// With terms.window > 0 a row attends only its last `window` keys (sliding-window layers) and the first `keep_first`.
+// With terms.all_values blockIdx.y is the key/value head whose values the row's weights are applied to.
 #include <math.h>
 
 #include "attention.cuh"
@@ -23,7 +24,8 @@ attention_generic_kernel(AttentionArgs a, float scale) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int D = a.head_dim, DV = a.value_dim;
   const T* q = static_cast<const T*>(a.q) + row * a.q_stride + static_cast<int64_t>(head) * D;
-  T* out = static_cast<T*>(a.out) + row * a.out_stride + static_cast<int64_t>(head) * DV;
+  const int kv_head = head / (a.q_heads / a.kv_heads), v_head = a.terms.all_values ? static_cast<int>(blockIdx.y) : kv_head;
+  T* out = static_cast<T*>(a.out) + row * a.out_stride + static_cast<int64_t>(a.terms.all_values ? head * a.kv_heads + v_head : head) * DV;
 
   int table_row, len;
   resolve_row(a, row, &table_row, &len);
@@ -32,7 +34,6 @@ attention_generic_kernel(AttentionArgs a, float scale) {
     return;
   }
   const int32_t* table = a.block_tables + static_cast<int64_t>(table_row) * a.table_width;
-  const int kv_head = head / (a.q_heads / a.kv_heads);
   const T* kc = static_cast<const T*>(a.key_cache);
   const T* vc = static_cast<const T*>(a.value_cache);
 
@@ -43,16 +44,18 @@ attention_generic_kernel(AttentionArgs a, float scale) {
     qr[j] = d < D ? Elem<T>::to_float(q[d]) : 0.0f;
     o[j] = 0.0f;
   }
-  const float row_scale = scale * query_temperature(a.terms, len), slope = distance_slope(a.terms, head, a.q_heads);
+  const float row_scale = scale * query_temperature(a.terms, len) * (a.terms.head_scale != nullptr ? a.terms.head_scale[head] : 1.0f), slope = distance_slope(a.terms, head, a.q_heads);
   float m = -INFINITY, l = 0.0f;
   const int first = window > 0 && len > window ? len - window : 0;
-  for (int t = first + warp; t < len; t += kWarps) {
+  const int kept = min(a.terms.keep_first, first);           // keys 0 .. kept - 1, then first ..
+  for (int i = warp; i < kept + len - first; i += kWarps) {
+    const int t = i < kept ? i : first + i - kept;
     const int64_t page = table[t / a.block_size];
     if (page < 0 || page >= a.num_blocks) continue;  // corrupt table entry: never dereferenced
     const int64_t base = page * a.block_stride + static_cast<int64_t>(t % a.block_size) * a.token_stride +
                          static_cast<int64_t>(kv_head) * D;
     const int64_t v_base = page * a.v_block_stride + static_cast<int64_t>(t % a.block_size) * a.v_token_stride +
-                           static_cast<int64_t>(kv_head) * DV;
+                           static_cast<int64_t>(v_head) * DV;
     float s = 0.0f;
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) {
@@ -62,6 +65,7 @@ attention_generic_kernel(AttentionArgs a, float scale) {
 #pragma unroll
     for (int x = 16; x > 0; x >>= 1) s += __shfl_xor_sync(0xffffffffu, s, x);
     s = fmaf(s, row_scale, -slope * static_cast<float>(len - 1 - t));
+    if (a.terms.softcap > 0.0f) s = a.terms.softcap * tanhf(s / a.terms.softcap);
     const float m_new = fmaxf(m, s);
     const float alpha = m == -INFINITY ? 0.0f : expf(m - m_new);
     const float p = expf(s - m_new);
@@ -112,9 +116,10 @@ int launch_attention_generic(const AttentionArgs& a, cudaStream_t stream) {
     return RLT_ERR_INVALID;
   }
   const float scale = score_scale(a);
+  const dim3 grid(static_cast<unsigned>(ctas), a.terms.all_values ? static_cast<unsigned>(a.kv_heads) : 1u);
   RLT_DISPATCH_DTYPE(a.dtype, T, {
-    if (widest <= 256) attention_generic_kernel<T, 8><<<static_cast<unsigned>(ctas), kThreads, 0, stream>>>(a, scale);
-    else attention_generic_kernel<T, 20><<<static_cast<unsigned>(ctas), kThreads, 0, stream>>>(a, scale);
+    if (widest <= 256) attention_generic_kernel<T, 8><<<grid, kThreads, 0, stream>>>(a, scale);
+    else attention_generic_kernel<T, 20><<<grid, kThreads, 0, stream>>>(a, scale);
   });
   return launch_status("attention_generic_kernel");
 }

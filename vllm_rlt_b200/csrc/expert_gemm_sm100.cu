@@ -8,7 +8,8 @@
 //   warp 0      TMA: 64 columns of the weight tile and of the token tile per stage, several stages ahead
 //   warp 1      tcgen05.mma into one of two accumulators in tensor memory (N = the tile's rows, rounded up to 16)
 //   warps 2..5  the other accumulator: activation, and the transpose on the way out — lane = output, column = token, so
-//               neighbouring lanes trade halves of two columns and store pairs of outputs, 64 bytes per token and warp
+//               neighbouring lanes trade halves of two columns and store pairs of outputs, 64 bytes per token and warp; where a pair
+//               of outputs is a gate and what it multiplies, a lane stores their one result of its token
 // Tiles are dealt round-robin in the order expert, rows, outputs: CTAs that run together share token tiles and weights in L2.
 #include "experts.cuh"
 #include "sm100_primitives.cuh"
@@ -150,11 +151,22 @@ expert_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
       if (!__all_sync(0xffffffffu, mbar_wait(smem_u32(&sm.done[buffer]), parity))) { failed = true; break; }
       tcgen05_after_sync();
       const int pair = tile.output + quarter * 32 + (lane & ~1);   // this lane stores outputs pair, pair + 1 of every second token
-      __nv_bfloat16* y = static_cast<__nv_bfloat16*>(g.y) + static_cast<int64_t>(tile.row) * g.y_stride + pair;
+      __nv_bfloat16* y = static_cast<__nv_bfloat16*>(g.y) + static_cast<int64_t>(tile.row) * g.y_stride + (g.paired ? pair / 2 : pair);
       for (int c = 0; c < tile.count; c += 32) {
         uint32_t r[32];
         tmem_load32(rows + buffer * kTokens + c, r);
         tmem_load_wait();
+        if (g.paired) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            const uint32_t give = (lane & 1) ? r[i] : r[i + 1], keep = (lane & 1) ? r[i + 1] : r[i];
+            const float got = __uint_as_float(__shfl_xor_sync(0xffffffffu, give, 1)), mine = __uint_as_float(keep);
+            const float gate = (lane & 1) ? got : mine, up = (lane & 1) ? mine : got;
+            const int token = c + i + (lane & 1);
+            if (token < tile.count && pair < g.out) y[token * g.y_stride] = __float2bfloat16_rn(activate<__nv_bfloat16>(gate, g.act) * up);
+          }
+          continue;
+        }
         if (g.act == kActSquaredRelu) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {

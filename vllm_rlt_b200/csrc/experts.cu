@@ -1,11 +1,11 @@
 // Mixture of experts: every token uses `top` of many small feed-forward layers.
 //
-//   expert_route_kernel   one warp per token: softmax of the router's fp32 logits, the `top` largest of score +
-//                         correction, weights = the chosen scores over their sum, and the token's place in each chosen
+//   expert_route_kernel   one warp per token: softmax of the router's fp32 logits (and a bias), the `top` largest of score +
+//                         correction (without one: of the logits), weights = the chosen scores over their sum, and the token's place in each chosen
 //                         expert's queue (atomic counts, a CTA's rows together: the order inside an expert is arbitrary, and no result depends on it)
 //   expert_gather_kernel  copies each token's row behind the others of its experts: rows sorted by expert, expert e from
 //                         counts[0] + .. + counts[e - 1] on
-//   expert_gemm_*         y = act(x W_e^T) over the sorted rows, every expert its own weights; tcgen05 in 16 bits
+//   expert_gemm_*         y = act(x W_e^T), or with weight rows in pairs (gate, up) y = act(gate) up, over the sorted rows, every expert its own weights; tcgen05 in 16 bits
 //                         (expert_gemm_sm100.cu), the tile kernel below for 32 bits and shapes outside it
 //
 // The weighted sum over a token's experts is taken where it is added to the residual (stream_mix.cu).
@@ -23,7 +23,7 @@ constexpr int kRowsPerWarp = 8;         // at most: a CTA counts its rows in sha
 
 template <int kPerLane>
 __global__ void __launch_bounds__(kThreads)
-expert_route_kernel(const float* __restrict__ logits, int64_t logit_stride, const float* __restrict__ correction, int rows, int experts,
+expert_route_kernel(const float* __restrict__ logits, int64_t logit_stride, const float* __restrict__ bias, const float* __restrict__ correction, int rows, int experts,
                     int top, float floor_sum, int per_warp, int32_t* __restrict__ counts, int32_t* __restrict__ chosen, int32_t* __restrict__ rank,
                     float* __restrict__ weights) {
   __shared__ int queued[32 * kMaxPerLane];    // rows of this CTA per expert, then where they start in the expert's queue
@@ -42,7 +42,8 @@ expert_route_kernel(const float* __restrict__ logits, int64_t logit_stride, cons
 #pragma unroll
     for (int j = 0; j < kPerLane; ++j) {
       const int e = lane + 32 * j;
-      s[j] = e < experts ? z[e] : -INFINITY;
+      s[j] = e < experts ? z[e] + (bias != nullptr ? bias[e] : 0.0f) : -INFINITY;
+      choice[j] = s[j];
       m = fmaxf(m, s[j]);
     }
 #pragma unroll
@@ -59,7 +60,7 @@ expert_route_kernel(const float* __restrict__ logits, int64_t logit_stride, cons
     for (int j = 0; j < kPerLane; ++j) {
       const int e = lane + 32 * j;
       s[j] /= total;
-      choice[j] = e < experts ? s[j] + (correction != nullptr ? correction[e] : 0.0f) : -INFINITY;
+      if (correction != nullptr) choice[j] = e < experts ? s[j] + correction[e] : -INFINITY;
     }
     float mine = 0.0f, sum = 0.0f;        // the weight of choice `lane`, and of all
     int mine_expert = 0;
@@ -165,6 +166,13 @@ expert_gemm_simple_kernel(ExpertGemm g) {
     }
     __syncthreads();
   }
+  if (g.paired) {
+    T* y = static_cast<T*>(g.y) + (static_cast<int64_t>(first) + row0) * g.y_stride + out0 / 2;
+    for (int i = 0; i < 4; ++i)
+      for (int j = 0; j < 4; j += 2)
+        if (tr + i < live_rows && tc + j < live_out) y[(tr + i) * g.y_stride + (tc + j) / 2] = Elem<T>::from_float(activate<T>(acc[i][j], g.act) * acc[i][j + 1]);
+    return;
+  }
   T* y = static_cast<T*>(g.y) + (static_cast<int64_t>(first) + row0) * g.y_stride + out0;
   for (int i = 0; i < 4; ++i)
     for (int j = 0; j < 4; ++j)
@@ -175,7 +183,7 @@ expert_gemm_simple_kernel(ExpertGemm g) {
 }  // namespace
 }  // namespace rlt
 
-extern "C" RLT_API int rlt_expert_route(const float* logits, int64_t logit_stride, const float* correction, int rows, int experts, int top,
+extern "C" RLT_API int rlt_expert_route(const float* logits, int64_t logit_stride, const float* bias, const float* correction, int rows, int experts, int top,
                                         float floor_sum, int32_t* counts, int32_t* chosen, int32_t* rank, float* weights, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(rows >= 0 && experts > 0 && top > 0 && top <= experts && logit_stride >= experts, "expert_route: invalid shape");
@@ -188,7 +196,7 @@ extern "C" RLT_API int rlt_expert_route(const float* logits, int64_t logit_strid
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int per_warp = rows >= 4096 ? kRowsPerWarp : 1;
   const unsigned grid = static_cast<unsigned>((rows + kWarps * per_warp - 1) / (kWarps * per_warp));
-#define RLT_ROUTE(P) expert_route_kernel<P><<<grid, kThreads, 0, s>>>(logits, logit_stride, correction, rows, experts, top, floor_sum, per_warp, counts, chosen, rank, weights)
+#define RLT_ROUTE(P) expert_route_kernel<P><<<grid, kThreads, 0, s>>>(logits, logit_stride, bias, correction, rows, experts, top, floor_sum, per_warp, counts, chosen, rank, weights)
   if (experts <= 32) RLT_ROUTE(1);
   else if (experts <= 64) RLT_ROUTE(2);
   else if (experts <= 128) RLT_ROUTE(4);
@@ -220,16 +228,17 @@ extern "C" RLT_API int rlt_expert_gather(const void* x, int64_t x_stride, const 
 }
 
 extern "C" RLT_API int rlt_expert_gemm(const void* x, int64_t x_stride, const void* w, void* y, int64_t y_stride, const int32_t* counts, int rows,
-                                       int experts, int in, int out, int act, int dtype, void* workspace, rlt_stream_t stream) {
+                                       int experts, int in, int out, int act, int paired, int dtype, void* workspace, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "expert_gemm: dtype must be float32, float16 or bfloat16");
-  RLT_REQUIRE(rows >= 0 && experts > 0 && in > 0 && out > 0 && x_stride >= in && y_stride >= out, "expert_gemm: invalid shape");
+  RLT_REQUIRE(rows >= 0 && experts > 0 && in > 0 && out > 0 && x_stride >= in && y_stride >= (paired != 0 ? out / 2 : out), "expert_gemm: invalid shape");
+  RLT_REQUIRE(paired == 0 || (out % 2 == 0 && act != 0), "expert_gemm: pairs of a gate and a value need an activation");
   RLT_REQUIRE(act == 0 || act_valid(act), "expert_gemm: unknown activation");
   if (rows == 0) return RLT_OK;
   RLT_REQUIRE(x && w && y && counts, "expert_gemm: null pointer");
   ExpertGemm g;
   g.x = x; g.x_stride = x_stride; g.w = w; g.y = y; g.y_stride = y_stride; g.counts = counts; g.rows = rows; g.experts = experts;
-  g.in = in; g.out = out; g.act = act; g.dtype = dtype; g.error = static_cast<unsigned*>(workspace);
+  g.in = in; g.out = out; g.act = act; g.paired = paired != 0; g.dtype = dtype; g.error = static_cast<unsigned*>(workspace);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (expert_gemm_sm100_supported(g)) {
     const int status = launch_expert_gemm_sm100(g, s);

@@ -12,6 +12,7 @@ struct ExpertGemm {
   const int32_t* counts;                // rows of every expert
   int rows, experts, in, out;           // rows: their sum
   int act;                              // Activation of the result, 0: none
+  bool paired;                          // weight rows 2i and 2i + 1 are a gate and what it multiplies: y [rows, out / 2] = act(gate) up
   int dtype;
   unsigned* error;                      // set when a bounded wait gave up (tcgen05 kernel)
 };

@@ -3,7 +3,7 @@
 //
 //   latent_write_kernel   the stacked down projections of a row: the query latent normed into the next GEMM's operand,
 //                         the key/value latent normed and the key part rotated into the row's page
-//   rotate_heads_kernel   the rotated part of every query head, in place or into another operand
+//   rotate_heads_kernel   the rotated part of every head, in place or into another operand; the last heads may be scaled on the way
 //   latent_gather_kernel  the cache rows of a range of positions of every sequence, side by side: what a prompt expands
 //                         into keys and values
 //
@@ -134,7 +134,8 @@ latent_write_kernel(LatentArgs a, int rows, int parts) {
 template <typename T, int kVec, bool kHalves>
 __global__ void __launch_bounds__(kThreads)
 rotate_heads_kernel(const T* src, int64_t src_row, int64_t src_head, T* dst, int64_t dst_row, int64_t dst_head, int heads, int dim,
-                    int rot_dims, const double* __restrict__ frequencies, float amplitude, const int32_t* __restrict__ positions, int rows, int per_cta) {
+                    int rot_dims, const double* __restrict__ frequencies, float amplitude, float scale, int scaled_from, const int32_t* __restrict__ positions, int rows,
+                    int per_cta) {
   extern __shared__ float2 turns[];
   const int pairs = rot_dims / 2, first = blockIdx.x * per_cta, count = min(per_cta, rows - first);
   for (int i = threadIdx.x; i < count * pairs; i += kThreads)
@@ -147,6 +148,7 @@ rotate_heads_kernel(const T* src, int64_t src_row, int64_t src_head, T* dst, int
     const int r = i / per_row, rest = i - r * per_row, head = rest / pieces, piece = rest - head * pieces;
     const T* from = src + (first + r) * src_row + head * src_head;
     T* to = dst + (first + r) * dst_row + head * dst_head;
+    const float factor = head >= scaled_from ? scale : 1.0f;
     if (kHalves && piece < joint) {
       const int d = piece * kVec;
       float u[kVec], v[kVec];
@@ -156,8 +158,8 @@ rotate_heads_kernel(const T* src, int64_t src_row, int64_t src_head, T* dst, int
       for (int e = 0; e < kVec; ++e) {
         const float2 t = turns[r * pairs + d + e];
         const float x = u[e];
-        u[e] = x * t.x - v[e] * t.y;
-        v[e] = v[e] * t.x + x * t.y;
+        u[e] = (x * t.x - v[e] * t.y) * factor;
+        v[e] = (v[e] * t.x + x * t.y) * factor;
       }
       store_floats<T, kVec>(to + d, u);
       store_floats<T, kVec>(to + pairs + d, v);
@@ -181,6 +183,8 @@ rotate_heads_kernel(const T* src, int64_t src_row, int64_t src_head, T* dst, int
           v[e + 1] = v[e + 1] * t.x + u * t.y;
         }
     }
+#pragma unroll
+    for (int e = 0; e < kStep; ++e) v[e] *= factor;
     if constexpr (kVec > 1) {
       store_floats<T, kVec>(to + d, v);
     } else {
@@ -252,8 +256,8 @@ extern "C" RLT_API int rlt_latent_write(const void* proj, int64_t proj_stride, i
 }
 
 extern "C" RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head, void* dst, int64_t dst_row, int64_t dst_head,
-                                        int heads, int dim, int rot_dims, const double* frequencies, int halves, float amplitude, const int32_t* positions,
-                                        int rows, int dtype, rlt_stream_t stream) {
+                                        int heads, int dim, int rot_dims, const double* frequencies, int halves, float amplitude, float scale, int scaled_from,
+                                        const int32_t* positions, int rows, int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "rotate_heads: dtype must be float32, float16 or bfloat16");
   RLT_REQUIRE(rows >= 0 && heads > 0 && dim >= 0 && rot_dims >= 0 && rot_dims <= dim && rot_dims % 2 == 0 && rot_dims <= 4096, "rotate_heads: invalid shape");
@@ -268,7 +272,7 @@ extern "C" RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_
   const size_t smem = static_cast<size_t>(per_cta) * (rot_dims / 2) * sizeof(float2);
   const unsigned grid = static_cast<unsigned>((rows + per_cta - 1) / per_cta);
 #define RLT_LAUNCH(T, V, H) rotate_heads_kernel<T, V, H><<<grid, kThreads, smem, s>>>(static_cast<const T*>(src), src_row, src_head, static_cast<T*>(dst), dst_row, \
-                                                                                     dst_head, heads, dim, rot_dims, frequencies, amplitude, positions, rows, per_cta)
+                                                                                     dst_head, heads, dim, rot_dims, frequencies, amplitude, scale, scaled_from, positions, rows, per_cta)
   RLT_DISPATCH_DTYPE(dtype, T, {
     constexpr int kWide = static_cast<int>(16 / sizeof(T));
     if (halves != 0) { if (wide) RLT_LAUNCH(T, kWide, true); else RLT_LAUNCH(T, 1, true); }

@@ -4,11 +4,12 @@
 //
 //   residual_norm_kernel   residual += delta (or residual = embed[token]), h = rmsnorm(residual) * (offset + w):
 //                          the tail of one layer and the head of the next in one pass over the row; for models with a norm
-//                          on both sides of a sublayer residual += scale * norm(delta) * w', and layer norms for RMS norms
+//                          on both sides of a sublayer residual += scale * norm(delta) * w', and layer norms for RMS norms;
+//                          the weighted sum over a token's experts joins the delta here, and without w the row goes on as it is
 //   block_epilogue_kernel  columns of the stacked input projection: keys and values to their pages,
 //                          the feed-forward columns through their activation into the stacked output operand
 //   gated_norm_kernel      y * silu(z), RMS-normed in equal parts, into the stacked output operand; or y RMS-normed first
-//                          and gated by sigmoid(z) behind the norm
+//                          and gated by sigmoid(z) or silu(z) behind the norm; a warp per part where the parts are heads
 //
 // All three are streaming kernels: every input is read once and every output written once.  Sums, norms
 // and activations are fp32; only the stored operand of the next GEMM is rounded to the model dtype.
@@ -27,6 +28,7 @@ struct NormArgs {
   const int64_t* row_index; int store_residual;
   const float* weight; float weight_offset;
   const float* delta_weight; float delta_scale;   // null: delta is added as it is
+  const void* part_values; const int32_t* part_rows; const float* part_weights; int parts;   // delta += sum_p weights[p] values[rows[p]]
   int centred;
   void* out; int width; float eps;
 };
@@ -52,8 +54,25 @@ residual_norm_kernel(NormArgs a) {
     if (at(k) < width) {
       if (emb != nullptr) load_floats<T, kVec>(emb + at(k), v[k]);
       else load_floats<float, kVec>(res + at(k), v[k]);
-      if (a.delta != nullptr) load_floats<T, kVec>(static_cast<const T*>(a.delta) + source * width + at(k), d[k]);
+      if (a.delta != nullptr) {
+        load_floats<T, kVec>(static_cast<const T*>(a.delta) + source * width + at(k), d[k]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < kVec; ++e) d[k][e] = 0.0f;
+      }
     }
+  for (int p = 0; p < a.parts; ++p) {
+    const float w = a.part_weights[source * a.parts + p];
+    const T* part = static_cast<const T*>(a.part_values) + static_cast<int64_t>(a.part_rows[source * a.parts + p]) * width;
+#pragma unroll
+    for (int k = 0; k < kPer; ++k)
+      if (at(k) < width) {
+        float y[kVec];
+        load_floats<T, kVec>(part + at(k), y);
+#pragma unroll
+        for (int e = 0; e < kVec; ++e) d[k][e] = fmaf(w, y[e], d[k][e]);
+      }
+  }
   // the row minus its mean (`centred`), and 1 / sqrt(mean of squares + eps) of it; deviations from the mean, not differences of sums
   auto normalise = [&](float (&x)[kPer][kVec]) {
     float sum = 0.0f;
@@ -79,7 +98,7 @@ residual_norm_kernel(NormArgs a) {
       }
     return 1.0f / sqrtf(block_sum<kThreads>(sum, scratch) / static_cast<float>(width) + a.eps);
   };
-  if (a.delta != nullptr) {
+  if (a.delta != nullptr || a.parts > 0) {
     if (a.delta_weight != nullptr) {
       const float r = normalise(d) * a.delta_scale;
 #pragma unroll
@@ -101,8 +120,14 @@ residual_norm_kernel(NormArgs a) {
     for (int k = 0; k < kPer; ++k)
       if (at(k) < width) store_floats<float, kVec>(res + at(k), v[k]);
   }
-  const float r = normalise(v);
   T* out = static_cast<T*>(a.out) + static_cast<int64_t>(blockIdx.x) * width;
+  if (a.weight == nullptr) {
+#pragma unroll
+    for (int k = 0; k < kPer; ++k)
+      if (at(k) < width) store_floats<T, kVec>(out + at(k), v[k]);
+    return;
+  }
+  const float r = normalise(v);
 #pragma unroll
   for (int k = 0; k < kPer; ++k)
     if (at(k) < width) {
@@ -159,10 +184,15 @@ block_epilogue_kernel(EpilogueArgs a) {
   }
 }
 
+enum Gate { kGateInFront = 0, kSigmoidBehind = 1, kSiluBehind = 2 };
+
+template <typename T>
+__device__ __forceinline__ float gate_behind(float z, int gate) { return gate == kSiluBehind ? activate<T>(z, kActSilu) : sigmoid<T>(z); }
+
 template <typename T, int kVec, bool kGateBehind>
 __global__ void __launch_bounds__(kThreads)
 gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z, int64_t z_stride,
-                  const float* __restrict__ weight, T* __restrict__ out, int64_t out_stride, int part, float eps) {
+                  const float* __restrict__ weight, T* __restrict__ out, int64_t out_stride, int part, float eps, int gate) {
   extern __shared__ __align__(16) float row_values[];
   __shared__ float scratch[kThreads / 32];
   const int64_t row = blockIdx.x;
@@ -186,16 +216,68 @@ gated_norm_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict
   for (int i = threadIdx.x * kVec; i < part; i += kThreads * kVec) {   // each thread reads back what it staged itself
     float v[kVec], w[kVec];
     load_floats<float, kVec>(row_values + i, v);
-    load_floats<float, kVec>(weight + first + i, w);
+    if (weight != nullptr) {
+      load_floats<float, kVec>(weight + first + i, w);
+    } else {
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) w[e] = 1.0f;
+    }
 #pragma unroll
     for (int e = 0; e < kVec; ++e) v[e] *= r * w[e];
     if (kGateBehind) {
       float g[kVec];
       load_floats<T, kVec>(zr + i, g);
 #pragma unroll
-      for (int e = 0; e < kVec; ++e) v[e] *= sigmoid<T>(g[e]);
+      for (int e = 0; e < kVec; ++e) v[e] *= gate_behind<T>(g[e], gate);
     }
     store_floats<T, kVec>(dst + i, v);
+  }
+}
+
+// A warp per (row, part), kPer accesses of kVec elements per lane: parts as small as a head.
+template <typename T, int kVec, int kPer>
+__global__ void __launch_bounds__(kThreads)
+gated_norm_parts_kernel(const T* __restrict__ y, int64_t y_stride, const T* __restrict__ z, int64_t z_stride, const float* __restrict__ weight,
+                        T* __restrict__ out, int64_t out_stride, int64_t rows, int parts, int part, float eps, int gate) {
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * (kThreads / 32) + (threadIdx.x >> 5);
+  if (item >= rows * parts) return;
+  const int64_t row = item / parts;
+  const int first = static_cast<int>(item - row * parts) * part, lane = threadIdx.x & 31;
+  float v[kPer][kVec], g[kPer][kVec], ss = 0.0f;
+#pragma unroll
+  for (int k = 0; k < kPer; ++k) {
+    const int i = (k * 32 + lane) * kVec;
+    if (i < part) {
+      load_floats<T, kVec>(y + row * y_stride + first + i, v[k]);
+      load_floats<T, kVec>(z + row * z_stride + first + i, g[k]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) v[k][e] = g[k][e] = 0.0f;
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kPer; ++k)
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) {
+      if (gate == kGateInFront) v[k][e] *= silu(g[k][e]);
+      ss = fmaf(v[k][e], v[k][e], ss);
+    }
+#pragma unroll
+  for (int x = 16; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+  const float r = 1.0f / sqrtf(ss / static_cast<float>(part) + eps);
+#pragma unroll
+  for (int k = 0; k < kPer; ++k) {
+    const int i = (k * 32 + lane) * kVec;
+    if (i >= part) continue;
+    if (weight != nullptr) {
+      float w[kVec];
+      load_floats<float, kVec>(weight + first + i, w);
+#pragma unroll
+      for (int e = 0; e < kVec; ++e) v[k][e] *= w[e];
+    }
+#pragma unroll
+    for (int e = 0; e < kVec; ++e) v[k][e] *= gate == kGateInFront ? r : r * gate_behind<T>(g[k][e], gate);
+    store_floats<T, kVec>(out + row * out_stride + first + i, v[k]);
   }
 }
 
@@ -207,13 +289,15 @@ constexpr size_t kMaxRowBytes = 48u * 1024u;   // a staged row of fp32 values
 
 extern "C" RLT_API int rlt_residual_norm(float* residual, const void* delta, const int64_t* tokens, const void* embed,
                                          int64_t vocab, const int64_t* row_index, int store_residual, const float* weight,
-                                         float weight_offset, const float* delta_weight, float delta_scale, int centred, void* out,
+                                         float weight_offset, const float* delta_weight, float delta_scale, int centred,
+                                         const void* part_values, const int32_t* part_rows, const float* part_weights, int parts, void* out,
                                          int rows, int width, float eps, int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "residual_norm: dtype must be float32, float16 or bfloat16");
   RLT_REQUIRE(rows >= 0 && width > 0 && eps >= 0.0f, "residual_norm: invalid shape or eps");
   if (rows == 0) return RLT_OK;
-  RLT_REQUIRE(residual && weight && out, "residual_norm: null pointer");
+  RLT_REQUIRE(residual && out, "residual_norm: null pointer");
+  RLT_REQUIRE(parts == 0 || (parts > 0 && part_values && part_rows && part_weights), "residual_norm: parts need values, rows and weights");
   RLT_REQUIRE((tokens == nullptr) == (embed == nullptr) && (tokens == nullptr || vocab > 0), "residual_norm: tokens and embed go together");
   if (width > kMaxPer * kThreads * 4) {
     set_last_error_text("residual_norm: widths above 12288 are not supported");
@@ -222,10 +306,11 @@ extern "C" RLT_API int rlt_residual_norm(float* residual, const void* delta, con
   NormArgs a;
   a.residual = residual; a.delta = delta; a.tokens = tokens; a.embed = embed; a.vocab = vocab; a.row_index = row_index;
   a.store_residual = store_residual; a.weight = weight; a.weight_offset = weight_offset; a.delta_weight = delta_weight;
-  a.delta_scale = delta_scale; a.centred = centred; a.out = out; a.width = width; a.eps = eps;
+  a.delta_scale = delta_scale; a.centred = centred; a.part_values = part_values; a.part_rows = part_rows; a.part_weights = part_weights;
+  a.parts = parts; a.out = out; a.width = width; a.eps = eps;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const bool wide = width % 4 == 0 && aligned16(residual) && aligned16(weight) && aligned16(delta) && aligned16(embed) && aligned16(out) &&
-                    aligned16(delta_weight);
+                    aligned16(delta_weight) && aligned16(part_values);
   const int per = (width + kThreads * 4 - 1) / (kThreads * 4);
   RLT_DISPATCH_DTYPE(dtype, T, {
     if (!wide && per == 1) residual_norm_kernel<T, 1, 4><<<rows, kThreads, 0, s>>>(a);
@@ -286,29 +371,46 @@ extern "C" RLT_API int rlt_block_epilogue(const void* proj, int64_t proj_stride,
 }
 
 extern "C" RLT_API int rlt_gated_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight,
-                                      void* out, int64_t out_stride, int rows, int width, int parts, float eps, int gate_behind,
+                                      void* out, int64_t out_stride, int rows, int width, int parts, float eps, int gate,
                                       int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "gated_norm: dtype must be float32, float16 or bfloat16");
   RLT_REQUIRE(rows >= 0 && width > 0 && parts > 0 && width % parts == 0 && eps >= 0.0f, "gated_norm: the width must be a whole number of parts");
   if (rows == 0) return RLT_OK;
-  RLT_REQUIRE(y && z && weight && out, "gated_norm: null pointer");
+  RLT_REQUIRE(y && z && out, "gated_norm: null pointer");
+  RLT_REQUIRE(gate >= kGateInFront && gate <= kSiluBehind, "gated_norm: unknown gate");
   const int part = width / parts;
   const size_t smem = static_cast<size_t>(part) * sizeof(float);
   if (smem > kMaxRowBytes - 1024) {
     set_last_error_text("gated_norm: parts above 12032 elements are not supported");
     return RLT_ERR_UNSUPPORTED;
   }
+  RLT_REQUIRE(parts <= 65535, "gated_norm: too many parts");
   const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>(parts));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const size_t bytes = 4 * dtype_size(dtype);
   auto aligned = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
   const bool wide = part % 4 == 0 && y_stride % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 && aligned(y) && aligned(z) && aligned(out) && aligned16(weight);
+  const int64_t warps = static_cast<int64_t>(rows) * parts;
+  if (parts > 1 && part <= (wide ? 512 : 128) && warps <= 0x7fffffff) {
+    const unsigned ctas = static_cast<unsigned>((warps + kThreads / 32 - 1) / (kThreads / 32));
+#define RLT_LAUNCH(T, V, P)                                                                                                                  \
+  gated_norm_parts_kernel<T, V, P><<<ctas, kThreads, 0, s>>>(static_cast<const T*>(y), y_stride, static_cast<const T*>(z), z_stride, weight,  \
+      static_cast<T*>(out), out_stride, rows, parts, part, eps, gate)
+    RLT_DISPATCH_DTYPE(dtype, T, {
+      if (!wide) RLT_LAUNCH(T, 1, 4);
+      else if (part <= 128) RLT_LAUNCH(T, 4, 1);
+      else if (part <= 256) RLT_LAUNCH(T, 4, 2);
+      else RLT_LAUNCH(T, 4, 4);
+    });
+#undef RLT_LAUNCH
+    return launch_status("gated_norm_parts_kernel");
+  }
 #define RLT_LAUNCH(T, V, G)                                                                                               \
   gated_norm_kernel<T, V, G><<<grid, kThreads, smem, s>>>(static_cast<const T*>(y), y_stride, static_cast<const T*>(z),    \
-      z_stride, weight, static_cast<T*>(out), out_stride, part, eps)
+      z_stride, weight, static_cast<T*>(out), out_stride, part, eps, gate)
   RLT_DISPATCH_DTYPE(dtype, T, {
-    if (gate_behind) { if (wide) RLT_LAUNCH(T, 4, true); else RLT_LAUNCH(T, 1, true); }
+    if (gate != kGateInFront) { if (wide) RLT_LAUNCH(T, 4, true); else RLT_LAUNCH(T, 1, true); }
     else { if (wide) RLT_LAUNCH(T, 4, false); else RLT_LAUNCH(T, 1, false); }
   });
 #undef RLT_LAUNCH

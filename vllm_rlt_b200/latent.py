@@ -71,10 +71,10 @@ def latent_write(proj, q_col: int, kv_col: int, q_weight, kv_weight, eps: float,
     return q
 
 
-def rotate_heads(src, dst, frequencies, positions, *, halves: bool = False, amplitude: float = 1.0):
+def rotate_heads(src, dst, frequencies, positions, *, halves: bool = False, amplitude: float = 1.0, scale: float = 1.0, scaled_from: int = 0):
     """Pairs (2i, 2i + 1) of every head — with `halves` pairs (i, i + n) of n frequencies — turned by position * frequency_i and
     multiplied by `amplitude`; src and dst `[rows, heads, dim]` with any row and head strides (dst may be src); the dimensions
-    behind the turned ones are copied."""
+    behind the turned ones are copied.  Heads from `scaled_from` on are multiplied by `scale`, all of their elements."""
     _capi.require_cuda(src, dst, frequencies, positions)
     rows, heads, dim = src.shape
     if dst.shape != src.shape or dst.dtype != src.dtype or src.stride(2) != 1 or dst.stride(2) != 1 or src.dtype not in _capi.DTYPE_CODES:
@@ -86,7 +86,7 @@ def rotate_heads(src, dst, frequencies, positions, *, halves: bool = False, ampl
     with torch.cuda.device(src.device):
         code = _capi.load().rlt_rotate_heads(_capi.ptr(src), src.stride(0), src.stride(1), _capi.ptr(dst), dst.stride(0), dst.stride(1), heads,
                                              dim, 2 * frequencies.numel(), _capi.ptr(frequencies), int(halves), float(amplitude),
-                                             _capi.ptr(positions), rows, _capi.DTYPE_CODES[src.dtype], _capi.stream_of(src))
+                                             float(scale), int(scaled_from), _capi.ptr(positions), rows, _capi.DTYPE_CODES[src.dtype], _capi.stream_of(src))
     _capi.check(code, "rotate_heads")
     return dst
 

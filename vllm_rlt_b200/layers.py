@@ -105,24 +105,31 @@ ACTIVATIONS = {"gelu": 1, "gelu_tanh": 2, "silu": 3, "squared_relu": 4}      # g
 
 
 def residual_norm(residual, weight, eps: float, dtype, *, delta=None, tokens=None, embed=None, row_index=None,
-                  weight_offset: float = 0.0, store: bool = True, behind=None, centred: bool = False):
+                  weight_offset: float = 0.0, store: bool = True, behind=None, centred: bool = False, parts=None):
     """The 32-bit residual stream and the norm that opens a layer or sublayer, in one pass:
 
         r = embed[tokens] or residual;  r += delta;  residual <- r (with `store`)
         returns norm(r) * (weight_offset + weight), in `dtype`
 
     norm(r) = r / sqrt(mean(r^2) + eps), with `centred` (a layer norm) of r minus its mean.  behind = (weight, scale): the sublayer has a
-    norm behind it too, r += scale * norm(delta) * weight.  residual: float32 [rows, width], updated in place.  `row_index` (int64)
+    norm behind it too, r += scale * norm(delta) * weight.  parts = (values, rows, weights): the weighted sum of rows of
+    `values` (rows int32, weights float32, both `[rows, k]`: a token's experts) joins the delta.  weight None: r itself is returned.  residual: float32 [rows, width], updated in place.  `row_index` (int64)
     selects rows: the result has one row per entry, and the residual is not stored.  `weight`: float32 [width]
     (`weight_offset` 1 for weights stored around zero)."""
     delta_weight, delta_scale = behind if behind is not None else (None, 1.0)
-    _capi.require_cuda(residual, weight, delta, tokens, embed, row_index, delta_weight)
+    _capi.require_cuda(residual, weight, delta, tokens, embed, row_index, delta_weight, *(parts or ()))
     if residual.dim() != 2 or residual.dtype != torch.float32 or not residual.is_contiguous():
         raise ValueError("residual must be contiguous float32 [rows, width]")
     rows, width = residual.shape
-    if weight.dtype != torch.float32 or weight.shape != (width,) or not weight.is_contiguous():
+    if weight is not None and (weight.dtype != torch.float32 or weight.shape != (width,) or not weight.is_contiguous()):
         raise ValueError("weight must be contiguous float32 [width]")
-    if delta_weight is not None and (delta is None or delta_weight.dtype != torch.float32 or delta_weight.shape != (width,)
+    part_values, part_rows, part_weights = parts if parts is not None else (None, None, None)
+    k = 0 if parts is None else part_rows.shape[1]
+    if parts is not None and (part_values.dtype != dtype or part_values.dim() != 2 or part_values.shape[1] != width or not part_values.is_contiguous()
+                              or part_rows.dtype != torch.int32 or part_weights.dtype != torch.float32 or part_rows.shape != (rows, k)
+                              or part_weights.shape != (rows, k) or not part_rows.is_contiguous() or not part_weights.is_contiguous()):
+        raise ValueError("parts must be contiguous values [n, width] of the model dtype, int32 rows and float32 weights [rows, k]")
+    if delta_weight is not None and ((delta is None and parts is None) or delta_weight.dtype != torch.float32 or delta_weight.shape != (width,)
                                      or not delta_weight.is_contiguous()):
         raise ValueError("the norm behind a sublayer needs a delta and a contiguous float32 [width] weight")
     if dtype not in _capi.DTYPE_CODES:
@@ -149,7 +156,7 @@ def residual_norm(residual, weight, eps: float, dtype, *, delta=None, tokens=Non
         code = _capi.load().rlt_residual_norm(
             _capi.ptr(residual), _capi.ptr(delta), _capi.ptr(tokens), _capi.ptr(embed), 0 if embed is None else embed.shape[0],
             _capi.ptr(row_index), int(store), _capi.ptr(weight), float(weight_offset), _capi.ptr(delta_weight), float(delta_scale),
-            int(centred), _capi.ptr(out), count, width, float(eps), _capi.DTYPE_CODES[dtype], _capi.stream_of(residual))
+            int(centred), _capi.ptr(part_values), _capi.ptr(part_rows), _capi.ptr(part_weights), k, _capi.ptr(out), count, width, float(eps), _capi.DTYPE_CODES[dtype], _capi.stream_of(residual))
     _capi.check(code, "residual_norm")
     return out
 
@@ -316,6 +323,61 @@ def head_gate(y, gate, out=None):
         code = _capi.load().rlt_head_gate(_capi.ptr(y), y.stride(0), _capi.ptr(gate), gate.stride(0), _capi.ptr(out), out.stride(0), rows, heads,
                                           dim, int(per_head(gate, heads, dim)), _capi.DTYPE_CODES[y.dtype], _capi.stream_of(y))
     _capi.check(code, "head_gate")
+    return out
+
+
+def norm_rotate(proj, columns, q_weight, k_weight, eps: float, frequencies, q_out, key_cache, value_cache, batch, *, halves: bool = False):
+    """What stands between an attention layer's projections and its scores: q and k of every head divided by their root mean square times
+    their weight (float32 `[dim]`, None: no norm), their first dimensions turned by the position as in `rotate_heads`, k and v into the
+    pages of their positions, q into q_out.
+
+    proj `[rows, columns]` holds q, k and v from the three `columns` on; q_out `[rows, heads, dim]`; the caches `[pages, block, kv_heads, dim]`
+    views; frequencies float64 (an empty tensor: no rotation)."""
+    _capi.require_cuda(proj, q_weight, k_weight, frequencies, q_out, key_cache, value_cache, batch.row_seq, batch.positions)
+    rows, heads, key_dim = q_out.shape
+    kv_heads, value_dim = value_cache.shape[2], value_cache.shape[3]
+    if proj.dim() != 2 or proj.shape[0] != rows or proj.stride(1) != 1 or proj.dtype not in _capi.DTYPE_CODES \
+            or any(t.dtype != proj.dtype for t in (q_out, key_cache, value_cache)):
+        raise ValueError("proj must be [rows, columns] with unit inner stride; q_out and caches of its dtype")
+    if key_cache.shape != (*value_cache.shape[:3], key_dim) or any(c.stride(3) != 1 or c.stride(2) != c.shape[3] for c in (key_cache, value_cache)):
+        raise ValueError("caches must be [pages, block, kv_heads, dim] with a contiguous tail, keys as wide as queries")
+    if any(at + n > proj.shape[1] for at, n in zip(columns, (heads * key_dim, kv_heads * key_dim, kv_heads * value_dim))):
+        raise ValueError("q, k and v must lie in the projection")
+    for w in (q_weight, k_weight):
+        if w is not None and (w.dtype != torch.float32 or w.shape != (key_dim,) or not w.is_contiguous()):
+            raise ValueError("weights must be contiguous float32 [dim]")
+    if frequencies.dtype != torch.float64 or 2 * frequencies.numel() > key_dim or q_out.stride(2) != 1 or q_out.stride(1) != key_dim:
+        raise ValueError("frequencies must be float64 of at most dim / 2 pairs, q_out [rows, heads, dim] with heads side by side")
+    if rows == 0:
+        return q_out
+    tables = batch.tables[0]
+    with torch.cuda.device(proj.device):
+        code = _capi.load().rlt_norm_rotate(
+            _capi.ptr(proj), proj.stride(0), *columns, heads, kv_heads, key_dim, value_dim, _capi.ptr(q_weight), _capi.ptr(k_weight), float(eps),
+            _capi.ptr(frequencies), 2 * frequencies.numel(), int(halves), _capi.ptr(batch.row_seq), _capi.ptr(batch.positions), _capi.ptr(q_out),
+            q_out.stride(0), _capi.ptr(key_cache), key_cache.stride(0), key_cache.stride(1), _capi.ptr(value_cache), value_cache.stride(0),
+            value_cache.stride(1), key_cache.shape[0], key_cache.shape[1], _capi.ptr(tables), tables.shape[1], rows,
+            _capi.DTYPE_CODES[proj.dtype], _capi.stream_of(proj))
+    _capi.check(code, "norm_rotate")
+    return q_out
+
+
+def head_mix(y, talk, out, kv_heads: int):
+    """`out[:, h] = sum_g talk[h, g] * y[:, g, c(h)]`: y `[rows, heads, kv_heads * dim]` (every head over the values of every key/value head),
+    talk float32 `[heads, heads]`, out `[rows, heads, dim]`, c(h) = h // (heads // kv_heads)."""
+    _capi.require_cuda(y, talk, out)
+    rows, heads, dim = out.shape
+    if y.shape != (rows, heads, kv_heads * dim) or any(t.stride(2) != 1 or t.stride(1) != t.shape[2] for t in (y, out)) \
+            or y.dtype not in _capi.DTYPE_CODES or out.dtype != y.dtype:
+        raise ValueError("y must be [rows, heads, kv_heads * dim] and out [rows, heads, dim] of one dtype, heads side by side")
+    if talk.dtype != torch.float32 or talk.shape != (heads, heads) or not talk.is_contiguous() or heads % kv_heads:
+        raise ValueError("talk must be contiguous float32 [heads, heads], heads a multiple of kv_heads")
+    if rows == 0:
+        return out
+    with torch.cuda.device(y.device):
+        code = _capi.load().rlt_head_mix(_capi.ptr(y), y.stride(0), _capi.ptr(talk), _capi.ptr(out), out.stride(0), rows, heads, kv_heads, dim,
+                                         _capi.DTYPE_CODES[y.dtype], _capi.stream_of(y))
+    _capi.check(code, "head_mix")
     return out
 
 

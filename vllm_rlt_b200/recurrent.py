@@ -1,5 +1,5 @@
 """Recurrent layers over packed sequences with per-sequence state slots: short causal convolution (also as part of what prepares
-an attention layer's heads), the Mamba-2 state-space recurrence, linear attention with constant decays, and the gated norm behind them.
+an attention layer's heads), the Mamba-2 state-space recurrence, linear attention with constant decays, the gated delta rule, and the gated norm behind them.
 
 `group` arguments are a step's sequence group (`StepGroup`): `cu` (int32 [n + 1], row offsets into the step's
 rows), `starts` (position of each portion's first token), `slots`, and the host-side bound `max_new`.
@@ -156,19 +156,59 @@ def decay_table(decays, device) -> torch.Tensor:
     return torch.stack([d, torch.log2(d.clamp_min(2.0 ** -100))]).to(device=device, dtype=torch.float32)
 
 
-def gated_norm(y, z, weight, out, parts: int, eps: float, *, gate_behind: bool = False):
-    """`out = rmsnorm(y * silu(z)) * weight`, or with `gate_behind` `rmsnorm(y) * weight * sigmoid(z)`; the row normed in
-    `parts` equal parts; all `[rows, width]`, any row stride."""
+def delta_scan(q, k, v, decay, beta, dt_bias, a_log, state, out, group):
+    """The gated delta rule with a decay per head and key channel (`rlt_delta_scan`); q and k are made unit vectors here.
+
+    q, k `[rows, kv_heads * dim]`, v, out `[rows, heads * vdim]` (q, k and v slices of rows of one stride), raw decay `[rows, heads * dim]` and
+    beta `[rows, heads]`, dt_bias float32 `[heads * dim]`, a_log float32 `[heads]`, state float32 `[slots, heads, dim, vdim]`, updated in
+    place.  The tensors hold all rows of a step; the group's sequences are worked on."""
+    device = _capi.require_cuda(q, k, v, decay, beta, dt_bias, a_log, state, out, group.cu, group.starts, group.slots)
+    if state.dim() != 4 or state.dtype != torch.float32 or not state.is_contiguous():
+        raise ValueError("state must be contiguous float32 [slots, heads, dim, vdim]")
+    slots, heads, dim, vdim = state.shape
+    rows, kv_heads = q.shape[0], q.shape[1] // dim
+    if q.shape != (rows, kv_heads * dim) or kv_heads < 1 or heads % kv_heads or k.shape != q.shape or v.shape != (rows, heads * vdim) \
+            or out.shape != v.shape or decay.shape != (rows, heads * dim) or beta.shape != (rows, heads):
+        raise ValueError("q / k [rows, kv_heads * dim], v / out [rows, heads * vdim], decay [rows, heads * dim], beta [rows, heads]")
+    if q.stride(0) != k.stride(0) or k.stride(0) != v.stride(0) or any(t.stride(1) != 1 for t in (q, k, v, decay, beta, out)):
+        raise ValueError("q, k and v must be column slices of the same rows")
+    if q.dtype not in (torch.float32, torch.bfloat16) or any(t.dtype != q.dtype for t in (k, v, decay, beta, out)):
+        raise ValueError("q, k, v, decay, beta and out must share float32 or bfloat16")
+    for name, t, n in (("dt_bias", dt_bias, heads * dim), ("a_log", a_log, heads)):
+        if t.dtype != torch.float32 or t.shape != (n,) or not t.is_contiguous():
+            raise ValueError(f"{name} must be contiguous float32 [{n}]")
+    if group.sequences == 0:
+        return out
+    lib, dtype = _capi.load(), _capi.DTYPE_CODES[q.dtype]
+    count = group.rows.stop - group.rows.start
+    with torch.cuda.device(device):
+        nbytes = lib.rlt_delta_scan_workspace_bytes(group.sequences, group.max_new, count, heads, dim, vdim, dtype)
+        workspace = torch.empty(nbytes, dtype=torch.uint8, device=device)
+        code = lib.rlt_delta_scan(
+            _capi.ptr(q), _capi.ptr(k), _capi.ptr(v), q.stride(0), _capi.ptr(decay), decay.stride(0), _capi.ptr(beta), beta.stride(0),
+            _capi.ptr(dt_bias), _capi.ptr(a_log), _capi.ptr(out), out.stride(0), _capi.ptr(state), slots, _capi.ptr(group.cu),
+            _capi.ptr(group.starts), _capi.ptr(group.slots), group.sequences, group.max_new, count, heads, kv_heads, dim, vdim, dtype,
+            _capi.ptr(workspace), nbytes, _capi.stream_of(q))
+    _capi.check(code, "delta_scan")
+    return out
+
+
+GATES = {False: 0, True: 1, "sigmoid": 1, "silu": 2}
+
+
+def gated_norm(y, z, weight, out, parts: int, eps: float, *, gate_behind: bool | str = False):
+    """`out = rmsnorm(y * silu(z)) * weight`, or with `gate_behind` `rmsnorm(y) * weight * sigmoid(z)` ("silu": silu(z)); the row normed in
+    `parts` equal parts; all `[rows, width]`, any row stride; weight None: ones."""
     device = _capi.require_cuda(y, z, weight, out)
     rows, width = y.shape
-    if z.shape != y.shape or out.shape != y.shape or weight.shape != (width,) or weight.dtype != torch.float32 \
+    if z.shape != y.shape or out.shape != y.shape or (weight is not None and (weight.shape != (width,) or weight.dtype != torch.float32)) \
             or any(t.stride(1) != 1 for t in (y, z, out)) or y.dtype not in _capi.DTYPE_CODES or z.dtype != y.dtype or out.dtype != y.dtype:
         raise ValueError("y, z and out must be [rows, width] of one dtype with unit inner stride, weight float32 [width]")
     if rows == 0:
         return out
     with torch.cuda.device(device):
         code = _capi.load().rlt_gated_norm(_capi.ptr(y), y.stride(0), _capi.ptr(z), z.stride(0), _capi.ptr(weight), _capi.ptr(out),
-                                           out.stride(0), rows, width, parts, float(eps), int(gate_behind), _capi.DTYPE_CODES[y.dtype],
+                                           out.stride(0), rows, width, parts, float(eps), GATES[gate_behind], _capi.DTYPE_CODES[y.dtype],
                                            _capi.stream_of(y))
     _capi.check(code, "gated_norm")
     return out

@@ -19,6 +19,7 @@ import torch
 from .checkpoint import read_config, read_weights
 from .hybrid_lm import HybridLM, HybridLMConfig
 from .looped_lm import LoopedLM, LoopedLMConfig
+from .postnorm_lm import PostNormLM, PostNormLMConfig
 from .sandwich_lm import SandwichLM, SandwichLMConfig
 from .stream_lm import StreamLM, StreamLMConfig
 
@@ -63,3 +64,4 @@ register_model("OuroForCausalLM", LoopedLMConfig.from_json, LoopedLM)
 register_model("Sobipel", HybridLMConfig.from_json, HybridLM)
 register_model("Sugosun", StreamLMConfig.from_json, StreamLM)
 register_model("Kezuvik", SandwichLMConfig.from_json, SandwichLM)
+register_model("Degavik", PostNormLMConfig.from_json, PostNormLM)
