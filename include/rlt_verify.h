@@ -716,7 +716,7 @@ RLT_API int rlt_head_mix(const void* y, int64_t y_stride, const float* talk, voi
  *   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  out = S^T q
  * q, k [rows][kv_heads * dim] and v [rows][heads * vdim] are column slices of rows of one stride; head h reads q and k of head
  * h / (heads / kv_heads).  decay [rows][heads * dim], beta [rows][heads], dt_bias fp32 [heads * dim], a_log fp32 [heads].  Sequences and slots
- * as in rlt_ssd_scan; rows: rows of all sequences together. */
+ * as in rlt_ssd_scan; rows: no fewer than all sequences have together. */
 RLT_API size_t rlt_delta_scan_workspace_bytes(int sequences, int max_tokens, int rows, int heads, int dim, int vdim, int dtype);
 RLT_API int rlt_delta_scan(const void* q, const void* k, const void* v, int64_t qkv_stride, const void* decay, int64_t decay_stride,
                    const void* beta, int64_t beta_stride, const float* dt_bias, const float* a_log, void* out, int64_t out_stride,

@@ -7,6 +7,8 @@
 // step kernel    one token after the other: decoding (bytes: the state, read and written once), short portions, 32-bit models.  A warp
 //                owns eight columns of a head's state and all its rows, so the two sums of a token are shuffles:
 //                S^T k and S^T q are taken together before the write, o = S^T q + u (k . q).
+// chunk kernels  longer portions in 16 bits, 64 tokens at a time: delta_chunk.cu, delta_chunk_sm100.cu.  A call whose chunks' operands would
+//                not fit the workspace goes over its sequences in passes of a few chunks each.
 //
 // q and k arrive as the convolution left them: lengths, decays and strengths are formed here, in fp32.
 #include "delta_scan.cuh"
@@ -169,11 +171,32 @@ int launch_step(const DeltaArgs& a, int sequences, cudaStream_t stream) {
   return launch_status("delta_step_kernel");
 }
 
+constexpr int kStepTokens = 16;                          // portions up to this many go one token after the other
+constexpr int64_t kMaxRecordBytes = 1024ll << 20;        // of one pass
+
+bool chunked(int max_tokens, int dim, int vdim, int dtype) {
+  return dtype == RLT_BF16 && max_tokens > kStepTokens && dim % 8 == 0 && vdim % 8 == 0 && dim <= 128 && vdim <= 128;
+}
+
+// Chunks per sequence and pass, and the records that takes.
+int pass_chunks(int sequences, int max_tokens, int rows, int heads, int dim, int64_t* records) {
+  const int64_t longest = (max_tokens + kChunk - 1) / kChunk, exact = static_cast<int64_t>(rows) / kChunk + sequences;
+  const int64_t fit = kMaxRecordBytes / (static_cast<int64_t>(delta_record_bytes(dim)) * heads);
+  int64_t per = longest;
+  if (exact > fit && longest * sequences > fit) per = fit / sequences < 1 ? 1 : (fit / sequences < longest ? fit / sequences : longest);
+  *records = exact < per * sequences ? exact : per * sequences;
+  return static_cast<int>(per);
+}
+
 }  // namespace
 }  // namespace rlt
 
 extern "C" RLT_API size_t rlt_delta_scan_workspace_bytes(int sequences, int max_tokens, int rows, int heads, int dim, int vdim, int dtype) {
-  return 256;
+  using namespace rlt;
+  if (sequences <= 0 || max_tokens <= 0 || rows <= 0 || heads <= 0 || dim <= 0 || !chunked(max_tokens, dim, vdim, dtype)) return 256;
+  int64_t records;
+  pass_chunks(sequences, max_tokens, rows, heads, dim, &records);
+  return static_cast<size_t>(records) * heads * delta_record_bytes(dim) + 256;
 }
 
 extern "C" RLT_API int rlt_delta_scan(const void* q, const void* k, const void* v, int64_t qkv_stride, const void* decay, int64_t decay_stride,
@@ -189,7 +212,7 @@ extern "C" RLT_API int rlt_delta_scan(const void* q, const void* k, const void* 
   RLT_REQUIRE(q && k && v && decay && beta && dt_bias && a_log && out && state && cu_seqlens && starts && slot_of, "delta_scan: null pointer");
   RLT_REQUIRE(qkv_stride >= static_cast<int64_t>(kv_heads) * dim && decay_stride >= static_cast<int64_t>(heads) * dim && beta_stride >= heads &&
                   out_stride >= static_cast<int64_t>(heads) * vdim, "delta_scan: row strides smaller than a row");
-  if (dim > 256 || sequences > 65535 || (vdim + kTileCols - 1) / kTileCols > 65535) {
+  if (dim > 256 || sequences > 65535 || (max_tokens + kChunk - 1) / kChunk > 65535 || (vdim + kTileCols - 1) / kTileCols > 65535) {
     set_last_error_text("delta_scan: key sizes above 256 are not supported");
     return RLT_ERR_UNSUPPORTED;
   }
@@ -200,5 +223,23 @@ extern "C" RLT_API int rlt_delta_scan(const void* q, const void* k, const void* 
   a.q_scale = static_cast<float>(1.0 / sqrt(static_cast<double>(dim)));
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == RLT_F32) return launch_step<float>(a, sequences, s);
+  if (chunked(max_tokens, dim, vdim, dtype) && delta_chunks_supported(a, dtype)) {
+    if (workspace == nullptr || (reinterpret_cast<uintptr_t>(workspace) & 15u) != 0 ||
+        workspace_bytes < rlt_delta_scan_workspace_bytes(sequences, max_tokens, rows, heads, dim, vdim, dtype)) {
+      set_last_error_text("delta_scan: workspace missing, misaligned or too small");
+      return RLT_ERR_WORKSPACE;
+    }
+    a.error = static_cast<unsigned*>(workspace);         // workspace: an error word (256 bytes), then the records
+    a.records = static_cast<unsigned char*>(workspace) + 256;
+    int64_t records;
+    a.chunk_count = pass_chunks(sequences, max_tokens, rows, heads, dim, &records);
+    RLT_CUDA_TRY(cudaMemsetAsync(a.error, 0, sizeof(unsigned), s));
+    for (a.first_chunk = 0; a.first_chunk * kChunk < max_tokens; a.first_chunk += a.chunk_count) {
+      int status = launch_delta_prepare(a, sequences, s);
+      if (status == RLT_OK) status = launch_delta_states(a, sequences, s);
+      if (status != RLT_OK) return status;
+    }
+    return RLT_OK;
+  }
   return launch_step<__nv_bfloat16>(a, sequences, s);
 }

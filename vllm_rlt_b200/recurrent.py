@@ -180,14 +180,13 @@ def delta_scan(q, k, v, decay, beta, dt_bias, a_log, state, out, group):
     if group.sequences == 0:
         return out
     lib, dtype = _capi.load(), _capi.DTYPE_CODES[q.dtype]
-    count = group.rows.stop - group.rows.start
     with torch.cuda.device(device):
-        nbytes = lib.rlt_delta_scan_workspace_bytes(group.sequences, group.max_new, count, heads, dim, vdim, dtype)
+        nbytes = lib.rlt_delta_scan_workspace_bytes(group.sequences, group.max_new, rows, heads, dim, vdim, dtype)
         workspace = torch.empty(nbytes, dtype=torch.uint8, device=device)
         code = lib.rlt_delta_scan(
             _capi.ptr(q), _capi.ptr(k), _capi.ptr(v), q.stride(0), _capi.ptr(decay), decay.stride(0), _capi.ptr(beta), beta.stride(0),
             _capi.ptr(dt_bias), _capi.ptr(a_log), _capi.ptr(out), out.stride(0), _capi.ptr(state), slots, _capi.ptr(group.cu),
-            _capi.ptr(group.starts), _capi.ptr(group.slots), group.sequences, group.max_new, count, heads, kv_heads, dim, vdim, dtype,
+            _capi.ptr(group.starts), _capi.ptr(group.slots), group.sequences, group.max_new, rows, heads, kv_heads, dim, vdim, dtype,
             _capi.ptr(workspace), nbytes, _capi.stream_of(q))
     _capi.check(code, "delta_scan")
     return out

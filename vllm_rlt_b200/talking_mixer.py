@@ -58,6 +58,15 @@ class TalkingAttentionConfig:
         return {prefix + name: shape for name, shape in shapes.items()}
 
 
+def talking_attention(kernels, q, key, value, out, group, terms: ScoreTerms, talk):
+    """Attention of a group's portions over the pages with score terms, heads mixed by `talk` (float32 `[heads, heads]`) behind the softmax;
+    q `[rows, heads, dim]`, out `[rows, heads, vdim]` of the group's rows."""
+    rows, heads, vdim = out.shape
+    spread = torch.empty(rows, heads, value.shape[2] * vdim, dtype=q.dtype, device=q.device)
+    kernels.scored(q, spread, key, value, group.tables, group.lengths, group.local_cu, group.max_new, terms, all_values=True)
+    return head_mix(spread, talk, out, value.shape[2])
+
+
 class TalkingAttention:
     """One layer's stacked weights, and its step.  `take(name, dtype=None)` gives a parameter on the device."""
 
@@ -78,8 +87,5 @@ class TalkingAttention:
         norm_rotate(proj, self.columns, self.q_norm, self.k_norm, self.eps, self.frequencies, q, key, value, batch, halves=m.rotation.halves)
         out = torch.empty(rows, m.heads, m.vdim, dtype=h.dtype, device=h.device)
         for group in batch.groups:
-            part = group.rows
-            spread = torch.empty(part.stop - part.start, m.heads, m.kv_heads * m.vdim, dtype=h.dtype, device=h.device)
-            self.kernels.scored(q[part], spread, key, value, group.tables, group.lengths, group.local_cu, group.max_new, self.terms, all_values=True)
-            head_mix(spread, self.talk, out[part], m.kv_heads)
+            talking_attention(self.kernels, q[group.rows], key, value, out[group.rows], group, self.terms, self.talk)
         return F.linear(out.view(rows, -1), self.w_o)
