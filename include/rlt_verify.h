@@ -634,10 +634,11 @@ RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_t src_head,
                      int64_t dst_head, int heads, int dim, int rot_dims, const double* frequencies, int halves,
                      float amplitude, float scale, int scaled_from, const int32_t* positions, int rows, int dtype, rlt_stream_t stream);
 
-/* Cache rows of positions first[s] .. of every sequence s, packed: row cu[s] + i holds position first[s] + i. */
+/* Cache rows of positions first[s] .. of every sequence s, packed behind its first n = min(keep, first[s]) positions: row cu[s] + i holds
+ * position i for i < n, and first[s] + i - n from there on. */
 RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks,
                       int block_size, int row_width, const int32_t* tables, int table_width, const int32_t* first,
-                      const int32_t* cu, int sequences, int rows, void* out, int dtype, rlt_stream_t stream);
+                      const int32_t* cu, int sequences, int rows, int keep, void* out, int dtype, rlt_stream_t stream);
 
 /* Prompt attention over packed keys and values (bf16): expanded from latents, or gathered from the pages of a windowed layer.
  * q [rows][heads][dim + rot_dim]; keys [key_rows][kv_heads][dim], values [key_rows][kv_heads][vdim] (strides between rows); shared_keys
@@ -710,6 +711,30 @@ RLT_API int rlt_norm_rotate(const void* proj, int64_t proj_stride, int q_col, in
  * [heads][heads], out [rows][heads * dim]. */
 RLT_API int rlt_head_mix(const void* y, int64_t y_stride, const float* talk, void* out, int64_t out_stride, int rows, int heads, int kv_heads,
                  int dim, int dtype, rlt_stream_t stream);
+
+/* Windowed attention with kept first tokens, bounded scores and heads that talk behind the softmax (bf16):
+ *   score = softcap * tanh((q . k) * scale * head_scale[h] / softcap) over keys j <= p with p - j < window (0: all) or j < keep_first
+ *   out[h] = sum_g talk[h][g] (softmax weights of head g, applied to the values of key/value head h / (heads / kv_heads))
+ * rlt_talking_attention: over pages, for short portions; tables, lengths and packing as in rlt_scored_attention; keys: a host-side bound on
+ * the keys a row sees, which sizes the split of a context (any bound gives the same result but for rounding).
+ * rlt_talking_prompt: over packed keys [key_rows][kv_heads][dim] and values [key_rows][kv_heads * value_dim], for long portions; spread
+ * [rows][heads][kv_heads * value_dim] receives every head over the values of every key/value head (rlt_head_mix takes it).  tiles as in
+ * rlt_latent_prompt_attention, at most 128 rows each, with the number of kept positions in front of the packed row in the sixth word.
+ * workspace: 256 bytes, the first word is set when a bounded wait gave up. */
+RLT_API int rlt_talking_attention_supported(int heads, int kv_heads, int dim, int value_dim, float softcap, int dtype);
+RLT_API size_t rlt_talking_attention_workspace_bytes(int rows, int sequences, int max_new, int heads, int kv_heads, int dim, int value_dim,
+                                             int64_t keys);
+RLT_API int rlt_talking_attention(const void* q, int64_t q_stride, void* out, int64_t out_stride, const void* key_cache, int64_t k_block_stride,
+                          int64_t k_token_stride, const void* value_cache, int64_t v_block_stride, int64_t v_token_stride, int64_t num_blocks,
+                          int block_size, int heads, int kv_heads, int dim, int value_dim, int dtype, const int32_t* block_tables, int sequences,
+                          int table_width, const int32_t* context_lengths, const int32_t* cu_seqlens_q, int rows, int max_new, float scale,
+                          int window, int keep_first, float softcap, const float* head_scale, const float* talk, int64_t keys, void* workspace,
+                          size_t workspace_bytes, rlt_stream_t stream);
+RLT_API int rlt_talking_prompt_supported(int heads, int kv_heads, int dim, int value_dim, float softcap, int dtype);
+RLT_API int rlt_talking_prompt(const void* q, int64_t q_stride, const void* keys, int64_t key_stride, const void* values, int64_t value_stride,
+                       void* spread, int64_t spread_stride, int rows, int key_rows, int heads, int kv_heads, int dim, int value_dim,
+                       const int32_t* tiles, int tile_count, float scale, int window, int keep_first, float softcap, const float* head_scale,
+                       int dtype, void* workspace, rlt_stream_t stream);
 
 /* The gated delta rule with a decay per head and key channel, state fp32 [slots][heads][dim][vdim], updated in place.  Per head, with k and q
  * divided by sqrt(sum of squares + 1e-6), q also by sqrt(dim), g = exp(-exp(a_log) softplus(decay + dt_bias)) and beta sigmoid of its raw value:

@@ -9,6 +9,8 @@ import plain_postnorm as plain
 import vllm_rlt_b200 as rlt
 from test_gpu_hybrid_kernels import BLOCK, DTYPES, close, group_of, paged_case
 from test_gpu_stream_kernels import larger_pages
+from vllm_rlt_b200.engine import KeyRanges
+from vllm_rlt_b200.talking_mixer import talking_attention
 
 pytestmark = pytest.mark.gpu
 
@@ -140,8 +142,8 @@ def run_talking(case, contexts, portions, terms, talk, heads, vdim):
     group = SimpleNamespace(sequences=len(portions), max_new=max(portions), tables=to(tables), cu=cu, local_cu=cu,
                             lengths=torch.tensor(contexts, dtype=torch.int32, device="cuda"), rows=slice(0, rows),
                             portions=[(c - n, n) for c, n in zip(contexts, portions)])
-    group.key_ranges = lambda window, keep=0: rlt.engine.KeyRanges.of(group.portions, window, torch.device("cuda"), keep)
-    rlt.talking_mixer.talking_attention(rlt.B200PagedAttention(), torch.cat(q).cuda(), to(key), to(value), out, group, terms, talk.cuda())
+    group.key_ranges = lambda *which: KeyRanges.of(group.portions, which[0], torch.device("cuda"), *which[1:])
+    talking_attention(rlt.B200PagedAttention(), torch.cat(q).cuda(), to(key), to(value), out, group, terms, talk.cuda())
     return out
 
 
@@ -173,7 +175,7 @@ def test_talking_attention(dtype, heads, kv_heads, dim, vdim, window, keep, cap,
             key, tables = larger_pages(case[3], case[5], page)
             value, _ = larger_pages(case[4], case[5], page)
             case = (*case[:3], key, value, tables)
-        close(run_talking(case, contexts, portions, terms, talk, heads, vdim), want, dtype, 2.5)
+        close(run_talking(case, contexts, portions, terms, talk, heads, vdim), want, dtype, 3 * float(talk.norm(dim=1).max()))    # mixing adds up roundings
 
 
 @pytest.mark.parametrize("dtype", DTYPES)

@@ -68,7 +68,7 @@ SIGNATURES = {
     "rlt_latent_write": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _I, _F, _P, _L, _P, _L, _L, _L, _I, _P, _I, _P, _P, _I, _I,
                               _P]),
     "rlt_rotate_heads": (_I, [_P, _L, _L, _P, _L, _L, _I, _I, _I, _P, _I, _F, _F, _I, _P, _I, _I, _P]),
-    "rlt_latent_gather": (_I, [_P, _L, _L, _L, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _P]),
+    "rlt_latent_gather": (_I, [_P, _L, _L, _L, _I, _I, _P, _I, _P, _P, _I, _I, _I, _P, _I, _P]),
     "rlt_latent_prompt_supported": (_I, [_I, _I, _I, _I]),
     "rlt_latent_prompt_attention": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _I, _F, _I, _P, _P, _L, _I,
                                          _I, _P, _P]),
@@ -84,6 +84,12 @@ SIGNATURES = {
     "rlt_norm_rotate": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _P, _L, _P, _L, _L, _P, _L, _L, _L, _I, _P, _I,
                              _I, _I, _P]),
     "rlt_head_mix": (_I, [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P]),
+    "rlt_talking_attention_supported": (_I, [_I, _I, _I, _I, _F, _I]),
+    "rlt_talking_attention_workspace_bytes": (_Z, [_I, _I, _I, _I, _I, _I, _I, _L]),
+    "rlt_talking_attention": (_I, [_P, _L, _P, _L, _P, _L, _L, _P, _L, _L, _L, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _I, _I, _F, _I, _I, _F,
+                                   _P, _P, _L, _P, _Z, _P]),
+    "rlt_talking_prompt_supported": (_I, [_I, _I, _I, _I, _F, _I]),
+    "rlt_talking_prompt": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P, _I, _F, _I, _I, _F, _P, _I, _P, _P]),
     "rlt_delta_scan_workspace_bytes": (_Z, [_I, _I, _I, _I, _I, _I, _I]),
     "rlt_delta_scan": (_I, [_P, _P, _P, _L, _P, _L, _P, _L, _P, _P, _P, _L, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _Z, _P]),
     "rlt_rollback": (_I, [_P, _P, _I, _P, _I, _I, _I, _P, _P, _L, _P, _I, _P, _P, _P, _P, _P, _P]),

@@ -9,8 +9,8 @@
 //
 // A product over channels with a decay between two tokens is split at a token r between them, i after r >= j: 2^(G_i - G_r) belongs to the
 // row and 2^(G_r - G_j) to the column, and neither exceeds one, however strong the decay.  So the chunk is halved again and again: the
-// block (later half, earlier half) of every pair of neighbours of 32, 16, 8, 4, 2 and 1 tokens is a product of its own on tensor cores,
-// sixteen rows at a time (eight keys over eight queries).  q and k are 16-bit (outputs of the convolution), their lengths are applied to
+// block (later half, earlier half) of every pair of neighbours of 32, 16 and 8 tokens is a product of its own on tensor cores,
+// sixteen rows at a time (eight keys over eight queries); inside eight tokens the decays are multiplied up one by one.  q and k are 16-bit (outputs of the convolution), their lengths are applied to
 // the products; what is computed here enters its product as the sum of two 16-bit numbers, so nothing of the recurrence is rounded to 16
 // bits.  The triangular system is solved in fp32: 16 x 16 blocks by substitution, joined by block products.
 #include "delta_scan.cuh"
@@ -37,19 +37,19 @@ struct PrepareShared {
     uint16_t v[kChunk][kValuePitch];           // later
   };
   float l[kChunk][kMatrix], t[kChunk][kMatrix];
-  unsigned char p[2][kChunk * 128];              // high and low halves
   float beta[kChunk], rq[kChunk], rk[kChunk];
 };
 
 __device__ __forceinline__ void copy_piece(uint32_t dst, const void* src, bool live) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
 }
+__device__ __forceinline__ float2 unpack(uint32_t x) { return make_float2(__uint_as_float(x << 16), __uint_as_float(x & 0xffff0000u)); }
 __device__ __forceinline__ void split_pair(float a, float b, uint32_t* hi, uint32_t* lo) {
   const uint32_t h = pack2<true>(a, b);
   *hi = h;
-  *lo = pack2<true>(a - __uint_as_float(h << 16), b - __uint_as_float(h & 0xffff0000u));
+  const float2 rest = sub_pair(make_float2(a, b), unpack(h));
+  *lo = pack2<true>(rest.x, rest.y);
 }
-__device__ __forceinline__ float2 unpack(uint32_t x) { return make_float2(__uint_as_float(x << 16), __uint_as_float(x & 0xffff0000u)); }
 __device__ __forceinline__ int swizzled(int row, int piece) { return row * 128 + ((piece ^ (row & 7)) << 4); }
 __device__ __forceinline__ void mma_split(float (&acc)[4], const uint32_t (&a_hi)[4], const uint32_t (&a_lo)[4], const uint32_t (&b_hi)[2], const uint32_t (&b_lo)[2]) {
   mma_16816<true>(acc, a_hi, b_hi[0], b_hi[1]);
@@ -59,8 +59,8 @@ __device__ __forceinline__ void mma_split(float (&acc)[4], const uint32_t (&a_hi
 
 // Two channels of a token times 2^(exponents).
 __device__ __forceinline__ void decayed(uint32_t raw, float2 factor, uint32_t* hi, uint32_t* lo) {
-  const float2 x = unpack(raw);
-  split_pair(x.x * factor.x, x.y * factor.y, hi, lo);
+  const float2 x = mul_pair(unpack(raw), factor);
+  split_pair(x.x, x.y, hi, lo);
 }
 
 template <int kDim, int kVal>
@@ -102,18 +102,16 @@ delta_prepare_kernel(DeltaArgs a) {
     const T* raw = static_cast<const T*>(a.decay) + row * a.decay_stride + static_cast<int64_t>(head) * a.dim + (live ? c : 0);
     const float bias = live ? a.dt_bias[static_cast<int64_t>(head) * a.dim + c] : 0.0f, rate = -kLog2e * expf(a.a_log[head]);
     float sum = 0.0f;
-#pragma unroll 8
+    T value[kRun];                             // all loads before the first use
+#pragma unroll
+    for (int i = 0; i < kRun; ++i)
+      if (live && from + i < count) value[i] = raw[(from + i) * a.decay_stride];
+#pragma unroll
     for (int i = 0; i < kRun; ++i) {
-      const int token = from + i;
-      if (live && token < count) sum = fmaf(rate, softplus(Elem<T>::to_float(raw[token * a.decay_stride]) + bias), sum);
-      sm.g[token][c] = sum;
+      if (live && from + i < count) sum = fmaf(rate, softplus_series(Elem<T>::to_float(value[i]) + bias), sum);
+      sm.g[from + i][c] = sum;
     }
   }
-  for (int i = threadIdx.x; i < kChunk * kMatrix; i += kThreads) {
-    (&sm.l[0][0])[i] = 0.0f;
-    (&sm.t[0][0])[i] = 0.0f;
-  }
-  for (int i = threadIdx.x; i < kChunk * 16; i += kThreads) reinterpret_cast<uint4*>(sm.p)[i] = make_uint4(0u, 0u, 0u, 0u);
   asm volatile("cp.async.wait_all;" ::: "memory");
   __syncthreads();
   {
@@ -148,19 +146,20 @@ delta_prepare_kernel(DeltaArgs a) {
   // acc: rows of eight tokens from `later` (keys, then queries) x eight tokens from `earlier`; elements 0, 1: (key g, token 2 t + e), 2, 3: queries
   auto store_products = [&](int later, int earlier, const float (&acc)[4]) {
     const int i = later + g;
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int j = earlier + 2 * t + e;
-      if (j < i) sm.l[i][j] = sm.beta[i] * sm.rk[i] * sm.rk[j] * acc[e];
-    }
     const int j = earlier + 2 * t;
-    const float p0 = j <= i ? sm.rq[i] * sm.rk[j] * acc[2] : 0.0f, p1 = j + 1 <= i ? sm.rq[i] * sm.rk[j + 1] * acc[3] : 0.0f;
+    const float2 r = *reinterpret_cast<const float2*>(&sm.rk[j]);
+    const float scale = sm.beta[i] * sm.rk[i];
+    *reinterpret_cast<float2*>(&sm.l[i][j]) = make_float2(scale * r.x * acc[0], scale * r.y * acc[1]);
+    const float p0 = sm.rq[i] * r.x * acc[2], p1 = sm.rq[i] * r.y * acc[3];
     const int at = swizzled(i, j >> 3) + (j & 7) * 2;
-    split_pair(p0, p1, reinterpret_cast<uint32_t*>(sm.p[0] + at), reinterpret_cast<uint32_t*>(sm.p[1] + at));
+    split_pair(p0, p1, reinterpret_cast<uint32_t*>(record + Record::kP + at), reinterpret_cast<uint32_t*>(record + Record::kP + Record::kBlock + at));
   };
   auto pair_at = [](const uint16_t* p) { return *reinterpret_cast<const uint32_t*>(p); };
   auto floats_at = [](const float* p) { return *reinterpret_cast<const float2*>(p); };
-  auto power = [](float2 x, float2 y) { return make_float2(fast_exp2(x.x - y.x), fast_exp2(x.y - y.y)); };
+  auto power = [](float2 x, float2 y) {
+    const float2 d = sub_pair(x, y);
+    return make_float2(fast_exp2(d.x), fast_exp2(d.y));
+  };
   // one block of eight later tokens against kN blocks of eight earlier ones, split at token `split`
   auto block_products = [&](int later, int earlier, int split, auto blocks) {
     constexpr int kN = decltype(blocks)::value;
@@ -197,47 +196,87 @@ delta_prepare_kernel(DeltaArgs a) {
   block_products((warp >> 2) * 32 + 16 + 8 * ((warp >> 1) & 1), (warp >> 2) * 32 + 8 * (warp & 1), (warp >> 2) * 32 + 15, std::integral_constant<int, 1>());
   if (warp < 4) block_products(warp * 16 + 8, warp * 16, warp * 16 + 7, std::integral_constant<int, 1>());                     // halves of 8
   {
-    // inside a block of eight: a lane's token is both its row and its column; at every level it is on one side of the split
-    const int block = warp * 8, i = block + g;
-    float sum[4] = {0.f, 0.f, 0.f, 0.f};
+    // Inside a block of eight: a lane owns kOwn channels, walks from every token back to the block's first one, and carries the decay
+    // along as a product of the tokens' own.  64 sums (28 of keys with keys, 36 of queries with keys) over the warp, two per lane.
+    constexpr int kOwn = kDim / 32;
+    const int block = warp * 8, c = lane * kOwn;
+    float kv[8][kOwn], qv[8][kOwn], step[8][kOwn];
 #pragma unroll
-    for (int half_size = 4; half_size > 0; half_size >>= 1) {
-      const bool later = (g & half_size) != 0;
-      const int split = block + (g & ~(2 * half_size - 1)) + half_size - 1;
-      float acc[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 2
-      for (int ks = 0; ks < kDim / 16; ++ks) {
-        uint32_t a_hi[4], a_lo[4], b_hi[2], b_lo[2];
+    for (int i = 0; i < 8; ++i) {
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int c = ks * 16 + half * 8 + 2 * t;
-          const float2 mine = floats_at(&sm.g[i][c]), at = floats_at(&sm.g[split][c]);
-          const float side = later ? 1.0f : -1.0f;
-          const float2 f = make_float2(fast_exp2(side * (mine.x - at.x)), fast_exp2(side * (mine.y - at.y)));
-          uint32_t hi, lo;
-          decayed(pair_at(&sm.k[i][c]), f, &hi, &lo);
-          a_hi[2 * half] = later ? hi : 0u; a_lo[2 * half] = later ? lo : 0u;
-          b_hi[half] = later ? 0u : hi; b_lo[half] = later ? 0u : lo;
-          decayed(pair_at(&sm.q[i][c]), f, &hi, &lo);
-          a_hi[2 * half + 1] = later ? hi : 0u; a_lo[2 * half + 1] = later ? lo : 0u;
-        }
-        mma_split(acc, a_hi, a_lo, b_hi, b_lo);
+      for (int e = 0; e < kOwn; e += 2) {
+        const float2 x = unpack(pair_at(&sm.k[block + i][c + e])), y = unpack(pair_at(&sm.q[block + i][c + e])), d = floats_at(&sm.g[block + i][c + e]);
+        kv[i][e] = x.x; kv[i][e + 1] = x.y;
+        qv[i][e] = y.x; qv[i][e + 1] = y.y;
+        step[i][e] = d.x; step[i][e + 1] = d.y;
       }
-#pragma unroll
-      for (int e = 0; e < 2; ++e)
-        if ((g & ~(2 * half_size - 1)) == ((2 * t + e) & ~(2 * half_size - 1))) { sum[e] += acc[e]; sum[2 + e] += acc[2 + e]; }
-    }
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};                 // a query with its own key: no decay, 16-bit operands as they are
-#pragma unroll
-    for (int ks = 0; ks < kDim / 16; ++ks) {
-      const int c = ks * 16 + 2 * t;
-      const uint32_t rows[4] = {0u, pair_at(&sm.q[i][c]), 0u, pair_at(&sm.q[i][c + 8])};
-      mma_16816<true>(acc, rows, pair_at(&sm.k[i][c]), pair_at(&sm.k[i][c + 8]));
     }
 #pragma unroll
-    for (int e = 0; e < 2; ++e)
-      if (g == 2 * t + e) sum[2 + e] += acc[2 + e];
-    store_products(block, block, sum);
+    for (int i = 7; i > 0; --i)
+#pragma unroll
+      for (int e = 0; e < kOwn; ++e) step[i][e] = fast_exp2(step[i][e] - step[i - 1][e]);
+    float sums[64];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      float kd[kOwn], qd[kOwn];
+#pragma unroll
+      for (int e = 0; e < kOwn; ++e) { kd[e] = kv[i][e]; qd[e] = qv[i][e]; }
+#pragma unroll
+      for (int j = i; j >= 0; --j) {
+        float ks = 0.0f, qs = 0.0f;
+#pragma unroll
+        for (int e = 0; e < kOwn; ++e) {
+          if (j < i) {
+            kd[e] *= step[j + 1][e];
+            qd[e] *= step[j + 1][e];
+            ks = fmaf(kd[e], kv[j][e], ks);
+          }
+          qs = fmaf(qd[e], kv[j][e], qs);
+        }
+        if (j < i) sums[i * (i - 1) / 2 + j] = ks;
+        sums[28 + i * (i + 1) / 2 + j] = qs;
+      }
+    }
+#pragma unroll
+    for (int step_lanes = 16, n = 32; step_lanes > 0; step_lanes >>= 1, n >>= 1)
+#pragma unroll
+      for (int m = 0; m < 32; ++m)
+        if (m < n) {
+          const bool odd = (lane & step_lanes) != 0;
+          const float keep = odd ? sums[2 * m + 1] : sums[2 * m], give = odd ? sums[2 * m] : sums[2 * m + 1];
+          sums[m] = keep + __shfl_xor_sync(0xffffffffu, give, step_lanes);
+        }
+    const int mine = static_cast<int>(__brev(static_cast<unsigned>(lane)) >> 27);
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      const int n = 32 * m + mine;
+      const bool key = n < 28;
+      const int p = key ? n : n - 28;
+      int i = (p >= 1) + (p >= 3) + (p >= 6) + (p >= 10) + (p >= 15) + (p >= 21) + (p >= 28);
+      const int j = block + p - i * (i + 1) / 2;
+      i += block + (key ? 1 : 0);
+      if (key) {
+        sm.l[i][j] = sm.beta[i] * sm.rk[i] * sm.rk[j] * sums[m];
+      } else {
+        const float x = sm.rq[i] * sm.rk[j] * sums[m];
+        const __nv_bfloat16 hi = __float2bfloat16_rn(x);
+        unsigned char* at = record + Record::kP + swizzled(i, j >> 3) + (j & 7) * 2;
+        *reinterpret_cast<__nv_bfloat16*>(at) = hi;
+        *reinterpret_cast<__nv_bfloat16*>(at + Record::kBlock) = __float2bfloat16_rn(x - __bfloat162float(hi));
+      }
+    }
+    // the diagonal block's own upper half, and every block right of it, are zero
+    for (int n = lane; n < 64; n += 32) {
+      const int i = block + (n >> 3), j = block + (n & 7);
+      if (j > i)
+#pragma unroll
+        for (int half = 0; half < 2; ++half)
+          *reinterpret_cast<uint16_t*>(record + Record::kP + half * Record::kBlock + swizzled(i, j >> 3) + (j & 7) * 2) = 0;
+      if ((n & 7) > warp)
+#pragma unroll
+        for (int half = 0; half < 2; ++half)
+          *reinterpret_cast<uint4*>(record + Record::kP + half * Record::kBlock + swizzled(i, n & 7)) = make_uint4(0u, 0u, 0u, 0u);
+    }
   }
 
   // ---- decayed operands ----
@@ -272,7 +311,7 @@ delta_prepare_kernel(DeltaArgs a) {
     k_hi[n] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
     k_lo[n] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   }
-  __syncthreads();                                       // decays and queries have been read, L and P are complete
+  __syncthreads();                                       // decays and queries have been read, L is complete
 #pragma unroll
   for (int n = 0; n < kPieces; ++n) {
     const int i = n * kThreads + threadIdx.x, r = i / (kDim / 8), c = (i % (kDim / 8)) * 8;
@@ -284,8 +323,6 @@ delta_prepare_kernel(DeltaArgs a) {
     const bool live = r < count && c < a.vdim;
     copy_piece(smem_u32(&sm.v[r][c]), live ? vg + r * a.qkv_stride + c : vg, live);
   }
-  for (int i = threadIdx.x; i < kChunk * 16; i += kThreads)
-    *reinterpret_cast<uint4*>(record + Record::kP + i * 16) = reinterpret_cast<const uint4*>(sm.p)[i];
 
   // ---- T = (I + L)^-1 ----
   if (threadIdx.x < kChunk) {                            // a column of a 16 x 16 block on the diagonal
@@ -308,9 +345,10 @@ delta_prepare_kernel(DeltaArgs a) {
     const bool mine = I < 4;
     float m[4] = {0.f, 0.f, 0.f, 0.f};
     if (mine) {
-      for (int k = J * 16; k < I * 16; ++k) {
-        const float x = sm.l[I * 16 + r][k];
-        const float4 y = *reinterpret_cast<const float4*>(&sm.t[k][J * 16 + c]);
+#pragma unroll 16
+      for (int k = 0; k < distance * 16; ++k) {
+        const float x = sm.l[I * 16 + r][J * 16 + k];
+        const float4 y = *reinterpret_cast<const float4*>(&sm.t[J * 16 + k][J * 16 + c]);
         m[0] = fmaf(x, y.x, m[0]); m[1] = fmaf(x, y.y, m[1]); m[2] = fmaf(x, y.z, m[2]); m[3] = fmaf(x, y.w, m[3]);
       }
       *reinterpret_cast<float4*>(&sm.t[I * 16 + r][J * 16 + c]) = make_float4(m[0], m[1], m[2], m[3]);

@@ -12,7 +12,8 @@ struct PromptTile {
   int position;    // of the first row in its sequence
   int key_row;     // packed key row of position key_first
   int key_first;   // first position of the sequence that is among the packed keys
-  int pad[3];
+  int kept;        // positions 0 .. kept - 1 are packed in front of key_row
+  int pad[2];
 };
 
 struct LatentPromptArgs {

@@ -4,7 +4,7 @@
 //   latent_write_kernel   the stacked down projections of a row: the query latent normed into the next GEMM's operand,
 //                         the key/value latent normed and the key part rotated into the row's page
 //   rotate_heads_kernel   the rotated part of every head, in place or into another operand; the last heads may be scaled on the way
-//   latent_gather_kernel  the cache rows of a range of positions of every sequence, side by side: what a prompt expands
+//   latent_gather_kernel  the cache rows of a range of positions of every sequence (and of its first few), side by side: what a prompt expands
 //                         into keys and values
 //
 // Rotation: dimensions 2i and 2i + 1 — in the `halves` layout i and i + rot_dims / 2 — are a pair, turned by position * frequency_i
@@ -199,7 +199,7 @@ template <typename V>
 __global__ void __launch_bounds__(kThreads)
 latent_gather_kernel(const unsigned char* __restrict__ cache, int64_t block_bytes, int64_t token_bytes, int64_t num_blocks, int block_size,
                      int row_bytes, const int32_t* __restrict__ tables, int table_width, const int32_t* __restrict__ first,
-                     const int32_t* __restrict__ cu, int sequences, int rows, unsigned char* __restrict__ out) {
+                     const int32_t* __restrict__ cu, int sequences, int rows, int keep, unsigned char* __restrict__ out) {
   const int row = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= rows) return;
   int lo = 0, hi = sequences - 1;             // last sequence with cu <= row
@@ -207,7 +207,8 @@ latent_gather_kernel(const unsigned char* __restrict__ cache, int64_t block_byte
     const int mid = (lo + hi + 1) >> 1;
     if (cu[mid] <= row) lo = mid; else hi = mid - 1;
   }
-  const int position = first[lo] + row - cu[lo];
+  const int from = first[lo], kept = min(keep, from), place = row - cu[lo];
+  const int position = place < kept ? place : from + place - kept;
   const int page_index = position / block_size;
   int64_t page = -1;
   if (position >= 0 && page_index < table_width) page = tables[static_cast<int64_t>(lo) * table_width + page_index];
@@ -284,10 +285,10 @@ extern "C" RLT_API int rlt_rotate_heads(const void* src, int64_t src_row, int64_
 
 extern "C" RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride, int64_t token_stride, int64_t num_blocks, int block_size,
                                          int row_width, const int32_t* tables, int table_width, const int32_t* first, const int32_t* cu,
-                                         int sequences, int rows, void* out, int dtype, rlt_stream_t stream) {
+                                         int sequences, int rows, int keep, void* out, int dtype, rlt_stream_t stream) {
   using namespace rlt;
   RLT_REQUIRE(dtype_valid(dtype), "latent_gather: dtype must be float32, float16 or bfloat16");
-  RLT_REQUIRE(rows >= 0 && row_width > 0 && block_size > 0 && num_blocks > 0 && sequences >= 0 && table_width > 0, "latent_gather: invalid shape");
+  RLT_REQUIRE(rows >= 0 && row_width > 0 && block_size > 0 && num_blocks > 0 && sequences >= 0 && table_width > 0 && keep >= 0, "latent_gather: invalid shape");
   if (rows == 0) return RLT_OK;
   RLT_REQUIRE(cache && tables && first && cu && out && sequences > 0, "latent_gather: null pointer");
   const int64_t size = static_cast<int64_t>(dtype_size(dtype));
@@ -298,8 +299,8 @@ extern "C" RLT_API int rlt_latent_gather(const void* cache, int64_t block_stride
   const unsigned char* from = static_cast<const unsigned char*>(cache);
   unsigned char* to = static_cast<unsigned char*>(out);
   if (row_bytes % 16 == 0 && block_bytes % 16 == 0 && token_bytes % 16 == 0 && aligned16(cache) && aligned16(out))
-    latent_gather_kernel<uint4><<<grid, kThreads, 0, s>>>(from, block_bytes, token_bytes, num_blocks, block_size, row_bytes, tables, table_width, first, cu, sequences, rows, to);
+    latent_gather_kernel<uint4><<<grid, kThreads, 0, s>>>(from, block_bytes, token_bytes, num_blocks, block_size, row_bytes, tables, table_width, first, cu, sequences, rows, keep, to);
   else
-    latent_gather_kernel<uint16_t><<<grid, kThreads, 0, s>>>(from, block_bytes, token_bytes, num_blocks, block_size, row_bytes, tables, table_width, first, cu, sequences, rows, to);
+    latent_gather_kernel<uint16_t><<<grid, kThreads, 0, s>>>(from, block_bytes, token_bytes, num_blocks, block_size, row_bytes, tables, table_width, first, cu, sequences, rows, keep, to);
   return launch_status("latent_gather_kernel");
 }

@@ -32,35 +32,38 @@ class StepEntry:
 
 @dataclass
 class KeyRanges:
-    """Positions `first[s]` .. of every sequence, packed: those of sequence s are rows cu[s] .. cu[s + 1] - 1.
+    """Positions `first[s]` .. of every sequence, packed: those of sequence s are rows cu[s] .. cu[s + 1] - 1, behind the first
+    min(keep, first[s]) positions of the sequence, which a window may keep.
 
-    tiles: the portions in runs of up to TILE_ROWS query rows, those with the most keys first, as records (first query row, rows,
-    position of the first row, packed row of position first[s], first[s], 0, 0, 0)."""
+    tiles: the portions in runs of up to `tile_rows` query rows, those with the most keys first, as records (first query row, rows,
+    position of the first row, packed row of position first[s], first[s], kept positions in front of it, 0, 0)."""
 
     first: torch.Tensor      # int32 [n]
     cu: torch.Tensor         # int32 [n + 1]
     rows: int
     tiles: torch.Tensor      # int32 [tiles, 8]
+    keep: int = 0
 
     TILE_ROWS = 256
 
     @classmethod
-    def of(cls, portions, window: int, device) -> "KeyRanges":
+    def of(cls, portions, window: int, device, keep: int = 0, tile_rows: int = TILE_ROWS) -> "KeyRanges":
         first = [max(start - window + 1, 0) if window else 0 for start, _ in portions]
         cu = [0]
         for f, (start, n) in zip(first, portions):
-            cu.append(cu[-1] + start + n - f)
+            cu.append(cu[-1] + min(keep, f) + start + n - f)
         tiles, row = [], 0
         for s, (start, n) in enumerate(portions):
-            for at in range(0, n, cls.TILE_ROWS):
-                tiles.append((row + at, min(n - at, cls.TILE_ROWS), start + at, cu[s], first[s], 0, 0, 0))
+            kept = min(keep, first[s])
+            for at in range(0, n, tile_rows):
+                tiles.append((row + at, min(n - at, tile_rows), start + at, cu[s] + kept, first[s], kept, 0, 0))
             row += n
         tiles.sort(key=lambda t: min(t[2] + t[1], window + t[1]) if window else t[2] + t[1], reverse=True)
         host = torch.tensor([x for t in tiles for x in t] + first + cu, dtype=torch.int32)
         if device.type == "cuda":
             host = host.pin_memory()
         tile_words, rest = host.to(device, non_blocking=True).split((8 * len(tiles), len(first) + len(cu)))
-        return cls(rest[:len(first)], rest[len(first):], cu[-1], tile_words.view(-1, 8))
+        return cls(rest[:len(first)], rest[len(first):], cu[-1], tile_words.view(-1, 8), keep)
 
 
 @dataclass
@@ -79,11 +82,13 @@ class StepGroup:
     portions: list | None = None   # host side: (start, tokens) of every sequence; None in a captured step
     _ranges: dict = field(default_factory=dict)
 
-    def key_ranges(self, window: int) -> "KeyRanges":
-        """The positions the group's rows see in a layer with this window (0: all), for kernels that want them packed."""
-        if window not in self._ranges:
-            self._ranges[window] = KeyRanges.of(self.portions, window, self.cu.device)
-        return self._ranges[window]
+    def key_ranges(self, window: int, keep: int = 0, tile_rows: int = KeyRanges.TILE_ROWS) -> "KeyRanges":
+        """The positions the group's rows see in a layer with this window (0: all) and so many kept first tokens, for kernels that want
+        them packed."""
+        key = window, keep, tile_rows
+        if key not in self._ranges:
+            self._ranges[key] = KeyRanges.of(self.portions, window, self.cu.device, keep, tile_rows)
+        return self._ranges[key]
 
 
 @dataclass

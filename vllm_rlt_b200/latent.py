@@ -92,7 +92,7 @@ def rotate_heads(src, dst, frequencies, positions, *, halves: bool = False, ampl
 
 
 def latent_gather(cache, tables, ranges):
-    """The cache rows of `ranges` (KeyRanges) side by side: `[ranges.rows, row width]`."""
+    """The cache rows of `ranges` (KeyRanges, with the first tokens it keeps) side by side: `[ranges.rows, row width]`."""
     _capi.require_cuda(cache, tables, ranges.first, ranges.cu)
     if cache.dim() != 4 or cache.shape[2] != 1 or cache.stride(3) != 1 or tables.dtype != torch.int32 or not tables.is_contiguous():
         raise ValueError("cache must be [pages, block, 1, width], tables contiguous int32 [sequences, pages]")
@@ -100,7 +100,7 @@ def latent_gather(cache, tables, ranges):
     with torch.cuda.device(cache.device):
         code = _capi.load().rlt_latent_gather(_capi.ptr(cache), cache.stride(0), cache.stride(1), cache.shape[0], cache.shape[1], cache.shape[3],
                                               _capi.ptr(tables), tables.shape[1], _capi.ptr(ranges.first), _capi.ptr(ranges.cu),
-                                              tables.shape[0], ranges.rows, _capi.ptr(out), _capi.DTYPE_CODES[cache.dtype],
+                                              tables.shape[0], ranges.rows, ranges.keep, _capi.ptr(out), _capi.DTYPE_CODES[cache.dtype],
                                               _capi.stream_of(cache))
     _capi.check(code, "latent_gather")
     return out

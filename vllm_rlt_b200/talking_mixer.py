@@ -1,9 +1,11 @@
 """Windowed attention with kept first tokens, bounded scores and heads that talk behind the softmax, as a mixer of the model classes.
 
     GEMM (q, k, v), norm_rotate (norms of q and k, rotation, keys and values to their pages), then
-    attention of every head over the values of every key/value head, head_mix;   GEMM (output)
+    long portions:  gathered keys and values of the window and the kept tokens, attention of every head over the values of every
+                    key/value head, head_mix, and
+    short ones:     the same over the pages, heads mixed where the splits of a context are merged;   GEMM (output)
 
-Every key and value stays in its page.
+Every key and value stays in its page.  32-bit models and sizes outside the kernels' alignment take the general attention and head_mix.
 """
 
 from __future__ import annotations
@@ -13,12 +15,16 @@ from dataclasses import dataclass
 import torch
 import torch.nn.functional as F
 
-from .attention import ScoreTerms
-from .latent import rotation_frequencies
-from .latent_mixer import RotationConfig
+from . import _capi
+from .attention import ScoreTerms, check_sink
+from .latent import latent_gather, rotation_frequencies
+from .latent_mixer import SHORT_PORTION, RotationConfig
 from .layers import head_mix, norm_rotate
 from .model_parts import check_positive, stack_blocks, take_keys
 from .sequence_cache import KVSpec
+
+
+PROMPT_ROWS = 128        # query rows of a tile of the prompt kernel
 
 
 @dataclass(frozen=True)
@@ -62,9 +68,76 @@ def talking_attention(kernels, q, key, value, out, group, terms: ScoreTerms, tal
     """Attention of a group's portions over the pages with score terms, heads mixed by `talk` (float32 `[heads, heads]`) behind the softmax;
     q `[rows, heads, dim]`, out `[rows, heads, vdim]` of the group's rows."""
     rows, heads, vdim = out.shape
-    spread = torch.empty(rows, heads, value.shape[2] * vdim, dtype=q.dtype, device=q.device)
-    kernels.scored(q, spread, key, value, group.tables, group.lengths, group.local_cu, group.max_new, terms, all_values=True)
-    return head_mix(spread, talk, out, value.shape[2])
+    kv_heads, dim = key.shape[2], q.shape[2]
+    shape = heads, kv_heads, dim, vdim, float(terms.softcap), _capi.DTYPE_CODES[q.dtype]
+    short = group.max_new <= SHORT_PORTION or group.portions is None
+    if short and _capi.load().rlt_talking_attention_supported(*shape):
+        return _over_pages(q, key, value, out, group, terms, talk)
+    spread = torch.empty(rows, heads, kv_heads * vdim, dtype=q.dtype, device=q.device)
+    if not short and _capi.load().rlt_talking_prompt_supported(*shape):
+        ranges = group.key_ranges(terms.window, terms.keep_first, PROMPT_ROWS)
+        keys, values = (latent_gather(cache.flatten(2).unsqueeze(2), group.tables, ranges) for cache in (key, value))
+        _over_packed(q, keys, values, spread, ranges, terms, kv_heads)
+    else:
+        kernels.scored(q, spread, key, value, group.tables, group.lengths, group.local_cu, group.max_new, terms, all_values=True)
+    return head_mix(spread, talk, out, kv_heads)
+
+
+def _check(q, out, terms: ScoreTerms, talk=None) -> None:
+    heads = q.shape[1]
+    check_sink(terms.head_scale, heads, "head_scale")
+    if terms.sink is not None or terms.distance_bias or terms.temp_coef:
+        raise ValueError("talking attention takes a window, kept first tokens, a soft cap and a scale per head")
+    if talk is not None and (talk.dtype != torch.float32 or talk.shape != (heads, heads) or not talk.is_contiguous()):
+        raise ValueError("talk must be contiguous float32 [heads, heads]")
+    if any(t.stride(2) != 1 or t.stride(1) != t.shape[2] for t in (q, out)) or out.dtype != q.dtype:
+        raise ValueError("q and out must have heads side by side and one dtype")
+
+
+def _over_pages(q, key, value, out, group, terms: ScoreTerms, talk):
+    """`rlt_talking_attention`: short portions over the pages."""
+    _capi.require_cuda(q, key, value, out, talk, terms.head_scale, group.tables, group.lengths, group.local_cu)
+    _check(q, out, terms, talk)
+    rows, heads, dim = q.shape
+    pages, block, kv_heads, vdim = value.shape
+    if key.shape != (pages, block, kv_heads, dim) or any(c.stride(3) != 1 or c.stride(2) != c.shape[3] or c.dtype != q.dtype for c in (key, value)):
+        raise ValueError("caches must be [pages, block, kv_heads, dim] of q's dtype with a contiguous tail")
+    if rows == 0:
+        return out
+    lib, width = _capi.load(), group.tables.shape[1]
+    seen = min(width * block, terms.window + terms.keep_first + group.max_new) if terms.window else width * block
+    sizes = rows, group.sequences, group.max_new, heads, kv_heads, dim, vdim, seen
+    with torch.cuda.device(q.device):
+        nbytes = lib.rlt_talking_attention_workspace_bytes(*sizes)
+        workspace = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
+        code = lib.rlt_talking_attention(
+            _capi.ptr(q), q.stride(0), _capi.ptr(out), out.stride(0), _capi.ptr(key), key.stride(0), key.stride(1), _capi.ptr(value), value.stride(0),
+            value.stride(1), pages, block, heads, kv_heads, dim, vdim, _capi.DTYPE_CODES[q.dtype], _capi.ptr(group.tables), group.sequences, width,
+            _capi.ptr(group.lengths), _capi.ptr(group.local_cu), rows, group.max_new, float(terms.scale), int(terms.window), int(terms.keep_first),
+            float(terms.softcap), _capi.ptr(terms.head_scale), _capi.ptr(talk), seen, _capi.ptr(workspace), nbytes, _capi.stream_of(q))
+    _capi.check(code, "talking_attention")
+    return out
+
+
+def _over_packed(q, keys, values, spread, ranges, terms: ScoreTerms, kv_heads: int):
+    """`rlt_talking_prompt`: long portions over packed keys `[ranges.rows, kv_heads * dim]` and values `[ranges.rows, kv_heads * vdim]`."""
+    _capi.require_cuda(q, keys, values, spread, terms.head_scale, ranges.tiles)
+    _check(q, spread, terms)
+    rows, heads, dim = q.shape
+    if keys.shape != (ranges.rows, kv_heads * dim) or values.shape[0] != ranges.rows or spread.shape != (rows, heads, values.shape[1]) \
+            or values.shape[1] % kv_heads or any(t.stride(1) != 1 or t.dtype != q.dtype for t in (keys, values)):
+        raise ValueError("keys [packed, kv_heads * dim], values [packed, kv_heads * vdim], spread [rows, heads, kv_heads * vdim] of one dtype")
+    if rows == 0:
+        return spread
+    workspace = torch.empty(256, dtype=torch.uint8, device=q.device)
+    with torch.cuda.device(q.device):
+        code = _capi.load().rlt_talking_prompt(
+            _capi.ptr(q), q.stride(0), _capi.ptr(keys), keys.stride(0), _capi.ptr(values), values.stride(0), _capi.ptr(spread), spread.stride(0), rows,
+            ranges.rows, heads, kv_heads, dim, values.shape[1] // kv_heads, _capi.ptr(ranges.tiles), ranges.tiles.shape[0], float(terms.scale),
+            int(terms.window), int(terms.keep_first), float(terms.softcap), _capi.ptr(terms.head_scale), _capi.DTYPE_CODES[q.dtype],
+            _capi.ptr(workspace), _capi.stream_of(q))
+    _capi.check(code, "talking_prompt")
+    return spread
 
 
 class TalkingAttention:
