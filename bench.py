@@ -1590,6 +1590,211 @@ def run_sandwich_workload(args):
     print(json.dumps(report))
 
 
+# Layer shapes of the postnorm workload: the windowed attention of the sandwich workload, recurrent layers with heads of the same size, and the
+# dense and mixture-of-experts feed-forwards of the stream workload.
+POSTNORM_SIZES = {
+    "2048": dict(width=2048, heads=16, kv_heads=4, rank=128, window=1024, keep=4, taps=4, ff=5632, experts=64, top=8, expert_ff=704, layers=8, vocab=49152),
+    "4096": dict(width=4096, heads=32, kv_heads=8, rank=128, window=1024, keep=4, taps=4, ff=9600, experts=32, top=4, expert_ff=2400, layers=6, vocab=49152),
+}
+
+
+def postnorm_config(size, pattern):
+    """config.json of a Degavik model whose layers repeat `pattern`: pairs of a mixer ('c' gated delta rule, 'r' retention, 't' talking attention)
+    and a feed-forward ('d' dense, 'e' experts with a shared one)."""
+    heads = size["heads"]
+    rot = {"base": 10000.0, "dims": HEAD_DIM}
+    mixers = {"c": ("channel_delta", {"heads": heads, "kv_heads": heads, "dim": HEAD_DIM, "vdim": HEAD_DIM, "conv": size["taps"]}),
+              "r": ("retention", {"heads": heads, "dim": HEAD_DIM, "vdim": HEAD_DIM, "rot": rot, "decay": [1 - 2.0 ** -(2 + 8 * h / heads) for h in range(heads)]}),
+              "t": ("attention", {"heads": heads, "kv_heads": size["kv_heads"], "dim": HEAD_DIM, "vdim": HEAD_DIM, "scale": HEAD_DIM ** -0.5, "softcap": 20.0,
+                                  "rot": dict(rot, dims=HEAD_DIM // 2), "mask": {"size": size["window"], "keep_first": size["keep"]}})}
+    feeds = {"d": {"kind": "dense", "ff": size["ff"]},
+             "e": {"kind": "moe", "router": {"experts": size["experts"], "top": size["top"]}, "expert": {"ff": size["expert_ff"]}, "shared": {"ff": size["expert_ff"]}}}
+    layers = []
+    for i in range(size["layers"]):
+        mixer, feed = pattern[i % len(pattern)]
+        layers.append({"type": mixers[mixer][0], "mixer": mixers[mixer][1], "mlp": feeds[feed]})
+    return {"architecture": "Degavik", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6}, "layers": layers}
+
+
+@torch.no_grad()
+def postnorm_kernel_rows(size, steps):
+    """Every kernel of a Degavik layer at prefill (16384 rows: 8 x 2048) and decode (64 rows, context 2048), with its algorithmic bytes
+    or flops against the measured peak, beside the like kernel of the nearest model (Kezuvik, Sugosun, Sobipel).  Talking attention's flops are
+    those of mixing the weights first: two products and a heads x heads matrix per pair."""
+    from types import SimpleNamespace
+
+    import vllm_rlt_b200 as rlt
+    from vllm_rlt_b200.engine import KeyRanges
+
+    device = torch.device("cuda", 0)
+    width, heads, kv_heads, rank, ff = (size[k] for k in ("width", "heads", "kv_heads", "rank", "ff"))
+    window, keep, taps, experts, top, expert_ff = (size[k] for k in ("window", "keep", "taps", "experts", "top", "expert_ff"))
+    inner, kv_inner = heads * HEAD_DIM, kv_heads * HEAD_DIM
+    bf16 = lambda *shape: torch.randn(*shape, device=device).to(torch.bfloat16)
+    f32 = lambda *shape: torch.randn(*shape, device=device)
+    add = KernelRows(steps)
+    terms = rlt.ScoreTerms(HEAD_DIM ** -0.5, window=window, keep_first=keep, softcap=20.0, head_scale=1 + 0.1 * f32(heads))
+    talk = torch.eye(heads, device=device) + 0.1 * f32(heads, heads)
+    for phase, seqs, new, context in (("prefill", 8, 2048, 2048), ("decode", 64, 1, 2048)):
+        rows, page = seqs * new, 64
+        pages = context // page
+        tables = torch.randperm(seqs * pages, device=device).int().view(seqs, pages)
+        lengths = torch.full((seqs,), context, dtype=torch.int32, device=device)
+        cu = (torch.arange(seqs + 1, device=device) * new).int()
+        positions = (torch.arange(rows, device=device) % new).int() + (context - new)
+        row_seq = torch.arange(seqs, device=device, dtype=torch.int32).repeat_interleave(new)
+        batch = SimpleNamespace(tables=tables[None], row_seq=row_seq, positions=positions)
+        group = SimpleNamespace(sequences=seqs, max_new=new, cu=cu, local_cu=cu, starts=lengths - new, slots=torch.arange(seqs, device=device, dtype=torch.int32),
+                                lengths=lengths, tables=tables, portions=[(0, new)] * seqs if new > 1 else None)
+        kernels = rlt.B200PagedAttention()
+        small = lambda nbytes: max(2, min(48, int(400e6 // nbytes) + 1))
+
+        # attention
+        seen = sum(min(p + 1, window) + max(min(keep, p + 1 - window), 0) for p in range(context - new, context)) * seqs
+        stored = seqs * min(context, new + window + keep - 1)
+        q, out = [bf16(rows, heads, HEAD_DIM) for _ in range(2)], bf16(rows, heads, HEAD_DIM)
+        kv_bytes, qo_bytes = stored * kv_inner * 4.0, rows * inner * 4.0
+        if new > 1:
+            ranges, plain_ranges = KeyRanges.of([(0, new)] * seqs, window, device, keep, 128), KeyRanges.of([(0, new)] * seqs, window, device)
+            k, v, gate = bf16(ranges.rows, kv_inner), bf16(ranges.rows, kv_inner), bf16(rows, inner)
+            spread = bf16(rows, heads, kv_inner)
+            add("talking attention, spread output", phase, "windowed attention (Kezuvik)",
+                lambda i: (lambda: rlt.talking_prompt(q[i % 2], k, v, spread, ranges, terms, kv_heads)), kv_bytes + qo_bytes, seen * heads * (4.0 * HEAD_DIM + 2 * heads), copies=4)
+            add("head_mix", phase, "head_gate (Kezuvik)", lambda i: (lambda: rlt.head_mix(spread, talk, out, kv_heads)), rows * (heads * kv_inner + inner) * 2.0, copies=2)
+
+            def whole(i):
+                def call():
+                    rlt.talking_prompt(q[i % 2], k, v, spread, ranges, terms, kv_heads)
+                    rlt.head_mix(spread, talk, out, kv_heads)
+                return call
+            add("talking attention and head_mix together", phase, "windowed attention (Kezuvik)", whole, kv_bytes + qo_bytes, seen * heads * (4.0 * HEAD_DIM + 2 * heads), copies=4)
+            cut = lambda t: t.unflatten(1, (kv_heads, HEAD_DIM))
+            add("windowed attention (Kezuvik)", phase, None,
+                lambda i: (lambda: rlt.packed_attention(q[i % 2], cut(k)[:plain_ranges.rows], cut(v)[:plain_ranges.rows], out, plain_ranges, HEAD_DIM ** -0.5, window, gate=gate)),
+                kv_bytes + 1.5 * qo_bytes, 4.0 * seen * inner, copies=4)
+            y = bf16(rows, heads, HEAD_DIM)
+            add("head_gate (Kezuvik)", phase, None, lambda i: (lambda: rlt.head_gate(y, gate)), rows * inner * 6.0, copies=2)
+            del k, v, gate, spread, y
+        else:
+            copies = small(kv_bytes)
+            pools = [bf16(2, seqs * pages, page, kv_heads, HEAD_DIM) for _ in range(copies)]
+            add("talking attention, heads mixed", phase, "windowed attention (Kezuvik)",
+                lambda i: (lambda: rlt.talking_attention(kernels, q[i % 2], pools[i][0], pools[i][1], out, group, terms, talk)), kv_bytes + qo_bytes, copies=copies)
+            plain = rlt.ScoreTerms(HEAD_DIM ** -0.5, window=window)
+            add("windowed attention (Kezuvik)", phase, None,
+                lambda i: (lambda: kernels.scored(q[i % 2], out, pools[i][0], pools[i][1], tables, lengths, cu, 1, plain)), kv_bytes + qo_bytes, copies=copies)
+            del pools
+        del q, out
+        channels = inner + 2 * kv_inner
+        copies = small(rows * channels * 2)
+        proj, q_out, cache = [bf16(rows, channels) for _ in range(copies)], bf16(rows, heads, HEAD_DIM), bf16(2, seqs * pages, page, kv_heads, HEAD_DIM)
+        norm_w, frequencies = f32(HEAD_DIM), rlt.rotation_frequencies(10000.0, HEAD_DIM // 2, device)
+        add("norm_rotate", phase, "conv_heads (Kezuvik)", lambda i: (lambda: rlt.norm_rotate(proj[i], (0, inner, inner + kv_inner), norm_w, norm_w, 1e-6, frequencies, q_out,
+                                                                                             cache[0], cache[1], batch)), rows * channels * 4.0, copies=copies)
+        weight, state = f32(taps, channels), torch.zeros(seqs, taps - 1, channels, dtype=torch.bfloat16, device=device)
+        add("conv_heads (Kezuvik)", phase, None, lambda i: (lambda: rlt.conv_heads(proj[i], (0, inner, inner + kv_inner), weight, 1e-6, state, q_out, cache[0], cache[1], group)),
+            rows * channels * 4.0 + (state.numel() * 4.0 if new == 1 else 0.0), copies=copies)
+        del proj, q_out, cache
+
+        # recurrent layers
+        copies = small(rows * inner * 8)
+        qkv, raw, beta, y = [bf16(rows, 3 * inner) for _ in range(copies)], [bf16(rows, inner) for _ in range(copies)], bf16(rows, heads), bf16(rows, inner)
+        thirds = lambda t: (t[:, :inner], t[:, inner:2 * inner], t[:, 2 * inner:])
+        sets = 2 if new > 1 else 4
+        dt_bias, a_log, states = f32(inner) - 3, f32(heads), [torch.zeros(seqs, heads, HEAD_DIM, HEAD_DIM, device=device) for _ in range(sets)]
+        add("delta_scan", phase, "ssd_scan (Sobipel)", lambda i: (lambda: rlt.delta_scan(*thirds(qkv[i % copies]), raw[i % copies], beta, dt_bias, a_log, states[i % sets], y, group)),
+            rows * (5 * inner + heads) * 2.0 + 2 * states[0].numel() * 4.0, copies=max(copies, 4))
+        table = rlt.decay_table([1 - 2.0 ** -(2 + 8 * h / heads) for h in range(heads)], device)
+        add("decay_scan", phase, "decay_scan (Sugosun: the same kernel)", lambda i: (lambda: rlt.decay_scan(*thirds(qkv[i % copies]), table, states[i % sets], y, group)),
+            rows * 4 * inner * 2.0 + 2 * states[0].numel() * 4.0, copies=max(copies, 4))
+        conv_w, conv_b, conv_state, mixed = f32(3 * inner, taps), f32(3 * inner), torch.zeros(seqs, taps - 1, 3 * inner, dtype=torch.bfloat16, device=device), bf16(rows, 3 * inner)
+        add("causal_conv", phase, "causal_conv (Sobipel: the same kernel)", lambda i: (lambda: rlt.causal_conv(qkv[i], conv_w, conv_b, conv_state, mixed, group)),
+            rows * 3 * inner * 4.0 + (conv_state.numel() * 4.0 if new == 1 else 0.0), copies=copies)
+        turn = rlt.rotation_frequencies(10000.0, HEAD_DIM, device)
+        pair = lambda t: t[:, :2 * inner].unflatten(1, (2 * heads, HEAD_DIM))
+        add("rotate_heads (halves, keys scaled)", phase, "rotate_heads (Kezuvik)", lambda i: (lambda: rlt.rotate_heads(
+            pair(qkv[i]), pair(qkv[i]), turn, positions, halves=True, scale=HEAD_DIM ** -0.5, scaled_from=heads)), rows * inner * 8.0, copies=copies)
+        add("rotate_heads (Kezuvik)", phase, None, lambda i: (lambda: rlt.rotate_heads(pair(qkv[i]), pair(qkv[i]), turn, positions, halves=True)), rows * inner * 8.0, copies=copies)
+        w_all, gated = f32(inner), bf16(rows, inner)
+        for name, like, weight, parts, gate in (("gated_norm per head (sigmoid)", "gated_norm (Sugosun)", w_all, heads, True), ("gated_norm per head (silu)", "gated_norm (Sugosun)", None, heads, "silu"),
+                                                ("gated_norm (Sugosun)", None, w_all, 1, True)):
+            add(name, phase, like, lambda i: (lambda: rlt.gated_norm(qkv[i][:, :inner], raw[i], weight, gated, parts, 1e-6, gate_behind=gate)), rows * inner * 6.0, copies=copies)
+        del qkv, raw, y, states, conv_state, mixed, gated
+        m_heads, vdim, n, groups = 2 * heads, 64, 128, 1 if heads == 16 else 8
+        x, dt, y = [bf16(rows, m_heads * vdim + 2 * groups * n) for _ in range(copies)], bf16(rows, m_heads), bf16(rows, m_heads * vdim)
+        ssm, dt_bias, a_log, d = [torch.zeros(seqs, m_heads, n, vdim, device=device) for _ in range(sets)], f32(m_heads) - 3, f32(m_heads), f32(m_heads)
+        add("ssd_scan (Sobipel)", phase, None, lambda i: (lambda: rlt.ssd_scan(*x[i % copies].split((m_heads * vdim, groups * n, groups * n), 1), dt, dt_bias, a_log, d, ssm[i % sets], y, group)),
+            rows * (2 * m_heads * vdim + 2 * groups * n + m_heads) * 2.0 + 2 * ssm[0].numel() * 4.0, copies=max(copies, 4))
+        del x, dt, y, ssm
+
+        # between the sublayers
+        copies = small(rows * width * 12.0)
+        residual, delta, w = [f32(rows, width) for _ in range(copies)], [bf16(rows, width) for _ in range(copies)], f32(width)
+        add("residual_norm, norm behind", phase, "residual_norm (Sobipel)", lambda i: (lambda: rlt.residual_norm(residual[i], None, 1e-6, torch.bfloat16, delta=delta[i], behind=(w, 1.0))),
+            rows * width * 12.0, copies=copies)
+        add("residual_norm (Sobipel)", phase, None, lambda i: (lambda: rlt.residual_norm(residual[i], w, 1e-6, torch.bfloat16, delta=delta[i])), rows * width * 12.0, copies=copies)
+        logits, bias = [f32(rows, experts) for _ in range(4)], 0.1 * f32(experts)
+        routing = rlt.expert_route(logits[0], None, top, bias=bias, floor_sum=0.0)
+        add("expert_route (biased logits)", phase, "expert_route (Sugosun)", lambda i: (lambda: rlt.expert_route(logits[i % 4], None, top, bias=bias, floor_sum=0.0)), rows * (experts * 4.0 + top * 12), copies=8)
+        add("expert_route (Sugosun)", phase, None, lambda i: (lambda: rlt.expert_route(logits[i % 4], bias, top)), rows * (experts * 4.0 + top * 12), copies=8)
+        x = rlt.expert_gather(delta[0], routing)
+        parts = (bf16(rows * top, width), routing.places, routing.weights)
+        add("residual_norm, norm behind experts and a shared one", phase, "residual_norm (Sobipel)",
+            lambda i: (lambda: rlt.residual_norm(residual[i], None, 1e-6, torch.bfloat16, delta=delta[i], parts=parts, behind=(w, 1.0))), rows * width * (12.0 + 2 * top), copies=copies)
+        del residual, delta, parts
+        used = int((routing.counts > 0).sum())
+        nbytes, flops = used * width * expert_ff * 2.0 + rows * top * (width + expert_ff) * 2.0, 2.0 * rows * top * width * expert_ff
+        wide, downs = [bf16(experts, 2 * expert_ff, width) for _ in range(2)], [bf16(experts, width, expert_ff) for _ in range(2)]
+        add("expert_gemm, gate and up in pairs", phase, "expert_gemm, up and squared relu (Sugosun)",
+            lambda i: (lambda: rlt.expert_gemm(x, wide[i % 2], routing.counts, "silu", paired=True)), nbytes + used * width * expert_ff * 2.0, 2 * flops, copies=4)
+        add("expert_gemm, up and squared relu (Sugosun)", phase, None, lambda i: (lambda: rlt.expert_gemm(x, wide[i % 2], routing.counts, "squared_relu")),
+            2 * nbytes - rows * top * width * 2.0, 2 * flops, copies=4)
+        act = bf16(rows * top, expert_ff)
+        add("expert_gemm, down", phase, "expert_gemm, up and squared relu (Sugosun)", lambda i: (lambda: rlt.expert_gemm(act, downs[i % 2], routing.counts)), nbytes, flops, copies=4)
+        del x, act, wide, downs
+        copies = small(rows * ff * 6)
+        gate_up = [bf16(rows, 2 * ff) for _ in range(copies)]
+        add("gated_unit (silu)", phase, "gated_unit (Kezuvik)", lambda i: (lambda: rlt.gated_unit(gate_up[i], ff, ff, "silu")), rows * ff * 6.0, copies=copies)
+        add("gated_unit (Kezuvik)", phase, None, lambda i: (lambda: rlt.gated_unit(gate_up[i], ff, ff, "gelu_tanh")), rows * ff * 6.0, copies=copies)
+        del gate_up
+    return add.rows
+
+
+def run_postnorm_workload(args):
+    """`--workload postnorm`: one JSON line with throughput rows, kernel rows and the clocks under them."""
+    import vllm_rlt_b200 as rlt
+    from vllm_rlt_b200.hybrid_lm import parameter_shapes as hybrid_shapes
+    from vllm_rlt_b200.postnorm_lm import parameter_shapes as postnorm_shapes
+    from vllm_rlt_b200.sandwich_lm import parameter_shapes as sandwich_shapes
+    from vllm_rlt_b200.stream_lm import parameter_shapes as stream_shapes
+
+    torch.cuda.set_device(0)
+    device = torch.device("cuda", 0)
+    report = {"workload": "postnorm", "data": "synthetic, random weights", "dtype": "bf16", "steps": args.steps, "sizes": {}}
+    with ClockSampler(0) as clocks:
+        for name, size in POSTNORM_SIZES.items():
+            rows = []
+            builds = [(f"Degavik, {label}", lambda pattern=pattern: rlt.PostNormLM(config := rlt.PostNormLMConfig.from_json(postnorm_config(size, pattern)),
+                                                                                   device_weights(postnorm_shapes(config, lambda tensor: size["rank"]), device), device))
+                      for label, pattern in (("gated delta rule and dense", ["cd"]), ("retention and dense", ["rd"]), ("talking attention and dense", ["td"]),
+                                             ("talking attention and experts", ["te"]), ("2 delta, attention, retention, half experts", ["cd", "te", "rd", "ce"]))]
+            builds.append(("Kezuvik, windowed attention", lambda: rlt.SandwichLM(
+                config := rlt.SandwichLMConfig.from_json(sandwich_config(SANDWICH_SIZES[name], "w")), device_weights(sandwich_shapes(config), device), device)))
+            builds.append(("Sugosun, lightning and dense", lambda: rlt.StreamLM(
+                config := rlt.StreamLMConfig.from_json(stream_config(STREAM_SIZES[name], ["ld"])), device_weights(stream_shapes(config), device), device)))
+            builds.append(("Sobipel, Mamba-2 layers", lambda: rlt.HybridLM(
+                config := rlt.HybridLMConfig.from_json(hybrid_config(dict(HYBRID_SIZES[name], layers=size["layers"]), "m")), device_weights(hybrid_shapes(config), device), device)))
+            for label, build in builds:
+                model = build()
+                rows += hybrid_model_rows(label, model, args.steps, args.warmup)
+                del model
+                torch.cuda.empty_cache()
+            report["sizes"][name] = {"shape": dict(size), "throughput": rows, "kernels": postnorm_kernel_rows(size, args.steps)}
+            torch.cuda.empty_cache()
+    report["clocks"] = clocks.summary()
+    print(json.dumps(report))
+
+
 def balanced_shards(lengths, world: int):
     """Longest-first greedy assignment of requests to ranks by prompt length: returns one list of request
     indices per rank whose total lengths differ by at most one request's length."""
@@ -1882,7 +2087,7 @@ def main():
     parser.add_argument("--no-cpu-baseline", action="store_true")
     parser.add_argument("--only", default=None, choices=["attention", "accept", "silu", "prefill"],
                         help="profiling aid: run only this kernel family (not a bench line)")
-    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded", "hybrid", "stream", "sandwich"],
+    parser.add_argument("--workload", default="rounds", choices=["rounds", "decode", "sharded", "hybrid", "stream", "sandwich", "postnorm"],
                         help="rounds: timed speculative rounds (the bench line); decode: one complete generation; "
                              "sharded: a fixed request set shared out over the ranks, decoded to completion")
     parser.add_argument("--engine", default="b200", choices=["b200", "reference"],
@@ -1930,6 +2135,9 @@ def main():
             setattr(args, name, sharded_default if sharded else decode_default)
     if sharded:
         run_sharded_workload(args)
+        return
+    if args.workload == "postnorm":
+        run_postnorm_workload(args)
         return
     if args.workload == "sandwich":
         run_sandwich_workload(args)

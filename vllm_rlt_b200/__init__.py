@@ -30,6 +30,7 @@ from .runner import (B200SpeculativeRunner, KVCacheManagerView, ModelRunnerOutpu
                      SchedulerOutput, SpeculativeConfig, SpeculativeRoundTicket, SpeculativeStats)
 from .sandwich_lm import SandwichLM, SandwichLMConfig
 from .stream_lm import StreamLM, StreamLMConfig
+from .talking_mixer import talking_attention, talking_decode, talking_prompt
 from .sequence_cache import CacheFull, CacheSpec, KVSpec, SequenceCache, StateSpec
 from .speculative import (PipelineState, SpeculativeResult, accept_greedy, accept_rejection, argmax_rows,
                           decode_result, pipeline_shift, probabilities, raise_for_status, round_uniforms,
@@ -50,4 +51,5 @@ __all__ = [
     "latent_gather", "latent_prompt_attention", "latent_prompt_supported", "latent_write", "rotate_heads", "rotation_frequencies", "stream_mix",
     "SandwichLM", "SandwichLMConfig", "YarnScaling", "conv_heads", "gated_unit", "head_gate", "packed_attention", "soft_cap",
     "PostNormLM", "PostNormLMConfig", "delta_scan", "head_mix", "norm_rotate", "paired_rows",
+    "talking_attention", "talking_decode", "talking_prompt",
 ]

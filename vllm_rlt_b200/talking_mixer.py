@@ -72,12 +72,12 @@ def talking_attention(kernels, q, key, value, out, group, terms: ScoreTerms, tal
     shape = heads, kv_heads, dim, vdim, float(terms.softcap), _capi.DTYPE_CODES[q.dtype]
     short = group.max_new <= SHORT_PORTION or group.portions is None
     if short and _capi.load().rlt_talking_attention_supported(*shape):
-        return _over_pages(q, key, value, out, group, terms, talk)
+        return talking_decode(q, key, value, out, group, terms, talk)
     spread = torch.empty(rows, heads, kv_heads * vdim, dtype=q.dtype, device=q.device)
     if not short and _capi.load().rlt_talking_prompt_supported(*shape):
         ranges = group.key_ranges(terms.window, terms.keep_first, PROMPT_ROWS)
         keys, values = (latent_gather(cache.flatten(2).unsqueeze(2), group.tables, ranges) for cache in (key, value))
-        _over_packed(q, keys, values, spread, ranges, terms, kv_heads)
+        talking_prompt(q, keys, values, spread, ranges, terms, kv_heads)
     else:
         kernels.scored(q, spread, key, value, group.tables, group.lengths, group.local_cu, group.max_new, terms, all_values=True)
     return head_mix(spread, talk, out, kv_heads)
@@ -94,7 +94,7 @@ def _check(q, out, terms: ScoreTerms, talk=None) -> None:
         raise ValueError("q and out must have heads side by side and one dtype")
 
 
-def _over_pages(q, key, value, out, group, terms: ScoreTerms, talk):
+def talking_decode(q, key, value, out, group, terms: ScoreTerms, talk):
     """`rlt_talking_attention`: short portions over the pages."""
     _capi.require_cuda(q, key, value, out, talk, terms.head_scale, group.tables, group.lengths, group.local_cu)
     _check(q, out, terms, talk)
@@ -119,7 +119,7 @@ def _over_pages(q, key, value, out, group, terms: ScoreTerms, talk):
     return out
 
 
-def _over_packed(q, keys, values, spread, ranges, terms: ScoreTerms, kv_heads: int):
+def talking_prompt(q, keys, values, spread, ranges, terms: ScoreTerms, kv_heads: int):
     """`rlt_talking_prompt`: long portions over packed keys `[ranges.rows, kv_heads * dim]` and values `[ranges.rows, kv_heads * vdim]`."""
     _capi.require_cuda(q, keys, values, spread, terms.head_scale, ranges.tiles)
     _check(q, spread, terms)
