@@ -721,9 +721,9 @@ RLT_API int rlt_head_mix(const void* y, int64_t y_stride, const float* talk, voi
  * [rows][heads][kv_heads * value_dim] receives every head over the values of every key/value head (rlt_head_mix takes it).  tiles as in
  * rlt_latent_prompt_attention, at most 128 rows each, with the number of kept positions in front of the packed row in the sixth word.
  * workspace: 256 bytes, the first word is set when a bounded wait gave up. */
-RLT_API int rlt_talking_attention_supported(int heads, int kv_heads, int dim, int value_dim, float softcap, int dtype);
+RLT_API int rlt_talking_attention_supported(int heads, int kv_heads, int dim, int value_dim, int block_size, float softcap, int dtype);
 RLT_API size_t rlt_talking_attention_workspace_bytes(int rows, int sequences, int max_new, int heads, int kv_heads, int dim, int value_dim,
-                                             int64_t keys);
+                                             int block_size, int64_t keys);
 RLT_API int rlt_talking_attention(const void* q, int64_t q_stride, void* out, int64_t out_stride, const void* key_cache, int64_t k_block_stride,
                           int64_t k_token_stride, const void* value_cache, int64_t v_block_stride, int64_t v_token_stride, int64_t num_blocks,
                           int block_size, int heads, int kv_heads, int dim, int value_dim, int dtype, const int32_t* block_tables, int sequences,

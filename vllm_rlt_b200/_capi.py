@@ -84,8 +84,8 @@ SIGNATURES = {
     "rlt_norm_rotate": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _P, _L, _P, _L, _L, _P, _L, _L, _L, _I, _P, _I,
                              _I, _I, _P]),
     "rlt_head_mix": (_I, [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P]),
-    "rlt_talking_attention_supported": (_I, [_I, _I, _I, _I, _F, _I]),
-    "rlt_talking_attention_workspace_bytes": (_Z, [_I, _I, _I, _I, _I, _I, _I, _L]),
+    "rlt_talking_attention_supported": (_I, [_I, _I, _I, _I, _I, _F, _I]),
+    "rlt_talking_attention_workspace_bytes": (_Z, [_I, _I, _I, _I, _I, _I, _I, _I, _L]),
     "rlt_talking_attention": (_I, [_P, _L, _P, _L, _P, _L, _L, _P, _L, _L, _L, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _I, _I, _F, _I, _I, _F,
                                    _P, _P, _L, _P, _Z, _P]),
     "rlt_talking_prompt_supported": (_I, [_I, _I, _I, _I, _F, _I]),

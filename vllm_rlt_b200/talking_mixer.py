@@ -69,12 +69,12 @@ def talking_attention(kernels, q, key, value, out, group, terms: ScoreTerms, tal
     q `[rows, heads, dim]`, out `[rows, heads, vdim]` of the group's rows."""
     rows, heads, vdim = out.shape
     kv_heads, dim = key.shape[2], q.shape[2]
-    shape = heads, kv_heads, dim, vdim, float(terms.softcap), _capi.DTYPE_CODES[q.dtype]
+    sizes, rest = (heads, kv_heads, dim, vdim), (float(terms.softcap), _capi.DTYPE_CODES[q.dtype])
     short = group.max_new <= SHORT_PORTION or group.portions is None
-    if short and _capi.load().rlt_talking_attention_supported(*shape):
+    if short and _capi.load().rlt_talking_attention_supported(*sizes, key.shape[1], *rest):
         return talking_decode(q, key, value, out, group, terms, talk)
     spread = torch.empty(rows, heads, kv_heads * vdim, dtype=q.dtype, device=q.device)
-    if not short and _capi.load().rlt_talking_prompt_supported(*shape):
+    if not short and _capi.load().rlt_talking_prompt_supported(*sizes, *rest):
         ranges = group.key_ranges(terms.window, terms.keep_first, PROMPT_ROWS)
         keys, values = (latent_gather(cache.flatten(2).unsqueeze(2), group.tables, ranges) for cache in (key, value))
         talking_prompt(q, keys, values, spread, ranges, terms, kv_heads)
@@ -106,7 +106,7 @@ def talking_decode(q, key, value, out, group, terms: ScoreTerms, talk):
         return out
     lib, width = _capi.load(), group.tables.shape[1]
     seen = min(width * block, terms.window + terms.keep_first + group.max_new) if terms.window else width * block
-    sizes = rows, group.sequences, group.max_new, heads, kv_heads, dim, vdim, seen
+    sizes = rows, group.sequences, group.max_new, heads, kv_heads, dim, vdim, block, seen
     with torch.cuda.device(q.device):
         nbytes = lib.rlt_talking_attention_workspace_bytes(*sizes)
         workspace = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
