@@ -1,17 +1,14 @@
 // Prompt attention with bounded scores over packed keys and values, every head applied to the values of every key/value head, on the
 // 5th-generation tensor cores, bf16 (head_mix.cu says what the spread output is for): windows with kept first tokens.
 //
-// Scores are bounded by the soft cap, so weights are exp(score) as they are: no running maximum, no rescaling of the output, and four groups
-// of softmax warps can take the stages of keys in turn.  128 query tokens of one head per CTA, up to 256 columns of the values of all
-// key/value heads (several CTAs along the columns otherwise), 19 warps:
-//   warps 4 i .. 4 i + 3  the softmax rows (row = TMEM lane) of stages i, i + 4, ..
-//   warp 16               issues Q K^T into the stage's scores,      warp 17  O += P V
-//   warp 18               the copies: Q once, then the stages of 64 keys
-// TMEM columns: 64 for the scores of each group, whose first half the weights overwrite, and O from 256 on.
-//
-// Where two query heads share a key/value head, their CTAs work as a pair on the same query tokens (talking_pair_kernel): one product of 256
-// rows for both, each CTA copying half of the stage's keys and half of the value columns.  The copies are what this attention is bound by:
-// a stage's values serve one head of 128 tokens only.  The CTA of rank 0 issues; the other one's warps 16 and 17 pass on what has arrived.
+// Scores are bounded by the soft cap, so weights are exp(score) as they are: no running maximum, no rescaling of the output, and groups of
+// softmax warps can take the stages of keys in turn.  An item is 128 query tokens of one head and up to 256 columns of the values of all
+// key/value heads; a CTA per SM goes from item to item.  Stages are counted through all of them, so copies and scores of the next item run
+// under the end of the one before; only its O += P V waits until O has been read.  11 warps:
+//   warps 0..3, 4..7  the softmax rows (row = TMEM lane) of every second stage
+//   warp 8            issues Q K^T into the stage's scores,      warp 9  O += P V
+//   warp 10           the copies: Q of every item, then its stages of 64 keys
+// TMEM columns: four buffers of 64 for the scores of a stage, whose first half its weights overwrite, and O from 256 on.
 //
 // Stages hold first the kept keys that lie in front of every row's window, then the window's keys from the first one that any row sees.
 #include "latent_attention.cuh"
@@ -22,15 +19,18 @@ namespace rlt {
 namespace {
 
 constexpr int kRows = 128, kKeys = 64;
-constexpr int kSides = 4;                                        // groups of softmax warps
+constexpr int kSides = 2;                                        // groups of softmax warps
+constexpr int kBuffers = 4;                                      // of scores: a group's next ones are ready when it comes to them
 constexpr int kSoftmaxWarps = kSides * 4, kThreads = (kSoftmaxWarps + 3) * 32;
 constexpr int kBlock = kKeys * 128, kQBlock = kRows * 128;       // 64-wide blocks of a stage's operand and of Q
-constexpr int kMaxBlocks = 4;                                    // of value columns per CTA
-constexpr uint32_t kColumns = 512, kSideCols = 64, kColO = 256;
+constexpr int kStaging = 32 * 64;                                // 32 output rows of 32 columns per warp
+constexpr int kMaxBlocks = 4;                                    // of value columns per item
+constexpr uint32_t kColumns = 512, kBufferCols = 64, kColO = 256;
 
 struct TalkingPromptArgs {
   __nv_bfloat16* out; int64_t out_stride;        // [rows][heads][columns]
   const PromptTile* tiles;
+  int slabs, items;                              // tiles x heads x slabs, the last fastest
   int heads, share, columns;                     // columns of the values of all key/value heads
   int window, keep;
   float factor, cap_log2;                        // tanh argument per unit of q . k and head scale; the cap in log2 units
@@ -41,57 +41,71 @@ struct TalkingPromptArgs {
 template <int kK, int kV>
 struct SpreadShared {
   static constexpr int kStageBytes = (kK + kV) * kBlock;
-  static constexpr int kFit = (222 * 1024 - kK * kQBlock) / kStageBytes;
+  static constexpr int kFit = (220 * 1024 - kK * kQBlock - kSoftmaxWarps * kStaging) / kStageBytes;
   static constexpr int kStages = kFit < 6 ? kFit : 6;
-  static_assert(kStages >= 3 && kStages * kStageBytes + kK * kQBlock >= kSoftmaxWarps * 4096, "the output is staged where Q, keys and values were");
+  static_assert(kStages >= 3, "copies run ahead of the products");
   unsigned char q[kK][kQBlock];
   unsigned char k[kStages][kK][kBlock];
   unsigned char v[kStages][kV][kBlock];
-  unsigned long long full_q, full_k[kStages], full_v[kStages], free_k[kStages], free_v[kStages];
-  unsigned long long s_ready[kSides], p_ready[kSides], p_free[kSides], o_done;
-  float sums[kSides][kRows];
+  unsigned char staging[kSoftmaxWarps][kStaging];
+  unsigned long long full_q, q_free, full_k[kStages], full_v[kStages], free_k[kStages], free_v[kStages];
+  unsigned long long s_ready[kBuffers], p_ready[kBuffers], p_free[kBuffers], o_done, o_free;
+  float sums[2][kSides][kRows];                  // of this item and the one before
   uint32_t tmem_base;
 };
 
-// cap tanh(x) in log2 units of 32 scores with arguments x = s factor.  tanh(x) = 1 - 2 / (e^2x + 1); where no argument exceeds one, x
-// times a polynomial in x^2 instead (a minimax fit, relative error 5e-8): multiplications, and the special-function unit is left to
-// the exponentials.
-__device__ __forceinline__ void bounded_scores(float (&s)[32], float factor, float cap_log2) {
+// exp(cap tanh(x)) by a polynomial: tanh(x) is x times a polynomial in x^2 where |x| does not exceed what it was fitted for.  Products of
+// pairs and exponentials alternate, so both units are busy.
+template <int kTerms>
+__device__ __forceinline__ void polynomial_weights(float (&s)[32], const float (&fit)[kTerms], float factor, float cap_log2) {
+  float2 c[kTerms];
+#pragma unroll
+  for (int i = 0; i < kTerms; ++i) c[i] = make_float2(fit[i] * cap_log2, fit[i] * cap_log2);
+  const float2 f = make_float2(factor, factor);
+#pragma unroll
+  for (int e = 0; e < 32; e += 2) {
+    const float2 x = mul_pair(make_float2(s[e], s[e + 1]), f), y = mul_pair(x, x);
+    float2 p = c[kTerms - 1];
+#pragma unroll
+    for (int i = kTerms - 2; i >= 0; --i) p = fma_pair(p, y, c[i]);
+    p = mul_pair(p, x);
+    s[e] = fast_exp2(p.x);
+    s[e + 1] = fast_exp2(p.y);
+  }
+}
+// The weights exp(cap tanh(x)) of 32 scores, x = s factor.  tanh(x) = 1 - 2 / (e^2x + 1) takes two operations of the special-function unit, which
+// the exponentials need already; where no argument of the warp exceeds 0.6 (or 1), a minimax polynomial of relative error 7e-8 (5e-8) instead.
+__device__ __forceinline__ void bounded_weights(float (&s)[32], float factor, float cap_log2) {
   float top[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
   for (int e = 0; e < 32; e += 8)
 #pragma unroll
     for (int c = 0; c < 4; ++c) top[c] = max3(top[c], fabsf(s[e + 2 * c]), fabsf(s[e + 2 * c + 1]));
   const float most = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3])) * fabsf(factor);
-  if (__all_sync(0xffffffffu, most <= 1.0f)) {
+  if (__all_sync(0xffffffffu, most <= 0.6f)) {
+    constexpr float kFit[5] = {0.9999999269f, -0.3333230997f, 0.1331017365f, -0.05210147962f, 0.01547542681f};
+    polynomial_weights(s, kFit, factor, cap_log2);
+  } else if (__all_sync(0xffffffffu, most <= 1.0f)) {
     constexpr float kFit[7] = {0.9999999502f, -0.3333283915f, 0.1332520406f, -0.05345702907f, 0.02028997947f, -0.006203378259f, 0.001041022353f};
-    const float2 f2 = make_float2(factor, factor);
-    const float2 c2 = make_float2(cap_log2, cap_log2);
-#pragma unroll
-    for (int e = 0; e < 32; e += 2) {
-      const float2 x = mul_pair(make_float2(s[e], s[e + 1]), f2), y = mul_pair(x, x);
-      float2 p = make_float2(kFit[6], kFit[6]);
-#pragma unroll
-      for (int i = 5; i >= 0; --i) p = fma_pair(p, y, make_float2(kFit[i], kFit[i]));
-      p = mul_pair(p, mul_pair(x, c2));
-      s[e] = p.x; s[e + 1] = p.y;
-    }
+    polynomial_weights(s, kFit, factor, cap_log2);
   } else {
     const float twice = 2.0f * kLog2e * factor;
 #pragma unroll
     for (int e = 0; e < 32; ++e) {
       const float u = fast_exp2(fminf(s[e] * twice, 100.0f));
-      s[e] = cap_log2 * (1.0f - __fdividef(2.0f, u + 1.0f));
+      s[e] = fast_exp2(cap_log2 * (1.0f - __fdividef(2.0f, u + 1.0f)));
     }
   }
 }
 
-// What a CTA walks over.
+// An item and its stages.
 struct Walk {
   PromptTile tile;
-  int window, count, from, kept, kept_stages, stages;
+  int head, slab0, window, count, from, kept, kept_stages, stages;
 
-  __device__ __forceinline__ Walk(const TalkingPromptArgs& a, int index) : tile(a.tiles[index]) {
+  __device__ __forceinline__ Walk(const TalkingPromptArgs& a, int item, int slab_columns) : tile(a.tiles[item / a.slabs / a.heads]) {
+    head = item / a.slabs % a.heads;
+    slab0 = item % a.slabs * slab_columns;
     window = a.window > 0 ? a.window : 0x40000000;
     count = min(tile.count, kRows);
     // positions: kept ones 0 .. kept - 1 in stages 0 .. kept_stages - 1, then from .. last in the others
@@ -105,99 +119,6 @@ struct Walk {
   }
 };
 
-// The softmax rows of every fourth stage, then a block of 64 output columns per group.  p_ready(side): the weights of a stage are stored.
-template <int kV, typename Shared, typename Ready>
-__device__ __forceinline__ bool softmax_rows(Shared& sm, const TalkingPromptArgs& a, const Walk& w, uint32_t tmem, int head, int slab0, Ready p_ready) {
-  const int lane = threadIdx.x & 31, warp = __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0);
-  const PromptTile& tile = w.tile;
-  const int count = w.count, window = w.window, kept = w.kept, kept_stages = w.kept_stages, from = w.from, stages = w.stages;
-  bool failed = false;
-  auto wait_all = [&](unsigned long long* bar, uint32_t parity) {
-    const bool ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(bar), parity));
-    tcgen05_after_sync();
-    return ok;
-  };
-  const int side = warp >> 2, warp_row = (warp & 3) * 32, row = warp_row + lane;
-  const bool live = row < count;
-  const int position = tile.position + row;
-  const int seen_end = live ? position + 1 : 0, seen_begin = position - window + 1;   // keys seen_begin .. seen_end - 1, and those below keep
-  const uint32_t tmem_row = tmem + (static_cast<uint32_t>(warp_row) << 16), s_col = tmem_row + side * kSideCols;
-  const float factor = a.factor * (a.head_scale != nullptr ? a.head_scale[head] : 1.0f);
-  float2 sum4[4] = {{0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}};
-  for (int j = side; j < stages; j += kSides) {
-    if (!wait_all(&sm.s_ready[side], (j / kSides) & 1)) { failed = true; break; }
-    const bool in_kept = j < kept_stages;
-    const int end = in_kept ? (live ? kept : 0) : seen_end;
-    uint32_t packed[32];
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      float s[32];
-      {
-        uint32_t r[32];
-        tmem_load32(s_col + half * 32, r);
-        tmem_load_wait();
-#pragma unroll
-        for (int e = 0; e < 32; ++e) s[e] = __uint_as_float(r[e]);
-      }
-      bounded_scores(s, factor, a.cap_log2);
-      const int first_key = (in_kept ? j * kKeys : from + (j - kept_stages) * kKeys) + half * 32;
-      if (first_key + 32 > end) {
-#pragma unroll
-        for (int e = 0; e < 32; ++e)
-          if (first_key + e >= end) s[e] = -INFINITY;
-      }
-      if (!in_kept && first_key < seen_begin) {
-#pragma unroll
-        for (int e = 0; e < 32; ++e)
-          if (first_key + e < seen_begin && first_key + e >= a.keep) s[e] = -INFINITY;
-      }
-#pragma unroll
-      for (int e = 0; e < 16; ++e) {
-        const float2 p = make_float2(fast_exp2(s[2 * e]), fast_exp2(s[2 * e + 1]));
-        sum4[e & 3] = add_pair(sum4[e & 3], p);
-        packed[half * 16 + e] = pack2<true>(p.x, p.y);
-      }
-    }
-    tmem_store32(s_col, packed);
-    tmem_store_wait();
-    tcgen05_before_sync();
-    __syncwarp();
-    if (lane == 0) p_ready(side);
-  }
-  const float2 sum2 = add_pair(add_pair(sum4[0], sum4[1]), add_pair(sum4[2], sum4[3]));
-  sm.sums[side][row] = sum2.x + sum2.y;
-  if (!failed && !wait_all(&sm.o_done, 0)) failed = true;
-  asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxWarps * 32) : "memory");
-  failed = __any_sync(0xffffffffu, failed);
-  if (!failed && side < kV) {
-    // a block of 64 output columns per group, through shared memory that nothing reads any more
-    const float total = (sm.sums[0][row] + sm.sums[1][row]) + (sm.sums[2][row] + sm.sums[3][row]), inv = total > 0.0f ? 1.0f / total : 0.0f;
-    unsigned char* staging = &sm.q[0][0] + warp * 4096;
-    const int64_t first_out = static_cast<int64_t>(tile.q_row) + warp_row;
-    const int warp_count = min(max(count - warp_row, 0), 32);
-    __nv_bfloat16* dst = a.out + first_out * a.out_stride + static_cast<int64_t>(head) * a.columns + slab0 + side * 64;
-    uint32_t r0[32], r1[32];
-    tmem_load32(tmem_row + kColO + side * 64, r0);
-    tmem_load32(tmem_row + kColO + side * 64 + 32, r1);
-    tmem_load_wait();
-#pragma unroll
-    for (int c = 0; c < 8; ++c) {
-      const float* f = reinterpret_cast<const float*>(c < 4 ? &r0[c * 8] : &r1[(c - 4) * 8]);
-      *reinterpret_cast<uint4*>(staging + lane * 128 + ((c ^ (lane & 7)) << 4)) =
-          make_uint4(pack2<true>(f[0] * inv, f[1] * inv), pack2<true>(f[2] * inv, f[3] * inv),
-                     pack2<true>(f[4] * inv, f[5] * inv), pack2<true>(f[6] * inv, f[7] * inv));
-    }
-    __syncwarp();
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int r = 4 * i + (lane >> 3);
-      if (r < warp_count && slab0 + side * 64 + (lane & 7) * 8 < a.columns)
-        reinterpret_cast<uint4*>(dst + r * a.out_stride)[lane & 7] = *reinterpret_cast<const uint4*>(staging + r * 128 + (((lane & 7) ^ (r & 7)) << 4));
-    }
-  }
-  return failed;
-}
-
 template <int kK, int kV>
 __global__ void __launch_bounds__(kThreads, 1)
 talking_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
@@ -207,21 +128,20 @@ talking_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
   extern __shared__ unsigned char smem_raw[];
   Shared& sm = *reinterpret_cast<Shared*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const int lane = threadIdx.x & 31, warp = __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0);
-  const int head = blockIdx.x, slab0 = blockIdx.y * kV * 64;     // neighbouring CTAs read the same keys and values
-  const Walk w(a, blockIdx.z);
-  const int stages = w.stages;
 
-  if ((blockIdx.x | blockIdx.y | blockIdx.z) == 0 && threadIdx.x == 0) *a.error = 0;   // a wait gives up seconds later
+  if (blockIdx.x == 0 && threadIdx.x == 0) *a.error = 0;   // a wait gives up seconds later
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(&sm.full_q), 1);
+    mbar_init(smem_u32(&sm.q_free), 1);
     mbar_init(smem_u32(&sm.o_done), 1);
+    mbar_init(smem_u32(&sm.o_free), kSoftmaxWarps);
     for (int s = 0; s < kStages; ++s) {
       mbar_init(smem_u32(&sm.full_k[s]), 1);
       mbar_init(smem_u32(&sm.full_v[s]), 1);
       mbar_init(smem_u32(&sm.free_k[s]), 1);
       mbar_init(smem_u32(&sm.free_v[s]), 1);
     }
-    for (int b = 0; b < kSides; ++b) {
+    for (int b = 0; b < kBuffers; ++b) {
       mbar_init(smem_u32(&sm.s_ready[b]), 1);
       mbar_init(smem_u32(&sm.p_ready[b]), kRows / 32);
       mbar_init(smem_u32(&sm.p_free[b]), 1);
@@ -239,67 +159,189 @@ talking_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
   constexpr uint32_t kIdesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kRows >> 4) << 24);
   constexpr uint32_t kIdescQK = kIdesc | (static_cast<uint32_t>(kKeys >> 3) << 17);                     // N = 64 keys
   constexpr uint32_t kIdescPV = kIdesc | (static_cast<uint32_t>(kV * 64 >> 3) << 17) | (1u << 16);       // N = value columns, B MN-major
-  bool failed = false;
+  bool failed = false;       // a wait that gave up is a role's last one
   auto wait_all = [&](unsigned long long* bar, uint32_t parity) {
-    const bool ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(bar), parity));
+    if (!failed && !__all_sync(0xffffffffu, mbar_wait(smem_u32(bar), parity))) failed = true;
     tcgen05_after_sync();
-    return ok;
+    return !failed;
   };
+  int done = 0;              // stages of the items before
 
   if (warp == kSoftmaxWarps + 2) {
     if (lane == 0) {
-      mbar_expect_tx(smem_u32(&sm.full_q), kK * kQBlock);
+      auto wait = [&](unsigned long long* bar, int use) {        // for the use before this one to be over
+        if (use > 0 && !mbar_wait(smem_u32(bar), (use - 1) & 1)) failed = true;
+        return !failed;
+      };
+      for (int item = blockIdx.x, n = 0; item < a.items && !failed; item += gridDim.x, ++n) {
+        const Walk w(a, item, kV * 64);
+        if (!wait(&sm.q_free, n)) break;
+        mbar_expect_tx(smem_u32(&sm.full_q), kK * kQBlock);
 #pragma unroll
-      for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.q[b][0]), &q_map, b * 64, head, w.tile.q_row, smem_u32(&sm.full_q));
-      for (int j = 0; j < stages && !failed; ++j) {
-        const int stage = j % kStages, use = j / kStages, row = w.key_row(j);
-        if (use > 0 && !mbar_wait(smem_u32(&sm.free_k[stage]), (use - 1) & 1)) { failed = true; break; }
-        uint32_t bar = smem_u32(&sm.full_k[stage]);
-        mbar_expect_tx(bar, kK * kBlock);
+        for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.q[b][0]), &q_map, b * 64, w.head, w.tile.q_row, smem_u32(&sm.full_q));
+        for (int j = 0; j < w.stages; ++j) {
+          const int stage = (done + j) % kStages, use = (done + j) / kStages, row = w.key_row(j);
+          if (!wait(&sm.free_k[stage], use)) break;
+          uint32_t bar = smem_u32(&sm.full_k[stage]);
+          mbar_expect_tx(bar, kK * kBlock);
 #pragma unroll
-        for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.k[stage][b][0]), &k_map, b * 64, head / a.share, row, bar);
-        if (use > 0 && !mbar_wait(smem_u32(&sm.free_v[stage]), (use - 1) & 1)) { failed = true; break; }
-        bar = smem_u32(&sm.full_v[stage]);
-        mbar_expect_tx(bar, kV * kBlock);
+          for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.k[stage][b][0]), &k_map, b * 64, w.head / a.share, row, bar);
+          if (!wait(&sm.free_v[stage], use)) break;
+          bar = smem_u32(&sm.full_v[stage]);
+          mbar_expect_tx(bar, kV * kBlock);
 #pragma unroll
-        for (int b = 0; b < kV; ++b) tma_load_2d(smem_u32(&sm.v[stage][b][0]), &v_map, slab0 + b * 64, row, bar);
+          for (int b = 0; b < kV; ++b) tma_load_2d(smem_u32(&sm.v[stage][b][0]), &v_map, w.slab0 + b * 64, row, bar);
+        }
+        done += w.stages;
       }
     }
     __syncwarp();
   } else if (warp == kSoftmaxWarps) {
     const uint64_t q_desc = umma_desc(smem_u32(&sm.q[0][0]), 16, 1024);
-    if (!wait_all(&sm.full_q, 0)) failed = true;
-    for (int j = 0; j < stages && !failed; ++j) {
-      const int b = j % kSides, stage = j % kStages;
-      if ((j >= kSides && !wait_all(&sm.p_free[b], (j / kSides - 1) & 1)) || !wait_all(&sm.full_k[stage], (j / kStages) & 1)) { failed = true; break; }
-      const uint64_t k_desc = umma_desc(smem_u32(&sm.k[stage][0][0]), 16, 1024);
-      if (elect_one()) {
+    for (int item = blockIdx.x, n = 0; item < a.items && !failed; item += gridDim.x, ++n) {
+      const Walk w(a, item, kV * 64);
+      if (!wait_all(&sm.full_q, n & 1)) break;
+      for (int j = 0; j < w.stages; ++j) {
+        const int g = done + j, b = g % kBuffers, stage = g % kStages;
+        if ((g >= kBuffers && !wait_all(&sm.p_free[b], (g / kBuffers - 1) & 1)) || !wait_all(&sm.full_k[stage], (g / kStages) & 1)) break;
+        const uint64_t k_desc = umma_desc(smem_u32(&sm.k[stage][0][0]), 16, 1024);
+        if (elect_one()) {
 #pragma unroll
-        for (int ks = 0; ks < 4 * kK; ++ks)
-          umma_issue(tmem + b * kSideCols, q_desc + static_cast<uint64_t>(((ks >> 2) * kQBlock + (ks & 3) * 32) >> 4),
-                     k_desc + static_cast<uint64_t>(((ks >> 2) * kBlock + (ks & 3) * 32) >> 4), kIdescQK, ks > 0);
-        umma_commit(smem_u32(&sm.s_ready[b]));
-        umma_commit(smem_u32(&sm.free_k[stage]));
+          for (int ks = 0; ks < 4 * kK; ++ks)
+            umma_issue(tmem + b * kBufferCols, q_desc + static_cast<uint64_t>(((ks >> 2) * kQBlock + (ks & 3) * 32) >> 4),
+                       k_desc + static_cast<uint64_t>(((ks >> 2) * kBlock + (ks & 3) * 32) >> 4), kIdescQK, ks > 0);
+          umma_commit(smem_u32(&sm.s_ready[b]));
+          umma_commit(smem_u32(&sm.free_k[stage]));
+          if (j + 1 == w.stages) umma_commit(smem_u32(&sm.q_free));
+        }
+        __syncwarp();
       }
-      __syncwarp();
+      done += w.stages;
     }
   } else if (warp == kSoftmaxWarps + 1) {
-    for (int j = 0; j < stages; ++j) {
-      const int b = j % kSides, stage = j % kStages;
-      if (!wait_all(&sm.full_v[stage], (j / kStages) & 1) || !wait_all(&sm.p_ready[b], (j / kSides) & 1)) { failed = true; break; }
-      const uint64_t v_desc = umma_desc(smem_u32(&sm.v[stage][0][0]), kBlock, 1024);
-      if (elect_one()) {
+    for (int item = blockIdx.x, n = 0; item < a.items && !failed; item += gridDim.x, ++n) {
+      const Walk w(a, item, kV * 64);
+      for (int j = 0; j < w.stages; ++j) {
+        const int g = done + j, b = g % kBuffers, stage = g % kStages;
+        if (!wait_all(&sm.full_v[stage], (g / kStages) & 1) || !wait_all(&sm.p_ready[b], (g / kBuffers) & 1)) break;
+        if (j == 0 && n > 0 && !wait_all(&sm.o_free, (n - 1) & 1)) break;
+        const uint64_t v_desc = umma_desc(smem_u32(&sm.v[stage][0][0]), kBlock, 1024);
+        if (elect_one()) {
 #pragma unroll
-        for (int ks = 0; ks < 4; ++ks)
-          umma_issue_ts(tmem + kColO, tmem + b * kSideCols + ks * 8, v_desc + static_cast<uint64_t>((ks * 2048) >> 4), kIdescPV, (j > 0 || ks > 0) ? 1u : 0u);
-        umma_commit(smem_u32(&sm.p_free[b]));
-        umma_commit(smem_u32(&sm.free_v[stage]));
-        if (j + 1 == stages) umma_commit(smem_u32(&sm.o_done));
+          for (int ks = 0; ks < 4; ++ks)
+            umma_issue_ts(tmem + kColO, tmem + b * kBufferCols + ks * 8, v_desc + static_cast<uint64_t>((ks * 2048) >> 4), kIdescPV, (j > 0 || ks > 0) ? 1u : 0u);
+          umma_commit(smem_u32(&sm.p_free[b]));
+          umma_commit(smem_u32(&sm.free_v[stage]));
+          if (j + 1 == w.stages) umma_commit(smem_u32(&sm.o_done));
+        }
+        __syncwarp();
       }
-      __syncwarp();
+      done += w.stages;
     }
   } else {
-    failed = softmax_rows<kV>(sm, a, w, tmem, head, slab0, [&](int side) { mbar_arrive(smem_u32(&sm.p_ready[side])); });
+    // ---- softmax rows of every second stage, then blocks of 64 output columns ----
+    const int side = warp >> 2, warp_row = (warp & 3) * 32, row = warp_row + lane;
+    const uint32_t tmem_row = tmem + (static_cast<uint32_t>(warp_row) << 16);
+    unsigned char* staging = sm.staging[warp];
+    for (int item = blockIdx.x, n = 0; item < a.items; item += gridDim.x, ++n) {
+      const Walk w(a, item, kV * 64);
+      const bool live = row < w.count;
+      const int position = w.tile.position + row;
+      const int seen_end = live ? position + 1 : 0, seen_begin = position - w.window + 1;   // keys seen_begin .. seen_end - 1, and those below keep
+      const float factor = a.factor * (a.head_scale != nullptr ? a.head_scale[w.head] : 1.0f);
+      float2 sum4[4] = {{0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}};
+      for (int j = (side - done % kSides + kSides) % kSides; j < w.stages; j += kSides) {
+        const int buffer = (done + j) % kBuffers;
+        const uint32_t s_col = tmem_row + buffer * kBufferCols;
+        wait_all(&sm.s_ready[buffer], ((done + j) / kBuffers) & 1);
+        const bool in_kept = j < w.kept_stages;
+        const int end = in_kept ? (live ? w.kept : 0) : seen_end;
+        uint32_t packed[32];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          float s[32];
+          {
+            uint32_t r[32];
+            tmem_load32(s_col + half * 32, r);
+            tmem_load_wait();
+#pragma unroll
+            for (int e = 0; e < 32; ++e) s[e] = __uint_as_float(r[e]);
+          }
+          bounded_weights(s, factor, a.cap_log2);
+          const int first_key = (in_kept ? j * kKeys : w.from + (j - w.kept_stages) * kKeys) + half * 32;
+          if (first_key + 32 > end) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e)
+              if (first_key + e >= end) s[e] = 0.0f;
+          }
+          if (!in_kept && first_key < seen_begin) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e)
+              if (first_key + e < seen_begin && first_key + e >= a.keep) s[e] = 0.0f;
+          }
+#pragma unroll
+          for (int e = 0; e < 16; ++e) {
+            const float2 p = make_float2(s[2 * e], s[2 * e + 1]);
+            sum4[e & 3] = add_pair(sum4[e & 3], p);
+            packed[half * 16 + e] = pack2<true>(p.x, p.y);
+          }
+        }
+        tmem_store32(s_col, packed);
+        tmem_store_wait();
+        tcgen05_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&sm.p_ready[buffer]));
+      }
+      done += w.stages;
+      const float2 sum2 = add_pair(add_pair(sum4[0], sum4[1]), add_pair(sum4[2], sum4[3]));
+      float (&sums)[kSides][kRows] = sm.sums[n & 1];
+      sums[side][row] = sum2.x + sum2.y;
+      wait_all(&sm.o_done, n & 1);
+      asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxWarps * 32) : "memory");
+      float total = 0.0f;
+#pragma unroll
+      for (int b = 0; b < kSides; ++b) total += sums[b][row];
+      const float inv = total > 0.0f ? 1.0f / total : 0.0f;
+      const int64_t first_out = static_cast<int64_t>(w.tile.q_row) + warp_row;
+      const int warp_count = min(max(w.count - warp_row, 0), 32);
+#pragma unroll
+      for (int turn = 0; turn < (kV + kSides - 1) / kSides; ++turn) {
+        const int block = side + turn * kSides;
+        uint32_t r0[32], r1[32];
+        if (block < kV) {
+          tmem_load32(tmem_row + kColO + block * 64, r0);
+          tmem_load32(tmem_row + kColO + block * 64 + 32, r1);
+          tmem_load_wait();
+        }
+        if (turn + 1 == (kV + kSides - 1) / kSides) {        // the warp has seen the last of O
+          tcgen05_before_sync();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(smem_u32(&sm.o_free));
+        }
+        if (block >= kV) continue;
+        // 32 columns at a time through shared memory, so that whole pieces of a row leave together
+        const int column0 = w.slab0 + block * 64;
+        __nv_bfloat16* dst = a.out + first_out * a.out_stride + static_cast<int64_t>(w.head) * a.columns + column0;
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const float* f = reinterpret_cast<const float*>(half == 0 ? &r0[c * 8] : &r1[c * 8]);
+            *reinterpret_cast<uint4*>(staging + lane * 64 + ((c ^ ((lane >> 1) & 3)) << 4)) =
+                make_uint4(pack2<true>(f[0] * inv, f[1] * inv), pack2<true>(f[2] * inv, f[3] * inv),
+                           pack2<true>(f[4] * inv, f[5] * inv), pack2<true>(f[6] * inv, f[7] * inv));
+          }
+          __syncwarp();
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int r = 8 * i + (lane >> 2), piece = lane & 3;
+            if (r < warp_count && column0 + half * 32 + piece * 8 < a.columns)
+              *reinterpret_cast<uint4*>(dst + r * a.out_stride + half * 32 + piece * 8) = *reinterpret_cast<const uint4*>(staging + r * 64 + ((piece ^ ((r >> 1) & 3)) << 4));
+          }
+          __syncwarp();
+        }
+      }
+    }
   }
   if (failed && lane == 0) atomicOr(a.error, 1u);
   tcgen05_before_sync();
@@ -307,160 +349,15 @@ talking_prompt_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
   if (warp == kSoftmaxWarps) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kColumns) : "memory");
 }
 
-// A stage of a pair: each CTA holds 32 of the 64 keys and half of the value columns.
 template <int kK, int kV>
-struct PairShared {
-  static constexpr int kKeyBlock = kKeys / 2 * 128, kStageBytes = kK * kKeyBlock + kV / 2 * kBlock;
-  static constexpr int kFit = (222 * 1024 - kK * kQBlock) / kStageBytes;
-  static constexpr int kStages = kFit < 6 ? kFit : 6;
-  static_assert(kV % 2 == 0 && kStages >= 3 && kStages * kStageBytes + kK * kQBlock >= kSoftmaxWarps * 4096, "the output is staged where Q, keys and values were");
-  unsigned char q[kK][kQBlock];
-  unsigned char k[kStages][kK][kKeyBlock];
-  unsigned char v[kStages][kV / 2][kBlock];
-  unsigned long long full_q, full_k[kStages], full_v[kStages], free_k[kStages], free_v[kStages];
-  unsigned long long s_ready[kSides], p_ready[kSides], p_free[kSides], o_done;
-  float sums[kSides][kRows];
-  uint32_t tmem_base;
-};
-
-template <int kK, int kV>
-__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads, 1)
-talking_pair_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
-                    TalkingPromptArgs a) {
-  using Shared = PairShared<kK, kV>;
-  constexpr int kStages = Shared::kStages, kKeyBlock = Shared::kKeyBlock;
-  extern __shared__ unsigned char smem_raw[];
-  Shared& sm = *reinterpret_cast<Shared*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-  const int lane = threadIdx.x & 31, warp = __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0);
-  const int head = blockIdx.x, slab0 = blockIdx.y * kV * 64;
-  const uint32_t rank = cluster_rank();
-  const bool leader = rank == 0;
-  const Walk w(a, blockIdx.z);
-  const int stages = w.stages;
-
-  if ((blockIdx.x | blockIdx.y | blockIdx.z) == 0 && threadIdx.x == 0) *a.error = 0;   // a wait gives up seconds later
-  if (threadIdx.x == 0) {
-    mbar_init(smem_u32(&sm.full_q), 1);
-    mbar_init(smem_u32(&sm.o_done), 1);
-    for (int s = 0; s < kStages; ++s) {
-      mbar_init(smem_u32(&sm.full_k[s]), leader ? 2 : 1);      // the leader's own copies, and word from the other CTA
-      mbar_init(smem_u32(&sm.full_v[s]), leader ? 2 : 1);
-      mbar_init(smem_u32(&sm.free_k[s]), 1);
-      mbar_init(smem_u32(&sm.free_v[s]), 1);
-    }
-    for (int b = 0; b < kSides; ++b) {
-      mbar_init(smem_u32(&sm.s_ready[b]), 1);
-      mbar_init(smem_u32(&sm.p_ready[b]), 2 * kRows / 32);     // both CTAs' rows; the leader's barrier is the one that counts
-      mbar_init(smem_u32(&sm.p_free[b]), 1);
-    }
-    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-  }
-  if (warp == kSoftmaxWarps) {
-    asm volatile("tcgen05.alloc.cta_group::2.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&sm.tmem_base)), "r"(kColumns) : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::2.sync.aligned;" ::: "memory");
-  }
-  tcgen05_before_sync();
-  __syncthreads();
-  cluster_sync();                              // the other CTA's barriers exist
-  tcgen05_after_sync();
-  const uint32_t tmem = sm.tmem_base;
-  constexpr uint32_t kIdesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(2 * kRows >> 4) << 24);
-  constexpr uint32_t kIdescQK = kIdesc | (static_cast<uint32_t>(kKeys >> 3) << 17);                     // N = 64 keys
-  constexpr uint32_t kIdescPV = kIdesc | (static_cast<uint32_t>(kV * 64 >> 3) << 17) | (1u << 16);       // N = value columns, B MN-major
-  bool failed = false;
-  auto wait_all = [&](unsigned long long* bar, uint32_t parity) {
-    const bool ok = __all_sync(0xffffffffu, mbar_wait_cluster(smem_u32(bar), parity));
-    tcgen05_after_sync();
-    return ok;
-  };
-
-  if (warp == kSoftmaxWarps + 2) {
-    if (lane == 0) {
-      mbar_expect_tx(smem_u32(&sm.full_q), kK * kQBlock);
-#pragma unroll
-      for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.q[b][0]), &q_map, b * 64, head, w.tile.q_row, smem_u32(&sm.full_q));
-      for (int j = 0; j < stages && !failed; ++j) {
-        const int stage = j % kStages, use = j / kStages, row = w.key_row(j);
-        if (use > 0 && !mbar_wait_cluster(smem_u32(&sm.free_k[stage]), (use - 1) & 1)) { failed = true; break; }
-        uint32_t bar = smem_u32(&sm.full_k[stage]);
-        mbar_expect_tx(bar, kK * kKeyBlock);
-#pragma unroll
-        for (int b = 0; b < kK; ++b) tma_load_3d(smem_u32(&sm.k[stage][b][0]), &k_map, b * 64, head / a.share, row + static_cast<int>(rank) * (kKeys / 2), bar);
-        if (use > 0 && !mbar_wait_cluster(smem_u32(&sm.free_v[stage]), (use - 1) & 1)) { failed = true; break; }
-        bar = smem_u32(&sm.full_v[stage]);
-        mbar_expect_tx(bar, kV / 2 * kBlock);
-#pragma unroll
-        for (int b = 0; b < kV / 2; ++b) tma_load_2d(smem_u32(&sm.v[stage][b][0]), &v_map, slab0 + (static_cast<int>(rank) * (kV / 2) + b) * 64, row, bar);
-      }
-    }
-    __syncwarp();
-  } else if (warp >= kSoftmaxWarps && !leader) {
-    const bool keys = warp == kSoftmaxWarps;
-    if (keys && !wait_all(&sm.full_q, 0)) failed = true;
-    for (int j = 0; j < stages && !failed; ++j) {
-      unsigned long long* bar = keys ? &sm.full_k[j % kStages] : &sm.full_v[j % kStages];
-      if (!wait_all(bar, (j / kStages) & 1)) { failed = true; break; }
-      if (lane == 0) mbar_arrive_at(smem_u32(bar), 0);
-      __syncwarp();
-    }
-  } else if (warp == kSoftmaxWarps) {
-    const uint64_t q_desc = umma_desc(smem_u32(&sm.q[0][0]), 16, 1024);
-    if (!wait_all(&sm.full_q, 0)) failed = true;
-    for (int j = 0; j < stages && !failed; ++j) {
-      const int b = j % kSides, stage = j % kStages;
-      if ((j >= kSides && !wait_all(&sm.p_free[b], (j / kSides - 1) & 1)) || !wait_all(&sm.full_k[stage], (j / kStages) & 1)) { failed = true; break; }
-      const uint64_t k_desc = umma_desc(smem_u32(&sm.k[stage][0][0]), 16, 1024);
-      if (elect_one()) {
-#pragma unroll
-        for (int ks = 0; ks < 4 * kK; ++ks)
-          umma_pair_issue(tmem + b * kSideCols, q_desc + static_cast<uint64_t>(((ks >> 2) * kQBlock + (ks & 3) * 32) >> 4),
-                          k_desc + static_cast<uint64_t>(((ks >> 2) * kKeyBlock + (ks & 3) * 32) >> 4), kIdescQK, ks > 0);
-        umma_pair_commit(smem_u32(&sm.s_ready[b]));
-        umma_pair_commit(smem_u32(&sm.free_k[stage]));
-      }
-      __syncwarp();
-    }
-  } else if (warp == kSoftmaxWarps + 1) {
-    for (int j = 0; j < stages; ++j) {
-      const int b = j % kSides, stage = j % kStages;
-      if (!wait_all(&sm.full_v[stage], (j / kStages) & 1) || !wait_all(&sm.p_ready[b], (j / kSides) & 1)) { failed = true; break; }
-      const uint64_t v_desc = umma_desc(smem_u32(&sm.v[stage][0][0]), kBlock, 1024);
-      if (elect_one()) {
-#pragma unroll
-        for (int ks = 0; ks < 4; ++ks)
-          umma_pair_issue_ts(tmem + kColO, tmem + b * kSideCols + ks * 8, v_desc + static_cast<uint64_t>((ks * 2048) >> 4), kIdescPV, (j > 0 || ks > 0) ? 1u : 0u);
-        umma_pair_commit(smem_u32(&sm.p_free[b]));
-        umma_pair_commit(smem_u32(&sm.free_v[stage]));
-        if (j + 1 == stages) umma_pair_commit(smem_u32(&sm.o_done));
-      }
-      __syncwarp();
-    }
-  } else {
-    failed = softmax_rows<kV>(sm, a, w, tmem, head, slab0, [&](int side) { mbar_arrive_at(smem_u32(&sm.p_ready[side]), 0); });
-  }
-  if (failed && lane == 0) atomicOr(a.error, 1u);
-  tcgen05_before_sync();
-  __syncthreads();
-  cluster_sync();                              // neither CTA leaves while the other may read its memory or arrive at its barriers
-  tcgen05_after_sync();
-  if (warp == kSoftmaxWarps) asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kColumns) : "memory");
-}
-
-template <int kK, int kV>
-int launch_pair(const TalkingPromptArgs& a, const CUtensorMap (&maps)[3], int slabs, int tile_count, cudaStream_t stream) {
-  auto kernel = talking_pair_kernel<kK, kV>;
-  const size_t smem = sizeof(PairShared<kK, kV>) + 1024;
-  RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-  kernel<<<dim3(static_cast<unsigned>(a.heads), static_cast<unsigned>(slabs), static_cast<unsigned>(tile_count)), kThreads, smem, stream>>>(maps[0], maps[1], maps[2], a);
-  return launch_status("talking_pair_kernel");
-}
-
-template <int kK, int kV>
-int launch(const TalkingPromptArgs& a, const CUtensorMap (&maps)[3], int slabs, int tile_count, cudaStream_t stream) {
+int launch(const TalkingPromptArgs& a, const CUtensorMap (&maps)[3], cudaStream_t stream) {
+  DeviceInfo info;
+  const int status = current_device_info(&info);
+  if (status != RLT_OK) return status;
   auto kernel = talking_prompt_kernel<kK, kV>;
   const size_t smem = sizeof(SpreadShared<kK, kV>) + 1024;
   RLT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-  kernel<<<dim3(static_cast<unsigned>(a.heads), static_cast<unsigned>(slabs), static_cast<unsigned>(tile_count)), kThreads, smem, stream>>>(maps[0], maps[1], maps[2], a);
+  kernel<<<static_cast<unsigned>(a.items < info.sm_count ? a.items : info.sm_count), kThreads, smem, stream>>>(maps[0], maps[1], maps[2], a);
   return launch_status("talking_prompt_kernel");
 }
 
@@ -495,27 +392,23 @@ extern "C" RLT_API int rlt_talking_prompt(const void* q, int64_t q_stride, const
   a.factor = static_cast<float>(static_cast<double>(scale) / static_cast<double>(softcap));
   a.cap_log2 = static_cast<float>(1.4426950408889634 * static_cast<double>(softcap));
   a.head_scale = head_scale; a.error = static_cast<unsigned*>(workspace);
-  const bool pair = a.share % 2 == 0;              // two heads that share a key/value head
   const int blocks = (columns + 63) / 64, slabs = (blocks + kMaxBlocks - 1) / kMaxBlocks, per = (blocks + slabs - 1) / slabs;
-  RLT_REQUIRE(slabs <= 65535 && tile_count <= 65535, "talking_prompt: batch exceeds the grid limits");
+  RLT_REQUIRE(static_cast<int64_t>(slabs) * heads * tile_count <= 0x7fffffff, "talking_prompt: batch too large");
+  a.slabs = slabs; a.items = slabs * heads * tile_count;
   CUtensorMap maps[3];
   if (make_box_map<3>(&maps[0], q, {dim, heads, rows}, {1, dim, q_stride}, {64, 1, kRows}) != RLT_OK ||
-      make_box_map<3>(&maps[1], keys, {dim, kv_heads, key_rows}, {1, dim, key_stride}, {64, 1, pair ? kKeys / 2 : kKeys}) != RLT_OK ||
+      make_box_map<3>(&maps[1], keys, {dim, kv_heads, key_rows}, {1, dim, key_stride}, {64, 1, kKeys}) != RLT_OK ||
       make_box_map<2>(&maps[2], values, {columns, key_rows}, {1, value_stride}, {64, kKeys}) != RLT_OK) {
     set_last_error_text("talking_prompt: cuTensorMapEncodeTiled rejected the operands");
     return RLT_ERR_UNSUPPORTED;
   }
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (pair) {
-    if (dim <= 64) return per <= 2 ? launch_pair<1, 2>(a, maps, slabs, tile_count, s) : launch_pair<1, 4>(a, maps, slabs, tile_count, s);
-    return per <= 2 ? launch_pair<2, 2>(a, maps, slabs, tile_count, s) : launch_pair<2, 4>(a, maps, slabs, tile_count, s);
-  }
 #define RLT_SPREAD(K)                                                        \
   switch (per) {                                                             \
-    case 1: return launch<K, 1>(a, maps, slabs, tile_count, s);              \
-    case 2: return launch<K, 2>(a, maps, slabs, tile_count, s);              \
-    case 3: return launch<K, 3>(a, maps, slabs, tile_count, s);              \
-    default: return launch<K, 4>(a, maps, slabs, tile_count, s);             \
+    case 1: return launch<K, 1>(a, maps, s);  \
+    case 2: return launch<K, 2>(a, maps, s);  \
+    case 3: return launch<K, 3>(a, maps, s);  \
+    default: return launch<K, 4>(a, maps, s); \
   }
   if (dim <= 64) { RLT_SPREAD(1) }
   RLT_SPREAD(2)

@@ -214,48 +214,6 @@ __device__ __forceinline__ void umma_issue_ts(uint32_t tmem_d, uint32_t tmem_a, 
                ::"r"(tmem_d), "r"(tmem_a), "l"(b), "r"(idesc), "r"(accumulate) : "memory");
 }
 
-// ---- two CTAs of a cluster on one product (cta_group::2) ------------------------------------
-// Each brings its rows of A and half of B's columns and receives its rows of D; the CTA of rank 0 issues for both.
-__device__ __forceinline__ uint32_t cluster_rank() {
-  uint32_t r;
-  asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
-  return r;
-}
-__device__ __forceinline__ void cluster_sync() {
-  asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-// Arrival at the barrier of the same offset in the CTA of rank `rank`.
-__device__ __forceinline__ void mbar_arrive_at(uint32_t bar, uint32_t rank) {
-  asm volatile("{\n.reg .b32 a;\nmapa.shared::cluster.u32 a, %0, %1;\nmbarrier.arrive.release.cluster.shared::cluster.b64 _, [a];\n}\n" ::"r"(bar), "r"(rank) : "memory");
-}
-// Bounded wait for a barrier at which other CTAs of the cluster arrive.
-__device__ __forceinline__ bool mbar_wait_cluster(uint32_t bar, uint32_t parity) {
-  const long long t0 = clock64();
-  for (;;) {
-    for (int i = 0; i < 64; ++i) {
-      uint32_t ok;
-      asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\nselp.u32 %0, 1, 0, p;\n}\n"
-                   : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-      if (ok != 0) return true;
-    }
-    if (clock64() - t0 > kWaitCycles) return false;
-  }
-}
-__device__ __forceinline__ void umma_pair_issue(uint32_t tmem_d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile("{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-               "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n}\n"
-               ::"r"(tmem_d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void umma_pair_issue_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile("{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-               "tcgen05.mma.cta_group::2.kind::f16 [%0], [%1], %2, %3, p;\n}\n"
-               ::"r"(tmem_d), "r"(tmem_a), "l"(b), "r"(idesc), "r"(accumulate) : "memory");
-}
-// Arrival at the barrier of the same offset in both CTAs when the products issued so far are complete.
-__device__ __forceinline__ void umma_pair_commit(uint32_t bar) {
-  asm volatile("tcgen05.commit.cta_group::2.mbarrier::arrive::one.shared::cluster.multicast::cluster.b64 [%0], %1;" ::"r"(bar), "h"(static_cast<uint16_t>(3)) : "memory");
-}
-
 // Packed fp32 pairs and the three-input maximum of sm_100: half the instructions for the scaling,
 // the sums and the row maximum of the softmax, whose warps are bound by issue slots and latency.
 __device__ __forceinline__ float2 fma_pair(float2 a, float2 b, float2 c) {
