@@ -1005,7 +1005,10 @@ class KernelRows:
     def __call__(self, kernel, phase, like, make, nbytes=0.0, flops=0.0, copies=None):
         """make(i) -> a call on the i-th set of tensors."""
         copies = copies or max(2, min(48, int(400e6 // max(nbytes, 1)) + 1))
-        us = ring_us([make(i) for i in range(copies)], self.steps)
+        calls = [make(i) for i in range(copies)]
+        torch.cuda.synchronize()
+        time.sleep(0.25)       # a row is timed in isolation, like the peaks: the clock has come back from the row before it
+        us = ring_us(calls, self.steps)
         tensor = flops / self.peak_tflops / 1e6 > nbytes / self.peak_gbs / 1e3
         frac = flops / us / 1e6 / self.peak_tflops if tensor else nbytes / us / 1e3 / self.peak_gbs
         self.rows.append({"kernel": kernel, "phase": phase, "like": like, "us": us, "bound": "tensor" if tensor else "hbm", "roofline_frac": frac})
